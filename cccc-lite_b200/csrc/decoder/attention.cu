@@ -1,0 +1,227 @@
+// What precedes attention (unit RMS of q and k, value mixing, cache append) and the plain attention kernel of the float
+// mode.
+#include "attention.cuh"
+
+namespace b200
+{
+
+// One CTA per token, one warp per head at a time: q heads, then k heads, then v heads.
+template <class T>
+__global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams p)
+{
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int i = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int e = p.token_entry[i];
+    const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
+    if (row >= p.T_max) { return; }
+    T* x = (T*)p.qkvg + (size_t)i * p.ld;
+    const size_t kv0 = (size_t)p.slot[e] * p.Hkv;
+    for (unsigned int h = warp; h < p.H + 2 * p.Hkv; h += warps)
+    {
+        if (h < p.H + p.Hkv)
+        {
+            const bool is_q = h < p.H;
+            const unsigned int kh = h - p.H;
+            T* src = is_q ? x + (size_t)h * p.dim : x + p.k_off + (size_t)kh * p.dim;
+            T* dst = is_q ? src : (T*)p.k_cache + ((kv0 + kh) * p.T_max + row) * p.k_ld;
+            if (is_q && !p.qk_norm) { continue; }
+            float inv = 1.f;
+            if (p.qk_norm)
+            {
+                float sq = 0.f;
+                for (unsigned int d = lane; d < p.dim; d += 32)
+                {
+                    const float v = Elem<T>::get(src[d]);
+                    sq += v * v;
+                }
+                inv = 1.0f / sqrtf(warp_sum(sq) / (float)p.dim + p.eps);
+            }
+            for (unsigned int d = lane; d < p.dim; d += 32) { dst[d] = Elem<T>::put(Elem<T>::get(src[d]) * inv); }
+        }
+        else
+        {
+            const unsigned int vh = h - p.H - p.Hkv;
+            const T* src = x + p.v_off + (size_t)vh * p.vdim;
+            T* dst = (T*)p.v_cache + ((kv0 + vh) * p.T_max + row) * p.v_ld;
+            T* first = p.v_mix ? (T*)p.v_first + (size_t)i * p.v_first_ld + (size_t)vh * p.vdim : nullptr;
+            for (unsigned int d = lane; d < p.vdim; d += 32)
+            {
+                float v = Elem<T>::get(src[d]);
+                if (p.v_mix == 1) { first[d] = src[d]; }
+                else if (p.v_mix == 2) { v = (1.0f - p.lambda) * v + p.lambda * Elem<T>::get(first[d]); }
+                dst[d] = Elem<T>::put(v);
+            }
+        }
+    }
+}
+
+constexpr unsigned int AP_KEYS = 128;
+
+// One CTA per (token, kv head): its G query heads against the cache in chunks of 128 keys with a running softmax.
+template <class T>
+__global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p)
+{
+    extern __shared__ float ap_smem[];
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int i = blockIdx.x, kvh = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int e = p.token_entry[i];
+    const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
+    const unsigned int keys = min(row + 1u, p.T_max), G = p.G;
+    float* q = ap_smem;                     // [G][dim]
+    float* sc = q + G * p.dim;              // [G][128]
+    float* acc = sc + G * AP_KEYS;          // [G][vdim]
+    float* ml = acc + G * p.vdim;           // [G][3]: maximum, sum, correction
+    const T* x = (const T*)p.qkvg + (size_t)i * p.ld;
+    const T* K = (const T*)p.k_cache + (((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max) * p.k_ld;
+    const T* V = (const T*)p.v_cache + (((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max) * p.v_ld;
+    for (unsigned int j = tid; j < G * p.dim; j += 128) { q[j] = Elem<T>::get(x[(size_t)kvh * G * p.dim + j]); }
+    for (unsigned int j = tid; j < G * p.vdim; j += 128) { acc[j] = 0.f; }
+    for (unsigned int g = tid; g < G; g += 128)
+    {
+        ml[3 * g] = -INFINITY;
+        ml[3 * g + 1] = 0.f;
+    }
+    __syncthreads();
+    for (unsigned int k0 = 0; k0 < keys; k0 += AP_KEYS)
+    {
+        const unsigned int nk = min(AP_KEYS, keys - k0);
+        if (tid < nk)
+        {
+            const T* kr = K + (size_t)(k0 + tid) * p.k_ld;
+            for (unsigned int g = 0; g < G; g++)
+            {
+                float s = 0.f;
+                for (unsigned int d = 0; d < p.dim; d++) { s = fmaf(q[g * p.dim + d], Elem<T>::get(kr[d]), s); }
+                sc[g * AP_KEYS + tid] = s * p.scale;
+            }
+        }
+        __syncthreads();
+        for (unsigned int g = warp; g < G; g += 4)
+        {
+            float* s = sc + g * AP_KEYS;
+            float m = -INFINITY;
+            for (unsigned int j = lane; j < nk; j += 32) { m = fmaxf(m, s[j]); }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) { m = fmaxf(m, __shfl_xor_sync(0xFFFFFFFFu, m, o)); }
+            const float mo = ml[3 * g], mn = fmaxf(mo, m);
+            float l = 0.f;
+            for (unsigned int j = lane; j < nk; j += 32)
+            {
+                const float w = expf(s[j] - mn);
+                s[j] = w;
+                l += w;
+            }
+            l = warp_sum(l);
+            __syncwarp();
+            if (lane == 0)
+            {
+                const float c = expf(mo - mn);
+                ml[3 * g] = mn;
+                ml[3 * g + 1] = ml[3 * g + 1] * c + l;
+                ml[3 * g + 2] = c;
+            }
+        }
+        __syncthreads();
+        for (unsigned int j = tid; j < G * p.vdim; j += 128)
+        {
+            const unsigned int g = j / p.vdim, d = j % p.vdim;
+            const float* s = sc + g * AP_KEYS;
+            float o = acc[j] * ml[3 * g + 2];
+            for (unsigned int k = 0; k < nk; k++) { o = fmaf(s[k], Elem<T>::get(V[(size_t)(k0 + k) * p.v_ld + d]), o); }
+            acc[j] = o;
+        }
+        __syncthreads();
+    }
+    T* out = (T*)p.out + (size_t)i * p.ldo + (size_t)kvh * G * p.vdim;
+    for (unsigned int j = tid; j < G * p.vdim; j += 128)
+    {
+        float o = acc[j] / ml[3 * (j / p.vdim) + 1];
+        if (p.gate) { o *= sigmoid_f32(Elem<T>::get(x[p.g_off + (size_t)kvh * G * p.vdim + j])); }
+        out[j] = Elem<T>::put(o);
+    }
+}
+
+template <class T>
+static int attention_append(const AttnParams& p, unsigned int tokens, void* stream, bool pdl)
+{
+    const unsigned int heads = p.H + 2 * p.Hkv;
+    const unsigned int warps = heads < 8 ? heads : 8;
+    return launch_kernel("attention_append", attention_append_kernel<T>, dim3(tokens), dim3(32 * warps), 0, stream, pdl, p);
+}
+
+template <class T>
+static int attention_plain(const AttnParams& p, unsigned int tokens, void* stream, bool pdl)
+{
+    const size_t smem = (size_t)p.G * (p.dim + p.vdim + AP_KEYS + 3) * 4;
+    const DecoderDevice* dev = decoder_device();
+    if (!dev || smem > (size_t)dev->max_smem) { return -1; }
+    return launch_kernel("attention_plain", attention_plain_kernel<T>, dim3(tokens, p.Hkv), dim3(128), smem, stream, pdl, p);
+}
+
+}    // namespace b200
+
+using namespace b200;
+
+static unsigned int vdim_padded(unsigned int vdim) { return (vdim + 15) / 16 * 16; }
+
+C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim)
+{
+    return kAttnCounters * 4ull + (unsigned long long)kAttnPartials * 16 * (vdim_padded(vdim) + 2) * 4;
+}
+
+C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, const cuda_b200_batch* b, void* stream, unsigned int flags, int kernel)
+{
+    if (!a || !b) { return -1; }
+    if (b->tokens == 0 || b->entries == 0) { return 0; }
+    if (!a->qkvg || !a->out || !a->k_cache || !a->v_cache || !a->work || !b->slot || !b->pos || !b->start || !b->n || !b->token_entry) { return -1; }
+    if ((dtype != DT_BF16 && dtype != DT_FLOAT) || a->H == 0 || a->Hkv == 0 || (a->H % a->Hkv) || a->dim == 0 || a->vdim == 0 || a->k_ld < a->dim
+        || a->v_ld < a->vdim || (a->k_ld % 8) || (a->v_ld % 8) || a->T_max == 0 || (a->v_mix && !a->v_first))
+    {
+        return -1;
+    }
+    AttnParams p;
+    p.qkvg = a->qkvg;
+    p.out = a->out;
+    p.k_cache = a->k_cache;
+    p.v_cache = a->v_cache;
+    p.v_first = a->v_first;
+    p.counter = (int*)a->work;
+    p.partial = (float*)a->work + kAttnCounters;
+    p.slot = (const int*)b->slot;
+    p.pos = (const int*)b->pos;
+    p.start = (const int*)b->start;
+    p.n = (const int*)b->n;
+    p.token_entry = (const int*)b->token_entry;
+    p.ld = a->ld;
+    p.ldo = a->ldo;
+    p.k_off = a->k_off;
+    p.v_off = a->v_off;
+    p.g_off = a->g_off;
+    p.v_first_ld = a->v_first_ld;
+    p.H = a->H;
+    p.Hkv = a->Hkv;
+    p.G = a->H / a->Hkv;
+    p.dim = a->dim;
+    p.vdim = a->vdim;
+    p.k_ld = a->k_ld;
+    p.v_ld = a->v_ld;
+    p.T_max = a->T_max;
+    p.splits = p.row_tiles = 1;
+    p.v_mix = a->v_mix;
+    p.qk_norm = a->qk_norm;
+    p.gate = a->gate;
+    p.lambda = a->lambda;
+    p.eps = a->eps;
+    p.scale = a->scale;
+    const bool pdl = (flags & 1u) != 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    int rc = dtype == DT_BF16 ? attention_append<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_append<float>(p, b->tokens, st, pdl);
+    if (rc) { return rc; }
+    if (dtype == DT_FLOAT) { return attention_plain<float>(p, b->tokens, st, pdl); }
+    if (kernel == 0) { kernel = p.dim > 256 || p.vdim > 256 ? 3 : (b->max_n * p.G <= 64 || b->max_n <= 4 ? 1 : 2); }
+    if (kernel == 1) { return launch_attention_split(p, b->entries, b->max_n, b->max_len, st, pdl); }
+    if (kernel == 2) { return launch_attention_tiled(p, b->entries, b->max_n, st, pdl); }
+    return attention_plain<__nv_bfloat16>(p, b->tokens, st, pdl);
+}

@@ -1,0 +1,481 @@
+// BF16 attention on mma.sync: a warp holds 16 query rows (a row is one query head of one token; the heads that share a
+// kv head are packed together) as A fragments and walks keys with a running softmax in float.  Keys arrive through
+// cp.async into padded shared-memory rows; K is the B operand as it lies, V through transposed ldmatrix.  Softmax weights
+// enter the value product as the sum of two BF16 numbers, so that they keep 16 significant bits.
+//   split : few query rows.  A CTA's four warps take 16-key tiles of one split of the sequence in turn, each through a
+//           ring of its own; their partial results meet in shared memory, the splits' in global memory, where the last
+//           CTA to arrive adds them in split order.
+//   tiled : prompts.  Four warps with 16 rows each share 64-key tiles, double buffered.
+#pragma once
+
+#include "attention.cuh"
+#include "../gemv_decode.cuh"
+
+namespace b200
+{
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid)
+{
+    const int bytes = valid ? 16 : 0;    // 0: sixteen zero bytes
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait()
+{
+    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr)
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr)
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"(addr));
+}
+
+// 16 query rows of one warp and their running softmax.
+template <int DK, int DV>
+struct RowTile
+{
+    uint32_t q[DK / 16][4];
+    float o[DV / 8][4];
+    float m[2], l[2];    // rows lane / 4 and lane / 4 + 8, in units of log2
+
+    // r0: first packed row of the tile inside entry e
+    __device__ __forceinline__ void init(const AttnParams& p, const __nv_bfloat16* qkvg, unsigned int start, unsigned int n, unsigned int kvh,
+        unsigned int r0, unsigned int lane)
+    {
+        const unsigned int rows = n * p.G;
+        const __nv_bfloat16* src[2];
+        bool ok[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+        {
+            const unsigned int r = r0 + (lane >> 2) + 8 * h;
+            ok[h] = r < rows;
+            const unsigned int rr = ok[h] ? r : 0;
+            src[h] = qkvg + (size_t)(start + rr / p.G) * p.ld + (size_t)(kvh * p.G + rr % p.G) * p.dim;
+            m[h] = -INFINITY;
+            l[h] = 0.f;
+        }
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; kk++)
+        {
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                const int h = j & 1;
+                const unsigned int d = kk * 16 + (lane & 3) * 2 + (j >> 1) * 8;
+                uint32_t lo = 0, hi = 0;
+                if (ok[h] && d < p.dim) { lo = __bfloat16_as_ushort(src[h][d]); }
+                if (ok[h] && d + 1 < p.dim) { hi = __bfloat16_as_ushort(src[h][d + 1]); }
+                q[kk][j] = lo | (hi << 16);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < DV / 8; i++)
+        {
+#pragma unroll
+            for (int j = 0; j < 4; j++) { o[i][j] = 0.f; }
+        }
+    }
+
+    // KT keys (a multiple of 16) at shared addresses ks / vs, the first being key k0 of the sequence; row h sees keys
+    // below lim[h].  scale2 = scale * log2(e).
+    template <int KT>
+    __device__ __forceinline__ void step(uint32_t ks, uint32_t vs, unsigned int k0, const unsigned int (&lim)[2], bool masked, float scale2,
+        unsigned int dim, unsigned int vdim, unsigned int lane)
+    {
+        constexpr int KS = (DK + 8) * 2, VS = (DV + 8) * 2;
+        float s[KT / 8][4];
+#pragma unroll
+        for (int i = 0; i < KT / 8; i++)
+        {
+#pragma unroll
+            for (int j = 0; j < 4; j++) { s[i][j] = 0.f; }
+        }
+        // lanes 0-7: keys 0-7, k 0-7; 8-15: keys 0-7, k 8-15; 16-23: keys 8-15, k 0-7; 24-31: keys 8-15, k 8-15
+        const uint32_t kb = ks + ((lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 16;
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; kk++)
+        {
+            if (kk * 16 < (int)dim)
+            {
+#pragma unroll
+                for (int i = 0; i < KT / 16; i++)
+                {
+                    uint32_t b[4];
+                    ldmatrix_x4(b, kb + i * 16 * KS + kk * 32);
+                    mma_bf16_16816(s[2 * i], q[kk][0], q[kk][1], q[kk][2], q[kk][3], b[0], b[1]);
+                    mma_bf16_16816(s[2 * i + 1], q[kk][0], q[kk][1], q[kk][2], q[kk][3], b[2], b[3]);
+                }
+            }
+        }
+        float mx[2] = { -INFINITY, -INFINITY };
+#pragma unroll
+        for (int i = 0; i < KT / 8; i++)
+        {
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                s[i][j] *= scale2;
+                if (masked && k0 + i * 8 + (lane & 3) * 2 + (j & 1) >= lim[j >> 1]) { s[i][j] = -INFINITY; }
+                mx[j >> 1] = fmaxf(mx[j >> 1], s[i][j]);
+            }
+        }
+        float base[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+        {
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xFFFFFFFFu, mx[h], 1));
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xFFFFFFFFu, mx[h], 2));
+            const float mn = fmaxf(m[h], mx[h]);
+            base[h] = mn == -INFINITY ? 0.f : mn;
+            const float c = exp2f(m[h] - base[h]);    // 0 while nothing has been seen
+            m[h] = mn;
+            l[h] *= c;
+#pragma unroll
+            for (int i = 0; i < DV / 8; i++)
+            {
+                o[i][2 * h] *= c;
+                o[i][2 * h + 1] *= c;
+            }
+        }
+        const uint32_t vb = vs + (lane & 15) * VS + (lane >> 4) * 16;
+#pragma unroll
+        for (int i = 0; i < KT / 16; i++)
+        {
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                // a0: row g, keys 0-7; a1: row g + 8, keys 0-7; a2, a3: keys 8-15
+                float* c = &s[2 * i + (j >> 1)][(j & 1) * 2];
+                const int h = j & 1;
+                const float p0 = exp2f(c[0] - base[h]), p1 = exp2f(c[1] - base[h]);
+                l[h] += p0 + p1;
+                hi[j] = pack_bf16x2(p0, p1);
+                lo[j] = pack_bf16x2(p0 - __uint_as_float(hi[j] << 16), p1 - __uint_as_float(hi[j] & 0xFFFF0000u));
+            }
+#pragma unroll
+            for (int d = 0; d < DV / 16; d++)
+            {
+                if (d * 16 < (int)vdim)
+                {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, vb + i * 16 * VS + d * 32);
+                    mma_bf16_16816(o[2 * d], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+                    mma_bf16_16816(o[2 * d + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+                    mma_bf16_16816(o[2 * d], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+                    mma_bf16_16816(o[2 * d + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+                }
+            }
+        }
+    }
+    // the row sums are held per lane until here
+    __device__ __forceinline__ void finish()
+    {
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+        {
+            l[h] += __shfl_xor_sync(0xFFFFFFFFu, l[h], 1);
+            l[h] += __shfl_xor_sync(0xFFFFFFFFu, l[h], 2);
+        }
+    }
+};
+
+__device__ __forceinline__ void attention_store(const AttnParams& p, const __nv_bfloat16* qkvg, unsigned int start, unsigned int kvh, unsigned int r,
+    unsigned int d, float v)
+{
+    const unsigned int col = (kvh * p.G + r % p.G) * p.vdim + d;
+    const size_t tok = start + r / p.G;
+    if (p.gate) { v *= sigmoid_f32(__bfloat162float(qkvg[tok * p.ld + p.g_off + col])); }
+    ((__nv_bfloat16*)p.out)[tok * p.ldo + col] = __float2bfloat16_rn(v);
+}
+
+constexpr int AS_WARPS = 4, AS_KT = 16;
+__host__ __device__ constexpr int as_stages(int dk, int dv) { return dk + dv <= 256 ? 4 : 3; }
+__host__ __device__ constexpr int as_tile_bytes(int dk, int dv) { return AS_KT * ((dk + 8) + (dv + 8)) * 2; }
+__host__ __device__ constexpr int as_smem(int dk, int dv)
+{
+    const int ring = AS_WARPS * as_stages(dk, dv) * as_tile_bytes(dk, dv), meet = AS_WARPS * 16 * (dv + 2) * 4;
+    return ring > meet ? ring : meet;
+}
+
+// grid (splits, Hkv * row_tiles, entries)
+template <int DK, int DV>
+__global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const AttnParams p)
+{
+    extern __shared__ __align__(16) unsigned char as_raw[];
+    constexpr int ST = as_stages(DK, DV), TB = as_tile_bytes(DK, DV), KS = (DK + 8) * 2, VS = (DV + 8) * 2;
+    __shared__ float ml[AS_WARPS][16][2];
+    __shared__ int last;
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const unsigned int split = blockIdx.x, kvh = blockIdx.y % p.Hkv, rt = blockIdx.y / p.Hkv, e = blockIdx.z;
+    const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e], r0 = rt * 16;
+    const unsigned int rows = n * p.G;
+    if (r0 >= rows) { return; }
+    const __nv_bfloat16* qkvg = (const __nv_bfloat16*)p.qkvg;
+    const size_t seq = ((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max;
+    const __nv_bfloat16* K = (const __nv_bfloat16*)p.k_cache + seq * p.k_ld;
+    const __nv_bfloat16* V = (const __nv_bfloat16*)p.v_cache + seq * p.v_ld;
+    // keys that any row of the tile sees, cut into equal runs of whole tiles
+    const unsigned int last_row = min(r0 + 15u, rows - 1);
+    const unsigned int T = min(pos + last_row / p.G + 1, p.T_max);
+    const unsigned int tiles = (T + AS_KT - 1) / AS_KT, per = (tiles + p.splits - 1) / p.splits;
+    const unsigned int tile0 = min(split * per, tiles), tile1 = min(tile0 + per, tiles);
+    const unsigned int first_lim = pos + r0 / p.G + 1;    // every row sees the keys below
+
+    RowTile<DK, DV> w;
+    w.init(p, qkvg, start, n, kvh, r0, lane);
+    unsigned int lim[2];
+#pragma unroll
+    for (int h = 0; h < 2; h++) { lim[h] = min(pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1, T); }
+
+    const uint32_t ring = smem_u32(as_raw) + warp * (ST * TB);
+    auto fetch = [&](unsigned int i) {    // i-th tile of this warp
+        const unsigned int tile = tile0 + warp + i * AS_WARPS;
+        if (tile < tile1)
+        {
+            const uint32_t ks = ring + (i % ST) * TB, vs = ks + AS_KT * KS;
+            for (unsigned int c = lane; c < AS_KT * (DK / 8); c += 32)
+            {
+                const unsigned int r = c / (DK / 8), d = c % (DK / 8), key = tile * AS_KT + r;
+                const bool ok = key < T && d * 8 < p.k_ld;
+                cp_async16(ks + r * KS + d * 16, K + (ok ? (size_t)key * p.k_ld + d * 8 : 0), ok);
+            }
+            for (unsigned int c = lane; c < AS_KT * (DV / 8); c += 32)
+            {
+                const unsigned int r = c / (DV / 8), d = c % (DV / 8), key = tile * AS_KT + r;
+                const bool ok = key < T && d * 8 < p.v_ld;
+                cp_async16(vs + r * VS + d * 16, V + (ok ? (size_t)key * p.v_ld + d * 8 : 0), ok);
+            }
+        }
+        cp_async_commit();
+    };
+#pragma unroll
+    for (int i = 0; i < ST - 1; i++) { fetch(i); }
+    const float scale2 = p.scale * 1.44269504088896341f;
+    unsigned int i = 0;
+    for (unsigned int tile = tile0 + warp; tile < tile1; tile += AS_WARPS, i++)
+    {
+        fetch(i + ST - 1);
+        cp_async_wait<ST - 1>();
+        __syncwarp();
+        const uint32_t ks = ring + (i % ST) * TB;
+        w.template step<AS_KT>(ks, ks + AS_KT * KS, tile * AS_KT, lim, (tile + 1) * AS_KT > first_lim, scale2, p.dim, p.vdim, lane);
+        __syncwarp();
+    }
+    cp_async_wait<0>();
+    w.finish();
+    __syncthreads();    // the rings become the meeting place
+    float* om = reinterpret_cast<float*>(as_raw) + warp * 16 * DV;
+    const unsigned int gr = lane >> 2, gc = (lane & 3) * 2;
+#pragma unroll
+    for (int d = 0; d < DV / 8; d++)
+    {
+        *reinterpret_cast<float2*>(om + gr * DV + d * 8 + gc) = make_float2(w.o[d][0], w.o[d][1]);
+        *reinterpret_cast<float2*>(om + (gr + 8) * DV + d * 8 + gc) = make_float2(w.o[d][2], w.o[d][3]);
+    }
+    if ((lane & 3) == 0)
+    {
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+        {
+            ml[warp][gr + 8 * h][0] = w.m[h];
+            ml[warp][gr + 8 * h][1] = w.l[h];
+        }
+    }
+    __syncthreads();
+    const unsigned int live = min(16u, rows - r0);
+    auto combine = [&](unsigned int r, unsigned int d, float& m, float& l, float& o) {
+        m = fmaxf(fmaxf(ml[0][r][0], ml[1][r][0]), fmaxf(ml[2][r][0], ml[3][r][0]));
+        l = o = 0.f;
+        if (m == -INFINITY) { return; }
+#pragma unroll
+        for (int j = 0; j < AS_WARPS; j++)
+        {
+            const float c = exp2f(ml[j][r][0] - m);
+            l += c * ml[j][r][1];
+            o += c * reinterpret_cast<float*>(as_raw)[(j * 16 + r) * DV + d];
+        }
+    };
+    if (p.splits == 1)
+    {
+        for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
+        {
+            float m, l, o;
+            combine(j / p.vdim, j % p.vdim, m, l, o);
+            attention_store(p, qkvg, start, kvh, r0 + j / p.vdim, j % p.vdim, o / l);
+        }
+        return;
+    }
+    const unsigned int vp = (p.vdim + 15) / 16 * 16, stride = 16 * (vp + 2);
+    const unsigned int unit = (e * p.row_tiles + rt) * p.Hkv + kvh;
+    float* mine = p.partial + ((size_t)unit * p.splits + split) * stride;
+    for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
+    {
+        const unsigned int r = j / p.vdim, d = j % p.vdim;
+        float m, l, o;
+        combine(r, d, m, l, o);
+        mine[32 + r * vp + d] = o;
+        if (d == 0)
+        {
+            mine[2 * r] = m;
+            mine[2 * r + 1] = l;
+        }
+    }
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) { last = atomicAdd(p.counter + unit, 1) == (int)p.splits - 1; }
+    __syncthreads();
+    if (!last) { return; }
+    __threadfence();
+    const float* all = p.partial + (size_t)unit * p.splits * stride;
+    for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
+    {
+        const unsigned int r = j / p.vdim, d = j % p.vdim;
+        float m = -INFINITY, l = 0.f, o = 0.f;
+        for (unsigned int s = 0; s < p.splits; s++) { m = fmaxf(m, __ldcg(all + s * stride + 2 * r)); }
+        for (unsigned int s = 0; s < p.splits; s++)
+        {
+            const float c = exp2f(__ldcg(all + s * stride + 2 * r) - m);
+            l += c * __ldcg(all + s * stride + 2 * r + 1);
+            o += c * __ldcg(all + s * stride + 32 + r * vp + d);
+        }
+        attention_store(p, qkvg, start, kvh, r0 + r, d, o / l);
+    }
+    if (threadIdx.x == 0) { p.counter[unit] = 0; }
+}
+
+constexpr int AT_WARPS = 4, AT_KT = 64;
+__host__ __device__ constexpr int at_kt(int dk, int dv) { return dk + dv <= 256 ? 64 : 32; }
+__host__ __device__ constexpr int at_smem(int dk, int dv) { return 2 * at_kt(dk, dv) * ((dk + 8) + (dv + 8)) * 2; }
+
+// grid (row tiles of 64, Hkv, entries); the last rows of a prompt see the most keys and start first
+template <int DK, int DV>
+__global__ void __launch_bounds__(32 * AT_WARPS) attention_tiled_kernel(const AttnParams p)
+{
+    extern __shared__ __align__(16) unsigned char at_raw[];
+    constexpr int KT = at_kt(DK, DV), KS = (DK + 8) * 2, VS = (DV + 8) * 2, TB = KT * (KS + VS);
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const unsigned int kvh = blockIdx.y, e = blockIdx.z;
+    const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e];
+    const unsigned int rows = n * p.G, tiles_r = (rows + 16 * AT_WARPS - 1) / (16 * AT_WARPS);
+    if (blockIdx.x >= tiles_r) { return; }
+    const unsigned int t0 = (tiles_r - 1 - blockIdx.x) * 16 * AT_WARPS, r0 = t0 + warp * 16;
+    const __nv_bfloat16* qkvg = (const __nv_bfloat16*)p.qkvg;
+    const size_t seq = ((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max;
+    const __nv_bfloat16* K = (const __nv_bfloat16*)p.k_cache + seq * p.k_ld;
+    const __nv_bfloat16* V = (const __nv_bfloat16*)p.v_cache + seq * p.v_ld;
+    const unsigned int T = min(pos + min(t0 + 16u * AT_WARPS - 1, rows - 1) / p.G + 1, p.T_max);
+    const unsigned int tiles = (T + KT - 1) / KT;
+
+    RowTile<DK, DV> w;
+    w.init(p, qkvg, start, n, kvh, r0, lane);
+    unsigned int lim[2];
+#pragma unroll
+    for (int h = 0; h < 2; h++) { lim[h] = min(pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1, T); }
+    const unsigned int first_lim = pos + r0 / p.G + 1, last_lim = pos + (r0 + 15) / p.G + 1;
+
+    const uint32_t ring = smem_u32(at_raw);
+    auto fetch = [&](unsigned int tile) {
+        if (tile < tiles)
+        {
+            const uint32_t ks = ring + (tile & 1u) * TB, vs = ks + KT * KS;
+            for (unsigned int c = threadIdx.x; c < KT * (DK / 8); c += 32 * AT_WARPS)
+            {
+                const unsigned int r = c / (DK / 8), d = c % (DK / 8), key = tile * KT + r;
+                const bool ok = key < T && d * 8 < p.k_ld;
+                cp_async16(ks + r * KS + d * 16, K + (ok ? (size_t)key * p.k_ld + d * 8 : 0), ok);
+            }
+            for (unsigned int c = threadIdx.x; c < KT * (DV / 8); c += 32 * AT_WARPS)
+            {
+                const unsigned int r = c / (DV / 8), d = c % (DV / 8), key = tile * KT + r;
+                const bool ok = key < T && d * 8 < p.v_ld;
+                cp_async16(vs + r * VS + d * 16, V + (ok ? (size_t)key * p.v_ld + d * 8 : 0), ok);
+            }
+        }
+        cp_async_commit();
+    };
+    fetch(0);
+    const float scale2 = p.scale * 1.44269504088896341f;
+    for (unsigned int tile = 0; tile < tiles; tile++)
+    {
+        fetch(tile + 1);
+        cp_async_wait<1>();
+        __syncthreads();
+        if (tile * KT < last_lim)
+        {
+            const uint32_t ks = ring + (tile & 1u) * TB;
+            w.template step<KT>(ks, ks + KT * KS, tile * KT, lim, (tile + 1) * KT > first_lim, scale2, p.dim, p.vdim, lane);
+        }
+        __syncthreads();
+    }
+    w.finish();
+    const unsigned int gr = lane >> 2, gc = (lane & 3) * 2;
+#pragma unroll
+    for (int h = 0; h < 2; h++)
+    {
+        const unsigned int r = r0 + gr + 8 * h;
+        if (r < rows)
+        {
+            const float inv = 1.0f / w.l[h];
+#pragma unroll
+            for (int d = 0; d < DV / 8; d++)
+            {
+#pragma unroll
+                for (int j = 0; j < 2; j++)
+                {
+                    const unsigned int c = d * 8 + gc + j;
+                    if (c < p.vdim) { attention_store(p, qkvg, start, kvh, r, c, w.o[d][2 * h + j] * inv); }
+                }
+            }
+        }
+    }
+}
+
+template <int DK, int DV>
+int run_attention_split(const AttnParams& p, unsigned int entries, cudaStream_t stream, bool pdl)
+{
+    return launch_kernel("attention_split", attention_split_kernel<DK, DV>, dim3(p.splits, p.Hkv * p.row_tiles, entries), dim3(32 * AS_WARPS),
+        (size_t)as_smem(DK, DV), stream, pdl, p);
+}
+template <int DK, int DV>
+int run_attention_tiled(const AttnParams& p, unsigned int entries, unsigned int max_n, cudaStream_t stream, bool pdl)
+{
+    const unsigned int tiles = (max_n * p.G + 16 * AT_WARPS - 1) / (16 * AT_WARPS);
+    return launch_kernel("attention_tiled", attention_tiled_kernel<DK, DV>, dim3(tiles, p.Hkv, entries), dim3(32 * AT_WARPS), (size_t)at_smem(DK, DV),
+        stream, pdl, p);
+}
+
+// One translation unit per padded key size (64, 128, 256) instantiates these.
+template <int DK>
+int attention_split_dk(const AttnParams& p, unsigned int entries, cudaStream_t stream, bool pdl);
+template <int DK>
+int attention_tiled_dk(const AttnParams& p, unsigned int entries, unsigned int max_n, cudaStream_t stream, bool pdl);
+
+#define B200_ATTENTION_DK(DK)                                                                                                       \
+    template <>                                                                                                                     \
+    int attention_split_dk<DK>(const AttnParams& p, unsigned int entries, cudaStream_t stream, bool pdl)                            \
+    {                                                                                                                               \
+        if (p.vdim <= 64) { return run_attention_split<DK, 64>(p, entries, stream, pdl); }                                          \
+        if (p.vdim <= 128) { return run_attention_split<DK, 128>(p, entries, stream, pdl); }                                        \
+        return run_attention_split<DK, 256>(p, entries, stream, pdl);                                                               \
+    }                                                                                                                               \
+    template <>                                                                                                                     \
+    int attention_tiled_dk<DK>(const AttnParams& p, unsigned int entries, unsigned int max_n, cudaStream_t stream, bool pdl)        \
+    {                                                                                                                               \
+        if (p.vdim <= 64) { return run_attention_tiled<DK, 64>(p, entries, max_n, stream, pdl); }                                   \
+        if (p.vdim <= 128) { return run_attention_tiled<DK, 128>(p, entries, max_n, stream, pdl); }                                 \
+        return run_attention_tiled<DK, 256>(p, entries, max_n, stream, pdl);                                                        \
+    }
+
+}    // namespace b200

@@ -1,0 +1,37 @@
+// One linear of a launch as the kernels see it, and where its results go.
+#pragma once
+
+#include "decoder_common.cuh"
+
+namespace b200
+{
+
+constexpr unsigned int LINEAR_MAX_MEMBERS = 3;
+
+struct LinearMember
+{
+    const void *W, *X;
+    void* Y;
+    const float* row_scale;
+    const int *group_offset, *x_row, *active;
+    unsigned int rows, N, K, ldw, ldx, ldy;
+    unsigned int groups, group_rows, up_row;
+    unsigned int slots;              // groups the launch walks: 1, the groups, or the active list's length
+    unsigned int block0, fblocks;    // streaming kernel: first CTA, CTAs per group
+    int out_type, activation, accumulate;
+    float alpha;
+};
+
+__device__ __forceinline__ void linear_store(const LinearMember& m, unsigned int row, unsigned int f, float v)
+{
+    const size_t i = (size_t)row * m.ldy + f;
+    if (m.row_scale != nullptr) { v *= m.row_scale[row]; }
+    if (m.out_type == DT_BF16) { ((__nv_bfloat16*)m.Y)[i] = __float2bfloat16_rn(v); }
+    else if (m.accumulate) { ((float*)m.Y)[i] += v; }
+    else { ((float*)m.Y)[i] = v; }
+}
+
+// linear_tile.cu: more than a few rows, tcgen05
+int launch_linear_tile(const LinearMember& m, cudaStream_t stream, bool pdl);
+
+}    // namespace b200

@@ -182,73 +182,11 @@ void Cublas::gemm(MatrixTransType TransA, MatrixTransType TransB, int M, int N, 
         CUBLAS_GEMM_DEFAULT_TENSOR_OP);
 }
 
-// ------------------------------------------------------------------------------ GpuControl
-thread_local GpuControl* GpuControl::current_gpu_ = nullptr;
-
-int GpuControl::init(int device)
-{
-    int count = 0;
-    if (cudaGetDeviceCount(&count) != cudaSuccess || device < 0 || device >= count)
-    {
-        cudaGetLastError();
-        return 1;
-    }
-    device_ = device;
-    if (cudaSetDevice(device_) != cudaSuccess) { return 1; }
-    if (cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking) != cudaSuccess) { return 1; }
-    cublas_ = std::make_unique<Cublas>();
-    if (cublas_->init(stream_) != CUBLAS_STATUS_SUCCESS) { return 1; }
-    current_gpu_ = this;
-    return 0;
-}
-
-GpuControl::~GpuControl()
-{
-    if (device_ < 0) { return; }
-    cudaSetDevice(device_);
-    cublas_.reset();
-    for (auto& kv : allocs_) { cudaFree(kv.first); }
-    allocs_.clear();
-    if (stream_) { cudaStreamDestroy(stream_); }
-    if (current_gpu_ == this) { current_gpu_ = nullptr; }
-}
-
-void GpuControl::setAsCurrent()
-{
-    if (current_gpu_ != this || true)
-    {
-        cudaSetDevice(device_);
-        current_gpu_ = this;
-    }
-}
-
-void* GpuControl::malloc(size_t bytes)
-{
-    setAsCurrent();
-    void* p = nullptr;
-    if (cudaMalloc(&p, bytes ? bytes : 1) != cudaSuccess)
-    {
-        cudaGetLastError();
-        LOG_ERR("GpuControl::malloc: %zu bytes failed on device %d\n", bytes, device_);
-        return nullptr;
-    }
-    allocs_[p] = bytes;
-    allocated_ += bytes;
-    return p;
-}
-
-void GpuControl::free(void* p)
-{
-    auto it = allocs_.find(p);
-    if (it == allocs_.end()) { return; }
-    setAsCurrent();
-    cudaStreamSynchronize(stream_);
-    cudaFree(p);
-    allocated_ -= it->second;
-    allocs_.erase(it);
-}
-
-void GpuControl::synchronize() const { cudaStreamSynchronize(stream_); }
+// GpuControl::init makes its dispatcher through this, so that programs without quantised models need not link it.
+static const bool g_dispatcher_known = GpuControl::setDispatcherFactory([](cudaStream_t stream) {
+    auto c = std::make_shared<Cublas>();
+    return c->init(stream) == CUBLAS_STATUS_SUCCESS ? c : std::shared_ptr<Cublas>();
+});
 
 // ---------------------------------------------------------------------------------- Matrix
 size_t Matrix::getDataSizeInByte() const

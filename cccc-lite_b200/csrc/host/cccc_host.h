@@ -122,7 +122,10 @@ public:
     void free(void* p);
     size_t allocatedBytes() const { return allocated_; }
     void synchronize() const;
-    std::unique_ptr<Cublas> cublas_;
+    // The quantised GEMM dispatcher, made by the factory of the library that holds it (null where that is not loaded).
+    std::shared_ptr<Cublas> cublas_;
+    using DispatcherFactory = std::shared_ptr<Cublas> (*)(cudaStream_t);
+    static bool setDispatcherFactory(DispatcherFactory f);
 
 private:
     static thread_local GpuControl* current_gpu_;    // GpuControl.cpp:18

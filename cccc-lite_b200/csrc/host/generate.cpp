@@ -93,12 +93,17 @@ int sampleLogits(std::vector<float>& logits, const SamplerConfig& cfg, const std
 
 int Generator::prefill(const std::vector<int>& tokens, const GenerateConfig& cfg, const std::vector<int>& ctx_ids)
 {
-    // The reference prefills all rows in one pass of its prefill net; here the rows go through the decode step
-    // one after the other, which fills the same cache rows and ends with the same last-row logits.
+    // The reference prefills all rows in one pass of its prefill net.  Where the model offers none, the rows go through
+    // the decode step one after the other, which fills the same cache rows and ends with the same last-row logits.
     reset_();
     const bool want = cfg.sampler.needsLogits();
     int next = 0;
-    for (size_t i = 0; i < tokens.size(); i++)
+    if (prefill_ && !tokens.empty())
+    {
+        next = prefill_(tokens, want ? &logits_ : nullptr);
+        prefill_tokens_ += (int)tokens.size();
+    }
+    else for (size_t i = 0; i < tokens.size(); i++)
     {
         const bool last = i + 1 == tokens.size();
         next = step_(tokens[i], (int)i, (last && want) ? &logits_ : nullptr);

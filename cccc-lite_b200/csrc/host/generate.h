@@ -43,11 +43,15 @@ public:
     // One decode step: feed `token` at cache row `pos`; return the arg-max token, and when
     // logits_out is not null also fill it with the V float logits of that step.
     using StepFn = std::function<int(int token, int pos, std::vector<float>* logits_out)>;
+    // A whole prompt at once, after a reset: its last token's arg-max, and its logits as above.
+    using PrefillFn = std::function<int(const std::vector<int>& tokens, std::vector<float>* logits_out)>;
     // Clears the cache before a (re)prefill (Net::resetKVCache).
     using ResetFn = std::function<void()>;
 
     Generator(int vocab, StepFn step, ResetFn reset, unsigned int seed = 0) : V_(vocab), step_(std::move(step)), reset_(std::move(reset)), rng_(seed) {}
 
+    // Without one the prompt goes through the step, token by token.
+    void setPrefill(PrefillFn f) { prefill_ = std::move(f); }
     // Generates up to max_new_tokens after ctx_ids (which it extends, and truncates on a KV rebuild exactly
     // as run_generate does, cccc-llm.cpp:347-577).  Returns the generated ids, EOS excluded.
     std::vector<int> generate(std::vector<int>& ctx_ids, const GenerateConfig& cfg, int max_new_tokens);
@@ -62,6 +66,7 @@ private:
     int V_;
     StepFn step_;
     ResetFn reset_;
+    PrefillFn prefill_;
     std::mt19937 rng_;
     std::vector<float> logits_;
     int rebuilds_ = 0, decode_steps_ = 0, prefill_tokens_ = 0;

@@ -1,0 +1,67 @@
+#include "kv_cache.h"
+
+namespace cccc
+{
+
+bool KvCache::init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int elem_bytes, int slots, int rows, std::string* err)
+{
+    gpu_ = gpu;
+    rows_ = rows;
+    length_.assign((size_t)slots, 0);
+    open_.assign((size_t)slots, false);
+    for (const auto& s : layers)
+    {
+        Layer l;
+        l.k_ld = (s.k_dim + 7) / 8 * 8;
+        l.v_ld = (s.v_dim + 7) / 8 * 8;
+        const size_t per = (size_t)slots * s.kv_heads * rows * elem_bytes;
+        l.k_bytes = per * l.k_ld;
+        l.v_bytes = per * l.v_ld;
+        l.k = gpu->malloc(l.k_bytes);
+        l.v = gpu->malloc(l.v_bytes);
+        if (!l.k || !l.v)
+        {
+            if (err) { *err = "no device memory for the KV cache"; }
+            return false;
+        }
+        bytes_ += l.k_bytes + l.v_bytes;
+        layers_.push_back(l);
+    }
+    clear();
+    return true;
+}
+
+int KvCache::open()
+{
+    for (int s = 0; s < slots(); s++)
+    {
+        if (!open_[s])
+        {
+            open_[s] = true;
+            length_[s] = 0;
+            return s;
+        }
+    }
+    return -1;
+}
+
+void KvCache::close(int slot)
+{
+    if (!isOpen(slot)) { return; }
+    open_[slot] = false;
+    length_[slot] = 0;
+}
+
+void KvCache::clear()
+{
+    gpu_->setAsCurrent();
+    for (auto& l : layers_)
+    {
+        cudaMemsetAsync(l.k, 0, l.k_bytes, gpu_->stream());
+        cudaMemsetAsync(l.v, 0, l.v_bytes, gpu_->stream());
+    }
+    for (auto& n : length_) { n = 0; }
+    gpu_->synchronize();
+}
+
+}    // namespace cccc
