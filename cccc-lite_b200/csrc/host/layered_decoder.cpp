@@ -78,7 +78,7 @@ bool LayeredDecoder::load(const ModelOptions& o, const DecoderSpec& spec, Tensor
     if (o.max_context <= 0 || o.max_sequences <= 0 || o.max_step_tokens <= 0) { return fail(err, "context, sequences and step tokens must be positive"); }
     if (gpu_.init(o.device) != 0) { return fail(err, "cannot open CUDA device " + std::to_string(o.device)); }
     cap_ = std::max(std::min(o.max_step_tokens, o.max_context * o.max_sequences), std::min(o.max_sequences, kStreamRows));
-    if (!loadTensors(source, err) || !allocate(err)) { return false; }
+    if (!loadTensors(source, err) || !allocate(o, err)) { return false; }
     gpu_.synchronize();
     return cuda_b200_decoder_check("model load") == 0 ? true : fail(err, "a CUDA error while loading");
 }
@@ -197,7 +197,7 @@ bool LayeredDecoder::loadTensors(TensorSource& s, std::string* err)
     return true;
 }
 
-bool LayeredDecoder::allocate(std::string* err)
+bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
 {
     std::vector<KvLayerShape> shapes;
     int vdim = 0, qkvg = 0, att = 0, ff = 0, eff = 0, sff = 0, router = 0, first = 0;
@@ -220,6 +220,7 @@ bool LayeredDecoder::allocate(std::string* err)
             max_experts_ = std::max(max_experts_, (int)m.experts.size());
         }
     }
+    if (!cache_.init(&gpu_, shapes, (int)elem(), o.max_sequences, o.max_context, err)) { return false; }
     ldw_ = pad64(spec_.width);
     ld_qkvg_ = pad64(qkvg);
     ld_att_ = pad64(att);

@@ -116,7 +116,7 @@ private:
 
     bool check(std::string* err) const;
     bool loadTensors(TensorSource& s, std::string* err);
-    bool allocate(std::string* err);
+    bool allocate(const ModelOptions& o, std::string* err);
     bool packRows(TensorSource& s, const std::vector<std::pair<std::string, int>>& parts, int k, int align, Weight* out, std::string* err);
     bool loadNorm(TensorSource& s, const std::string& name, Norm* out, std::string* err);
     void* dmalloc(size_t bytes, bool zero);
