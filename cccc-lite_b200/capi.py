@@ -82,7 +82,8 @@ SYMBOLS["cuda_embed_fwd_bf16_to_fp8"] = (_i, [_vp, _vp, _vp, _i, _i, _i])
 class AttnDecode(C.Structure):
     """cuda_attn_decode of include/cccc_cuda_b200.h."""
     _fields_ = [(n, C.c_void_p) for n in ("q", "k", "v", "q_norm", "k_norm", "cos_tab", "sin_tab", "k_cache", "v_cache", "pos", "out")] + [
-        (n, C.c_uint) for n in ("ldq", "ldk", "ldv", "ldo", "B", "H", "Hkv", "head_dim", "T_max")] + [("epsilon", C.c_float), ("dk", C.c_float)]
+        (n, C.c_uint) for n in ("ldq", "ldk", "ldv", "ldo", "B", "H", "Hkv", "head_dim", "T_max")] + [("epsilon", C.c_float), ("dk", C.c_float),
+                                                                                                     ("slot", C.c_void_p)]
 
 
 SYMBOLS["cuda_rms_norm_bf16"] = (_i, [_vp, _vp, _vp, _vp, _vp, _u, _u, _f, _vp, _u])
@@ -353,11 +354,11 @@ def swiglu_bf16(gate, up, out, rows: int, cols: int, ld_gate=None, ld_up=None, l
 
 
 def make_attn_decode(*, q, k, v, k_cache, v_cache, pos, out, cos_tab, sin_tab, B: int, H: int, Hkv: int, head_dim: int, T_max: int,
-                     q_norm=None, k_norm=None, ldq=None, ldk=None, ldv=None, ldo=None, eps: float = 1e-6, dk: float = 0.0):
+                     q_norm=None, k_norm=None, ldq=None, ldk=None, ldv=None, ldo=None, eps: float = 1e-6, dk: float = 0.0, slot=None):
     """A cuda_attn_decode filled from tensors (it only holds pointers: keep the tensors alive)."""
     a = AttnDecode()
     for name, t in (("q", q), ("k", k), ("v", v), ("q_norm", q_norm), ("k_norm", k_norm), ("cos_tab", cos_tab), ("sin_tab", sin_tab),
-                    ("k_cache", k_cache), ("v_cache", v_cache), ("pos", pos), ("out", out)):
+                    ("k_cache", k_cache), ("v_cache", v_cache), ("pos", pos), ("out", out), ("slot", slot)):
         setattr(a, name, _ptr(t))
     a.ldq = H * head_dim if ldq is None else ldq
     a.ldk = Hkv * head_dim if ldk is None else ldk

@@ -369,6 +369,7 @@ C_EXPORT int cuda_attn_decode_bf16(const cuda_attn_decode* a, void* stream, unsi
     p.k_cache = (uint16_t*)a->k_cache;
     p.v_cache = (uint16_t*)a->v_cache;
     p.pos = (const int*)a->pos;
+    p.slot = (const int*)a->slot;
     p.out = (uint16_t*)a->out;
     p.ldq = a->ldq;
     p.ldk = a->ldk;

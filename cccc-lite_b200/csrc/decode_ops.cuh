@@ -102,14 +102,21 @@ struct AttnDecodeParams
     const uint16_t* k_norm;  // [HD] or nullptr
     const uint16_t* cos_tab; // [rows][HD/2]
     const uint16_t* sin_tab;
-    uint16_t* k_cache;       // [B][Hkv][T_max][HD]
+    uint16_t* k_cache;       // [slots][Hkv][T_max][HD]
     uint16_t* v_cache;
     const int* pos;          // [B]: where the new token goes = index of the newest valid row afterwards
     uint16_t* out;           // [B][ldo]: H heads of HD
+    const int* slot;         // [B]: the cache slot of each sequence, or nullptr: sequence b has slot b
     unsigned int ldq, ldk, ldv, ldo;
     unsigned int B, H, Hkv, T_max;
     float eps, scale;        // RMSNorm epsilon of the q/k norms; 1/sqrt(dk)
 };
+
+// First row of a (sequence, kv head) in the caches.
+__device__ __forceinline__ size_t attn_cache_row(const AttnDecodeParams& p, unsigned int b, unsigned int kvh)
+{
+    return ((size_t)(p.slot != nullptr ? (unsigned int)p.slot[b] : b) * p.Hkv + kvh) * p.T_max;
+}
 
 constexpr int kAttnRingK = 4;     // passes of 32 rows (8 KB at head_dim 128); even: the loop consumes two per turn
 constexpr int kAttnRingV = 8;     // passes of 16 rows (4 KB at head_dim 128)
@@ -270,8 +277,8 @@ __device__ __forceinline__ void attn_prologue(const AttnDecodeParams& p, AttnSme
     team_sync();
     if (owner && pos < p.T_max)
     {
-        uint16_t* kc = p.k_cache + (((size_t)b * p.Hkv + kvh) * p.T_max + pos) * HD;
-        uint16_t* vc = p.v_cache + (((size_t)b * p.Hkv + kvh) * p.T_max + pos) * HD;
+        uint16_t* kc = p.k_cache + (attn_cache_row(p, b, kvh) + pos) * HD;
+        uint16_t* vc = p.v_cache + (attn_cache_row(p, b, kvh) + pos) * HD;
         const uint16_t* v = p.v + (size_t)b * p.ldv + (size_t)kvh * HD;
         for (unsigned int i = tid; i < HD; i += kTeam)
         {
@@ -342,7 +349,7 @@ __device__ __forceinline__ void attn_scores_ring(const AttnDecodeParams& p, Attn
     constexpr int CPL = HD / 64;    // 16-byte pieces per lane
     constexpr int D = kAttnRingK;
     const unsigned int sub = tid & 7u, slot = tid >> 3;
-    const uint16_t* Kb = p.k_cache + ((size_t)b * p.Hkv + kvh) * p.T_max * HD;
+    const uint16_t* Kb = p.k_cache + attn_cache_row(p, b, kvh) * HD;
     const unsigned int n_pass = t1 > t0 ? (t1 - t0 + 31u) / 32u : 0u;
     auto issue = [&](unsigned int pass) {
         if (pass < n_pass)
@@ -477,7 +484,7 @@ __device__ __forceinline__ void attn_scores(const AttnDecodeParams& p, AttnSmem<
     {
     constexpr int CPL = HD / 64;    // 16-byte pieces per lane
     const unsigned int sub = tid & 7u, slot = tid >> 3;
-    const uint16_t* Kb = p.k_cache + ((size_t)b * p.Hkv + kvh) * p.T_max * HD;
+    const uint16_t* Kb = p.k_cache + attn_cache_row(p, b, kvh) * HD;
     uint4 kv[UNROLL][CPL];
     auto fetch = [&](unsigned int tb) {
 #pragma unroll
@@ -563,7 +570,7 @@ __device__ __forceinline__ void attn_pv(const AttnDecodeParams& p, AttnSmem<G, H
     constexpr int UNROLL = 8;
     const unsigned int n = t1 > t0 ? t1 - t0 : 0;
     const unsigned int sub = tid % LPR, slot = tid / LPR;
-    const uint16_t* Vb = p.v_cache + ((size_t)b * p.Hkv + kvh) * p.T_max * HD;
+    const uint16_t* Vb = p.v_cache + attn_cache_row(p, b, kvh) * HD;
     if constexpr (RING)
     {
         // The ring form (see attn_scores_ring): V rows by cp.async, kAttnRingV passes of SLOTS rows in flight, the first

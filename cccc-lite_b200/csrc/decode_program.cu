@@ -237,6 +237,7 @@ C_EXPORT int cuda_decode_program_add_attention(cuda_decode_program* p, const cud
     A.k_cache = (uint16_t*)a->k_cache;
     A.v_cache = (uint16_t*)a->v_cache;
     A.pos = (const int*)a->pos;
+    A.slot = (const int*)a->slot;
     A.out = (uint16_t*)a->out;
     A.ldq = a->ldq;
     A.ldk = a->ldk;

@@ -212,7 +212,7 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     p.v_mix = a->v_mix;
     p.qk_norm = a->qk_norm;
     p.gate = a->gate;
-    p.lambda = a->lambda;
+    p.lambda = a->mix;
     p.eps = a->eps;
     p.scale = a->scale;
     const bool pdl = (flags & 1u) != 0;

@@ -380,6 +380,7 @@ bool DecodeStep::load(GpuControl* gpu, const BinFile& file, const ModelConfig& c
     std::vector<int> z(max_batch, 0);
     cudaMemcpy(d_ids_, z.data(), (size_t)max_batch * 4, cudaMemcpyHostToDevice);
     cudaMemcpy(d_pos_, z.data(), (size_t)max_batch * 4, cudaMemcpyHostToDevice);
+    cudaMemcpy(d_slot_, z.data(), (size_t)max_batch * 4, cudaMemcpyHostToDevice);
     if (tp_) { tp_->barrier(); }
     const int rc = issue(1, gpu_->stream());
     gpu_->synchronize();
@@ -419,14 +420,8 @@ bool DecodeStep::loadTensors(const BinFile& file, std::string* err)
             return false;
         }
         if (!cfg.qk_norm) { L.q_norm = L.k_norm = nullptr; }
-        const size_t cache = (size_t)max_batch * Hkv_ * cfg.max_context * cfg.head_dim * 2;
-        L.k_cache = (uint16_t*)dmalloc(cache);
-        L.v_cache = (uint16_t*)dmalloc(cache);
-        if (!L.k_cache || !L.v_cache) { return fail(err, "no device memory for the KV cache"); }
-        cudaMemset(L.k_cache, 0, cache);
-        cudaMemset(L.v_cache, 0, cache);
-        cache_bytes_ += 2 * cache;
     }
+    if (!cache_.init(gpu_, std::vector<KvLayerShape>((size_t)cfg.layers, { Hkv_, cfg.head_dim, cfg.head_dim }), 2, max_batch, cfg.max_context, err)) { return false; }
     if (!loadLinear(file, "W_lm_head", cfg.vocab, cfg.hidden, 'c', &lm_head_, err)) { return false; }
     if (!loadBf16(file, "W_emb", (size_t)cfg.vocab * cfg.hidden, &emb_, true, err) || !loadBf16(file, "W_rms_final", cfg.hidden, &final_norm_, true, err))
     {
@@ -465,12 +460,14 @@ bool DecodeStep::loadTensors(const BinFile& file, std::string* err)
     logits_ = (uint16_t*)dmalloc(B * vocab_loc_ * 2);
     d_ids_ = (int*)dmalloc(B * 4);
     d_pos_ = (int*)dmalloc(B * 4);
+    d_slot_ = (int*)dmalloc(B * 4);
     d_best_ = (float*)dmalloc(B * 4);
-    if (!x_ || !xn_ || !tmp_ || !qkv_ || !att_ || !gu_ || !h_ || !logits_ || !d_ids_ || !d_pos_ || !d_best_) { return fail(err, "no device memory for the step's buffers"); }
-    // one pinned block: ids in, positions in, ids out, best out
-    if (cudaMallocHost((void**)&h_ids_, B * 16) != cudaSuccess) { return fail(err, "no pinned memory"); }
+    if (!x_ || !xn_ || !tmp_ || !qkv_ || !att_ || !gu_ || !h_ || !logits_ || !d_ids_ || !d_pos_ || !d_slot_ || !d_best_) { return fail(err, "no device memory for the step's buffers"); }
+    // one pinned block: ids in, positions in, slots in, ids out, best out
+    if (cudaMallocHost((void**)&h_ids_, B * 20) != cudaSuccess) { return fail(err, "no pinned memory"); }
     h_pos_ = h_ids_ + B;
-    h_out_ = h_pos_ + B;
+    h_slot_ = h_pos_ + B;
+    h_out_ = h_slot_ + B;
     h_best_ = (float*)(h_out_ + B);
     if (cudaMallocHost((void**)&h_logits_, B * vocab_loc_ * 2) != cudaSuccess) { return fail(err, "no pinned memory for the logits"); }
     if (world_ > 1)
@@ -486,17 +483,7 @@ bool DecodeStep::loadTensors(const BinFile& file, std::string* err)
     return true;
 }
 
-void DecodeStep::resetCache()
-{
-    gpu_->setAsCurrent();
-    const size_t cache = (size_t)max_batch_ * Hkv_ * cfg_.max_context * cfg_.head_dim * 2;
-    for (auto& L : layers_)
-    {
-        cudaMemsetAsync(L.k_cache, 0, cache, gpu_->stream());
-        cudaMemsetAsync(L.v_cache, 0, cache, gpu_->stream());
-    }
-    gpu_->synchronize();
-}
+void DecodeStep::resetCache() { cache_.clear(); }
 
 int DecodeStep::issue(int M, cudaStream_t st)
 {
@@ -522,8 +509,9 @@ int DecodeStep::issue(int M, cudaStream_t st)
     };
     ok(cuda_embed_bf16(d_ids_, emb_, x_, hid, M, cfg_.vocab, st, PDL));
     bool pending = false;
-    for (auto& L : layers_)
+    for (size_t i = 0; i < layers_.size(); i++)
     {
+        const Layer& L = layers_[i];
         norm(L.attn_norm, pending);
         cuda_wq_linear g[3] = {};
         const Linear* qkv[3] = { &L.q, &L.k, &L.v };
@@ -543,7 +531,7 @@ int DecodeStep::issue(int M, cudaStream_t st)
             off += qkv[j]->n;
         }
         ok(cuda_gemm_wq_bf16_group(wt, 3, g, xn_, M, hid, hid, st, PDL));
-        cuda_attn_decode a = attnArgs(L, M);
+        cuda_attn_decode a = attnArgs(i, M);
         ok(cuda_attn_decode_bf16(&a, st, PDL));
         row_linear(L.o, att_);
         norm(L.ffn_norm, tp);
@@ -573,8 +561,9 @@ int DecodeStep::issue(int M, cudaStream_t st)
     return bad ? -1 : n;
 }
 
-cuda_attn_decode DecodeStep::attnArgs(const Layer& L, int M) const
+cuda_attn_decode DecodeStep::attnArgs(size_t layer, int M) const
 {
+    const Layer& L = layers_[layer];
     cuda_attn_decode a = {};
     a.q = qkv_;
     a.k = qkv_ + q_loc_;
@@ -583,9 +572,10 @@ cuda_attn_decode DecodeStep::attnArgs(const Layer& L, int M) const
     a.k_norm = L.k_norm;
     a.cos_tab = cos_;
     a.sin_tab = sin_;
-    a.k_cache = L.k_cache;
-    a.v_cache = L.v_cache;
+    a.k_cache = cache_.k((int)layer);
+    a.v_cache = cache_.v((int)layer);
     a.pos = d_pos_;
+    a.slot = d_slot_;
     a.out = att_;
     a.ldq = a.ldk = a.ldv = qkv_ld_;
     a.ldo = q_loc_;
@@ -631,13 +621,13 @@ bool DecodeStep::buildProgram()
         in.epsilon = cfg_.eps;
         return in;
     };
-    for (auto& L : layers_)
+    for (size_t i = 0; i < layers_.size() && good; i++)
     {
-        if (!good) { break; }
+        const Layer& L = layers_[i];
         cuda_wq_linear g[3] = { lin(L.q, qkv_, hid, qkv_ld_, 0.f), lin(L.k, qkv_ + q_loc_, hid, qkv_ld_, 0.f), lin(L.v, qkv_ + q_loc_ + kv_loc_, hid, qkv_ld_, 0.f) };
         cuda_decode_input in = input(1, x_, hid, L.attn_norm);
         good = good && cuda_decode_program_add_linears(p, 3, g, &in, hid, 0) == 0;
-        cuda_attn_decode a = attnArgs(L, 1);
+        cuda_attn_decode a = attnArgs(i, 1);
         good = good && cuda_decode_program_add_attention(p, &a) == 0;
         cuda_wq_linear o = lin(L.o, x_, q_loc_, hid, 1.0f);
         in = input(0, att_, q_loc_, nullptr);
@@ -676,7 +666,7 @@ bool DecodeStep::useProgram(bool on)
     return use_program_;
 }
 
-int DecodeStep::step(const int* token_ids, const int* positions, int M, int* next_ids, float* best_logits, uint16_t* logits_host)
+int DecodeStep::step(const int* token_ids, const int* positions, int M, int* next_ids, float* best_logits, uint16_t* logits_host, const int* slots)
 {
     if (M < 1 || M > max_batch_) { return -1; }
     gpu_->setAsCurrent();
@@ -685,9 +675,11 @@ int DecodeStep::step(const int* token_ids, const int* positions, int M, int* nex
     {
         h_ids_[i] = token_ids[i];
         h_pos_[i] = positions[i];
+        h_slot_[i] = slots ? slots[i] : i;
     }
     cudaMemcpyAsync(d_ids_, h_ids_, (size_t)M * 4, cudaMemcpyHostToDevice, st);
     cudaMemcpyAsync(d_pos_, h_pos_, (size_t)M * 4, cudaMemcpyHostToDevice, st);
+    cudaMemcpyAsync(d_slot_, h_slot_, (size_t)M * 4, cudaMemcpyHostToDevice, st);
     int rc = 0;
     if (use_program_ && M == 1 && program_)
     {

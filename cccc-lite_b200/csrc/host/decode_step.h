@@ -13,6 +13,7 @@
 
 #include "bin_file.h"
 #include "cccc_host.h"
+#include "kv_cache.h"
 
 #include <condition_variable>
 #include <mutex>
@@ -89,14 +90,16 @@ public:
     bool load(GpuControl* gpu, const BinFile& file, const ModelConfig& cfg, int max_batch, TensorParallel* tp, int rank, std::string* err);
     // One step for M sequences: token ids and cache rows in, arg-max token ids out (global ids, the same on every
     // rank); logits_host (nullable) receives this rank's shard of the BF16 logits, [M][vocab / world].
-    int step(const int* token_ids, const int* positions, int M, int* next_ids, float* best_logits, uint16_t* logits_host);
+    // slots (nullable): the cache slot of each sequence; without it sequence i has slot i.
+    int step(const int* token_ids, const int* positions, int M, int* next_ids, float* best_logits, uint16_t* logits_host, const int* slots = nullptr);
+    KvCache& cache() { return cache_; }
     void resetCache();
     // One sequence, one GPU: run steps through the recorded decode program (one persistent kernel) when it takes the model.
     bool useProgram(bool on);
     int launchesPerStep() const { return launches_per_step_; }    // of the launch-per-op step
     int lastLaunches() const { return last_launches_; }         // of the step that ran last
     int quantisedOnLoad() const { return quantised_on_load_; }  // tensors that arrived as BF16 / half / float
-    size_t cacheBytes() const { return cache_bytes_; }
+    size_t cacheBytes() const { return cache_.bytes(); }
     // Writes the quantised tensors as a cache file of named weights (weight_<dtype>_<name>, scale_<name>,
     // blockscale_<name>: the keys cccc/Net.cpp:1324-1527 looks up), so that the next start loads them directly.
     // One rank only, after keepHostCopies(true) and load().
@@ -125,13 +128,12 @@ private:
     {
         Linear q, k, v, o, gate, up, down;
         uint16_t *attn_norm = nullptr, *ffn_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr;
-        uint16_t *k_cache = nullptr, *v_cache = nullptr;
     };
     bool loadTensors(const BinFile& file, std::string* err);
     bool loadLinear(const BinFile& f, const std::string& name, int N, int K, char kind, Linear* out, std::string* err);
     bool loadBf16(const BinFile& f, const std::string& name, size_t n, uint16_t** out, bool required, std::string* err);
     int issue(int M, cudaStream_t st);
-    cuda_attn_decode attnArgs(const Layer& L, int M) const;
+    cuda_attn_decode attnArgs(size_t layer, int M) const;
     bool buildProgram();
     void* dmalloc(size_t bytes);
     GpuControl* gpu_ = nullptr;
@@ -144,12 +146,12 @@ private:
     Linear lm_head_;
     uint16_t *emb_ = nullptr, *final_norm_ = nullptr, *cos_ = nullptr, *sin_ = nullptr;
     uint16_t *x_ = nullptr, *xn_ = nullptr, *tmp_ = nullptr, *qkv_ = nullptr, *att_ = nullptr, *gu_ = nullptr, *h_ = nullptr, *logits_ = nullptr;
-    int *d_ids_ = nullptr, *d_pos_ = nullptr, *h_ids_ = nullptr, *h_pos_ = nullptr, *h_out_ = nullptr;
+    int *d_ids_ = nullptr, *d_pos_ = nullptr, *d_slot_ = nullptr, *h_ids_ = nullptr, *h_pos_ = nullptr, *h_slot_ = nullptr, *h_out_ = nullptr;
     float *d_best_ = nullptr, *h_best_ = nullptr;
     uint16_t* h_logits_ = nullptr;
     std::vector<Matrix> quantised_;    // tensors quantised while loading own their device memory
     int quantised_on_load_ = 0, layers_loaded_ = 0, last_launches_ = 0;
-    size_t cache_bytes_ = 0;
+    KvCache cache_;
     void* seq_counters_ = nullptr;
     std::vector<void*> owned_;
     std::vector<Stored> stored_;

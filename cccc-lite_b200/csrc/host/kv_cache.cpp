@@ -3,6 +3,15 @@
 namespace cccc
 {
 
+KvCache::~KvCache()
+{
+    for (auto& l : layers_)
+    {
+        gpu_->free(l.k);
+        gpu_->free(l.v);
+    }
+}
+
 bool KvCache::init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int elem_bytes, int slots, int rows, std::string* err)
 {
     gpu_ = gpu;
@@ -19,13 +28,13 @@ bool KvCache::init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int
         l.v_bytes = per * l.v_ld;
         l.k = gpu->malloc(l.k_bytes);
         l.v = gpu->malloc(l.v_bytes);
+        layers_.push_back(l);
         if (!l.k || !l.v)
         {
             if (err) { *err = "no device memory for the KV cache"; }
             return false;
         }
         bytes_ += l.k_bytes + l.v_bytes;
-        layers_.push_back(l);
     }
     clear();
     return true;

@@ -18,6 +18,10 @@ struct KvLayerShape
 class KvCache
 {
 public:
+    KvCache() = default;
+    ~KvCache();
+    KvCache(const KvCache&) = delete;
+    KvCache& operator=(const KvCache&) = delete;
     // elem_bytes 2 or 4.  Rows are padded to eight elements; the padding is zero and stays so.
     bool init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int elem_bytes, int slots, int rows, std::string* err);
     void* k(int layer) const { return layers_[layer].k; }
@@ -41,7 +45,7 @@ private:
         int k_ld = 0, v_ld = 0;
         size_t k_bytes = 0, v_bytes = 0;
     };
-    GpuControl* gpu_ = nullptr;    // owns the memory
+    GpuControl* gpu_ = nullptr;
     std::vector<Layer> layers_;
     std::vector<int> length_;
     std::vector<bool> open_;

@@ -435,7 +435,7 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
         a.v_mix = L.v_mix;
         a.qk_norm = s.qk_norm;
         a.gate = !s.gate.empty();
-        a.lambda = L.lambda;
+        a.mix = L.lambda;
         a.eps = spec_.eps;
         a.scale = s.scale;
         ok(cuda_b200_attention_rows(act(), &a, &b, st, PDL, 0));

@@ -84,7 +84,7 @@ typedef struct cuda_b200_batch
 } cuda_b200_batch;
 
 /* Attention of a layer from its projections on.  First, for every token of the batch: q heads to unit RMS in place
- * (qk_norm), k heads to unit RMS and v (mixed with v_first: v = (1 - lambda) v + lambda v_first) appended to the caches,
+ * (qk_norm), k heads to unit RMS and v (mixed with v_first: v = (1 - mix) v + mix v_first) appended to the caches,
  * v_first stored.  Caches hold rows of k_ld / v_ld elements (multiples of 8) whose padding is zero.  A batch entry's
  * sequence must fit: pos + n <= T_max. */
 typedef struct cuda_b200_attention
@@ -99,7 +99,7 @@ typedef struct cuda_b200_attention
     unsigned int H, Hkv, dim, vdim, k_ld, v_ld, T_max;
     int v_mix;                 /* 0: plain, 1: this layer's values are the ones later layers mix in, 2: mix */
     int qk_norm, gate;         /* 1: unit RMS of q and k; multiply the output by sigmoid(gate) */
-    float lambda, eps, scale;
+    float mix, eps, scale;
 } cuda_b200_attention;
 C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
 /* Appends, then causal softmax attention over the caches (query head h reads kv head h / (H / Hkv)), then the output gate.

@@ -298,7 +298,8 @@ C_EXPORT int cuda_swiglu_bf16(const void* gate, const void* up, void* out, unsig
  * through distributed shared memory.  Query head h reads kv head h / (H / Hkv).
  *   q, k, v  : the projections' outputs, [B] rows of H*head_dim, Hkv*head_dim, Hkv*head_dim BF16
  *              values, row strides ldq/ldk/ldv in elements (they may be slices of one buffer)
- *   caches   : [B][Hkv][T_max][head_dim] BF16
+ *   caches   : [slots][Hkv][T_max][head_dim] BF16
+ *   slot     : DEVICE int32 [B]: the cache slot of each sequence; NULL = sequence b has slot b
  *   pos      : DEVICE int32 [B]: the row the new token is appended at (= tokens already cached);
  *              rows 0..pos are attended.  pos >= T_max appends nothing and attends T_max rows.
  *   tables   : RoPE cos / sin, [>= max pos + 1][head_dim / 2] BF16
@@ -321,6 +322,7 @@ typedef struct cuda_attn_decode
     unsigned int ldq, ldk, ldv, ldo;
     unsigned int B, H, Hkv, head_dim, T_max;
     float epsilon, dk;
+    const void* slot;
 } cuda_attn_decode;
 C_EXPORT int cuda_attn_decode_bf16(const cuda_attn_decode* a, void* stream, unsigned int flags);
 

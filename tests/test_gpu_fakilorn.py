@@ -1,0 +1,291 @@
+"""The Fakilorn decoder through the serving interface - registry, loader, cache slots, steps, scheduler, generation loop,
+command line - against the plain statement in oracle/fakilorn.py, on small random models."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+
+from __graft_entry__ import ROOT, load_package
+from oracle import fakilorn as F
+
+pytestmark = pytest.mark.gpu
+
+BAR = {"float32": 3e-5, "bfloat16": 0.03}     # rms of the logits' error over the logits' standard deviation
+
+
+def attn(heads, kv, dim, vdim, scale, mix=True):
+    return dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, scale=scale, v_mix=mix)
+
+
+def moe(experts, top, ff, shared=0):
+    m = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=ff))
+    if shared:
+        m["shared"] = dict(ff=shared)
+    return m
+
+
+def config(width, vocab, layers, eps=1e-4, embed=5.0, logit=1.5):
+    return dict(architecture="Fakilorn", width=width, vocab=vocab, embedding=dict(scale=embed), logit_scale=logit, norm=dict(eps=eps),
+                layers=[dict(type="attention", mixer=m, mlp=f) for m, f in layers])
+
+
+DENSE = lambda ff: dict(kind="dense", ff=ff)
+CONFIGS = {
+    # layers of unlike sizes, a layer without feed-forward, values mixed from the second layer on, no shared expert in one
+    "mixed": config(200, 331, [(attn(6, 2, 40, 24, 0.5, False), DENSE(136)), (attn(6, 3, 24, 16, 0.6), moe(5, 3, 56, 72)), (attn(4, 2, 32, 24, 0.4), None),
+                               (attn(8, 1, 16, 48, 0.7), moe(7, 2, 40))], eps=1e-2),
+    # sizes that are multiples of nothing
+    "odd": config(97, 53, [(attn(4, 4, 7, 5, 1.3), moe(1, 1, 19, 23)), (attn(5, 1, 11, 20, 1.0), DENSE(33))]),
+    # many query heads per kv head; every expert chosen
+    "wide": config(264, 640, [(attn(24, 1, 72, 136, 0.3), moe(4, 4, 64, 32)), (attn(24, 1, 80, 136, 0.3), moe(4, 1, 64, 32))], embed=1.0, logit=1.0),
+    # keys and values beyond the tensor-core kernels' sizes
+    "huge": config(128, 100, [(attn(2, 1, 264, 16, 0.1), DENSE(64)), (attn(2, 1, 16, 272, 0.5, False), DENSE(64))]),
+}
+
+
+@pytest.fixture(scope="module")
+def serve():
+    return load_package().serve
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    out = {}
+    for name, c in CONFIGS.items():
+        d = tmp_path_factory.mktemp(name)
+        w = F.random_weights(c, seed=len(name))
+        (d / "config.json").write_text(json.dumps(c))
+        F.write_safetensors(str(d / "model.safetensors"), w)
+        out[name] = (str(d), c, w)
+    return out
+
+
+def tokens_for(c, n, seed):
+    return [int(t) for t in np.random.default_rng(seed).integers(0, c["vocab"], n)]
+
+
+def error(got, want):
+    return float(np.sqrt(((got - want) ** 2).mean()) / want.std())
+
+
+def feed(m, slot, tokens, cuts):
+    rows, at = [], 0
+    for n in cuts:
+        n = min(n, len(tokens) - at)
+        if n <= 0:
+            break
+        lg, _ = m.step([(slot, tokens[at:at + n], range(n))])
+        rows.append(np.array(lg, np.float64).reshape(n, -1))
+        at += n
+    assert at == len(tokens)
+    return np.concatenate(rows)
+
+
+CUTS = {"whole": [10 ** 6], "tokens": [1] * 10 ** 4, "twos": [2, 3] * 10 ** 4, "unequal": [45, 2, 68, 33, 1, 1, 31, 64, 7] * 100, "prompt then tokens": [120] + [1] * 10 ** 4}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_logits_do_not_depend_on_the_cuts(serve, folders, name, dtype):
+    d, c, w = folders[name]
+    tokens = tokens_for(c, 210, 1)
+    want = F.forward(c, w, tokens)
+    m = serve.Model(d, dtype=dtype, max_context=256, max_sequences=2, max_step_tokens=160)      # the whole prompt takes two passes
+    ref = None
+    for how, cuts in CUTS.items():
+        slot = m.open_slot()
+        got = feed(m, slot, tokens, cuts)
+        assert m.slot_length(slot) == len(tokens)
+        m.close_slot(slot)
+        for part, rows in (("all", slice(None)), ("first", slice(0, 3)), ("last", slice(-3, None))):
+            assert error(got[rows], want[rows]) < BAR[dtype], (how, part, error(got[rows], want[rows]))
+        ref = got if ref is None else ref
+        assert error(got, ref) < BAR[dtype] / 2, how
+    m.close()
+
+
+def sharp(c, w, factor):
+    """The same model with attention that picks single keys: scores `factor` times as large."""
+    c = json.loads(json.dumps(c))
+    for L in c["layers"]:
+        L["mixer"]["scale"] *= factor
+    return c
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_sharp_attention_far_back(serve, tmp_path, dtype):
+    """Scores so large that a position reads one or two keys, anywhere in a long past; prompts and decoding."""
+    c = sharp(config(128, 200, [(attn(4, 2, 32, 24, 0.35), DENSE(96)), (attn(4, 2, 32, 24, 0.35), moe(6, 2, 48, 40))], embed=8.0), None, 2.0)
+    w = F.random_weights(c, 3)
+    (tmp_path / "config.json").write_text(json.dumps(c))
+    F.write_safetensors(str(tmp_path / "model.safetensors"), w)
+    # each token once, then once more: equal tokens match best
+    tokens = list(range(200)) + tokens_for(c, 700, 2)
+    want = F.forward(c, w, tokens)
+    m = serve.Model(str(tmp_path), dtype=dtype, max_context=1024)
+    for cuts in ([900], [833] + [1] * 67, [64] * 15):
+        slot = m.open_slot()
+        got = feed(m, slot, tokens, cuts)
+        m.close_slot(slot)
+        err = np.sqrt(((got - want) ** 2).mean(1)) / want.std()
+        assert np.median(err) < BAR[dtype] and err.max() < 10 * BAR[dtype], (np.median(err), err.max())
+    m.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_batches_slots_and_reuse(serve, folders, dtype):
+    """Requests of unequal length share steps, come and go, and take over slots: each gets the logits it gets alone."""
+    d, c, w = folders["mixed"]
+    rng = np.random.default_rng(9)
+    m = serve.Model(d, dtype=dtype, max_context=160, max_sequences=3, max_step_tokens=128)
+    todo = [tokens_for(c, n, 100 + n) for n in (1, 150, 37, 64, 5, 129, 90, 2, 160, 33)]
+    want = [F.forward(c, w, t) for t in todo]
+    live, queue, got, seen_slots = {}, list(range(len(todo))), {i: [] for i in range(len(todo))}, []
+    while live or queue:
+        while queue and len(live) < 3:
+            live[queue.pop(0)] = [m.open_slot(), 0]
+        entries, plan = [], []
+        for i, (slot, at) in live.items():
+            n = min(int(rng.choice([1, 1, 2, 3, 20, 70])), len(todo[i]) - at)
+            entries.append((slot, todo[i][at:at + n], range(n)))
+            plan.append((i, n))
+            seen_slots.append((i, slot))
+        lg, ch = m.step(entries, choice=True)
+        rows, k = np.array(lg, np.float64).reshape(-1, c["vocab"]), 0
+        assert list(np.argmax(rows, axis=1)) == ch
+        for i, n in plan:
+            got[i].append(rows[k:k + n])
+            k += n
+            live[i][1] += n
+            if live[i][1] == len(todo[i]):
+                m.close_slot(live[i][0])
+                del live[i]
+    assert len({s for _, s in seen_slots}) == 3 and len({(i, s) for i, s in seen_slots}) == len(todo)
+    for i in range(len(todo)):
+        assert error(np.concatenate(got[i]), want[i]) < BAR[dtype], i
+    # entries that cannot run leave everything as it is
+    slot = m.open_slot()
+    m.step([(slot, [1, 2], [])])
+    for bad in ([(slot, [c["vocab"]], [0])], [(slot, [-1], [0])], [(slot, [1] * 159, [0])], [(slot, [1], [1])], [(slot + 1, [1], [0])], [(slot, [1], [0]), (slot, [2], [0])]):
+        with pytest.raises(RuntimeError, match="cannot run"):
+            m.step(bad)
+    assert m.slot_length(slot) == 2
+    lg, _ = m.step([(slot, [3], [0])])
+    assert error(np.array(lg, np.float64), F.forward(c, w, [1, 2, 3])[2]) < BAR[dtype]
+    m.close()
+
+
+def test_decode_steps_replay_a_graph_over_growing_lengths(serve, folders):
+    """Long decoding past the lengths at which the split count changes."""
+    d, c, w = folders["odd"]
+    tokens = tokens_for(c, 300, 4)
+    want = F.forward(c, w, tokens)
+    m = serve.Model(d, max_context=300)
+    slot = m.open_slot()
+    got = feed(m, slot, tokens, [1] * 300)
+    assert error(got, want) < BAR["bfloat16"] and error(got[-20:], want[-20:]) < BAR["bfloat16"]
+    with pytest.raises(RuntimeError, match="cannot run"):
+        m.step([(slot, [0], [0])])
+    m.close()
+
+
+def greedy(c, w, prompt, n):
+    out = []
+    for _ in range(n):
+        z = F.forward(c, w, prompt + out)[-1]
+        out.append(int(np.argmax(z)))
+    return out
+
+
+def test_greedy_generation_loop_scheduler_and_command_line(serve, folders):
+    d, c, w = folders["mixed"]
+    prompts = [tokens_for(c, n, n) for n in (5, 61, 1, 18, 33)]
+    want = [greedy(c, w, p, 8) for p in prompts]
+    m = serve.Model(d, dtype="float32", max_context=128, max_sequences=2)
+    for p, g in zip(prompts, want):
+        ids, stats = m.generate(p, 8, portion=7)
+        assert ids == g and stats["prefill_tokens"] == len(p) and stats["rebuilds"] == 0
+    assert m.generate(prompts[0], 8, eos_ids=[want[0][3]])[0] == want[0][:want[0].index(want[0][3])]
+    for budget in (3, 40, 1000):
+        got, steps = m.generate_many(prompts + [[], [0] * 129], 8, step_tokens=budget)
+        assert got[:5] == want and got[5:] == [None, None]
+    # a sampler sees each request's own logits and seed
+    a, _ = m.generate_many(prompts, 6, seed=3, sampler=dict(temperature=0.9, top_k=12))
+    b, _ = m.generate_many(prompts, 6, seed=3, sampler=dict(temperature=0.9, top_k=12), step_tokens=5)
+    assert a == b and a != [g[:6] for g in want]
+    # a slot too small for all: the scheduler ends the sequence at the slot's last row, the loop rebuilds
+    small = serve.Model(d, dtype="float32", max_context=8)
+    got, _ = small.generate_many([prompts[0]], 8)
+    assert got[0] == want[0][:4]
+    ids, stats = small.generate(prompts[0], 8, sys_n=1, turn_n=1)
+    assert stats["rebuilds"] >= 1 and ids[:4] == want[0][:4]
+    small.close()
+    m.close()
+    cmd = [sys.executable, os.path.join(ROOT, "bin", "generate"), "--model", d, "--dtype", "float32", "--max-new", "8"]
+    for p in prompts[:2]:
+        cmd += ["--prompt", ",".join(map(str, p))]
+    out = subprocess.run(cmd, capture_output=True, text=True, timeout=300)
+    assert out.returncode == 0, out.stderr
+    assert [[int(x) for x in line.split(",")] for line in out.stdout.split()] == want[:2]
+
+
+def test_trace_runner(serve, folders, tmp_path):
+    d, c, w = folders["odd"]
+    a, b = tokens_for(c, 40, 7), tokens_for(c, 9, 8)
+    steps = [dict(step=0, entries=[dict(id="a", tokens=a[:33], want=[0, 32])], end=[]), dict(step=1, entries=[dict(id="b", tokens=b, want=[8])], end=["b"]),
+             dict(step=2, entries=[dict(id="a", tokens=a[33:39], want=[])], end=[]), dict(step=5, entries=[dict(id="a", tokens=a[39:], want=[0])], end=["a"])]
+    out = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", d, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "60"],
+                         input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=300)
+    assert out.returncode == 0, out.stderr
+    assert [x for x in out.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2", "done 5"]
+    za, zb = F.forward(c, w, a), F.forward(c, w, b)
+    for step, want in ((0, za[[0, 32]]), (1, zb[[8]]), (5, za[[39]])):
+        got = np.fromfile(tmp_path / f"{step}.f32", "<f4").reshape(-1, c["vocab"])
+        assert got.shape == want.shape and error(got, want) < BAR["float32"], step
+    assert not os.path.exists(tmp_path / "2.f32")
+
+
+def test_quantised_model_serves_through_the_same_interface(serve, tmp_path):
+    """The registry's other architecture: the same logits as its own step, its sequences in any slot."""
+    from oracle import oracle as O
+    from tests.test_gpu_decode_model import make_model
+    from tests.test_gpu_host_step import container_entries, small_cfg
+    from tests.test_loader_cpu import write_container
+
+    cfg = small_cfg(True)
+    w = make_model(O.FP8_E5M2, cfg, seed=21)
+    write_container(str(tmp_path / "model.bin"), container_entries(O.FP8_E5M2, cfg, w))
+    (tmp_path / "config.json").write_text(json.dumps(dict(architecture="cccc-llm", hidden=cfg.hidden, n_heads=cfg.n_heads, n_kv_heads=cfg.n_kv_heads,
+                                                          head_dim=cfg.head_dim, ffn=cfg.ffn, vocab=cfg.vocab, layers=cfg.layers, rope_theta=cfg.rope_theta,
+                                                          eps=cfg.eps, qk_norm=cfg.qk_norm)))
+    h = load_package().hostapi
+    L = h.lib()
+    g = L.cccc_host_gpu_create(0)
+    f = L.cccc_host_bin_open(str(tmp_path / "model.bin").encode())
+    own = h.HostDecodeStep(g, f, cfg, 64)
+    prompt = [11, 12, 13, 14, 15]
+    want, _ = own.generate(prompt, 10, T=32, T_kv=64)
+    m = serve.Model(str(tmp_path), max_context=64, max_sequences=3)
+    assert m.generate(prompt, 10)[0] == want
+    first = [m.open_slot(), m.open_slot()]
+    m.close_slot(first[0])                      # sequences run in slots 1 and 2, then in 0
+    third = m.open_slot()
+    lg, ch = m.step([(first[1], prompt, [4]), (third, prompt[:3], [2])], choice=True)
+    own.reset()
+    for i, t in enumerate(prompt):
+        nxt, _, z = own.step([t], [i], want_logits=True)
+        if i == 2:
+            z3, n3 = O.bf16_bits_to_f32(z)[0], nxt[0]
+    got = np.array(lg).reshape(2, -1)
+    ref = np.stack([O.bf16_bits_to_f32(z)[0], z3])
+    assert error(got.astype(np.float64), ref) < 0.02
+    assert ch == [int(np.argmax(r)) for r in got]
+    both, _ = m.generate_many([prompt], 10)
+    assert len(both[0]) == 10
+    m.close()
+    own.close()
+    L.cccc_host_bin_close(f)
+    L.cccc_host_gpu_destroy(g)
