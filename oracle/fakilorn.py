@@ -107,7 +107,7 @@ def attention_mixer(h, w, m, eps, v_first):
     q = unit_rms((h @ w["q"].T).reshape(T, H, d), eps)
     k = unit_rms((h @ w["k"].T).reshape(T, G, d), eps)
     own = (h @ w["v"].T).reshape(T, G, dv)
-    v = own if v_first is None else mix_values(own, v_first, float(w["vmix"]))
+    v = own if v_first is None else mix_values(own, v_first.reshape(own.shape), float(w["vmix"]))
     o = causal_attention(q, k, v, m["scale"], H // G).reshape(T, H * dv)
     o = o * sigmoid(h @ w["g"].T)
     return o @ w["o"].T, own
