@@ -215,13 +215,29 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     p.lambda = a->mix;
     p.eps = a->eps;
     p.scale = a->scale;
+    p.fused = 0;
     const bool pdl = (flags & 1u) != 0;
     cudaStream_t st = (cudaStream_t)stream;
+    const bool direct = p.dim <= 128 && p.vdim <= 128 && (p.k_ld % 16) == 0 && (p.v_ld % 16) == 0;
+    if (dtype == DT_FLOAT) { kernel = 3; }
+    if (kernel == 0)
+    {
+        if (p.dim > 256 || p.vdim > 256) { kernel = 3; }
+        else if (b->max_n * p.G <= 64 || b->max_n <= 4) { kernel = direct ? 4 : 1; }
+        else { kernel = 2; }
+    }
+    if (kernel == 4 && b->max_n == 1)
+    {
+        p.fused = 1;
+        return launch_attention_direct(p, b->entries, 1, b->max_len, st, pdl);
+    }
     int rc = dtype == DT_BF16 ? attention_append<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_append<float>(p, b->tokens, st, pdl);
     if (rc) { return rc; }
-    if (dtype == DT_FLOAT) { return attention_plain<float>(p, b->tokens, st, pdl); }
-    if (kernel == 0) { kernel = p.dim > 256 || p.vdim > 256 ? 3 : (b->max_n * p.G <= 64 || b->max_n <= 4 ? 1 : 2); }
-    if (kernel == 1) { return launch_attention_split(p, b->entries, b->max_n, b->max_len, st, pdl); }
-    if (kernel == 2) { return launch_attention_tiled(p, b->entries, b->max_n, st, pdl); }
-    return attention_plain<__nv_bfloat16>(p, b->tokens, st, pdl);
+    switch (kernel)
+    {
+    case 1: return launch_attention_split(p, b->entries, b->max_n, b->max_len, st, pdl);
+    case 2: return launch_attention_tiled(p, b->entries, b->max_n, st, pdl);
+    case 4: return launch_attention_direct(p, b->entries, b->max_n, b->max_len, st, pdl);
+    default: return dtype == DT_BF16 ? attention_plain<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_plain<float>(p, b->tokens, st, pdl);
+    }
 }

@@ -197,6 +197,128 @@ __device__ __forceinline__ void attention_store(const AttnParams& p, const __nv_
 }
 
 constexpr int AS_WARPS = 4, AS_KT = 16;
+constexpr unsigned int kMaxSplits = 32;
+
+// What the warps of a split CTA leave for each other, and the last CTA's weights of the splits.
+struct SplitMeet
+{
+    float ml[AS_WARPS][16][2];    // maximum (log2) and sum of every row
+    float weight[16][kMaxSplits];
+    float inv[16];
+    int last;
+};
+
+// Adds the four warps' results (om: [warp][RT][DV] floats, meet.ml) and, with several splits, the splits' - the last CTA of
+// a unit to arrive does, in split order, so that the bits do not depend on who that is.  All 128 threads call.
+template <int DV, int RT>
+__device__ __forceinline__ void split_finish(const AttnParams& p, SplitMeet& meet, const float* om, const __nv_bfloat16* qkvg, unsigned int e,
+    unsigned int start, unsigned int kvh, unsigned int rt, unsigned int r0, unsigned int rows)
+{
+    __syncthreads();
+    const unsigned int tid = threadIdx.x, live = min((unsigned int)RT, rows - r0);
+    if (tid < live)
+    {
+        float m = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int w = 0; w < AS_WARPS; w++) { m = fmaxf(m, meet.ml[w][tid][0]); }
+        float c[AS_WARPS];
+#pragma unroll
+        for (int w = 0; w < AS_WARPS; w++)
+        {
+            c[w] = m == -INFINITY ? 0.f : exp2f(meet.ml[w][tid][0] - m);
+            l += c[w] * meet.ml[w][tid][1];
+        }
+#pragma unroll
+        for (int w = 0; w < AS_WARPS; w++) { meet.ml[w][tid][0] = c[w]; }
+        meet.ml[0][tid][1] = m;
+        meet.ml[1][tid][1] = l;
+    }
+    __syncthreads();
+    auto sum = [&](unsigned int r, unsigned int d) {
+        float o = 0.f;
+#pragma unroll
+        for (int w = 0; w < AS_WARPS; w++) { o += meet.ml[w][r][0] * om[(w * RT + r) * DV + d]; }
+        return o;
+    };
+    if (p.splits == 1)
+    {
+        for (unsigned int j = tid; j < live * p.vdim; j += 32 * AS_WARPS)
+        {
+            const unsigned int r = j / p.vdim, d = j % p.vdim;
+            attention_store(p, qkvg, start, kvh, r0 + r, d, sum(r, d) / meet.ml[1][r][1]);
+        }
+        return;
+    }
+    const unsigned int vp = (p.vdim + 15) / 16 * 16, stride = 16 * (vp + 2), split = blockIdx.x;
+    const unsigned int unit = (e * p.row_tiles + rt) * p.Hkv + kvh;
+    float* all = p.partial + (size_t)unit * p.splits * stride;
+    float* mine = all + (size_t)split * stride;
+    for (unsigned int j = tid; j < live * p.vdim; j += 32 * AS_WARPS)
+    {
+        const unsigned int r = j / p.vdim, d = j % p.vdim;
+        mine[32 + r * vp + d] = sum(r, d);
+    }
+    if (tid < live)
+    {
+        mine[2 * tid] = meet.ml[0][tid][1];
+        mine[2 * tid + 1] = meet.ml[1][tid][1];
+    }
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) { meet.last = atomicAdd(p.counter + unit, 1) == (int)p.splits - 1; }
+    __syncthreads();
+    if (!meet.last) { return; }
+    __threadfence();
+    for (unsigned int j = tid; j < live * p.splits; j += 32 * AS_WARPS)
+    {
+        const unsigned int r = j / p.splits, s = j % p.splits;
+        meet.weight[r][s] = __ldcg(all + (size_t)s * stride + 2 * r);
+    }
+    __syncthreads();
+    // a warp per row: the rows' maxima over the splits, then weights and sums
+    for (unsigned int r = tid >> 5; r < live; r += AS_WARPS)
+    {
+        const unsigned int lane = tid & 31;
+        float m = -INFINITY, l = 0.f;
+        for (unsigned int s = lane; s < p.splits; s += 32) { m = fmaxf(m, meet.weight[r][s]); }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) { m = fmaxf(m, __shfl_xor_sync(0xFFFFFFFFu, m, o)); }
+        for (unsigned int s = lane; s < p.splits; s += 32)
+        {
+            const float c = exp2f(meet.weight[r][s] - m);
+            meet.weight[r][s] = c;
+            l += c * __ldcg(all + (size_t)s * stride + 2 * r + 1);
+        }
+        l = warp_sum(l);
+        if (lane == 0) { meet.inv[r] = 1.0f / l; }
+    }
+    __syncthreads();
+    // four columns per thread (the rows are padded to sixteen)
+    for (unsigned int j = tid; j < live * (vp / 4); j += 32 * AS_WARPS)
+    {
+        const unsigned int r = j / (vp / 4), d = (j % (vp / 4)) * 4;
+        const float* src = all + 32 + r * vp + d;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 16
+        for (unsigned int s = 0; s < p.splits; s++)
+        {
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * stride));
+            const float c = meet.weight[r][s];
+            o.x += c * x.x;
+            o.y += c * x.y;
+            o.z += c * x.z;
+            o.w += c * x.w;
+        }
+        const float out[4] = { o.x, o.y, o.z, o.w };
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+        {
+            if (d + i < p.vdim) { attention_store(p, qkvg, start, kvh, r0 + r, d + i, out[i] * meet.inv[r]); }
+        }
+    }
+    if (tid == 0) { p.counter[unit] = 0; }
+}
+
 __host__ __device__ constexpr int as_stages(int dk, int dv) { return dk + dv <= 256 ? 4 : 3; }
 __host__ __device__ constexpr int as_tile_bytes(int dk, int dv) { return AS_KT * ((dk + 8) + (dv + 8)) * 2; }
 __host__ __device__ constexpr int as_smem(int dk, int dv)
@@ -211,8 +333,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const At
 {
     extern __shared__ __align__(16) unsigned char as_raw[];
     constexpr int ST = as_stages(DK, DV), TB = as_tile_bytes(DK, DV), KS = (DK + 8) * 2, VS = (DV + 8) * 2;
-    __shared__ float ml[AS_WARPS][16][2];
-    __shared__ int last;
+    __shared__ SplitMeet meet;
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -287,73 +408,14 @@ __global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const At
 #pragma unroll
         for (int h = 0; h < 2; h++)
         {
-            ml[warp][gr + 8 * h][0] = w.m[h];
-            ml[warp][gr + 8 * h][1] = w.l[h];
+            meet.ml[warp][gr + 8 * h][0] = w.m[h];
+            meet.ml[warp][gr + 8 * h][1] = w.l[h];
         }
     }
-    __syncthreads();
-    const unsigned int live = min(16u, rows - r0);
-    auto combine = [&](unsigned int r, unsigned int d, float& m, float& l, float& o) {
-        m = fmaxf(fmaxf(ml[0][r][0], ml[1][r][0]), fmaxf(ml[2][r][0], ml[3][r][0]));
-        l = o = 0.f;
-        if (m == -INFINITY) { return; }
-#pragma unroll
-        for (int j = 0; j < AS_WARPS; j++)
-        {
-            const float c = exp2f(ml[j][r][0] - m);
-            l += c * ml[j][r][1];
-            o += c * reinterpret_cast<float*>(as_raw)[(j * 16 + r) * DV + d];
-        }
-    };
-    if (p.splits == 1)
-    {
-        for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
-        {
-            float m, l, o;
-            combine(j / p.vdim, j % p.vdim, m, l, o);
-            attention_store(p, qkvg, start, kvh, r0 + j / p.vdim, j % p.vdim, o / l);
-        }
-        return;
-    }
-    const unsigned int vp = (p.vdim + 15) / 16 * 16, stride = 16 * (vp + 2);
-    const unsigned int unit = (e * p.row_tiles + rt) * p.Hkv + kvh;
-    float* mine = p.partial + ((size_t)unit * p.splits + split) * stride;
-    for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
-    {
-        const unsigned int r = j / p.vdim, d = j % p.vdim;
-        float m, l, o;
-        combine(r, d, m, l, o);
-        mine[32 + r * vp + d] = o;
-        if (d == 0)
-        {
-            mine[2 * r] = m;
-            mine[2 * r + 1] = l;
-        }
-    }
-    __threadfence();
-    __syncthreads();
-    if (threadIdx.x == 0) { last = atomicAdd(p.counter + unit, 1) == (int)p.splits - 1; }
-    __syncthreads();
-    if (!last) { return; }
-    __threadfence();
-    const float* all = p.partial + (size_t)unit * p.splits * stride;
-    for (unsigned int j = threadIdx.x; j < live * p.vdim; j += 32 * AS_WARPS)
-    {
-        const unsigned int r = j / p.vdim, d = j % p.vdim;
-        float m = -INFINITY, l = 0.f, o = 0.f;
-        for (unsigned int s = 0; s < p.splits; s++) { m = fmaxf(m, __ldcg(all + s * stride + 2 * r)); }
-        for (unsigned int s = 0; s < p.splits; s++)
-        {
-            const float c = exp2f(__ldcg(all + s * stride + 2 * r) - m);
-            l += c * __ldcg(all + s * stride + 2 * r + 1);
-            o += c * __ldcg(all + s * stride + 32 + r * vp + d);
-        }
-        attention_store(p, qkvg, start, kvh, r0 + r, d, o / l);
-    }
-    if (threadIdx.x == 0) { p.counter[unit] = 0; }
+    split_finish<DV, 16>(p, meet, reinterpret_cast<float*>(as_raw), qkvg, e, start, kvh, rt, r0, rows);
 }
 
-constexpr int AT_WARPS = 4, AT_KT = 64;
+constexpr int AT_WARPS = 4;
 __host__ __device__ constexpr int at_kt(int dk, int dv) { return dk + dv <= 256 ? 64 : 32; }
 __host__ __device__ constexpr int at_smem(int dk, int dv) { return 2 * at_kt(dk, dv) * ((dk + 8) + (dv + 8)) * 2; }
 

@@ -21,8 +21,8 @@ bool KvCache::init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int
     for (const auto& s : layers)
     {
         Layer l;
-        l.k_ld = (s.k_dim + 7) / 8 * 8;
-        l.v_ld = (s.v_dim + 7) / 8 * 8;
+        l.k_ld = (s.k_dim + 15) / 16 * 16;
+        l.v_ld = (s.v_dim + 15) / 16 * 16;
         const size_t per = (size_t)slots * s.kv_heads * rows * elem_bytes;
         l.k_bytes = per * l.k_ld;
         l.v_bytes = per * l.v_ld;

@@ -22,7 +22,7 @@ public:
     ~KvCache();
     KvCache(const KvCache&) = delete;
     KvCache& operator=(const KvCache&) = delete;
-    // elem_bytes 2 or 4.  Rows are padded to eight elements; the padding is zero and stays so.
+    // elem_bytes 2 or 4.  Rows are padded to sixteen elements; the padding is zero and stays so.
     bool init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int elem_bytes, int slots, int rows, std::string* err);
     void* k(int layer) const { return layers_[layer].k; }
     void* v(int layer) const { return layers_[layer].v; }

@@ -103,8 +103,9 @@ typedef struct cuda_b200_attention
 } cuda_b200_attention;
 C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
 /* Appends, then causal softmax attention over the caches (query head h reads kv head h / (H / Hkv)), then the output gate.
- * kernel: 0 = by shape, 1 = split-KV (few query rows), 2 = tiled (prompts), 3 = the plain kernel (always in float mode, and
- * for key or value sizes above 256). */
+ * kernel: 0 = by shape, 1 = split-KV through shared memory (few query rows), 2 = tiled (prompts), 3 = the plain kernel
+ * (always in float mode, and for key or value sizes above 256), 4 = split-KV straight into registers (sizes up to 128, k_ld
+ * and v_ld multiples of 16, caches 32-byte aligned; with one token per entry the append is part of it). */
 C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, const cuda_b200_batch* b, void* stream, unsigned int flags,
     int kernel);
 

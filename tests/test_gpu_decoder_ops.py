@@ -277,7 +277,7 @@ class Attn:
         row[:, k_off:k_off + G * d] = self.k.reshape(T, -1)
         row[:, v_off:v_off + G * dv] = self.v.reshape(T, -1)
         row[:, g_off:g_off + H * dv] = self.g.reshape(T, -1)
-        kl, vl = pad8(d), pad8(dv)
+        kl, vl = (n + (-n) % 16 for n in (d, dv))
         kc, vc = np.zeros(self.kc.shape[:3] + (kl,), np.float32), np.zeros(self.vc.shape[:3] + (vl,), np.float32)
         kc[..., :d], vc[..., :dv] = self.kc, self.vc
         self.x, self.K, self.V = dev(row, dt), dev(kc, dt), dev(vc, dt)
@@ -319,17 +319,20 @@ class Attn:
         return out * F.sigmoid(f8(self.g)) if self.gate else out
 
 
-KINDS = {FLOAT: [0], BF16: [1, 2, 3]}
+KINDS = {FLOAT: [0], BF16: [1, 2, 3, 4]}
 SIZES = [(6, 2, 40, 24), (4, 4, 7, 5), (24, 1, 72, 136), (8, 2, 64, 48), (2, 1, 128, 128), (3, 3, 200, 16), (5, 1, 16, 256), (12, 3, 256, 72)]
 
 
 @pytest.mark.parametrize("dtype", [FLOAT, BF16])
 @pytest.mark.parametrize("H,Hkv,dim,vdim", SIZES)
 def test_attention_sizes_and_ragged_batches(D, dtype, H, Hkv, dim, vdim):
-    for v_mix in (0, 1, 2):
-        a = Attn(D, dtype, H, Hkv, dim, vdim, [(2, 130, 3), (0, 0, 37), (3, 333, 1), (1, 64, 18)], scale=0.3, v_mix=v_mix, seed=H * dim)
+    ragged, decoding = [(2, 130, 3), (0, 0, 37), (3, 333, 1), (1, 64, 18)], [(1, 600, 1), (3, 0, 1), (0, 15, 1), (2, 16, 1)]
+    for v_mix, entries in ((0, ragged), (1, ragged), (2, ragged), (0, decoding), (1, decoding), (2, decoding)):
+        a = Attn(D, dtype, H, Hkv, dim, vdim, entries, scale=0.3, v_mix=v_mix, seed=H * dim)
         want = a.reference()
         for kind in KINDS[dtype]:
+            if kind == 4 and max(dim, vdim) > 128:
+                continue
             got = a.run(kind)
             close(got.reshape(a.T, -1), want.reshape(a.T, -1), dtype, (kind, v_mix), 10 if dtype == FLOAT else 1.5)
             # the caches: new rows in place, everything else untouched, padding zero
@@ -367,7 +370,7 @@ def test_one_key_stands_out(D, dtype, pos, n):
             a.k[spot - pos], a.v[spot - pos] = u, 5.0
         want = a.reference()
         for kind in KINDS[dtype]:
-            if kind == 1 and n > 100:
+            if kind in (1, 4) and n > 100:
                 continue
             got = a.run(kind)
             close(got.reshape(n, -1), want.reshape(n, -1), dtype, (kind, spot), 10 if dtype == FLOAT else 1.5)
@@ -382,7 +385,7 @@ def test_softmax_weights_are_not_rounded(D):
     a.vc[..., :] = 64.0 * np.where(np.arange(T) % 2, 1, -1)[None, None, :, None] + (np.arange(T) % 7 == 0)[None, None, :, None]
     a.vc = F.bf16_round(a.vc).reshape(a.vc.shape)
     want = a.reference()
-    for kind in (1, 2, 3):
+    for kind in (1, 2, 3, 4):
         assert np.abs(a.run(kind) - want).max() < 2.5e-3 * max(1.0, np.abs(want).max()), kind
 
 
@@ -393,5 +396,6 @@ def test_split_results_do_not_depend_on_the_splits(D):
     many.kc, many.vc = one.kc, one.vc
     for name in ("q", "k", "v", "g"):
         getattr(many, name)[3] = getattr(one, name)[0]
-    x, y = one.run(1)[0], many.run(1)[3]
-    assert np.abs(x - y).max() <= 2.0 ** -8 * np.abs(x).max()
+    for kind in (1, 4):
+        x, y = one.run(kind)[0], many.run(kind)[3]
+        assert np.abs(x - y).max() <= 2.0 ** -8 * np.abs(x).max()
