@@ -224,7 +224,7 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     {
         if (p.dim > 256 || p.vdim > 256) { kernel = 3; }
         else if (b->max_n * p.G <= 64 || b->max_n <= 4) { kernel = direct ? 4 : 1; }
-        else { kernel = 2; }
+        else { kernel = p.dim <= 128 && p.vdim <= 128 && a->slots != 0 ? 5 : 2; }
     }
     if (kernel == 4 && b->max_n == 1)
     {
@@ -237,6 +237,7 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     {
     case 1: return launch_attention_split(p, b->entries, b->max_n, b->max_len, st, pdl);
     case 2: return launch_attention_tiled(p, b->entries, b->max_n, st, pdl);
+    case 5: return launch_attention_tile(p, a->slots, b->entries, b->max_n, st, pdl);
     case 4: return launch_attention_direct(p, b->entries, b->max_n, b->max_len, st, pdl);
     default: return dtype == DT_BF16 ? attention_plain<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_plain<float>(p, b->tokens, st, pdl);
     }

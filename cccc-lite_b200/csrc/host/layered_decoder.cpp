@@ -432,6 +432,7 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
         a.k_ld = (unsigned int)cache_.kLd((int)i);
         a.v_ld = (unsigned int)cache_.vLd((int)i);
         a.T_max = (unsigned int)cache_.rows();
+        a.slots = (unsigned int)cache_.slots();
         a.v_mix = L.v_mix;
         a.qk_norm = s.qk_norm;
         a.gate = !s.gate.empty();

@@ -25,7 +25,7 @@ Linear = _struct("Linear", ("W", "X", "Y", "row_scale", "group_offset", "x_row",
                  ("alpha",))
 Batch = _struct("Batch", ("slot", "pos", "start", "n", "token_entry"), ("entries", "tokens", "max_n", "max_len"))
 Attention = _struct("Attention", ("qkvg", "out", "k_cache", "v_cache", "v_first", "work"),
-                    ("ld", "ldo", "k_off", "v_off", "g_off", "v_first_ld", "H", "Hkv", "dim", "vdim", "k_ld", "v_ld", "T_max"), ("v_mix", "qk_norm", "gate"),
+                    ("ld", "ldo", "k_off", "v_off", "g_off", "v_first_ld", "H", "Hkv", "dim", "vdim", "k_ld", "v_ld", "T_max", "slots"), ("v_mix", "qk_norm", "gate"),
                     ("mix", "eps", "scale"))
 Route = _struct("Route", ("logits", "pair_row", "pair_weight", "row_token", "group_offset", "active", "shared_weight", "choice", "counters"),
                 ("n", "ldl", "experts", "top", "active_cap"), ("sg_col",))

@@ -96,16 +96,17 @@ typedef struct cuda_b200_attention
     void* v_first;             /* [tokens][v_first_ld] dtype: written (v_mix 1) or read (v_mix 2) */
     void* work;                /* float scratch of cuda_b200_attention_work_bytes, zeroed once */
     unsigned int ld, ldo, k_off, v_off, g_off, v_first_ld;
-    unsigned int H, Hkv, dim, vdim, k_ld, v_ld, T_max;
+    unsigned int H, Hkv, dim, vdim, k_ld, v_ld, T_max, slots;
     int v_mix;                 /* 0: plain, 1: this layer's values are the ones later layers mix in, 2: mix */
     int qk_norm, gate;         /* 1: unit RMS of q and k; multiply the output by sigmoid(gate) */
     float mix, eps, scale;
 } cuda_b200_attention;
 C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
 /* Appends, then causal softmax attention over the caches (query head h reads kv head h / (H / Hkv)), then the output gate.
- * kernel: 0 = by shape, 1 = split-KV through shared memory (few query rows), 2 = tiled (prompts), 3 = the plain kernel
+ * kernel: 0 = by shape, 1 = split-KV through shared memory (few query rows), 2 = tiled on mma.sync, 3 = the plain kernel
  * (always in float mode, and for key or value sizes above 256), 4 = split-KV straight into registers (sizes up to 128, k_ld
- * and v_ld multiples of 16, caches 32-byte aligned; with one token per entry the append is part of it). */
+ * and v_ld multiples of 16, caches 32-byte aligned; with one token per entry the append is part of it), 5 = tiled on
+ * tcgen05 (prompts; sizes up to 128, caches 16-byte aligned, `slots` given: the caches end after that many). */
 C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, const cuda_b200_batch* b, void* stream, unsigned int flags,
     int kernel);
 
