@@ -5,7 +5,7 @@
 namespace b200
 {
 
-// One CTA per token, one warp per head at a time: q heads, then k heads, then v heads.
+// A warp per (token, head): q heads, then k heads, then v heads.
 template <class T>
 __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams p)
 {
@@ -17,7 +17,8 @@ __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams 
     if (row >= p.T_max) { return; }
     T* x = (T*)p.qkvg + (size_t)i * p.ld;
     const size_t kv0 = (size_t)p.slot[e] * p.Hkv;
-    for (unsigned int h = warp; h < p.H + 2 * p.Hkv; h += warps)
+    const unsigned int h = blockIdx.y * warps + warp;
+    if (h < p.H + 2 * p.Hkv)
     {
         if (h < p.H + p.Hkv)
         {
@@ -25,7 +26,7 @@ __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams 
             const unsigned int kh = h - p.H;
             T* src = is_q ? x + (size_t)h * p.dim : x + p.k_off + (size_t)kh * p.dim;
             T* dst = is_q ? src : (T*)p.k_cache + ((kv0 + kh) * p.T_max + row) * p.k_ld;
-            if (is_q && !p.qk_norm) { continue; }
+            if (is_q && !p.qk_norm) { return; }
             float inv = 1.f;
             if (p.qk_norm)
             {
@@ -148,7 +149,7 @@ static int attention_append(const AttnParams& p, unsigned int tokens, void* stre
 {
     const unsigned int heads = p.H + 2 * p.Hkv;
     const unsigned int warps = heads < 8 ? heads : 8;
-    return launch_kernel("attention_append", attention_append_kernel<T>, dim3(tokens), dim3(32 * warps), 0, stream, pdl, p);
+    return launch_kernel("attention_append", attention_append_kernel<T>, dim3(tokens, (heads + warps - 1) / warps), dim3(32 * warps), 0, stream, pdl, p);
 }
 
 template <class T>

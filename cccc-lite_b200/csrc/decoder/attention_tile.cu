@@ -4,8 +4,9 @@
 // A TMA lane streams keys and values from the cache (128-byte swizzle) through two-deep rings; the MMA lane issues
 // S = Q K^T (M = 128, N = 64) into tensor memory and, once the softmax warps have turned S into weights, O += P V with P as
 // the operand in tensor memory and V as it lies ([key][element], an MN-major operand).  The weights enter as the sum of two
-// BF16 numbers.  S of the next tile is computed while the value product of this one is being issued.  Four softmax warps own
-// one row per thread; the running maximum only moves when it grows by more than 2^8, so that O is seldom rescaled.
+// BF16 numbers and take the place of their scores.  There are two such places: the scores of the next tile are ready when the
+// softmax warps get to them.  Four softmax warps own one row per thread; the running maximum only moves when it grows by more
+// than 2^8, so that O is seldom rescaled.
 // Every wait is bounded; on expiry the status word is raised, the roles drain, tensor memory is freed and the CTA returns.
 #include "attention.cuh"
 #include "../gemm_stream.cuh"
@@ -18,7 +19,7 @@ constexpr int TA_THREADS = 192;
 constexpr int TA_BLOCK = TA_KT * 128;          // 64 keys x 64 elements
 constexpr int TA_QBLOCK = TA_ROWS * 128;       // 128 rows x 64 elements
 __host__ __device__ constexpr int ta_smem(int dk, int dv) { return 1024 + (dk / 64) * TA_QBLOCK + 2 * (dk / 64 + dv / 64) * TA_BLOCK + 1024; }
-constexpr uint32_t TA_TMEM = 256, TA_P = 64, TA_O = 128;    // columns: S 0-63, P high 64-95, P low 96-127, O from 128
+constexpr uint32_t TA_TMEM = 256, TA_O = 128;    // columns: two places of S (64) or P (32 high, 32 low), then O
 
 // An MN-major operand [k][64 elements] with the 128-byte swizzle: 8-k groups 1024 bytes apart, 64-element blocks TA_BLOCK apart.
 __device__ __forceinline__ uint64_t umma_desc_mnmajor_sw128(uint32_t smem_addr)
@@ -38,6 +39,9 @@ __device__ __forceinline__ float exp2_f32(float x)
     return y;
 }
 
+// A BF16 gate's sigmoid, by the hardware's exponential and reciprocal.
+__device__ __forceinline__ float gate_sigmoid(float z) { return __fdividef(1.0f, 1.0f + exp2_f32(-1.44269504088896341f * z)); }
+
 template <int DK, int DV>
 __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     const __grid_constant__ AttnParams p, unsigned int* status)
@@ -47,8 +51,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
     constexpr int KBY = (DK / 64) * TA_BLOCK, VBY = (DV / 64) * TA_BLOCK;
     uint64_t* k_full = reinterpret_cast<uint64_t*>(smem);
     uint64_t *k_empty = k_full + 2, *v_full = k_full + 4, *v_empty = k_full + 6;
-    uint64_t *q_ready = k_full + 8, *s_full = k_full + 9, *p_ready = k_full + 10, *pv_done = k_full + 11;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 12);
+    uint64_t *s_full = k_full + 8, *p_ready = k_full + 10, *q_ready = k_full + 12, *pv_done = k_full + 13;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 14);
     volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
     unsigned char* qs = smem + 1024;
     unsigned char* ks = qs + (DK / 64) * TA_QBLOCK;
@@ -57,10 +61,10 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0)
     {
-        for (int i = 0; i < 8; i++) { mbar_init(k_full + i, 1); }
+        for (int i = 0; i < 10; i++) { mbar_init(k_full + i, 1); }
         mbar_init(q_ready, 4);
-        mbar_init(s_full, 1);
-        mbar_init(p_ready, 4);
+        mbar_init(p_ready, 4);    // one per place: a warp may be a tile ahead of another
+        mbar_init(p_ready + 1, 4);
         mbar_init(pv_done, 1);
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -140,23 +144,22 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                 {
                     if (k * 16 < (int)p.dim)
                     {
-                        umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + (k / 4) * TA_QBLOCK + (k % 4) * 32),
+                        umma_bf16(tmem + (i & 1u) * 64, umma_desc_kmajor_sw128(q_addr + (k / 4) * TA_QBLOCK + (k % 4) * 32),
                             umma_desc_kmajor_sw128(k_addr + (i & 1u) * KBY + (k / 4) * TA_BLOCK + (k % 4) * 32), idesc_s, k != 0 ? 1u : 0u);
                     }
                 }
                 umma_commit(k_empty + (i & 1u));
-                umma_commit(s_full);
+                umma_commit(s_full + (i & 1u));
             }
             __syncwarp();
             return true;
         };
-        bool ok = tiles == 0 || (wait(q_ready, 0) && scores(0));
+        bool ok = tiles == 0 || (wait(q_ready, 0) && scores(0) && (tiles == 1 || scores(1)));
         for (unsigned int i = 0; i < tiles && ok; i++)
         {
-            ok = wait(p_ready, i);
+            ok = wait(p_ready + (i & 1u), i >> 1);
             if (!ok) { break; }
             tc_fence_after();
-            if (i + 1 < tiles && !scores(i + 1)) { ok = false; break; }
             if (!wait(v_full + (i & 1u), i >> 1)) { ok = false; break; }
             tc_fence_after();
             if (elect_one())
@@ -167,7 +170,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
 #pragma unroll
                     for (int k = 0; k < TA_KT / 16; k++)
                     {
-                        umma_bf16_ts(tmem + TA_O, tmem + TA_P + part * 32 + k * 8, umma_desc_mnmajor_sw128(v_addr + (i & 1u) * VBY + k * 2048), idesc_o,
+                        umma_bf16_ts(tmem + TA_O, tmem + (i & 1u) * 64 + part * 32 + k * 8, umma_desc_mnmajor_sw128(v_addr + (i & 1u) * VBY + k * 2048), idesc_o,
                             (i | (unsigned int)part | (unsigned int)k) != 0 ? 1u : 0u);
                     }
                 }
@@ -175,6 +178,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                 umma_commit(pv_done);
             }
             __syncwarp();
+            // into the place of the weights just issued: products of one thread run in the order of their issue
+            if (i + 2 < tiles && !scores(i + 2)) { ok = false; }
         }
         if (!ok)
         {
@@ -193,6 +198,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
         {
             const __nv_bfloat16* src = x + (size_t)head * p.dim;
             const bool vec = (p.dim % 8) == 0;
+            const uint32_t flip = p.scale < 0.f ? 0x80008000u : 0u;    // the maximum is taken before scaling
 #pragma unroll
             for (int c = 0; c < DK / 8; c++)
             {
@@ -208,6 +214,10 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                         v = make_uint4(u[0] | (u[1] << 16), u[2] | (u[3] << 16), u[4] | (u[5] << 16), u[6] | (u[7] << 16));
                     }
                 }
+                v.x ^= flip;
+                v.y ^= flip;
+                v.z ^= flip;
+                v.w ^= flip;
                 sts128(smem_u32(qs) + (c / 8) * TA_QBLOCK + rl * 128 + (((c % 8) ^ (rl & 7u)) * 16), v.x, v.y, v.z, v.w);
             }
             fence_proxy_async();
@@ -215,20 +225,19 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             if (lane == 0) { mbar_arrive(q_ready); }
         }
         const unsigned int lim = min(pos + r / p.G + 1, T), first_lim = pos + t0 / p.G + 1;
-        const float scale2 = p.scale * 1.44269504088896341f;
+        const float scale2 = fmaxf(fabsf(p.scale) * 1.44269504088896341f, 1e-30f);    // 0 times a masked -inf would be no number
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (unsigned int i = 0; i < tiles; i++)
         {
-            ok = __all_sync(0xFFFFFFFFu, wait(s_full, i));
+            const uint32_t place = lanes + (i & 1u) * 64;
+            ok = __all_sync(0xFFFFFFFFu, wait(s_full + (i & 1u), i >> 1));
             if (!ok) { break; }
             tc_fence_after();
             uint32_t s[TA_KT];
-            tmem_ld_32x32(lanes, *reinterpret_cast<uint32_t(*)[32]>(s));
-            tmem_ld_32x32(lanes + 32, *reinterpret_cast<uint32_t(*)[32]>(s + 32));
+            tmem_ld_32x32(place, *reinterpret_cast<uint32_t(*)[32]>(s));
+            tmem_ld_32x32(place + 32, *reinterpret_cast<uint32_t(*)[32]>(s + 32));
             tmem_ld_wait();
-#pragma unroll
-            for (int j = 0; j < TA_KT; j++) { s[j] = __float_as_uint(__uint_as_float(s[j]) * scale2); }
             if ((i + 1) * TA_KT > first_lim)
             {
 #pragma unroll
@@ -240,7 +249,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             float mx[4] = { -INFINITY, -INFINITY, -INFINITY, -INFINITY };    // four maxima in flight
 #pragma unroll
             for (int j = 0; j < TA_KT; j++) { mx[j & 3] = fmaxf(mx[j & 3], __uint_as_float(s[j])); }
-            const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+            const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale2;
             float c = 1.f;
             if (top > m + 8.f)
             {
@@ -253,43 +262,42 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
 #pragma unroll
             for (int j = 0; j < TA_KT / 2; j++)
             {
-                const float a = exp2_f32(__uint_as_float(s[2 * j]) - m), b = exp2_f32(__uint_as_float(s[2 * j + 1]) - m);
+                const float a = exp2_f32(fmaf(__uint_as_float(s[2 * j]), scale2, -m)), b = exp2_f32(fmaf(__uint_as_float(s[2 * j + 1]), scale2, -m));
                 sum[0] += a;
                 sum[1] += b;
                 hi[j] = pack_bf16x2(a, b);
                 lo[j] = pack_bf16x2(a - __uint_as_float(hi[j] << 16), b - __uint_as_float(hi[j] & 0xFFFF0000u));
             }
             l += sum[0] + sum[1];
-            if (i > 0)
+            if (i > 0 && __any_sync(0xFFFFFFFFu, c != 1.f))
             {
-                // the product before has read its weights and left O alone
+                // the product before leaves O alone (the one before that has: the scores of this tile came after it)
                 ok = __all_sync(0xFFFFFFFFu, wait(pv_done, i - 1));
                 if (!ok) { break; }
                 tc_fence_after();
-                if (__any_sync(0xFFFFFFFFu, c != 1.f))
+#pragma unroll
+                for (int d = 0; d < DV; d += 32)
                 {
+                    uint32_t o[32];
+                    tmem_ld_32x32(lanes + TA_O + d, o);
+                    tmem_ld_wait();
 #pragma unroll
-                    for (int d = 0; d < DV; d += 32)
-                    {
-                        uint32_t o[32];
-                        tmem_ld_32x32(lanes + TA_O + d, o);
-                        tmem_ld_wait();
-#pragma unroll
-                        for (int j = 0; j < 32; j++) { o[j] = __float_as_uint(__uint_as_float(o[j]) * c); }
-                        tmem_st_32x16(lanes + TA_O + d, o);
-                        tmem_st_32x16(lanes + TA_O + d + 16, o + 16);
-                    }
+                    for (int j = 0; j < 32; j++) { o[j] = __float_as_uint(__uint_as_float(o[j]) * c); }
+                    tmem_st_32x16(lanes + TA_O + d, o);
+                    tmem_st_32x16(lanes + TA_O + d + 16, o + 16);
                 }
             }
-            tmem_st_32x16(lanes + TA_P, hi);
-            tmem_st_32x16(lanes + TA_P + 16, hi + 16);
-            tmem_st_32x16(lanes + TA_P + 32, lo);
-            tmem_st_32x16(lanes + TA_P + 48, lo + 16);
+            tmem_st_32x16(place, hi);
+            tmem_st_32x16(place + 16, hi + 16);
+            tmem_st_32x16(place + 32, lo);
+            tmem_st_32x16(place + 48, lo + 16);
             tmem_st_wait();
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) { mbar_arrive(p_ready); }
+            if (lane == 0) { mbar_arrive(p_ready + (i & 1u)); }
         }
+        // in turn, since a wait tells only neighbouring phases apart (the scores of the last tile came after product tiles - 3)
+        if (tiles > 1) { ok = ok && __all_sync(0xFFFFFFFFu, wait(pv_done, tiles - 2)); }
         ok = ok && __all_sync(0xFFFFFFFFu, wait(pv_done, tiles - 1));
         if (ok)
         {
@@ -323,8 +331,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
 #pragma unroll
                                 for (int j = 0; j < 4; j++)
                                 {
-                                    v[2 * j] *= sigmoid_f32(__uint_as_float(gw[j] << 16));
-                                    v[2 * j + 1] *= sigmoid_f32(__uint_as_float(gw[j] & 0xFFFF0000u));
+                                    v[2 * j] *= gate_sigmoid(__uint_as_float(gw[j] << 16));
+                                    v[2 * j + 1] *= gate_sigmoid(__uint_as_float(gw[j] & 0xFFFF0000u));
                                 }
                             }
                             *reinterpret_cast<uint4*>(out + d + q) =

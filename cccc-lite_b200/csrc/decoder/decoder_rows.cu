@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(1024) route_small_kernel(const RouteParams p)
     }
 }
 
-constexpr unsigned int kRouteTokens = 32;    // tokens per CTA of the two-kernel form
+constexpr unsigned int kRouteTokens = 8;    // tokens per CTA of the two-kernel form
 
 __global__ void __launch_bounds__(256) route_choose_kernel(const RouteParams p)
 {
