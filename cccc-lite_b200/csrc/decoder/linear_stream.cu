@@ -1,7 +1,7 @@
 // Linears of a few rows with BF16 weights (weight streaming, HBM-bound), and the linears of the float mode.
 //
-// The streaming kernel: a CTA of eight warps owns 16 (or 2 x 16) output features; its warps take the 64-wide k chunks in
-// turn.  A lane loads 32 bytes of weight row g and of row g + 8 straight into the A fragments of mma.m16n8k16 - the k order
+// The streaming kernel: eight warps, WK of which share 16 (or 2 x 16) output features and take the 64-wide k chunks in turn
+// (all eight, or two where k is short).  A lane loads 32 bytes of weight row g and of row g + 8 straight into the A fragments of mma.m16n8k16 - the k order
 // inside a chunk is permuted, identically for both operands, so that fragments are whole pieces of a row - and the rows of X
 // are the eight B columns.  The next chunks' weights are requested before the current ones are consumed, the first ones of
 // a dense member before the previous kernel of the stream has finished.  The warps' partial sums meet in shared memory.
@@ -28,9 +28,9 @@ __device__ __forceinline__ void ldg_stream(const void* p, uint4& a, uint4& b)
                  : "l"(p));
 }
 
-// NT: row groups of eight; RT: 16-feature tiles per warp; U: chunks per loop turn
-template <int NT, int RT, int U>
-__global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const __grid_constant__ LinearLaunch L)
+// NT: row groups of eight; RT: 16-feature tiles per warp; U: chunks per loop turn; WK: warps that share features
+template <int NT, int RT, int U, int WK>
+__global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_kernel(const __grid_constant__ LinearLaunch L)
 {
     constexpr int R = 16 * RT, C = 8 * NT;
     __shared__ float red[LS_WARPS][C][R + 1];
@@ -41,9 +41,10 @@ __global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const _
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const unsigned int b = blockIdx.x - m.block0;
     const bool gated = m.activation == B200_ACT_SILU_GATE;
-    const unsigned int F = gated ? R / 2 : R;    // output features of the CTA
+    const unsigned int F = gated ? R / 2 : R;    // output features of a warp
+    const unsigned int wk = warp % WK, wf = warp / WK;
     const unsigned int fb = b % m.fblocks, slot = b / m.fblocks;
-    const unsigned int f0 = fb * F;
+    const unsigned int fc = fb * F * (LS_WARPS / WK), f0 = fc + wf * F;    // first feature of the CTA, of the warp
     const bool grouped = m.group_offset != nullptr;
     grid_dependency_launch();
     unsigned int group = 0, row0 = 0, count = m.rows;
@@ -80,7 +81,7 @@ __global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const _
 #pragma unroll
         for (int u = 0; u < U; u++)
         {
-            const unsigned int c = c0 + u * LS_WARPS;
+            const unsigned int c = c0 + u * WK;
             if (c < chunks)
             {
 #pragma unroll
@@ -95,11 +96,11 @@ __global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const _
             }
         }
     };
-    load(a, warp);
+    load(a, wk);
     if (!grouped) { grid_dependency_wait(); }
     for (unsigned int n0 = 0; n0 < count; n0 += C)
     {
-        if (n0 != 0) { load(a, warp); }
+        if (n0 != 0) { load(a, wk); }
         const __nv_bfloat16* xr[NT];
         bool live[NT];
 #pragma unroll
@@ -122,27 +123,36 @@ __global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const _
                 for (int j = 0; j < 4; j++) { acc[r][nt][j] = 0.f; }
             }
         }
-        for (unsigned int c0 = warp; c0 < chunks; c0 += U * LS_WARPS)
+        for (unsigned int c0 = wk; c0 < chunks; c0 += U * WK)
         {
-            load(an, c0 + U * LS_WARPS);
+            load(an, c0 + U * WK);
 #pragma unroll
             for (int u = 0; u < U; u++)
             {
-                const unsigned int c = c0 + u * LS_WARPS;
+                const unsigned int c = c0 + u * WK;
                 if (c >= chunks) { break; }
+                uint4 x[NT][2];
 #pragma unroll
                 for (int nt = 0; nt < NT; nt++)
                 {
 #pragma unroll
                     for (int k = 0; k < 2; k++)
                     {
-                        uint4 x = make_uint4(0, 0, 0, 0);
-                        if (live[nt]) { x = *reinterpret_cast<const uint4*>(xr[nt] + c * 64 + k * 8); }
+                        x[nt][k] = make_uint4(0, 0, 0, 0);
+                        if (live[nt]) { x[nt][k] = *reinterpret_cast<const uint4*>(xr[nt] + c * 64 + k * 8); }
+                    }
+                }
+#pragma unroll
+                for (int nt = 0; nt < NT; nt++)
+                {
+#pragma unroll
+                    for (int k = 0; k < 2; k++)
+                    {
 #pragma unroll
                         for (int r = 0; r < RT; r++)
                         {
-                            mma_bf16_16816(acc[r][nt], a[u][r][0][k].x, a[u][r][1][k].x, a[u][r][0][k].y, a[u][r][1][k].y, x.x, x.y);
-                            mma_bf16_16816(acc[r][nt], a[u][r][0][k].z, a[u][r][1][k].z, a[u][r][0][k].w, a[u][r][1][k].w, x.z, x.w);
+                            mma_bf16_16816(acc[r][nt], a[u][r][0][k].x, a[u][r][1][k].x, a[u][r][0][k].y, a[u][r][1][k].y, x[nt][k].x, x[nt][k].y);
+                            mma_bf16_16816(acc[r][nt], a[u][r][0][k].z, a[u][r][1][k].z, a[u][r][0][k].w, a[u][r][1][k].w, x[nt][k].z, x[nt][k].w);
                         }
                     }
                 }
@@ -177,19 +187,20 @@ __global__ void __launch_bounds__(32 * LS_WARPS, 2) linear_stream_kernel(const _
         }
         __syncthreads();
         const unsigned int cols = min((unsigned int)C, count - n0);
-        for (unsigned int i = threadIdx.x; i < cols * F; i += 32 * LS_WARPS)
+        const unsigned int all = F * (LS_WARPS / WK);
+        for (unsigned int i = threadIdx.x; i < cols * all; i += 32 * LS_WARPS)
         {
-            const unsigned int f = i % F, n = i / F;
-            if (f0 + f >= m.N) { continue; }
+            const unsigned int f = i % all, n = i / all, w0 = f / F * WK, fl = f % F;
+            if (fc + f >= m.N) { continue; }
             float v = 0.f, up = 0.f;
 #pragma unroll
-            for (int w = 0; w < LS_WARPS; w++) { v += red[w][n][f]; }
+            for (int w = 0; w < WK; w++) { v += red[w0 + w][n][fl]; }
             if (gated)
             {
 #pragma unroll
-                for (int w = 0; w < LS_WARPS; w++) { up += red[w][n][16 + f]; }
+                for (int w = 0; w < WK; w++) { up += red[w0 + w][n][16 + fl]; }
             }
-            linear_store(m, row0 + n0 + n, f0 + f, linear_activation(m.activation, m.alpha * v, m.alpha * up));
+            linear_store(m, row0 + n0 + n, fc + f, linear_activation(m.activation, m.alpha * v, m.alpha * up));
         }
     }
 }
@@ -270,19 +281,28 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearMember m)
     }
 }
 
-template <int NT, int RT, int U>
-static int launch_stream(LinearLaunch& L, cudaStream_t st, bool pdl)
+template <int NT, int RT, int U, int WK>
+static int launch_stream_wk(LinearLaunch& L, cudaStream_t st, bool pdl)
 {
     unsigned int blocks = 0;
     for (unsigned int j = 0; j < L.count; j++)
     {
         LinearMember& m = L.m[j];
-        const unsigned int F = m.activation == B200_ACT_SILU_GATE ? 8 * RT : 16 * RT;
+        const unsigned int F = (m.activation == B200_ACT_SILU_GATE ? 8 * RT : 16 * RT) * (LS_WARPS / WK);
         m.fblocks = (m.N + F - 1) / F;
         m.block0 = blocks;
         blocks += m.fblocks * m.slots;
     }
-    return launch_kernel("linear_stream", linear_stream_kernel<NT, RT, U>, dim3(blocks), dim3(32 * LS_WARPS), 0, st, pdl, L);
+    return launch_kernel("linear_stream", linear_stream_kernel<NT, RT, U, WK>, dim3(blocks), dim3(32 * LS_WARPS), 0, st, pdl, L);
+}
+
+template <int NT, int RT, int U>
+static int launch_stream(LinearLaunch& L, cudaStream_t st, bool pdl)
+{
+    // eight warps over few chunks would leave some without any; the members of a launch take one form
+    unsigned int longest = 0;
+    for (unsigned int j = 0; j < L.count; j++) { longest = L.m[j].K > longest ? L.m[j].K : longest; }
+    return longest <= 1024 ? launch_stream_wk<NT, RT, U, 2>(L, st, pdl) : launch_stream_wk<NT, RT, U, 8>(L, st, pdl);
 }
 
 }    // namespace b200
@@ -295,8 +315,7 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
     if (!members || count > LINEAR_MAX_MEMBERS || (dtype != DT_BF16 && dtype != DT_FLOAT)) { return -1; }
     LinearLaunch L;
     memset(&L, 0, sizeof(L));
-    bool any_gated = false;
-    unsigned int most = 0;
+    unsigned int most = 0, group_max[LINEAR_MAX_MEMBERS] = {};
     for (unsigned int j = 0; j < count; j++)
     {
         const cuda_b200_linear& a = members[j];
@@ -332,7 +351,7 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         m.accumulate = a.accumulate;
         m.alpha = a.alpha;
         if (m.slots == 0) { return -1; }
-        any_gated = any_gated || a.activation == B200_ACT_SILU_GATE;
+        group_max[L.count - 1] = a.group_max;
         const unsigned int rows = a.group_offset ? a.group_max : a.rows;
         most = rows > most ? rows : most;
     }
@@ -355,9 +374,35 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
     }
     if (kernel == 1 || (kernel == 0 && most <= 32))
     {
-        if (most <= 8) { return any_gated ? launch_stream<1, 2, 1>(L, st, pdl) : launch_stream<1, 1, 2>(L, st, pdl); }
-        if (most <= 16) { return any_gated ? launch_stream<2, 2, 1>(L, st, pdl) : launch_stream<2, 1, 2>(L, st, pdl); }
-        return launch_stream<4, 2, 1>(L, st, pdl);
+        // Members whose groups hold about as many rows share a launch: 8, 16 or 32 rows at a time.  A group with more rows
+        // than that reads its weights again, so experts go by twice their mean.
+        for (unsigned int width = 8; width <= 32; width *= 2)
+        {
+            LinearLaunch part;
+            memset(&part, 0, sizeof(part));
+            bool gated = false;
+            for (unsigned int j = 0; j < L.count; j++)
+            {
+                const LinearMember& m = L.m[j];
+                unsigned int rows = m.rows;
+                if (m.group_offset)
+                {
+                    rows = 2 * ((m.rows + m.slots - 1) / m.slots);
+                    if (rows > group_max[j]) { rows = group_max[j]; }
+                }
+                if (width < 32 ? rows > width : false) { continue; }
+                if (width > 8 && rows <= width / 2) { continue; }
+                part.m[part.count++] = m;
+                gated = gated || m.activation == B200_ACT_SILU_GATE;
+            }
+            if (part.count == 0) { continue; }
+            int rc;
+            if (width == 8) { rc = gated ? launch_stream<1, 2, 1>(part, st, pdl) : launch_stream<1, 1, 2>(part, st, pdl); }
+            else if (width == 16) { rc = gated ? launch_stream<2, 2, 1>(part, st, pdl) : launch_stream<2, 1, 2>(part, st, pdl); }
+            else { rc = launch_stream<4, 2, 1>(part, st, pdl); }
+            if (rc) { return rc; }
+        }
+        return 0;
     }
     for (unsigned int j = 0; j < L.count; j++)
     {

@@ -66,7 +66,7 @@ typedef struct cuda_b200_linear
     float alpha;
 } cuda_b200_linear;
 /* Up to three independent members.  BF16: where no member has more than 32 rows (in one group), one launch of a weight-
- * streaming kernel runs all of them; else one tcgen05 launch per member (x_row not taken there).  kernel: 0 = by shape,
+ * streaming kernel runs all of them that hold about as many rows; else one tcgen05 launch per member (x_row not taken there).  kernel: 0 = by shape,
  * 1 = weight streaming, 2 = tcgen05 (tests and tuning). */
 C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b200_linear* members, void* stream, unsigned int flags, int kernel);
 
