@@ -22,6 +22,9 @@ With N>1 (launched under torchrun, one rank per GPU) the same token is computed 
 q/k/v/gate/up/lm_head split by output feature, o/down split by input feature with the all-reduce fused
 into their kernel, logits all-gathered; `value` stays whole-job bytes of the unsharded model per second.
 
+`--decoder` instead times decode and prefill steps of Fakilorn models (BF16 weights, random) with layers of a real
+model's size, beside the quantised model's at equal size.
+
 `--impl reference` times the reference's CPU form of the path (its types.h decode to float, then
 OpenBLAS sgemm) on all host cores, each step a bounded sample of the same workload.
 """
@@ -732,6 +735,97 @@ def gpu_arm(args):
         os._exit(0)
 
 
+# ---- Fakilorn beside the quantised model (--decoder) ----------------------------------------------------
+def decoder_cases(layers):
+    """Layers of a real model's size: `dense` has the headline model's own (its linears in BF16), `experts` a routed one's."""
+    q = QWEN
+    attn = dict(heads=q["HEADS"], kv_heads=q["KVHEADS"], dim=q["HD"], vdim=q["HD"], scale=q["HD"] ** -0.5, v_mix=True)
+    moe = dict(kind="moe", router=dict(experts=64, top=8), expert=dict(ff=768), shared=dict(ff=768))
+    base = lambda width, vocab, mixer, mlp: dict(architecture="Fakilorn", width=width, vocab=vocab, embedding=dict(scale=8.0), logit_scale=1.0, norm=dict(eps=1e-5),
+                                                 layers=[dict(type="attention", mixer=mixer, mlp=mlp)] * layers)
+    return {"dense": base(q["HIDDEN"], q["VOCAB"], attn, dict(kind="dense", ff=q["FFN"])),
+            "experts": base(2048, 65536, dict(attn, heads=16, kv_heads=4), moe)}
+
+
+def decoder_work(c, tokens, sequences, context):
+    """(bytes, linear flops, attention flops) of one step of `sequences` x `tokens` new tokens on `context` cached ones:
+    weights that are read (experts: the expected number of different ones), cache rows, the wanted rows' logits."""
+    T, W = tokens * sequences, c["width"]
+    nbytes, flops, aflops = 2 * c["vocab"] * W, 2 * c["vocab"] * W * sequences, 0
+    for L in c["layers"]:
+        m, f = L["mixer"], L["mlp"]
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        w = W * (H * d + G * d + G * dv + 2 * H * dv)
+        active = w
+        if f["kind"] == "dense":
+            w += 2 * W * f["ff"]
+            active = w
+        else:
+            E, top, e, s = f["router"]["experts"], f["router"]["top"], 3 * W * f["expert"]["ff"], 3 * W * f["shared"]["ff"]
+            active = w + E * W + s + top * e
+            w += E * W + s + E * (1 - (1 - top / E) ** T) * e
+        nbytes += 2 * w + 2 * sequences * (context + tokens) * G * (d + dv)
+        flops += 2 * active * T
+        aflops += 2 * H * (d + dv) * sequences * (tokens * context + tokens * (tokens + 1) // 2)
+    return nbytes, flops, aflops
+
+
+def decoder_arm(args):
+    """Fakilorn with random weights through the serving interface, and the quantised model's decode step and prefill linears
+    at the same layer sizes, in one JSON line."""
+    import importlib
+    import tempfile
+
+    import torch
+
+    from __graft_entry__ import load_package
+
+    watchdog = start_watchdog(args.watchdog)
+    pkg = load_package()
+    peaks = load_peaks()
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    layers = args.layers or 8
+    dev = torch.device("cuda:0")
+    torch.cuda.set_device(dev)
+    out = {"metric": "decoder_steps", "layers": layers, "context": CONTEXT, "data": "random weights", "dtype": "bf16",
+           "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": "measured" if peaks else "fallback"},
+           "timing": "CUDA events, fastest of 5 runs of 10 steps, weights larger than L2"}
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches = pkg.decoder_capi.launches()
+    for name, c in decoder_cases(layers).items():
+        with tempfile.TemporaryDirectory() as d:
+            with open(os.path.join(d, "config.json"), "w") as f:
+                json.dump(c, f)
+            m = pkg.serve.Model(d, max_context=CONTEXT, max_sequences=32, max_step_tokens=4096, noise_weights=True)
+        case = {}
+        for B in (1, 8, 32):
+            ms = m.time_step(B, 1, CONTEXT - 1)
+            nbytes, _, _ = decoder_work(c, 1, B, CONTEXT - 1)
+            case[f"decode_batch{B}"] = {"ms_per_step": round(ms, 4), "tok_per_s": round(B / ms * 1e3, 1), "gbs": round(nbytes / ms / 1e6, 1),
+                                        "frac_of_hbm": round(nbytes / ms / 1e6 / hbm, 4)}
+        for tokens in (512, 2048):
+            ms = m.time_step(1, tokens, 0, 5, 5)
+            _, fl, afl = decoder_work(c, tokens, 1, 0)
+            case[f"prefill_{tokens}"] = {"ms": round(ms, 4), "tok_per_s": round(tokens / ms * 1e3, 1), "tflops": round((fl + afl) / ms / 1e9, 1),
+                                         "frac_of_bf16": round((fl + afl) / ms / 1e9 / tf, 4)}
+        case["weight_bytes"] = m.info(4)
+        out[name] = case
+        m.close()
+    # the closest model at equal size: FP8 weights, RMSNorm, RoPE, SwiGLU; its decode step, and its prefill linears
+    capi, dm = pkg.capi, importlib.import_module("cccc_lite_b200.decode_model")
+    dims = model_dims("e5m2", layers)
+    wt, lin, bufs = build_model(torch, capi, dims, 32, "e5m2", 0, 1, dev)
+    model = decode_step_model(torch, capi, dm, dims, wt, lin, 1, 0, 32, dev, bufs)
+    stream = torch.cuda.Stream(dev)
+    out["quantised"] = {f"decode_batch{B}": time_decode_step(torch, None, capi, model, dims, B, "e5m2", 1, 20, dev, stream, 1) for B in (1, 8, 32)}
+    out["quantised"]["prefill_linears_2048"] = prefill_probe(torch, capi, dims, "e5m2", dev, peaks)
+    out["gpu_launches"] = pkg.decoder_capi.launches() - launches
+    out["clocks"] = sampler.stop()
+    print(json.dumps(out), flush=True)
+    watchdog.cancel()
+
+
 def prefill_probe(torch, capi, dims, wtype, dev, peaks):
     """The prefill configuration (config 4) in brief: M=2048 tokens through one layer's seven linears (tcgen05 kernels),
     q/k/v and gate/up as grouped calls on their shared input, timed with CUDA events; reported next to
@@ -1044,8 +1138,12 @@ def main():
                     help="headline chain through cuda_decode_program_* (one persistent kernel per token) instead of launch by launch")
     ap.add_argument("--watchdog", type=float, default=540.0, help="seconds after which a stuck run exits by itself")
     ap.add_argument("--no-cpu-baseline", action="store_true")
+    ap.add_argument("--decoder", action="store_true",
+                    help="instead of the headline: Fakilorn's decode and prefill steps beside the quantised model's at equal layer sizes")
     args = ap.parse_args()
-    if args.impl == "reference":
+    if args.decoder:
+        decoder_arm(args)
+    elif args.impl == "reference":
         reference_arm(args)
     else:
         gpu_arm(args)
