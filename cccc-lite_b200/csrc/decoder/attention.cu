@@ -28,6 +28,18 @@ __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams 
             T* dst = is_q ? src : (T*)p.k_cache + ((kv0 + kh) * p.T_max + row) * p.k_ld;
             if (is_q && !p.qk_norm) { return; }
             float inv = 1.f;
+            // rows of up to 128 elements in whole quads: one load and one store per lane
+            if ((p.dim % 4) == 0 && p.dim <= 128 && (p.ld % 4) == 0 && (p.k_off % 4) == 0)
+            {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (4 * lane < p.dim) { v = load4(src + 4 * lane); }
+                if (p.qk_norm)
+                {
+                    inv = 1.0f / sqrtf(warp_sum((v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w)) / (float)p.dim + p.eps);
+                }
+                if (4 * lane < p.dim) { store4(dst + 4 * lane, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv)); }
+                return;
+            }
             if (p.qk_norm)
             {
                 float sq = 0.f;
@@ -177,6 +189,8 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     if (!a || !b) { return -1; }
     if (b->tokens == 0 || b->entries == 0) { return 0; }
     if (!a->qkvg || !a->out || !a->k_cache || !a->v_cache || !a->work || !b->slot || !b->pos || !b->start || !b->n || !b->token_entry) { return -1; }
+    auto low = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) != 0; };
+    if (low(a->qkvg) || low(a->k_cache) || low(a->v_cache) || low(a->work)) { return -1; }
     if ((dtype != DT_BF16 && dtype != DT_FLOAT) || a->H == 0 || a->Hkv == 0 || (a->H % a->Hkv) || a->dim == 0 || a->vdim == 0 || a->k_ld < a->dim
         || a->v_ld < a->vdim || (a->k_ld % 8) || (a->v_ld % 8) || a->T_max == 0 || (a->v_mix && !a->v_first))
     {

@@ -7,6 +7,7 @@
 namespace b200
 {
 
+// Row strides are multiples of four elements: quads of columns, the last one possibly into the padding.
 template <class T>
 __global__ void __launch_bounds__(256) embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, unsigned int ldt,
     float* __restrict__ X, unsigned int ldx, unsigned int width, unsigned int vocab, float scale)
@@ -17,7 +18,16 @@ __global__ void __launch_bounds__(256) embed_f32_kernel(const int* __restrict__ 
     const bool ok = id >= 0 && (unsigned int)id < vocab;
     const T* src = table + (size_t)(ok ? id : 0) * ldt;
     float* dst = X + (size_t)blockIdx.x * ldx;
-    for (unsigned int i = threadIdx.x; i < width; i += blockDim.x) { dst[i] = ok ? Elem<T>::get(src[i]) * scale : 0.f; }
+#pragma unroll 4
+    for (unsigned int i = threadIdx.x; i < (width + 3) / 4; i += blockDim.x)
+    {
+        float4 v = ok ? load4(src + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v.x *= scale;
+        v.y *= scale;
+        v.z *= scale;
+        v.w *= scale;
+        store4(dst + 4 * i, v);
+    }
 }
 
 // ---- branch addition + norm ------------------------------------------------------------------------
@@ -29,22 +39,6 @@ __device__ __forceinline__ float block_sum(float v, float* part)
     if (lane == 0) { part[warp] = v; }
     __syncthreads();
     return warp_sum(lane < warps ? part[lane] : 0.f);
-}
-
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const __nv_bfloat16* p)
-{
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v)
-{
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    uint2 u;
-    u.x = *reinterpret_cast<const uint32_t*>(&a);
-    u.y = *reinterpret_cast<const uint32_t*>(&b);
-    *reinterpret_cast<uint2*>(p) = u;
 }
 
 struct NormParams
@@ -63,7 +57,7 @@ struct NormParams
 
 // One CTA per row.  The row lives in shared memory as floats; quads of columns per thread (row strides are multiples
 // of four elements, so the last quad may cover padding columns, which take no part in the sums and are not stored).
-template <class T>
+template <class T, bool SLOTS>
 __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormParams p)
 {
     extern __shared__ __align__(16) float nr_row[];
@@ -75,11 +69,13 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormParams p)
     const unsigned int quads = (p.width + 3) / 4;
     const T* Y = (const T*)p.Y;
     float sum = 0.f;
+#pragma unroll 4
     for (unsigned int i = threadIdx.x; i < quads; i += blockDim.x)
     {
         float4 v = load4(x + 4 * i);
-        if (p.slots != 0)
+        if (SLOTS)
         {
+#pragma unroll 4
             for (unsigned int s = 0; s < p.slots; s++)
             {
                 const float w = p.slot_weight[(size_t)blockIdx.x * p.slots + s];
@@ -350,15 +346,35 @@ __global__ void __launch_bounds__(1024) argmax_f32_kernel(const float* __restric
     const float* row = logits + (size_t)blockIdx.x * ld;
     float best = -INFINITY;
     int at = 0x7FFFFFFF;
-    for (unsigned int i = threadIdx.x; i < cols; i += blockDim.x)
-    {
-        const float v = row[i];
+    auto see = [&](float v, unsigned int i) {
         if (v > best || (v == best && at == 0x7FFFFFFF))    // the second case: a leading -inf
         {
             best = v;
             at = (int)i;
         }
+    };
+    unsigned int done = 0;
+    if ((ld % 4) == 0 && (reinterpret_cast<uintptr_t>(logits) & 15u) == 0)
+    {
+        // four quads of a thread in flight; its indices still grow, so that the first of equal values stays
+        const float4* quad = reinterpret_cast<const float4*>(row);
+        for (; done + 16 * blockDim.x <= cols; done += 16 * blockDim.x)
+        {
+            float4 v[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) { v[j] = quad[done / 4 + j * blockDim.x + threadIdx.x]; }
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                const unsigned int i = done + 4 * (j * blockDim.x + threadIdx.x);
+                see(v[j].x, i);
+                see(v[j].y, i + 1);
+                see(v[j].z, i + 2);
+                see(v[j].w, i + 3);
+            }
+        }
     }
+    for (unsigned int i = done + threadIdx.x; i < cols; i += blockDim.x) { see(row[i], i); }
     auto take = [&](float ov, int oi) {
         if (ov > best || (ov == best && oi < at))
         {
@@ -396,7 +412,7 @@ C_EXPORT int cuda_b200_embed_f32(int dtype, const void* ids, const void* table, 
     unsigned int width, unsigned int vocab, float scale, void* stream, unsigned int flags)
 {
     if (n == 0) { return 0; }
-    if (!ids || !table || !X) { return -1; }
+    if (!ids || !table || !X || (ld_table % 4) || (ldx % 4)) { return -1; }
     const bool pdl = (flags & 1u) != 0;
     if (dtype == DT_BF16)
     {
@@ -440,8 +456,9 @@ C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* strea
     unsigned int threads = a->n <= 64 ? 1024u : 256u;
     while (threads > 64 && threads / 2 * 4 >= a->width) { threads /= 2; }
     const bool pdl = (flags & 1u) != 0;
-    return dtype == DT_BF16 ? launch_kernel("norm_rows", norm_rows_kernel<__nv_bfloat16>, dim3(a->n), dim3(threads), smem, stream, pdl, p)
-                            : launch_kernel("norm_rows", norm_rows_kernel<float>, dim3(a->n), dim3(threads), smem, stream, pdl, p);
+    auto run = [&](auto kernel) { return launch_kernel("norm_rows", kernel, dim3(a->n), dim3(threads), smem, stream, pdl, p); };
+    if (dtype == DT_BF16) { return p.slots ? run(norm_rows_kernel<__nv_bfloat16, true>) : run(norm_rows_kernel<__nv_bfloat16, false>); }
+    return p.slots ? run(norm_rows_kernel<float, true>) : run(norm_rows_kernel<float, false>);
 }
 
 C_EXPORT int cuda_b200_route_rows(const cuda_b200_route* a, void* stream, unsigned int flags)

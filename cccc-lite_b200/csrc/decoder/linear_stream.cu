@@ -372,6 +372,12 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         }
         return 0;
     }
+    // a dense linear of 17 to 32 rows with a tile for every SM (a head over a vocabulary): tiles stream weights as fast
+    if (kernel == 0 && L.count == 1 && most > 16 && !L.m[0].group_offset && !L.m[0].x_row)
+    {
+        const DecoderDevice* dev = decoder_device();
+        if (dev && L.m[0].N >= 256u * (unsigned int)dev->sm_count) { kernel = 2; }
+    }
     if (kernel == 1 || (kernel == 0 && most <= 32))
     {
         // Members whose groups hold about as many rows share a launch: 8, 16 or 32 rows at a time.  A group with more rows

@@ -86,7 +86,7 @@ typedef struct cuda_b200_batch
 /* Attention of a layer from its projections on.  First, for every token of the batch: q heads to unit RMS in place
  * (qk_norm), k heads to unit RMS and v (mixed with v_first: v = (1 - mix) v + mix v_first) appended to the caches,
  * v_first stored.  Caches hold rows of k_ld / v_ld elements (multiples of 8) whose padding is zero.  A batch entry's
- * sequence must fit: pos + n <= T_max. */
+ * sequence must fit: pos + n <= T_max.  qkvg, the caches and work are 16-byte aligned. */
 typedef struct cuda_b200_attention
 {
     void* qkvg;                /* [tokens][ld] dtype: q at 0, k at k_off, v at v_off, output gate at g_off */
