@@ -221,15 +221,15 @@ def test_experts_from_router_to_stream(D, dtype, tokens, E, top, ff, width):
 
 def test_a_group_of_members_is_the_separate_launches(D):
     rng = np.random.default_rng(11)
-    x = rand(rng, 6, 320)
+    x = rand(rng, 6, 288)
     X = padded(x, BF16)
     members, outs, wants = [], [], []
     for j, (N, act) in enumerate(((70, 0), (48, 2), (130, 1))):
-        w = rand(rng, N * (2 if act == 2 else 1), 320, scale=0.05)
+        w = rand(rng, N * (2 if act == 2 else 1), 288, scale=0.05)
         W, Y = padded(w, BF16), padded(np.zeros((6, N)), FLOAT)
         full = x.astype(np.float64) @ w.T
         wants.append(act_ref(act, full[:, :N], full[:, N:]))
-        members.append(D.fill(D.Linear, W=W, X=X, Y=Y, rows=6, N=N, K=320, ldw=320, ldx=320, ldy=pad64(N), up_row=N, activation=act, alpha=1.0))
+        members.append(D.fill(D.Linear, W=W, X=X, Y=Y, rows=6, N=N, K=288, ldw=320, ldx=320, ldy=pad64(N), up_row=N, activation=act, alpha=1.0))
         outs.append((W, Y, N))
     before = D.launches()
     assert D.linear(BF16, members, flags=1) == 0 and D.launches() == before + 1
@@ -320,7 +320,7 @@ class Attn:
 
 
 KINDS = {FLOAT: [0], BF16: [1, 2, 3, 4, 5]}
-SIZES = [(6, 2, 40, 24), (4, 4, 7, 5), (24, 1, 72, 136), (8, 2, 64, 48), (2, 1, 128, 128), (3, 3, 200, 16), (5, 1, 16, 256), (12, 3, 256, 72)]
+SIZES = [(6, 2, 40, 24), (4, 4, 7, 5), (24, 1, 72, 136), (8, 2, 64, 56), (2, 1, 128, 128), (3, 3, 200, 16), (5, 1, 16, 256), (12, 3, 256, 72)]
 
 
 @pytest.mark.parametrize("dtype", [FLOAT, BF16])
@@ -391,8 +391,8 @@ def test_softmax_weights_are_not_rounded(D):
 
 def test_split_results_do_not_depend_on_the_splits(D):
     """The same query alone (many splits) and among thirty others (few): the same values up to float rounding."""
-    one = Attn(D, BF16, 8, 2, 64, 48, [(3, 650, 1)], seed=4)
-    many = Attn(D, BF16, 8, 2, 64, 48, [(s % 4, 100 + s, 1) for s in range(3)] + [(3, 650, 1)], slots=4, seed=5)
+    one = Attn(D, BF16, 8, 2, 64, 56, [(3, 650, 1)], seed=4)
+    many = Attn(D, BF16, 8, 2, 64, 56, [(s % 4, 100 + s, 1) for s in range(3)] + [(3, 650, 1)], slots=4, seed=5)
     many.kc, many.vc = one.kc, one.vc
     for name in ("q", "k", "v", "g"):
         getattr(many, name)[3] = getattr(one, name)[0]

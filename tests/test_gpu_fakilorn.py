@@ -40,7 +40,7 @@ CONFIGS = {
     # sizes that are multiples of nothing
     "odd": config(97, 53, [(attn(4, 4, 7, 5, 1.3), moe(1, 1, 19, 23)), (attn(5, 1, 11, 20, 1.0), DENSE(33))]),
     # many query heads per kv head; every expert chosen
-    "wide": config(264, 640, [(attn(24, 1, 72, 136, 0.3), moe(4, 4, 64, 32)), (attn(24, 1, 80, 136, 0.3), moe(4, 1, 64, 32))], embed=1.0, logit=1.0),
+    "wide": config(264, 610, [(attn(24, 1, 72, 136, 0.3), moe(4, 4, 64, 32)), (attn(24, 1, 80, 136, 0.3), moe(4, 1, 64, 32))], embed=1.0, logit=1.0),
     # keys and values beyond the tensor-core kernels' sizes
     "huge": config(128, 100, [(attn(2, 1, 264, 16, 0.1), DENSE(64)), (attn(2, 1, 16, 272, 0.5, False), DENSE(64))]),
 }
