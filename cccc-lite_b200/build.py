@@ -48,7 +48,8 @@ DECODER_LIB = os.path.join(HERE, "libcccc-b200-decoder.so")
 DECODER_DIR = os.path.join(CSRC, "decoder")
 OBJ_DIR = os.path.join(HERE, "build")    # git-ignored object files: only changed translation units are recompiled
 # the serving core; every other .cpp of csrc/host belongs to the host library
-CORE = ["gpu_control", "json", "tensor_source", "kv_cache", "language_model", "generate", "scheduler", "layered_decoder", "fakilorn", "model_capi"]
+CORE = ["gpu_control", "json", "tensor_source", "kv_cache", "language_model", "generate", "scheduler", "layered_decoder", "layered_mixers", "design_config",
+        "fakilorn", "tazunex", "model_capi"]
 
 
 def _mtime(paths) -> float:

@@ -1,5 +1,5 @@
-// What precedes attention (unit RMS of q and k, value mixing, cache append) and the plain attention kernel of the float
-// mode.
+// What precedes attention (norms and rotation of q and k, value mixing, cache append) and the plain attention kernel of the
+// float mode.
 #include "attention.cuh"
 
 namespace b200
@@ -11,7 +11,7 @@ __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams 
 {
     grid_dependency_launch();
     grid_dependency_wait();
-    const unsigned int i = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const unsigned int i = p.t0 + blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int e = p.token_entry[i];
     const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
     if (row >= p.T_max) { return; }
@@ -69,19 +69,86 @@ __global__ void __launch_bounds__(256) attention_append_kernel(const AttnParams 
     }
 }
 
+// A CTA per token and part (0: q, 1: k and v), for norms over a whole projection and rotations.  The part's row lives in shared
+// memory as floats.
+template <class T>
+__global__ void __launch_bounds__(512) attention_prepare_kernel(const AttnParams p)
+{
+    extern __shared__ float ar_row[];
+    __shared__ float sums[16];
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int i = p.t0 + blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+    const bool is_q = blockIdx.y == 0;
+    const int e = p.token_entry[i];
+    const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
+    if (row >= p.T_max) { return; }
+    T* x = (T*)p.qkvg + (size_t)i * p.ld;
+    const size_t kv0 = (size_t)p.slot[e] * p.Hkv;
+    const unsigned int heads = is_q ? p.H : p.Hkv, all = heads * p.dim;
+    const T* src = is_q ? x : x + p.k_off;
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    float sq = 0.f;
+    for (unsigned int d = tid; d < all; d += blockDim.x)
+    {
+        const float v = Elem<T>::get(src[d]);
+        ar_row[d] = v;
+        sq += v * v;
+    }
+    if (w != nullptr)
+    {
+        sq = warp_sum(sq);
+        if (lane == 0) { sums[warp] = sq; }
+        __syncthreads();
+        const float inv = 1.0f / sqrtf(warp_sum(lane < warps ? sums[lane] : 0.f) / (float)all + p.eps);
+        for (unsigned int d = tid; d < all; d += blockDim.x) { ar_row[d] *= inv * w[d]; }
+    }
+    __syncthreads();
+    if (p.qk_norm)
+    {
+        for (unsigned int h = warp; h < heads; h += warps)
+        {
+            float* r = ar_row + h * p.dim;
+            float s = 0.f;
+            for (unsigned int d = lane; d < p.dim; d += 32) { s += r[d] * r[d]; }
+            const float inv = 1.0f / sqrtf(warp_sum(s) / (float)p.dim + p.eps);
+            for (unsigned int d = lane; d < p.dim; d += 32) { r[d] *= inv; }
+        }
+        __syncthreads();
+    }
+    const float2* rot = p.rotary + (size_t)row * (p.rot_dims / 2);
+    for (unsigned int j = tid; j < all; j += blockDim.x)
+    {
+        const unsigned int h = j / p.dim, d = j % p.dim;
+        const float v = rotated(ar_row + h * p.dim, d, p.rot_dims, p.rot_interleaved != 0, rot);
+        T* dst = is_q ? x + j : (T*)p.k_cache + ((kv0 + h) * p.T_max + row) * p.k_ld + d;
+        *dst = Elem<T>::put(v);
+    }
+    if (is_q) { return; }
+    for (unsigned int j = tid; j < p.Hkv * p.vdim; j += blockDim.x)
+    {
+        const T raw = x[p.v_off + j];
+        float v = Elem<T>::get(raw);
+        if (p.v_mix == 1) { ((T*)p.v_first)[(size_t)i * p.v_first_ld + j] = raw; }
+        else if (p.v_mix == 2) { v = (1.0f - p.lambda) * v + p.lambda * Elem<T>::get(((const T*)p.v_first)[(size_t)i * p.v_first_ld + j]); }
+        ((T*)p.v_cache)[((kv0 + j / p.vdim) * p.T_max + row) * p.v_ld + j % p.vdim] = Elem<T>::put(v);
+    }
+}
+
 constexpr unsigned int AP_KEYS = 128;
 
-// One CTA per (token, kv head): its G query heads against the cache in chunks of 128 keys with a running softmax.
+// One CTA per (token, kv head, group of GB query heads): the heads against the cache in chunks of 128 keys with a running
+// softmax.
 template <class T>
-__global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p)
+__global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p, const unsigned int GB)
 {
     extern __shared__ float ap_smem[];
     grid_dependency_launch();
     grid_dependency_wait();
-    const unsigned int i = blockIdx.x, kvh = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const unsigned int i = p.t0 + blockIdx.x, kvh = blockIdx.y, g0 = blockIdx.z * GB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int e = p.token_entry[i];
     const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
-    const unsigned int keys = min(row + 1u, p.T_max), G = p.G;
+    const unsigned int keys = min(row + 1u, p.T_max), G = min(GB, p.G - g0), h0 = kvh * p.G + g0;
     float* q = ap_smem;                     // [G][dim]
     float* sc = q + G * p.dim;              // [G][128]
     float* acc = sc + G * AP_KEYS;          // [G][vdim]
@@ -89,7 +156,7 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p
     const T* x = (const T*)p.qkvg + (size_t)i * p.ld;
     const T* K = (const T*)p.k_cache + (((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max) * p.k_ld;
     const T* V = (const T*)p.v_cache + (((size_t)p.slot[e] * p.Hkv + kvh) * p.T_max) * p.v_ld;
-    for (unsigned int j = tid; j < G * p.dim; j += 128) { q[j] = Elem<T>::get(x[(size_t)kvh * G * p.dim + j]); }
+    for (unsigned int j = tid; j < G * p.dim; j += 128) { q[j] = Elem<T>::get(x[(size_t)(h0 + j / p.dim) * p.q_ld + j % p.dim]); }
     for (unsigned int j = tid; j < G * p.vdim; j += 128) { acc[j] = 0.f; }
     for (unsigned int g = tid; g < G; g += 128)
     {
@@ -97,7 +164,7 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p
         ml[3 * g + 1] = 0.f;
     }
     __syncthreads();
-    for (unsigned int k0 = 0; k0 < keys; k0 += AP_KEYS)
+    for (unsigned int k0 = first_key(p, (unsigned int)e, row + 1u); k0 < keys; k0 += AP_KEYS)
     {
         const unsigned int nk = min(AP_KEYS, keys - k0);
         if (tid < nk)
@@ -147,11 +214,14 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p
         }
         __syncthreads();
     }
-    T* out = (T*)p.out + (size_t)i * p.ldo + (size_t)kvh * G * p.vdim;
+    T* out = (T*)p.out + (size_t)i * p.ldo + (size_t)h0 * p.vdim;
     for (unsigned int j = tid; j < G * p.vdim; j += 128)
     {
-        float o = acc[j] / ml[3 * (j / p.vdim) + 1];
-        if (p.gate) { o *= sigmoid_f32(Elem<T>::get(x[p.g_off + (size_t)kvh * G * p.vdim + j])); }
+        const unsigned int g = j / p.vdim;
+        float l = ml[3 * g + 1];
+        if (p.sink != nullptr) { l += expf(p.sink[h0 + g] - ml[3 * g]); }
+        float o = acc[j] / l * head_factor<T>(p, i, h0 + g);
+        if (p.gate) { o *= sigmoid_f32(Elem<T>::get(x[p.g_off + (size_t)h0 * p.vdim + j])); }
         out[j] = Elem<T>::put(o);
     }
 }
@@ -159,6 +229,15 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const AttnParams p
 template <class T>
 static int attention_append(const AttnParams& p, unsigned int tokens, void* stream, bool pdl)
 {
+    if (p.q_norm || p.k_norm || p.rot_dims)
+    {
+        const unsigned int most = (p.H > p.Hkv ? p.H : p.Hkv) * p.dim;
+        unsigned int threads = 512;
+        while (threads > 64 && threads / 2 * 4 >= most) { threads /= 2; }
+        const DecoderDevice* dev = decoder_device();
+        if (!dev || (size_t)most * 4 > (size_t)dev->max_smem - 1024) { return -1; }
+        return launch_kernel("attention_prepare", attention_prepare_kernel<T>, dim3(tokens, 2), dim3(threads), (size_t)most * 4, stream, pdl, p);
+    }
     const unsigned int heads = p.H + 2 * p.Hkv;
     const unsigned int warps = heads < 8 ? heads : 8;
     return launch_kernel("attention_append", attention_append_kernel<T>, dim3(tokens, (heads + warps - 1) / warps), dim3(32 * warps), 0, stream, pdl, p);
@@ -167,10 +246,12 @@ static int attention_append(const AttnParams& p, unsigned int tokens, void* stre
 template <class T>
 static int attention_plain(const AttnParams& p, unsigned int tokens, void* stream, bool pdl)
 {
-    const size_t smem = (size_t)p.G * (p.dim + p.vdim + AP_KEYS + 3) * 4;
     const DecoderDevice* dev = decoder_device();
-    if (!dev || smem > (size_t)dev->max_smem) { return -1; }
-    return launch_kernel("attention_plain", attention_plain_kernel<T>, dim3(tokens, p.Hkv), dim3(128), smem, stream, pdl, p);
+    if (!dev) { return 1; }
+    const size_t head = (size_t)(p.dim + p.vdim + AP_KEYS + 3) * 4, fit = (size_t)dev->max_smem / head;
+    if (fit == 0) { return -1; }
+    const unsigned int GB = p.G < fit ? p.G : (unsigned int)fit;
+    return launch_kernel("attention_plain", attention_plain_kernel<T>, dim3(tokens, p.Hkv, (p.G + GB - 1) / GB), dim3(128), head * GB, stream, pdl, p, GB);
 }
 
 }    // namespace b200
@@ -192,7 +273,8 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     auto low = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) != 0; };
     if (low(a->qkvg) || low(a->k_cache) || low(a->v_cache) || low(a->work)) { return -1; }
     if ((dtype != DT_BF16 && dtype != DT_FLOAT) || a->H == 0 || a->Hkv == 0 || (a->H % a->Hkv) || a->dim == 0 || a->vdim == 0 || a->k_ld < a->dim
-        || a->v_ld < a->vdim || (a->k_ld % 8) || (a->v_ld % 8) || a->T_max == 0 || (a->v_mix && !a->v_first))
+        || a->v_ld < a->vdim || (a->k_ld % 8) || (a->v_ld % 8) || a->T_max == 0 || (a->v_mix && !a->v_first) || (a->rot_dims % 2) || a->rot_dims > a->dim
+        || (a->rot_dims && !a->rotary) || (!a->no_append && a->q_ld != 0 && a->q_ld != a->dim) || (a->q_ld != 0 && a->q_ld < a->dim))
     {
         return -1;
     }
@@ -209,6 +291,19 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     p.start = (const int*)b->start;
     p.n = (const int*)b->n;
     p.token_entry = (const int*)b->token_entry;
+    p.floor = (const int*)b->floor;
+    p.q_norm = (const float*)a->q_norm;
+    p.k_norm = (const float*)a->k_norm;
+    p.sink = (const float*)a->sink;
+    p.rotary = (const float2*)a->rotary;
+    p.head_gate = a->head_gate;
+    p.ld_gate = a->ld_gate;
+    p.rot_dims = a->rot_dims;
+    p.rot_interleaved = a->rot_interleaved;
+    p.window = a->window;
+    p.q_ld = a->q_ld ? a->q_ld : a->dim;
+    p.e0 = b->first_entry;
+    p.t0 = b->first_token;
     p.ld = a->ld;
     p.ldo = a->ldo;
     p.k_off = a->k_off;
@@ -241,12 +336,13 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
         else if (b->max_n * p.G <= 64 || b->max_n <= 4) { kernel = direct ? 4 : 1; }
         else { kernel = p.dim <= 128 && p.vdim <= 128 && a->slots != 0 ? 5 : 2; }
     }
-    if (kernel == 4 && b->max_n == 1)
+    const bool ready = a->no_append != 0, simple = !p.q_norm && !p.k_norm && p.rot_dims == 0;
+    if (kernel == 4 && b->max_n == 1 && !ready && simple)
     {
         p.fused = 1;
         return launch_attention_direct(p, b->entries, 1, b->max_len, st, pdl);
     }
-    int rc = dtype == DT_BF16 ? attention_append<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_append<float>(p, b->tokens, st, pdl);
+    int rc = ready ? 0 : dtype == DT_BF16 ? attention_append<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_append<float>(p, b->tokens, st, pdl);
     if (rc) { return rc; }
     switch (kernel)
     {

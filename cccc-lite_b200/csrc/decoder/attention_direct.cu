@@ -52,7 +52,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS, NR == 1 && DK + DV < 256 ? 3 : 
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    const unsigned int split = blockIdx.x, kvh = blockIdx.y % p.Hkv, rt = blockIdx.y / p.Hkv, e = blockIdx.z;
+    const unsigned int split = blockIdx.x, kvh = blockIdx.y % p.Hkv, rt = blockIdx.y / p.Hkv, e = p.e0 + blockIdx.z;
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e], r0 = rt * RT;
     const unsigned int rows = n * p.G;
     if (r0 >= rows) { return; }
@@ -62,9 +62,10 @@ __global__ void __launch_bounds__(32 * AS_WARPS, NR == 1 && DK + DV < 256 ? 3 : 
     __nv_bfloat16* V = (__nv_bfloat16*)p.v_cache + seq * p.v_ld;
     const unsigned int last_row = min(r0 + RT - 1u, rows - 1);
     const unsigned int T = min(pos + last_row / p.G + 1, p.T_max);
-    const unsigned int tiles = (T + 15) / 16, per = (tiles + p.splits - 1) / p.splits;
-    const unsigned int tile0 = min(split * per, tiles), tile1 = min(tile0 + per, tiles);
-    const unsigned int first_lim = pos + r0 / p.G + 1;
+    const unsigned int first_lim = pos + r0 / p.G + 1, last_low = first_key(p, e, pos + last_row / p.G + 1);
+    const unsigned int begin = first_key(p, e, first_lim) / 16;
+    const unsigned int tiles = (T + 15) / 16, per = (tiles - begin + p.splits - 1) / p.splits;
+    const unsigned int tile0 = min(begin + split * per, tiles), tile1 = min(tile0 + per, tiles);
 
     uint32_t k[2][KB][8], v[4][VR];
     auto load_k = [&](unsigned int tile) {
@@ -154,21 +155,22 @@ __global__ void __launch_bounds__(32 * AS_WARPS, NR == 1 && DK + DV < 256 ? 3 : 
 
     // queries: the same permuted element order as the keys
     uint32_t q[NR][KB][8];
-    unsigned int lim[NR];
+    unsigned int low[NR], lim[NR];
 #pragma unroll
     for (int h = 0; h < NR; h++)
     {
         const unsigned int r = r0 + g + 8 * h;
         const bool ok = r < rows;
         const unsigned int rr = ok ? r : 0;
-        const __nv_bfloat16* src = qkvg + (size_t)(start + rr / p.G) * p.ld + (size_t)(kvh * p.G + rr % p.G) * p.dim;
+        const __nv_bfloat16* src = qkvg + (size_t)(start + rr / p.G) * p.ld + (size_t)(kvh * p.G + rr % p.G) * p.q_ld;
+        low[h] = first_key(p, e, pos + r / p.G + 1);
         lim[h] = min(pos + r / p.G + 1, T);
         float f[KB][16], sq = 0.f;
 #pragma unroll
         for (int b = 0; b < KB; b++)
         {
             const unsigned int d0 = b * 64 + t * 16;
-            if ((p.dim % 16) == 0)
+            if ((p.dim % 16) == 0 && (p.q_ld % 16) == 0)
             {
                 uint32_t x[8];
                 ldg32(src + d0, x, ok && d0 < p.dim);
@@ -241,7 +243,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS, NR == 1 && DK + DV < 256 ? 3 : 
         }
         load_k(tile + AS_WARPS);
         prefetch(tile + 3 * AS_WARPS);
-        const bool masked = (tile + 1) * 16 > first_lim;
+        const bool masked = (tile + 1) * 16 > first_lim || tile * 16 < last_low;
         uint32_t hi[2 * NR], lo[2 * NR];    // [key half][row group]
 #pragma unroll
         for (int h = 0; h < NR; h++)
@@ -255,7 +257,8 @@ __global__ void __launch_bounds__(32 * AS_WARPS, NR == 1 && DK + DV < 256 ? 3 : 
                 {
                     float& z = s[i][2 * h + j];
                     z *= scale2;
-                    if (masked && tile * 16 + i * 8 + 2 * t + j >= lim[h]) { z = -INFINITY; }
+                    const unsigned int key = tile * 16 + i * 8 + 2 * t + j;
+                    if (masked && (key < low[h] || key >= lim[h])) { z = -INFINITY; }
                     mx = fmaxf(mx, z);
                 }
             }
@@ -340,7 +343,7 @@ int launch_attention_direct(const AttnParams& p0, unsigned int entries, unsigned
     const unsigned int nr = max_n * p.G <= 8 ? 1 : 2;
     p.row_tiles = (max_n * p.G + 8 * nr - 1) / (8 * nr);
     if ((unsigned long long)p.Hkv * p.row_tiles > 65535ull) { return -1; }
-    if (!plan_splits(p, entries, max_len, nr == 1 && (p.dim <= 64 || p.vdim <= 64) ? 3 : 2)) { return 1; }
+    if (!plan_splits(p, entries, max_n, max_len, nr == 1 && (p.dim <= 64 || p.vdim <= 64) ? 3 : 2)) { return 1; }
     if (p.dim <= 64) { return p.vdim <= 64 ? run_direct<64, 64>(p, entries, nr, stream, pdl) : run_direct<64, 128>(p, entries, nr, stream, pdl); }
     return p.vdim <= 64 ? run_direct<128, 64>(p, entries, nr, stream, pdl) : run_direct<128, 128>(p, entries, nr, stream, pdl);
 }

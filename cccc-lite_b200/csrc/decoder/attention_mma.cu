@@ -19,10 +19,11 @@ int attention_tiled_dk<256>(const AttnParams&, unsigned int, unsigned int, cudaS
 
 // How many splits a (sequence, kv head, row tile) is cut into: the least estimated time, a wave of CTAs taking a fixed part
 // and a part that goes with the keys of a split.
-bool plan_splits(AttnParams& p, unsigned int entries, unsigned int max_len, unsigned int ctas_per_sm)
+bool plan_splits(AttnParams& p, unsigned int entries, unsigned int max_n, unsigned int max_len, unsigned int ctas_per_sm)
 {
     const DecoderDevice* dev = decoder_device();
     if (!dev) { return false; }
+    if (p.window != 0 && max_len > p.window + max_n) { max_len = p.window + max_n; }
     p.splits = 1;
     const unsigned long long units = (unsigned long long)entries * p.Hkv * p.row_tiles, slots = (unsigned long long)dev->sm_count * ctas_per_sm;
     if (units > kAttnCounters) { return true; }
@@ -46,7 +47,7 @@ int launch_attention_split(const AttnParams& p0, unsigned int entries, unsigned 
     if (p.dim > 256 || p.vdim > 256 || entries > 65535u) { return -1; }
     p.row_tiles = (max_n * p.G + 15) / 16;
     if ((unsigned long long)p.Hkv * p.row_tiles > 65535ull) { return -1; }
-    if (!plan_splits(p, entries, max_len, 1)) { return 1; }
+    if (!plan_splits(p, entries, max_n, max_len, 1)) { return 1; }
     if (p.dim <= 64) { return attention_split_dk<64>(p, entries, stream, pdl); }
     if (p.dim <= 128) { return attention_split_dk<128>(p, entries, stream, pdl); }
     return attention_split_dk<256>(p, entries, stream, pdl);

@@ -57,7 +57,7 @@ struct RowTile
             const unsigned int r = r0 + (lane >> 2) + 8 * h;
             ok[h] = r < rows;
             const unsigned int rr = ok[h] ? r : 0;
-            src[h] = qkvg + (size_t)(start + rr / p.G) * p.ld + (size_t)(kvh * p.G + rr % p.G) * p.dim;
+            src[h] = qkvg + (size_t)(start + rr / p.G) * p.ld + (size_t)(kvh * p.G + rr % p.G) * p.q_ld;
             m[h] = -INFINITY;
             l[h] = 0.f;
         }
@@ -83,10 +83,10 @@ struct RowTile
         }
     }
 
-    // KT keys (a multiple of 16) at shared addresses ks / vs, the first being key k0 of the sequence; row h sees keys
-    // below lim[h].  scale2 = scale * log2(e).
+    // KT keys (a multiple of 16) at shared addresses ks / vs, the first being key k0 of the sequence; row h sees the keys
+    // from low[h] on and below lim[h].  scale2 = scale * log2(e).
     template <int KT>
-    __device__ __forceinline__ void step(uint32_t ks, uint32_t vs, unsigned int k0, const unsigned int (&lim)[2], bool masked, float scale2,
+    __device__ __forceinline__ void step(uint32_t ks, uint32_t vs, unsigned int k0, const unsigned int (&low)[2], const unsigned int (&lim)[2], bool masked, float scale2,
         unsigned int dim, unsigned int vdim, unsigned int lane)
     {
         constexpr int KS = (DK + 8) * 2, VS = (DV + 8) * 2;
@@ -122,7 +122,8 @@ struct RowTile
             for (int j = 0; j < 4; j++)
             {
                 s[i][j] *= scale2;
-                if (masked && k0 + i * 8 + (lane & 3) * 2 + (j & 1) >= lim[j >> 1]) { s[i][j] = -INFINITY; }
+                const unsigned int key = k0 + i * 8 + (lane & 3) * 2 + (j & 1);
+                if (masked && (key < low[j >> 1] || key >= lim[j >> 1])) { s[i][j] = -INFINITY; }
                 mx[j >> 1] = fmaxf(mx[j >> 1], s[i][j]);
             }
         }
@@ -192,6 +193,7 @@ __device__ __forceinline__ void attention_store(const AttnParams& p, const __nv_
 {
     const unsigned int col = (kvh * p.G + r % p.G) * p.vdim + d;
     const size_t tok = start + r / p.G;
+    v *= head_factor<__nv_bfloat16>(p, tok, kvh * p.G + r % p.G);
     if (p.gate) { v *= sigmoid_f32(__bfloat162float(qkvg[tok * p.ld + p.g_off + col])); }
     ((__nv_bfloat16*)p.out)[tok * p.ldo + col] = __float2bfloat16_rn(v);
 }
@@ -230,6 +232,7 @@ __device__ __forceinline__ void split_finish(const AttnParams& p, SplitMeet& mee
         }
 #pragma unroll
         for (int w = 0; w < AS_WARPS; w++) { meet.ml[w][tid][0] = c[w]; }
+        if (p.sink != nullptr && p.splits == 1) { l += exp2f(p.sink[kvh * p.G + (r0 + tid) % p.G] * 1.44269504088896341f - m); }
         meet.ml[0][tid][1] = m;
         meet.ml[1][tid][1] = l;
     }
@@ -250,7 +253,7 @@ __device__ __forceinline__ void split_finish(const AttnParams& p, SplitMeet& mee
         return;
     }
     const unsigned int vp = (p.vdim + 15) / 16 * 16, stride = 16 * (vp + 2), split = blockIdx.x;
-    const unsigned int unit = (e * p.row_tiles + rt) * p.Hkv + kvh;
+    const unsigned int unit = ((e - p.e0) * p.row_tiles + rt) * p.Hkv + kvh;
     float* all = p.partial + (size_t)unit * p.splits * stride;
     float* mine = all + (size_t)split * stride;
     for (unsigned int j = tid; j < live * p.vdim; j += 32 * AS_WARPS)
@@ -290,6 +293,7 @@ __device__ __forceinline__ void split_finish(const AttnParams& p, SplitMeet& mee
             l += c * __ldcg(all + (size_t)s * stride + 2 * r + 1);
         }
         l = warp_sum(l);
+        if (p.sink != nullptr) { l += exp2f(p.sink[kvh * p.G + (r0 + r) % p.G] * 1.44269504088896341f - m); }
         if (lane == 0) { meet.inv[r] = 1.0f / l; }
     }
     __syncthreads();
@@ -337,7 +341,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const At
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const unsigned int split = blockIdx.x, kvh = blockIdx.y % p.Hkv, rt = blockIdx.y / p.Hkv, e = blockIdx.z;
+    const unsigned int split = blockIdx.x, kvh = blockIdx.y % p.Hkv, rt = blockIdx.y / p.Hkv, e = p.e0 + blockIdx.z;
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e], r0 = rt * 16;
     const unsigned int rows = n * p.G;
     if (r0 >= rows) { return; }
@@ -348,15 +352,21 @@ __global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const At
     // keys that any row of the tile sees, cut into equal runs of whole tiles
     const unsigned int last_row = min(r0 + 15u, rows - 1);
     const unsigned int T = min(pos + last_row / p.G + 1, p.T_max);
-    const unsigned int tiles = (T + AS_KT - 1) / AS_KT, per = (tiles + p.splits - 1) / p.splits;
-    const unsigned int tile0 = min(split * per, tiles), tile1 = min(tile0 + per, tiles);
-    const unsigned int first_lim = pos + r0 / p.G + 1;    // every row sees the keys below
+    const unsigned int first_lim = pos + r0 / p.G + 1;    // no row ends before
+    const unsigned int begin = first_key(p, e, first_lim) / AS_KT, last_low = first_key(p, e, pos + last_row / p.G + 1);
+    const unsigned int tiles = (T + AS_KT - 1) / AS_KT, per = (tiles - begin + p.splits - 1) / p.splits;
+    const unsigned int tile0 = min(begin + split * per, tiles), tile1 = min(tile0 + per, tiles);
 
     RowTile<DK, DV> w;
     w.init(p, qkvg, start, n, kvh, r0, lane);
-    unsigned int lim[2];
+    unsigned int low[2], lim[2];
 #pragma unroll
-    for (int h = 0; h < 2; h++) { lim[h] = min(pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1, T); }
+    for (int h = 0; h < 2; h++)
+    {
+        const unsigned int end = pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1;
+        low[h] = first_key(p, e, end);
+        lim[h] = min(end, T);
+    }
 
     const uint32_t ring = smem_u32(as_raw) + warp * (ST * TB);
     auto fetch = [&](unsigned int i) {    // i-th tile of this warp
@@ -389,7 +399,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS) attention_split_kernel(const At
         cp_async_wait<ST - 1>();
         __syncwarp();
         const uint32_t ks = ring + (i % ST) * TB;
-        w.template step<AS_KT>(ks, ks + AS_KT * KS, tile * AS_KT, lim, (tile + 1) * AS_KT > first_lim, scale2, p.dim, p.vdim, lane);
+        w.template step<AS_KT>(ks, ks + AS_KT * KS, tile * AS_KT, low, lim, (tile + 1) * AS_KT > first_lim || tile * AS_KT < last_low, scale2, p.dim, p.vdim, lane);
         __syncwarp();
     }
     cp_async_wait<0>();
@@ -428,7 +438,7 @@ __global__ void __launch_bounds__(32 * AT_WARPS) attention_tiled_kernel(const At
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const unsigned int kvh = blockIdx.y, e = blockIdx.z;
+    const unsigned int kvh = blockIdx.y, e = p.e0 + blockIdx.z;
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e];
     const unsigned int rows = n * p.G, tiles_r = (rows + 16 * AT_WARPS - 1) / (16 * AT_WARPS);
     if (blockIdx.x >= tiles_r) { return; }
@@ -442,10 +452,16 @@ __global__ void __launch_bounds__(32 * AT_WARPS) attention_tiled_kernel(const At
 
     RowTile<DK, DV> w;
     w.init(p, qkvg, start, n, kvh, r0, lane);
-    unsigned int lim[2];
+    unsigned int low[2], lim[2];
 #pragma unroll
-    for (int h = 0; h < 2; h++) { lim[h] = min(pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1, T); }
+    for (int h = 0; h < 2; h++)
+    {
+        const unsigned int end = pos + (r0 + (lane >> 2) + 8 * h) / p.G + 1;
+        low[h] = first_key(p, e, end);
+        lim[h] = min(end, T);
+    }
     const unsigned int first_lim = pos + r0 / p.G + 1, last_lim = pos + (r0 + 15) / p.G + 1;
+    const unsigned int begin = first_key(p, e, pos + t0 / p.G + 1) / KT, first_low = first_key(p, e, first_lim), last_low = first_key(p, e, last_lim);
 
     const uint32_t ring = smem_u32(at_raw);
     auto fetch = [&](unsigned int tile) {
@@ -467,17 +483,17 @@ __global__ void __launch_bounds__(32 * AT_WARPS) attention_tiled_kernel(const At
         }
         cp_async_commit();
     };
-    fetch(0);
+    fetch(begin);
     const float scale2 = p.scale * 1.44269504088896341f;
-    for (unsigned int tile = 0; tile < tiles; tile++)
+    for (unsigned int tile = begin; tile < tiles; tile++)
     {
         fetch(tile + 1);
         cp_async_wait<1>();
         __syncthreads();
-        if (tile * KT < last_lim)
+        if (tile * KT < last_lim && (tile + 1) * KT > first_low)
         {
             const uint32_t ks = ring + (tile & 1u) * TB;
-            w.template step<KT>(ks, ks + KT * KS, tile * KT, lim, (tile + 1) * KT > first_lim, scale2, p.dim, p.vdim, lane);
+            w.template step<KT>(ks, ks + KT * KS, tile * KT, low, lim, (tile + 1) * KT > first_lim || tile * KT < last_low, scale2, p.dim, p.vdim, lane);
         }
         __syncthreads();
     }
@@ -489,7 +505,9 @@ __global__ void __launch_bounds__(32 * AT_WARPS) attention_tiled_kernel(const At
         const unsigned int r = r0 + gr + 8 * h;
         if (r < rows)
         {
-            const float inv = 1.0f / w.l[h];
+            float l = w.l[h];
+            if (p.sink != nullptr) { l += exp2f(p.sink[kvh * p.G + r % p.G] * 1.44269504088896341f - w.m[h]); }
+            const float inv = 1.0f / l;
 #pragma unroll
             for (int d = 0; d < DV / 8; d++)
             {

@@ -72,20 +72,21 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
     if (warp == 1) { tmem_alloc(tmem_slot, TA_TMEM); }
     grid_dependency_launch();
     grid_dependency_wait();
-    const unsigned int kvh = blockIdx.y, e = blockIdx.z;
+    const unsigned int kvh = blockIdx.y, e = p.e0 + blockIdx.z;
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e];
     const unsigned int rows = n * p.G, row_tiles = (rows + TA_ROWS - 1) / TA_ROWS;
     const bool idle = blockIdx.x >= row_tiles;    // a shorter entry than the longest one
     const unsigned int t0 = idle ? 0 : (row_tiles - 1 - blockIdx.x) * TA_ROWS;    // the rows that see the most keys first
     const unsigned int T = idle ? 0 : min(pos + min(t0 + TA_ROWS - 1u, rows - 1) / p.G + 1, p.T_max);
-    const unsigned int tiles = (T + TA_KT - 1) / TA_KT;
+    const unsigned int begin = idle ? 0 : first_key(p, e, pos + t0 / p.G + 1) / TA_KT;    // key tile the first row's window starts in
+    const unsigned int tiles = (T + TA_KT - 1) / TA_KT - begin;
     const unsigned int seq = ((unsigned int)p.slot[e] * p.Hkv + kvh) * p.T_max;
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
-    auto give_up = [&](unsigned int why) {
-        atomicMax(status, why);
+    auto give_up = [&](unsigned int role, unsigned int step) {
+        note_timeout(status, WAIT_ATTENTION_TILE, role, step);
         *abort_flag = 1;
     };
     auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             for (unsigned int i = 0; i < tiles && ok; i++)
             {
                 const unsigned int s = i & 1u;
-                const int y = (int)(seq + i * TA_KT);
+                const int y = (int)(seq + (begin + i) * TA_KT);
                 if (i >= 2 && !wait(k_empty + s, (i >> 1) - 1)) { ok = false; break; }
                 mbar_expect_tx(k_full + s, KBY);
 #pragma unroll
@@ -115,7 +116,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             }
             if (!ok)
             {
-                give_up((unsigned int)ST_TIMEOUT_EMPTY);
+                give_up(0, k_issued);
                 // wait (bounded) for the copies in flight before the CTA may leave
                 auto drain = [&](uint64_t* full, unsigned int issued) {
                     for (unsigned int j = issued > 2 ? issued - 2 : 0; j < issued; j++)
@@ -154,9 +155,11 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             __syncwarp();
             return true;
         };
+        unsigned int at = 0;    // product the lane is at
         bool ok = tiles == 0 || (wait(q_ready, 0) && scores(0) && (tiles == 1 || scores(1)));
         for (unsigned int i = 0; i < tiles && ok; i++)
         {
+            at = i + 1;
             ok = wait(p_ready + (i & 1u), i >> 1);
             if (!ok) { break; }
             tc_fence_after();
@@ -183,7 +186,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
         }
         if (!ok)
         {
-            if (lane == 0) { give_up((unsigned int)ST_TIMEOUT_FULL); }
+            if (lane == 0) { give_up(1, at); }
             if (elect_one()) { umma_commit(pv_done); }    // completes once the MMAs in flight have stopped reading shared memory
             __syncwarp();
         }
@@ -196,8 +199,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
         const unsigned int tok = start + (real ? r / p.G : 0), head = kvh * p.G + (real ? r % p.G : 0);
         const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg + (size_t)tok * p.ld;
         {
-            const __nv_bfloat16* src = x + (size_t)head * p.dim;
-            const bool vec = (p.dim % 8) == 0;
+            const __nv_bfloat16* src = x + (size_t)head * p.q_ld;
+            const bool vec = (p.dim % 8) == 0 && (p.q_ld % 8) == 0;
             const uint32_t flip = p.scale < 0.f ? 0x80008000u : 0u;    // the maximum is taken before scaling
 #pragma unroll
             for (int c = 0; c < DK / 8; c++)
@@ -224,7 +227,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             __syncwarp();
             if (lane == 0) { mbar_arrive(q_ready); }
         }
-        const unsigned int lim = min(pos + r / p.G + 1, T), first_lim = pos + t0 / p.G + 1;
+        const unsigned int low = first_key(p, e, pos + r / p.G + 1), lim = min(pos + r / p.G + 1, T);
+        const unsigned int first_lim = pos + t0 / p.G + 1, last_low = first_key(p, e, pos + (t0 + TA_ROWS - 1) / p.G + 1);
         const float scale2 = fmaxf(fabsf(p.scale) * 1.44269504088896341f, 1e-30f);    // 0 times a masked -inf would be no number
         float m = -INFINITY, l = 0.f;
         bool ok = true;
@@ -238,12 +242,13 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             tmem_ld_32x32(place, *reinterpret_cast<uint32_t(*)[32]>(s));
             tmem_ld_32x32(place + 32, *reinterpret_cast<uint32_t(*)[32]>(s + 32));
             tmem_ld_wait();
-            if ((i + 1) * TA_KT > first_lim)
+            const unsigned int key0 = (begin + i) * TA_KT;
+            if (key0 + TA_KT > first_lim || key0 < last_low)
             {
 #pragma unroll
                 for (int j = 0; j < TA_KT; j++)
                 {
-                    if (i * TA_KT + j >= lim) { s[j] = 0xFF800000u; }    // -inf
+                    if (key0 + j < low || key0 + j >= lim) { s[j] = 0xFF800000u; }    // -inf
                 }
             }
             float mx[4] = { -INFINITY, -INFINITY, -INFINITY, -INFINITY };    // four maxima in flight
@@ -257,12 +262,13 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                 m = top;
                 l *= c;
             }
+            const float base = m == -INFINITY ? 0.f : m;    // a window may start after this tile
             uint32_t hi[TA_KT / 2], lo[TA_KT / 2];
             float sum[2] = { 0.f, 0.f };
 #pragma unroll
             for (int j = 0; j < TA_KT / 2; j++)
             {
-                const float a = exp2_f32(fmaf(__uint_as_float(s[2 * j]), scale2, -m)), b = exp2_f32(fmaf(__uint_as_float(s[2 * j + 1]), scale2, -m));
+                const float a = exp2_f32(fmaf(__uint_as_float(s[2 * j]), scale2, -base)), b = exp2_f32(fmaf(__uint_as_float(s[2 * j + 1]), scale2, -base));
                 sum[0] += a;
                 sum[1] += b;
                 hi[j] = pack_bf16x2(a, b);
@@ -302,7 +308,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
         if (ok)
         {
             tc_fence_after();
-            const float inv = 1.0f / l;
+            if (p.sink != nullptr) { l += exp2_f32(fmaf(p.sink[head], 1.44269504088896341f, -m)); }
+            const float inv = head_factor<__nv_bfloat16>(p, tok, head) / l;
             const __nv_bfloat16* gate = x + p.g_off + (size_t)head * p.vdim;
             __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)tok * p.ldo + (size_t)head * p.vdim;
             const bool vec = (p.vdim % 8) == 0 && (p.g_off % 8) == 0;
@@ -355,7 +362,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                 __syncwarp();
             }
         }
-        else if (lane == 0) { give_up((unsigned int)ST_TIMEOUT_FULL); }
+        else if (lane == 0) { give_up(2 + quarter, tiles); }
     }
     tc_fence_before();
     __syncthreads();

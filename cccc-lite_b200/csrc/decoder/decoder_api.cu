@@ -68,7 +68,7 @@ C_EXPORT int cuda_b200_decoder_check(const char* label)
     unsigned int st = 0;
     if (w && cudaMemcpy(&st, w, sizeof(st), cudaMemcpyDeviceToHost) == cudaSuccess && st != 0)
     {
-        fprintf(stderr, "%s: a bounded wait ran out (status %u)\n", label ? label : "decoder", st);
+        fprintf(stderr, "%s: a bounded wait ran out (kernel %u, role %u, step %u)\n", label ? label : "decoder", st >> 28, (st >> 24) & 15u, st & 0xFFFFFFu);
         cudaMemset(w, 0, sizeof(st));
         return 1;
     }

@@ -11,6 +11,17 @@ namespace b200
 
 // The status word of this library's bounded waits (device memory, allocated once per device); nullptr on failure.
 unsigned int* decoder_status_word();
+// What the status word says of the first wait that ran out: which kernel, which of its roles, at which of the role's steps.
+enum : unsigned int
+{
+    WAIT_LINEAR_TILE = 1,
+    WAIT_ATTENTION_TILE = 2
+};
+__device__ __forceinline__ void note_timeout(unsigned int* status, unsigned int kernel, unsigned int role, unsigned int step)
+{
+    atomicCAS(status, 0u, kernel << 28 | role << 24 | (step & 0xFFFFFFu));
+}
+
 struct DecoderDevice
 {
     int sm_count = 0, max_smem = 0;
@@ -62,8 +73,12 @@ __device__ __forceinline__ float warp_sum(float v)
     return v;
 }
 
+__host__ __device__ __forceinline__ bool activation_gated(int activation) { return activation == B200_ACT_SILU_GATE || activation == B200_ACT_GELU_GATE; }
+
+__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
 // The part of a linear's epilogue that does not depend on where the result goes.
-__device__ __forceinline__ float linear_activation(int activation, float a, float up)
+__device__ __forceinline__ float linear_activation(int activation, float a, float up, float cap)
 {
     if (activation == B200_ACT_RELU2)
     {
@@ -71,7 +86,21 @@ __device__ __forceinline__ float linear_activation(int activation, float a, floa
         return a * a;
     }
     if (activation == B200_ACT_SILU_GATE) { return a * sigmoid_f32(a) * up; }
+    if (activation == B200_ACT_GELU_GATE) { return gelu_tanh_f32(a) * up; }
+    if (activation == B200_ACT_SOFTCAP) { return cap * tanhf(a / cap); }
     return a;
+}
+
+// Element d of a head after its first `dims` elements have been turned pair by pair (element i goes with i + dims / 2, or,
+// interleaved, 2i with 2i + 1); rot: (cos, sin) of the position's angles.
+__device__ __forceinline__ float rotated(const float* head, unsigned int d, unsigned int dims, bool interleaved, const float2* rot)
+{
+    if (d >= dims) { return head[d]; }
+    const unsigned int half = dims / 2, i = interleaved ? d / 2 : d % half;
+    const bool second = interleaved ? (d & 1u) != 0 : d >= half;
+    const float2 cs = rot[i];
+    const float u = head[interleaved ? 2 * i : i], v = head[interleaved ? 2 * i + 1 : i + half];
+    return second ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
 }
 
 template <class K, class... Args>

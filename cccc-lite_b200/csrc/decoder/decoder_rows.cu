@@ -1,5 +1,5 @@
-// Row operations of a decoder layer: scaled embedding, branch addition + norm, routing to experts, row gather, greedy
-// choice over float logits.
+// Row operations of a decoder layer: scaled embedding, branch addition + norm, table of rotations, routing to experts, row
+// gather, greedy choice over float logits.
 #include "decoder_common.cuh"
 
 #include <cfloat>
@@ -50,14 +50,22 @@ struct NormParams
     const int* slot_row;
     const float* slot_weight;
     const int* rows;
-    unsigned int width, ldx, ldo, ldy, slots;
+    const float *branch, *branch_weight;
+    unsigned int width, ldx, ldo, ldy, slots, ldb;
     int kind;
     float eps;
 };
 
 // One CTA per row.  The row lives in shared memory as floats; quads of columns per thread (row strides are multiples
 // of four elements, so the last quad may cover padding columns, which take no part in the sums and are not stored).
-template <class T, bool SLOTS>
+enum
+{
+    ADD_NOTHING,
+    ADD_SLOTS,     // experts' outputs
+    ADD_BRANCH     // a branch that is normalised itself
+};
+
+template <class T, int ADD>
 __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormParams p)
 {
     extern __shared__ __align__(16) float nr_row[];
@@ -68,12 +76,48 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormParams p)
     float* x = p.X + (size_t)r * p.ldx;
     const unsigned int quads = (p.width + 3) / 4;
     const T* Y = (const T*)p.Y;
+    float bmean = 0.f, binv = 0.f;
+    if (ADD == ADD_BRANCH)
+    {
+        const float* b = p.branch + (size_t)r * p.ldb;
+        auto live = [&](unsigned int i, int j) { return 4 * i + j < p.width; };
+        float s = 0.f;
+#pragma unroll 4
+        for (unsigned int i = threadIdx.x; i < quads; i += blockDim.x)
+        {
+            const float4 v = load4(b + 4 * i);
+            *reinterpret_cast<float4*>(nr_row + 4 * i) = v;
+            s += v.x + (live(i, 1) ? v.y : 0.f) + (live(i, 2) ? v.z : 0.f) + (live(i, 3) ? v.w : 0.f);
+        }
+        if (p.kind == B200_NORM_LAYER) { bmean = block_sum(s, part) / (float)p.width; }
+        s = 0.f;
+        for (unsigned int i = threadIdx.x; i < quads; i += blockDim.x)
+        {
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                const float v = nr_row[4 * i + j] - bmean;
+                if (live(i, j)) { s += v * v; }
+            }
+        }
+        binv = 1.0f / sqrtf(block_sum(s, part) / (float)p.width + p.eps);
+    }
     float sum = 0.f;
 #pragma unroll 4
     for (unsigned int i = threadIdx.x; i < quads; i += blockDim.x)
     {
         float4 v = load4(x + 4 * i);
-        if (SLOTS)
+        if (ADD == ADD_BRANCH)
+        {
+            const float4 b = *reinterpret_cast<float4*>(nr_row + 4 * i);
+            auto w = [&](int j) { return p.branch_weight && 4 * i + j < p.width ? p.branch_weight[4 * i + j] : 1.f; };
+            v.x += (b.x - bmean) * binv * w(0);
+            v.y += (b.y - bmean) * binv * w(1);
+            v.z += (b.z - bmean) * binv * w(2);
+            v.w += (b.w - bmean) * binv * w(3);
+            store4(x + 4 * i, v);
+        }
+        if (ADD == ADD_SLOTS)
         {
 #pragma unroll 4
             for (unsigned int s = 0; s < p.slots; s++)
@@ -128,6 +172,16 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormParams p)
         }
         if (whole) { store4(out + 4 * i, make_float4(a[0], a[1], a[2], a[3])); }
     }
+}
+
+// ---- rotations -------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) rotary_table_kernel(float2* __restrict__ table, unsigned int pairs, unsigned int dims, double base)
+{
+    const unsigned int i = blockIdx.y * blockDim.x + threadIdx.x;
+    if (i >= pairs) { return; }
+    double s, c;
+    sincos((double)blockIdx.x * pow(base, -2.0 * (double)i / (double)dims), &s, &c);
+    table[(size_t)blockIdx.x * pairs + i] = make_float2((float)c, (float)s);
 }
 
 // ---- routing ---------------------------------------------------------------------------------------
@@ -427,12 +481,22 @@ C_EXPORT int cuda_b200_embed_f32(int dtype, const void* ids, const void* table, 
     return -1;
 }
 
+C_EXPORT int cuda_b200_rotary_table(void* table, unsigned int rows, unsigned int dims, double base, void* stream)
+{
+    if (rows == 0 || dims == 0) { return 0; }
+    if (!table || (dims % 2) || !(base > 0.0)) { return -1; }
+    const unsigned int pairs = dims / 2, threads = pairs < 256 ? (pairs + 31) / 32 * 32 : 256;
+    return launch_kernel("rotary_table", rotary_table_kernel, dim3(rows, (pairs + threads - 1) / threads), dim3(threads), 0, stream, false, (float2*)table, pairs,
+        dims, base);
+}
+
 C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* stream, unsigned int flags)
 {
     if (!a || a->n == 0) { return a ? 0 : -1; }
     if (!a->X || a->width == 0 || (a->ldx % 4) || (a->out && (a->ldo % 4)) || (dtype != DT_BF16 && dtype != DT_FLOAT)) { return -1; }
     if (a->kind != B200_NORM_RMS && a->kind != B200_NORM_LAYER) { return -1; }
     if (a->slots && (!a->Y || !a->slot_row || !a->slot_weight || a->rows || (a->ldy % 4))) { return -1; }
+    if (a->branch && (a->slots || a->rows || (a->ldb % 4) || a->ldb < a->width)) { return -1; }
     const DecoderDevice* dev = decoder_device();
     const size_t smem = ((size_t)a->width + 3) / 4 * 16;
     if (!dev || smem > (size_t)dev->max_smem - 1024) { return -1; }
@@ -445,6 +509,9 @@ C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* strea
     p.slot_row = (const int*)a->slot_row;
     p.slot_weight = (const float*)a->slot_weight;
     p.rows = (const int*)a->rows;
+    p.branch = (const float*)a->branch;
+    p.branch_weight = (const float*)a->branch_weight;
+    p.ldb = a->ldb;
     p.width = a->width;
     p.ldx = a->ldx;
     p.ldo = a->ldo;
@@ -457,8 +524,12 @@ C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* strea
     while (threads > 64 && threads / 2 * 4 >= a->width) { threads /= 2; }
     const bool pdl = (flags & 1u) != 0;
     auto run = [&](auto kernel) { return launch_kernel("norm_rows", kernel, dim3(a->n), dim3(threads), smem, stream, pdl, p); };
-    if (dtype == DT_BF16) { return p.slots ? run(norm_rows_kernel<__nv_bfloat16, true>) : run(norm_rows_kernel<__nv_bfloat16, false>); }
-    return p.slots ? run(norm_rows_kernel<float, true>) : run(norm_rows_kernel<float, false>);
+    auto pick = [&](auto zero) {
+        using T = decltype(zero);
+        if (p.branch) { return run(norm_rows_kernel<T, ADD_BRANCH>); }
+        return p.slots ? run(norm_rows_kernel<T, ADD_SLOTS>) : run(norm_rows_kernel<T, ADD_NOTHING>);
+    };
+    return dtype == DT_BF16 ? pick(__nv_bfloat16()) : pick(0.f);
 }
 
 C_EXPORT int cuda_b200_route_rows(const cuda_b200_route* a, void* stream, unsigned int flags)

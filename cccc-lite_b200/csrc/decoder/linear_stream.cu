@@ -40,7 +40,7 @@ __global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_
     const LinearMember& m = L.m[mi];
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const unsigned int b = blockIdx.x - m.block0;
-    const bool gated = m.activation == B200_ACT_SILU_GATE;
+    const bool gated = activation_gated(m.activation);
     const unsigned int F = gated ? R / 2 : R;    // output features of a warp
     const unsigned int wk = warp % WK, wf = warp / WK;
     const unsigned int fb = b % m.fblocks, slot = b / m.fblocks;
@@ -62,7 +62,9 @@ __global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_
         count = (unsigned int)m.group_offset[group + 1] - row0;
         if (count == 0) { return; }
     }
+    if (m.blocks > 1) { group = slot; }
     const __nv_bfloat16* W = (const __nv_bfloat16*)m.W + (size_t)group * m.group_rows * m.ldw;
+    const unsigned int xcol = m.blocks > 1 ? group * m.x_step : 0u, ycol = m.blocks > 1 ? group * m.y_step : 0u;
     const __nv_bfloat16* wr[RT][2];
 #pragma unroll
     for (int r = 0; r < RT; r++)
@@ -110,7 +112,7 @@ __global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_
             live[nt] = n < count;
             unsigned int r = row0 + (live[nt] ? n : 0u);
             if (m.x_row != nullptr) { r = (unsigned int)m.x_row[r]; }
-            xr[nt] = (const __nv_bfloat16*)m.X + (size_t)r * m.ldx + t * 16;
+            xr[nt] = (const __nv_bfloat16*)m.X + (size_t)r * m.ldx + xcol + t * 16;
         }
         float acc[RT][NT][4];
 #pragma unroll
@@ -200,7 +202,8 @@ __global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_
 #pragma unroll
                 for (int w = 0; w < WK; w++) { up += red[w0 + w][n][16 + fl]; }
             }
-            linear_store(m, row0 + n0 + n, fc + f, linear_activation(m.activation, m.alpha * v, m.alpha * up));
+            const float y = linear_activation(m.activation, m.alpha * v, m.alpha * up, m.cap);
+            linear_store(m, row0 + n0 + n, ycol + fc + f, y * linear_row_factor<__nv_bfloat16>(m, row0 + n0 + n, group));
         }
     }
 }
@@ -224,7 +227,9 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearMember m)
     }
     const unsigned int f0 = blockIdx.x * LF_F, r0 = blockIdx.y * LF_R;
     if (r0 >= count) { return; }
+    if (m.blocks > 1) { group = blockIdx.z; }
     const float* W = (const float*)m.W + (size_t)group * m.group_rows * m.ldw;
+    const unsigned int xcol = m.blocks > 1 ? group * m.x_step : 0u, ycol = m.blocks > 1 ? group * m.y_step : 0u;
     const unsigned int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;    // 16 x 16 threads: 4 features x 2 rows each
     float acc[GATED ? 2 : 1][2][4] = {};
     for (unsigned int k0 = 0; k0 < m.K; k0 += LF_K)
@@ -244,7 +249,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearMember m)
             {
                 unsigned int xr = row0 + r0 + r;
                 if (m.x_row != nullptr) { xr = (unsigned int)m.x_row[xr]; }
-                v = ((const float*)m.X)[(size_t)xr * m.ldx + k0 + k];
+                v = ((const float*)m.X)[(size_t)xr * m.ldx + xcol + k0 + k];
             }
             xs[k][r] = v;
         }
@@ -275,7 +280,8 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearMember m)
             const unsigned int r = r0 + ty + 16 * i, f = f0 + tx + 16 * j;
             if (r < count && f < m.N)
             {
-                linear_store(m, row0 + r, f, linear_activation(m.activation, m.alpha * acc[0][i][j], GATED ? m.alpha * acc[GATED ? 1 : 0][i][j] : 0.f));
+                const float y = linear_activation(m.activation, m.alpha * acc[0][i][j], GATED ? m.alpha * acc[GATED ? 1 : 0][i][j] : 0.f, m.cap);
+                linear_store(m, row0 + r, ycol + f, y * linear_row_factor<float>(m, row0 + r, group));
             }
         }
     }
@@ -288,7 +294,7 @@ static int launch_stream_wk(LinearLaunch& L, cudaStream_t st, bool pdl)
     for (unsigned int j = 0; j < L.count; j++)
     {
         LinearMember& m = L.m[j];
-        const unsigned int F = (m.activation == B200_ACT_SILU_GATE ? 8 * RT : 16 * RT) * (LS_WARPS / WK);
+        const unsigned int F = (activation_gated(m.activation) ? 8 * RT : 16 * RT) * (LS_WARPS / WK);
         m.fblocks = (m.N + F - 1) / F;
         m.block0 = blocks;
         blocks += m.fblocks * m.slots;
@@ -322,12 +328,14 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         if (a.rows == 0 || a.N == 0) { continue; }
         auto bad_align = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 31u) != 0; };
         if (!a.W || !a.X || !a.Y || a.K == 0 || bad_align(a.W) || bad_align(a.X)) { return -1; }
-        if (a.activation < B200_ACT_NONE || a.activation > B200_ACT_SILU_GATE || (a.out_type != DT_FLOAT && a.out_type != DT_BF16)) { return -1; }
+        if (a.activation < B200_ACT_NONE || a.activation > B200_ACT_SOFTCAP || (a.out_type != DT_FLOAT && a.out_type != DT_BF16)) { return -1; }
         if (a.accumulate && a.out_type != DT_FLOAT) { return -1; }
         if (dtype == DT_FLOAT && a.out_type != DT_FLOAT) { return -1; }
         const unsigned int kp = (a.K + 63) / 64 * 64;
         if ((a.ldw % 64) || (a.ldx % 64) || a.ldw < kp || a.ldx < kp) { return -1; }
-        if (a.group_offset && (a.groups == 0 || a.group_max == 0)) { return -1; }
+        if (a.group_offset && (a.groups == 0 || a.group_max == 0 || a.blocks > 1)) { return -1; }
+        if (a.blocks > 1 && ((a.x_step % 8) || a.x_row)) { return -1; }
+        if (a.activation == B200_ACT_SOFTCAP && !(a.cap > 0.f)) { return -1; }
         LinearMember& m = L.m[L.count++];
         m.W = a.W;
         m.X = a.X;
@@ -345,7 +353,13 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         m.groups = a.group_offset ? a.groups : 1;
         m.group_rows = a.group_rows;
         m.up_row = a.up_row;
-        m.slots = a.group_offset ? (a.active ? a.active_cap : a.groups) : 1;
+        m.blocks = a.blocks > 1 ? a.blocks : 1;
+        m.x_step = a.x_step;
+        m.y_step = a.y_step;
+        m.head_gate = a.head_gate;
+        m.ld_gate = a.ld_gate;
+        m.cap = a.cap;
+        m.slots = a.group_offset ? (a.active ? a.active_cap : a.groups) : m.blocks;
         m.out_type = a.out_type;
         m.activation = a.activation;
         m.accumulate = a.accumulate;
@@ -364,16 +378,16 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         {
             const LinearMember& m = L.m[j];
             const unsigned int rows = m.group_offset ? (most < m.rows ? most : m.rows) : m.rows;
-            const dim3 grid((m.N + LF_F - 1) / LF_F, (rows + LF_R - 1) / LF_R, m.groups);
+            const dim3 grid((m.N + LF_F - 1) / LF_F, (rows + LF_R - 1) / LF_R, m.blocks > 1 ? m.blocks : m.groups);
             if (grid.y > 65535u || grid.z > 65535u) { return -1; }
-            const int rc = m.activation == B200_ACT_SILU_GATE ? launch_kernel("linear_f32", linear_f32_kernel<true>, grid, dim3(256), 0, st, pdl, m)
+            const int rc = activation_gated(m.activation) ? launch_kernel("linear_f32", linear_f32_kernel<true>, grid, dim3(256), 0, st, pdl, m)
                                                               : launch_kernel("linear_f32", linear_f32_kernel<false>, grid, dim3(256), 0, st, pdl, m);
             if (rc) { return rc; }
         }
         return 0;
     }
     // a dense linear of 17 to 32 rows with a tile for every SM (a head over a vocabulary): tiles stream weights as fast
-    if (kernel == 0 && L.count == 1 && most > 16 && !L.m[0].group_offset && !L.m[0].x_row)
+    if (kernel == 0 && L.count == 1 && most > 16 && L.m[0].blocks == 1 && !L.m[0].group_offset && !L.m[0].x_row)
     {
         const DecoderDevice* dev = decoder_device();
         if (dev && L.m[0].N >= 256u * (unsigned int)dev->sm_count) { kernel = 2; }
@@ -399,7 +413,7 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
                 if (width < 32 ? rows > width : false) { continue; }
                 if (width > 8 && rows <= width / 2) { continue; }
                 part.m[part.count++] = m;
-                gated = gated || m.activation == B200_ACT_SILU_GATE;
+                gated = gated || activation_gated(m.activation);
             }
             if (part.count == 0) { continue; }
             int rc;

@@ -26,10 +26,11 @@ __host__ __device__ constexpr int lt_header(void) { return (LT_HEADER + 1023) / 
 __host__ __device__ constexpr int lt_smem(int bn) { return lt_header() + lt_stages(bn) * lt_stage_bytes(bn) + 1024; }
 
 // 32 result columns of one row
-__device__ __forceinline__ void store_row32(const LinearMember& m, unsigned int row, unsigned int f, const float (&v)[32], bool vec)
+__device__ __forceinline__ void store_row32(const LinearMember& m, unsigned int row, unsigned int block, unsigned int f, const float (&v)[32], bool vec)
 {
-    const float s = m.row_scale != nullptr ? m.row_scale[row] : 1.f;
-    const size_t i = (size_t)row * m.ldy + f;
+    const float s = linear_row_factor<__nv_bfloat16>(m, row, block);
+    const unsigned int ycol = block * m.y_step;
+    const size_t i = (size_t)row * m.ldy + ycol + f;
     if (f + 32 <= m.N && vec)
     {
         if (m.out_type == DT_BF16)
@@ -65,7 +66,7 @@ __device__ __forceinline__ void store_row32(const LinearMember& m, unsigned int 
 #pragma unroll
     for (int j = 0; j < 32; j++)
     {
-        if (f + j < m.N) { linear_store(m, row, f + j, v[j]); }
+        if (f + j < m.N) { linear_store(m, row, ycol + f + j, s * v[j]); }
     }
 }
 
@@ -88,7 +89,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
     unsigned char* stages = smem + lt_header();
 
     const unsigned int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const bool gated = m.activation == B200_ACT_SILU_GATE;
+    const bool gated = activation_gated(m.activation);
     const unsigned int FT = gated ? BN / 2 : BN;    // result features per tile
     const unsigned int kblocks = (m.K + LT_BK - 1) / LT_BK;
 
@@ -134,11 +135,13 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
     const unsigned int row_tiles = m.group_offset != nullptr ? (unsigned int)first_tile[m.groups] : (m.rows + LT_M - 1) / LT_M;
-    const unsigned int total = row_tiles * ftiles;
+    const unsigned int total = row_tiles * ftiles * m.blocks;
 
-    // tile -> first weight row, first feature, first X / Y row, live rows.  Row tiles run fastest inside a group.
-    auto coords = [&](unsigned int t, unsigned int& w0, unsigned int& f0, unsigned int& r0, unsigned int& live) {
-        unsigned int g = 0, tiles = row_tiles, rel = t, base = 0, rows = m.rows;
+    // tile -> block, first weight row, first feature, first X / Y row, live rows.  Row tiles run fastest inside a group.
+    auto coords = [&](unsigned int t, unsigned int& block, unsigned int& w0, unsigned int& f0, unsigned int& r0, unsigned int& live) {
+        block = m.blocks > 1 ? t / (row_tiles * ftiles) : 0u;
+        t -= block * row_tiles * ftiles;
+        unsigned int g = block, tiles = row_tiles, rel = t, base = 0, rows = m.rows;
         if (m.group_offset != nullptr)
         {
             unsigned int lo = 0, hi = m.groups;    // the last group whose tiles start at or before t
@@ -169,8 +172,9 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
             unsigned int it = 0;
             for (unsigned int t = blockIdx.x; t < total && ok; t += gridDim.x)
             {
-                unsigned int w0, f0, r0, live;
-                coords(t, w0, f0, r0, live);
+                unsigned int block, w0, f0, r0, live;
+                coords(t, block, w0, f0, r0, live);
+                const unsigned int xcol = block * m.x_step;
                 const unsigned int w1 = gated ? w0 + m.up_row : w0 + BN / 2;
                 for (unsigned int kb = 0; kb < kblocks; kb++, it++)
                 {
@@ -178,13 +182,13 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
                     if (it >= NS && (*abort_flag != 0 || !mbar_wait_bounded(empty + s, ((it / NS) - 1u) & 1u)))
                     {
                         ok = false;
-                        atomicMax(status, (unsigned int)ST_TIMEOUT_EMPTY);
+                        note_timeout(status, WAIT_LINEAR_TILE, 0, it);
                         *abort_flag = 1;
                         break;
                     }
                     unsigned char* st = stages + s * STAGE;
                     mbar_expect_tx(full + s, STAGE);
-                    tma_load_2d(st, &tmX, (int)(kb * LT_BK), (int)r0, full + s);
+                    tma_load_2d(st, &tmX, (int)(xcol + kb * LT_BK), (int)r0, full + s);
                     tma_load_2d(st + LT_X_BYTES, &tmW, (int)(kb * LT_BK), (int)w0, full + s);
                     tma_load_2d(st + LT_X_BYTES + BN * LT_BK, &tmW, (int)(kb * LT_BK), (int)w1, full + s);
                     mbar_arrive(full + s);
@@ -239,7 +243,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
         {
             if (lane == 0)
             {
-                atomicMax(status, (unsigned int)ST_TIMEOUT_FULL);
+                note_timeout(status, WAIT_LINEAR_TILE, 1, it);
                 *abort_flag = 1;
             }
             // the barrier completes once the MMAs in flight have stopped reading shared memory
@@ -254,8 +258,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
         unsigned int n = 0;
         for (unsigned int t = blockIdx.x; t < total && ok; t += gridDim.x, n++)
         {
-            unsigned int w0, f0, r0, live;
-            coords(t, w0, f0, r0, live);
+            unsigned int block, w0, f0, r0, live;
+            coords(t, block, w0, f0, r0, live);
             const unsigned int a = n & 1u;
             ok = *abort_flag == 0 && mbar_wait_bounded(acc_full + a, (n >> 1) & 1u);
             ok = __all_sync(0xFFFFFFFFu, ok) && *abort_flag == 0;
@@ -264,7 +268,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
             {
                 if (lane == 0)
                 {
-                    atomicMax(status, (unsigned int)ST_TIMEOUT_FULL);
+                    note_timeout(status, WAIT_LINEAR_TILE, 2, n);
                     *abort_flag = 1;
                 }
                 break;
@@ -287,15 +291,15 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
 #pragma unroll
                     for (int j = 0; j < 32; j++)
                     {
-                        v[j] = linear_activation(B200_ACT_SILU_GATE, m.alpha * __uint_as_float(r[j]), m.alpha * __uint_as_float(u[j]));
+                        v[j] = linear_activation(m.activation, m.alpha * __uint_as_float(r[j]), m.alpha * __uint_as_float(u[j]), m.cap);
                     }
                 }
                 else
                 {
 #pragma unroll
-                    for (int j = 0; j < 32; j++) { v[j] = linear_activation(m.activation, m.alpha * __uint_as_float(r[j]), 0.f); }
+                    for (int j = 0; j < 32; j++) { v[j] = linear_activation(m.activation, m.alpha * __uint_as_float(r[j]), 0.f, m.cap); }
                 }
-                if (rl < live) { store_row32(m, r0 + rl, f0 + c, v, vec != 0); }
+                if (rl < live) { store_row32(m, r0 + rl, block, f0 + c, v, vec != 0); }
                 __syncwarp();
             }
             tc_fence_before();
@@ -313,19 +317,19 @@ static int launch_tile(const LinearMember& m, const DecoderDevice& dev, cudaStre
 {
     unsigned int* status = decoder_status_word();
     if (!status) { return 1; }
-    const bool gated = m.activation == B200_ACT_SILU_GATE;
+    const bool gated = activation_gated(m.activation);
     const unsigned int FT = gated ? BN / 2 : BN;
     const unsigned int ftiles = (m.N + FT - 1) / FT;
     // weight rows of all groups; rows past the end read as zeros, rows of a neighbouring group give results nobody stores
-    const unsigned long long wrows = (unsigned long long)(m.groups - 1) * m.group_rows + (gated ? m.up_row : 0u) + m.N;
+    const unsigned long long wrows = (unsigned long long)((m.blocks > 1 ? m.blocks : m.groups) - 1) * m.group_rows + (gated ? m.up_row : 0u) + m.N;
     CUtensorMap tx, tw;
-    if (!make_map_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, m.X, m.K, m.rows, (unsigned long long)m.ldx * 2, LT_BK, LT_M, true)
+    if (!make_map_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, m.X, (unsigned long long)(m.blocks - 1) * m.x_step + m.K, m.rows, (unsigned long long)m.ldx * 2, LT_BK, LT_M, true)
         || !make_map_2d(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, m.W, m.K, wrows, (unsigned long long)m.ldw * 2, LT_BK, BN / 2, true))
     {
         return -1;
     }
-    const bool vec = (reinterpret_cast<uintptr_t>(m.Y) & 15u) == 0 && (m.ldy % 8) == 0;
-    unsigned long long tiles = (unsigned long long)((m.rows + LT_M - 1) / LT_M + (m.groups > 1 ? m.groups : 0)) * ftiles;    // an upper bound
+    const bool vec = (reinterpret_cast<uintptr_t>(m.Y) & 15u) == 0 && (m.ldy % 8) == 0 && (m.y_step % 8) == 0;
+    unsigned long long tiles = (unsigned long long)((m.rows + LT_M - 1) / LT_M + (m.groups > 1 ? m.groups : 0)) * ftiles * m.blocks;    // an upper bound
     const unsigned int grid = (unsigned int)(tiles < (unsigned long long)dev.sm_count ? tiles : dev.sm_count);
     return launch_kernel("linear_tile", linear_tile_kernel<BN>, dim3(grid), dim3(LT_THREADS), (size_t)lt_smem(BN), stream, pdl, tx, tw, m, ftiles,
         vec ? 1 : 0, status);
@@ -337,11 +341,11 @@ int launch_linear_tile(const LinearMember& m, cudaStream_t stream, bool pdl)
     const DecoderDevice* dev = decoder_device();
     if (!dev) { return 1; }
     // the widest tile that still gives every SM one
-    const bool gated = m.activation == B200_ACT_SILU_GATE;
+    const bool gated = activation_gated(m.activation);
     const unsigned long long rt = (m.rows + LT_M - 1) / LT_M;
     auto tiles = [&](unsigned int bn) {
         const unsigned int ft = gated ? bn / 2 : bn;
-        return rt * ((m.N + ft - 1) / ft);
+        return rt * m.blocks * ((m.N + ft - 1) / ft);
     };
     if (tiles(256) >= (unsigned long long)dev->sm_count * 8 / 10) { return launch_tile<256>(m, *dev, stream, pdl); }
     if (tiles(128) >= (unsigned long long)dev->sm_count * 8 / 10) { return launch_tile<128>(m, *dev, stream, pdl); }

@@ -1,32 +1,13 @@
 // Fakilorn: attention without positions over unit-RMS queries and keys, values mixed with the first layer's, a sigmoid
 // output gate; dense squared-ReLU or mixture-of-experts feed-forwards; layer norms; a scaled, shared embedding table.
 // Reads config.json into a DecoderSpec; everything else is LayeredDecoder.
-#include "layered_decoder.h"
-
-#include <cstdio>
+#include "design_config.h"
 
 namespace cccc
 {
 
 namespace
 {
-bool fail(std::string* err, const std::string& what)
-{
-    if (err) { *err = what; }
-    return false;
-}
-
-// Members a reader does not know: said on stderr, since the model may mean something by them.
-void warnUnknown(const Json& j, const std::string& where, const std::vector<std::string>& known)
-{
-    for (const auto& m : j.members())
-    {
-        bool found = false;
-        for (const auto& k : known) { found = found || k == m.first; }
-        if (!found) { std::fprintf(stderr, "config.json: %s.%s is not known and ignored\n", where.c_str(), m.first.c_str()); }
-    }
-}
-
 ExpertSpec expert(const std::string& prefix, int ff) { return { ff, prefix + ".gate", prefix + ".up", prefix + ".down" }; }
 
 bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
@@ -34,7 +15,7 @@ bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
     if (!c["layers"].size() || c["embedding"]["scale"].type() != Json::NUMBER || c["norm"]["eps"].type() != Json::NUMBER
         || c["logit_scale"].type() != Json::NUMBER)
     {
-        return fail(err, "config.json: vocab, width, embedding.scale, norm.eps, logit_scale and layers are needed");
+        return configError(err, "vocab, width, embedding.scale, norm.eps, logit_scale and layers are needed");
     }
     s->vocab = (int)c["vocab"].number();
     s->width = (int)c["width"].number();
@@ -48,14 +29,14 @@ bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
     {
         const Json& j = c["layers"][i];
         const std::string at = "layers[" + std::to_string(i) + "]", p = "l" + std::to_string(i);
-        if (j["type"].string() != "attention") { return fail(err, "config.json: " + at + ": no mixer of type '" + j["type"].string() + "'"); }
+        if (j["type"].string() != "attention") { return configError(err, at + ": no mixer of type '" + j["type"].string() + "'"); }
         LayerSpec L;
         L.norm1 = p + ".norm1";
         L.norm2 = p + ".norm2";
         const Json& m = j["mixer"];
         warnUnknown(m, at + ".mixer", { "heads", "kv_heads", "dim", "vdim", "scale", "v_mix" });
-        if (m["scale"].type() != Json::NUMBER) { return fail(err, "config.json: " + at + ": mixer.scale is needed"); }
-        AttentionSpec& a = L.mixer;
+        if (m["scale"].type() != Json::NUMBER) { return configError(err, at + ": mixer.scale is needed"); }
+        AttentionSpec& a = L.attention;
         a.heads = (int)m["heads"].number();
         a.kv_heads = (int)m["kv_heads"].number();
         a.dim = (int)m["dim"].number();
@@ -77,7 +58,7 @@ bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
             warnUnknown(f, at + ".mlp", { "kind", "ff" });
             L.mlp.kind = MlpSpec::DENSE;
             L.mlp.activation = B200_ACT_RELU2;
-            L.mlp.dense = expert(p + ".mlp", (int)f["ff"].number());
+            L.mlp.dense = { (int)f["ff"].number(), "", p + ".mlp.up", p + ".mlp.down" };
         }
         else if (kind == "moe")
         {
@@ -95,32 +76,17 @@ bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
             if (!f["shared"].isNull())
             {
                 L.mlp.shared = expert(p + ".mlp.shared", (int)f["shared"]["ff"].number());
-                if (L.mlp.shared.ff <= 0) { return fail(err, "config.json: " + at + ": mlp.shared.ff must be positive"); }
+                if (L.mlp.shared.ff <= 0) { return configError(err, at + ": mlp.shared.ff must be positive"); }
                 L.mlp.shared_gate = p + ".mlp.shared.sg";
             }
         }
-        else { return fail(err, "config.json: " + at + ": no feed-forward of kind '" + kind + "'"); }
+        else { return configError(err, at + ": no feed-forward of kind '" + kind + "'"); }
         s->layers.push_back(L);
     }
     return true;
 }
 
-const bool g_registered = ModelRegistry::add("Fakilorn", [](const ModelOptions& o, const Json& config, std::string* err) {
-    std::unique_ptr<LayeredDecoder> m(new LayeredDecoder());
-    DecoderSpec spec;
-    if (!readSpec(config, &spec, err)) { return std::unique_ptr<LanguageModel>(); }
-    if (o.noise_weights)
-    {
-        NoiseSource noise(1);
-        if (!m->load(o, spec, noise, err)) { m.reset(); }
-    }
-    else
-    {
-        SafetensorsFile file;
-        if (!file.open(o.dir + "/model.safetensors", err) || !m->load(o, spec, file, err)) { m.reset(); }
-    }
-    return std::unique_ptr<LanguageModel>(std::move(m));
-});
+const bool g_registered = registerLayered("Fakilorn", readSpec);
 }    // namespace
 
 }    // namespace cccc

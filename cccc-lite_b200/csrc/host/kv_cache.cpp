@@ -9,6 +9,7 @@ KvCache::~KvCache()
     {
         gpu_->free(l.k);
         gpu_->free(l.v);
+        gpu_->free(l.state);
     }
 }
 
@@ -26,15 +27,17 @@ bool KvCache::init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int
         const size_t per = (size_t)slots * s.kv_heads * rows * elem_bytes;
         l.k_bytes = per * l.k_ld;
         l.v_bytes = per * l.v_ld;
-        l.k = gpu->malloc(l.k_bytes);
-        l.v = gpu->malloc(l.v_bytes);
+        l.state_bytes = (size_t)slots * s.state_floats * 4;
+        if (l.k_bytes) { l.k = gpu->malloc(l.k_bytes); }
+        if (l.v_bytes) { l.v = gpu->malloc(l.v_bytes); }
+        if (l.state_bytes) { l.state = (float*)gpu->malloc(l.state_bytes); }
         layers_.push_back(l);
-        if (!l.k || !l.v)
+        if ((l.k_bytes && !l.k) || (l.v_bytes && !l.v) || (l.state_bytes && !l.state))
         {
             if (err) { *err = "no device memory for the KV cache"; }
             return false;
         }
-        bytes_ += l.k_bytes + l.v_bytes;
+        bytes_ += l.k_bytes + l.v_bytes + l.state_bytes;
     }
     clear();
     return true;
@@ -66,8 +69,9 @@ void KvCache::clear()
     gpu_->setAsCurrent();
     for (auto& l : layers_)
     {
-        cudaMemsetAsync(l.k, 0, l.k_bytes, gpu_->stream());
-        cudaMemsetAsync(l.v, 0, l.v_bytes, gpu_->stream());
+        if (l.k) { cudaMemsetAsync(l.k, 0, l.k_bytes, gpu_->stream()); }
+        if (l.v) { cudaMemsetAsync(l.v, 0, l.v_bytes, gpu_->stream()); }
+        if (l.state) { cudaMemsetAsync(l.state, 0, l.state_bytes, gpu_->stream()); }
     }
     for (auto& n : length_) { n = 0; }
     gpu_->synchronize();

@@ -1,5 +1,7 @@
-// The KV cache of a decoder: per layer a key and a value array [slot][kv head][row][elements], one slot per live
-// sequence.  Slots are handed out and taken back here; their lengths say how many rows count.
+// What a decoder keeps of its live sequences, one slot each: per layer a key and a value array [slot][kv head][row][elements]
+// (or one array, where values are read from the key rows), or a recurrent state of fixed size, in floats.  Slots are handed out
+// and taken back here; their lengths say how many rows count.  A sequence of length 0 starts from an empty state, whatever its
+// slot's state memory holds.
 #pragma once
 
 #include "cccc_host.h"
@@ -12,7 +14,8 @@ namespace cccc
 
 struct KvLayerShape
 {
-    int kv_heads = 0, k_dim = 0, v_dim = 0;
+    int kv_heads = 0, k_dim = 0, v_dim = 0;    // v_dim 0: no value array
+    size_t state_floats = 0;                   // per slot
 };
 
 class KvCache
@@ -26,6 +29,7 @@ public:
     bool init(GpuControl* gpu, const std::vector<KvLayerShape>& layers, int elem_bytes, int slots, int rows, std::string* err);
     void* k(int layer) const { return layers_[layer].k; }
     void* v(int layer) const { return layers_[layer].v; }
+    float* state(int layer) const { return layers_[layer].state; }
     int kLd(int layer) const { return layers_[layer].k_ld; }
     int vLd(int layer) const { return layers_[layer].v_ld; }
     int slots() const { return (int)length_.size(); }
@@ -42,8 +46,9 @@ private:
     struct Layer
     {
         void *k = nullptr, *v = nullptr;
+        float* state = nullptr;
         int k_ld = 0, v_ld = 0;
-        size_t k_bytes = 0, v_bytes = 0;
+        size_t k_bytes = 0, v_bytes = 0, state_bytes = 0;
     };
     GpuControl* gpu_ = nullptr;
     std::vector<Layer> layers_;

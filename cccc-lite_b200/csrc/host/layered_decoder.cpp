@@ -21,6 +21,19 @@ float widen(uint16_t b)
     std::memcpy(&f, &u, 4);
     return f;
 }
+bool activationGated(int a) { return a == B200_ACT_SILU_GATE || a == B200_ACT_GELU_GATE; }
+// Do two layers have tensors of the same shapes?
+bool sameShape(const LayerSpec& a, const LayerSpec& b)
+{
+    auto key = [](const LayerSpec& l) {
+        const AttentionSpec& x = l.attention;
+        const LatentSpec& y = l.latent;
+        const MlstmSpec& z = l.mlstm;
+        return std::vector<int>{ (int)l.kind, x.heads, x.kv_heads, x.dim, x.vdim, y.heads, y.dim, y.rot_dim, y.vdim, y.q_rank, y.kv_rank, z.heads, z.dim, z.vdim,
+            (int)l.mlp.kind, l.mlp.dense.ff, (int)l.mlp.experts.size(), l.mlp.shared.ff };
+    };
+    return key(a) == key(b);
+}
 constexpr int kStreamRows = 32;    // rows up to which the weight-streaming kernels (and the graphs) run a pass
 }    // namespace
 
@@ -49,17 +62,19 @@ bool LayeredDecoder::check(std::string* err) const
     int mixed = -1;
     for (size_t i = 0; i < s.layers.size(); i++)
     {
-        const AttentionSpec& a = s.layers[i].mixer;
         const std::string at = "layer " + std::to_string(i) + ": ";
-        if (a.heads <= 0 || a.kv_heads <= 0 || a.dim <= 0 || a.vdim <= 0) { return fail(err, at + "heads, kv_heads, dim and vdim must be positive"); }
-        if (a.heads % a.kv_heads) { return fail(err, at + "heads must be a multiple of kv_heads"); }
-        if (a.v_mix)
+        // layers may share tensors through one another, but not in a circle
+        int own = (int)i;
+        for (size_t hops = 0; s.layers[own].weights_of != -1; hops++)
         {
-            if (mixed >= 0 && mixed != a.kv_heads * a.vdim) { return fail(err, at + "layers that mix values must have values of one size"); }
-            mixed = a.kv_heads * a.vdim;
+            own = s.layers[own].weights_of;
+            if (own < 0 || own >= (int)s.layers.size() || hops >= s.layers.size()) { return fail(err, at + "weights_of must lead to a layer with tensors"); }
         }
+        if (!sameShape(s.layers[i], s.layers[own])) { return fail(err, at + "differs from the layer whose tensors it uses"); }
+        if (!checkMixer(s.layers[i], at, &mixed, err)) { return false; }
         const MlpSpec& m = s.layers[i].mlp;
         if (m.kind == MlpSpec::DENSE && m.dense.ff <= 0) { return fail(err, at + "ff must be positive"); }
+        if (m.kind == MlpSpec::DENSE && activationGated(m.activation) != !m.dense.gate.empty()) { return fail(err, at + "a gated activation needs a gate, others take none"); }
         if (m.kind == MlpSpec::MOE)
         {
             if (m.experts.empty() || m.top <= 0 || m.top > (int)m.experts.size()) { return fail(err, at + "top must lie between 1 and the number of experts"); }
@@ -77,60 +92,95 @@ bool LayeredDecoder::load(const ModelOptions& o, const DecoderSpec& spec, Tensor
     if (!check(err)) { return false; }
     if (o.max_context <= 0 || o.max_sequences <= 0 || o.max_step_tokens <= 0) { return fail(err, "context, sequences and step tokens must be positive"); }
     if (gpu_.init(o.device) != 0) { return fail(err, "cannot open CUDA device " + std::to_string(o.device)); }
+    max_context_ = o.max_context;
     cap_ = std::max(std::min(o.max_step_tokens, o.max_context * o.max_sequences), std::min(o.max_sequences, kStreamRows));
     if (!loadTensors(source, err) || !allocate(o, err)) { return false; }
     gpu_.synchronize();
     return cuda_b200_decoder_check("model load") == 0 ? true : fail(err, "a CUDA error while loading");
 }
 
-// Tensors [rows][k] one below the other, every one padded to a multiple of `align` rows; rows padded to 64 columns; zeros.
-bool LayeredDecoder::packRows(TensorSource& s, const std::vector<std::pair<std::string, int>>& parts, int k, int align, Weight* out, std::string* err)
+// `rows` rows of k from the first-th element of `bits` to row `at` of w.
+bool LayeredDecoder::upload(const std::string& name, const std::vector<uint16_t>& bits, size_t first, int rows, int k, size_t at, const Weight& w, std::string* err)
 {
+    const size_t row_bytes = (size_t)w.ld * elem();
+    const void* src = bits.data() + first;
+    std::vector<float> wide;
+    if (dtype_ == FLOAT)
+    {
+        wide.resize((size_t)rows * k);
+        for (size_t i = 0; i < wide.size(); i++) { wide[i] = widen(bits[first + i]); }
+        src = wide.data();
+    }
+    weight_bytes_ += (size_t)rows * k * elem();
+    return cudaMemcpy2D((char*)w.w + at * row_bytes, row_bytes, src, (size_t)k * elem(), (size_t)k * elem(), (size_t)rows, cudaMemcpyHostToDevice) == cudaSuccess
+        || fail(err, "cannot copy '" + name + "' to the device");
+}
+
+// Tensors [rows][k] one below the other, every piece padded to a multiple of `align` rows; rows padded to 64 columns; zeros.
+bool LayeredDecoder::packRows(TensorSource& s, const std::vector<Rows>& parts, int k, int align, Weight* out, std::string* err)
+{
+    auto padded = [&](int n) { return (size_t)(n + align - 1) / align * align; };
     size_t rows = 0;
-    for (const auto& p : parts) { rows += (size_t)(p.second + align - 1) / align * align; }
+    for (const auto& p : parts) { rows += padded(p.rows / p.pieces) * p.pieces; }
     out->rows = (int)rows;
     out->k = k;
     out->ld = pad64(k);
-    const size_t row_bytes = (size_t)out->ld * elem();
-    out->w = dmalloc(rows * row_bytes, true);
-    if (!out->w) { return fail(err, "no device memory for '" + parts[0].first + "'"); }
+    out->w = dmalloc(rows * out->ld * elem(), true);
+    if (!out->w) { return fail(err, "no device memory for '" + parts[0].name + "'"); }
     gpu_.synchronize();
     std::vector<uint16_t> bits;
-    std::vector<float> wide;
     size_t at = 0;
     for (const auto& p : parts)
     {
-        if (!s.readBf16(p.first, { p.second, k }, &bits, err)) { return false; }
-        const void* src = bits.data();
-        if (dtype_ == FLOAT)
+        if (!s.readBf16(p.name, { p.rows, k }, &bits, err)) { return false; }
+        const int piece = p.rows / p.pieces;
+        for (int j = 0; j < p.pieces; j++)
         {
-            wide.resize(bits.size());
-            for (size_t i = 0; i < bits.size(); i++) { wide[i] = widen(bits[i]); }
-            src = wide.data();
+            if (!upload(p.name, bits, (size_t)j * piece * k, piece, k, at, *out, err)) { return false; }
+            at += padded(piece);
         }
-        if (cudaMemcpy2D((char*)out->w + at * row_bytes, row_bytes, src, (size_t)k * elem(), (size_t)k * elem(), (size_t)p.second, cudaMemcpyHostToDevice)
-            != cudaSuccess)
-        {
-            return fail(err, "cannot copy '" + p.first + "' to the device");
-        }
-        weight_bytes_ += bits.size() * elem();
-        at += (size_t)(p.second + align - 1) / align * align;
     }
     return true;
 }
 
+bool LayeredDecoder::packTransposed(TensorSource& s, const std::string& name, int pieces, int rows, int k, Weight* out, std::string* err)
+{
+    std::vector<uint16_t> bits, turned((size_t)pieces * rows * k);
+    if (!s.readBf16(name, { (int64_t)pieces * rows, k }, &bits, err)) { return false; }
+    for (int p = 0; p < pieces; p++)
+    {
+        for (int r = 0; r < rows; r++)
+        {
+            for (int c = 0; c < k; c++) { turned[((size_t)p * k + c) * rows + r] = bits[((size_t)p * rows + r) * k + c]; }
+        }
+    }
+    out->rows = pieces * k;
+    out->k = rows;
+    out->ld = pad64(rows);
+    out->w = dmalloc((size_t)out->rows * out->ld * elem(), true);
+    if (!out->w) { return fail(err, "no device memory for '" + name + "'"); }
+    gpu_.synchronize();
+    return upload(name, turned, 0, out->rows, rows, 0, *out, err);
+}
+
+// Vectors one behind the other, as floats.
+bool LayeredDecoder::loadVector(TensorSource& s, const std::vector<std::pair<std::string, int>>& parts, float** out, std::string* err)
+{
+    std::vector<float> f;
+    std::vector<uint16_t> bits;
+    for (const auto& p : parts)
+    {
+        if (!s.readBf16(p.first, { p.second }, &bits, err)) { return false; }
+        for (uint16_t b : bits) { f.push_back(widen(b)); }
+    }
+    *out = (float*)dmalloc(f.size() * 4, false);
+    return (*out && cudaMemcpy(*out, f.data(), f.size() * 4, cudaMemcpyHostToDevice) == cudaSuccess) || fail(err, "no device memory for '" + parts[0].first + "'");
+}
+
 bool LayeredDecoder::loadNorm(TensorSource& s, const std::string& name, Norm* out, std::string* err)
 {
-    auto vec = [&](const std::string& n, float** dst) {
-        std::vector<uint16_t> bits;
-        if (!s.readBf16(n, { spec_.width }, &bits, err)) { return false; }
-        std::vector<float> f(bits.size());
-        for (size_t i = 0; i < f.size(); i++) { f[i] = widen(bits[i]); }
-        *dst = (float*)dmalloc(f.size() * 4, false);
-        if (!*dst || cudaMemcpy(*dst, f.data(), f.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) { return fail(err, "no device memory for '" + n + "'"); }
-        return true;
-    };
-    return vec(name, &out->w) && (spec_.norm_kind != B200_NORM_LAYER || vec(name + ".b", &out->b));
+    return loadVector(s, { { name, spec_.width } }, &out->w, err)
+        && (spec_.norm_kind != B200_NORM_LAYER || loadVector(s, { { name + ".b", spec_.width } }, &out->b, err));
 }
 
 bool LayeredDecoder::loadTensors(TensorSource& s, std::string* err)
@@ -140,76 +190,72 @@ bool LayeredDecoder::loadTensors(TensorSource& s, std::string* err)
     head_ = embed_;
     if (spec_.head != spec_.embed && !packRows(s, { { spec_.head, spec_.vocab } }, W, 1, &head_, err)) { return false; }
     if (!loadNorm(s, spec_.final_norm, &final_norm_, err)) { return false; }
-    bool mixing = false;
     layers_.resize(spec_.layers.size());
     for (size_t i = 0; i < layers_.size(); i++)
     {
-        const LayerSpec& ls = spec_.layers[i];
-        const AttentionSpec& a = ls.mixer;
-        Layer& L = layers_[i];
-        if (!loadNorm(s, ls.norm1, &L.norm1, err)) { return false; }
-        std::vector<std::pair<std::string, int>> parts = { { a.q, a.heads * a.dim }, { a.k, a.kv_heads * a.dim }, { a.v, a.kv_heads * a.vdim } };
-        if (!a.gate.empty()) { parts.emplace_back(a.gate, a.heads * a.vdim); }
-        if (!packRows(s, parts, W, 8, &L.qkvg, err)) { return false; }
-        auto pad8 = [](int n) { return (n + 7) / 8 * 8; };
-        L.k_off = pad8(a.heads * a.dim);
-        L.v_off = L.k_off + pad8(a.kv_heads * a.dim);
-        L.g_off = L.v_off + pad8(a.kv_heads * a.vdim);
-        L.n_qkvg = L.qkvg.rows;
-        if (!packRows(s, { { a.o, W } }, a.heads * a.vdim, 1, &L.o, err)) { return false; }
-        if (a.v_mix)
+        if (spec_.layers[i].weights_of == -1 && !loadLayer(s, spec_.layers[i], &layers_[i], err)) { return false; }
+    }
+    bool mixing = false;
+    for (size_t i = 0; i < layers_.size(); i++)
+    {
+        size_t own = i;
+        while (spec_.layers[own].weights_of != -1) { own = (size_t)spec_.layers[own].weights_of; }
+        if (own != i) { layers_[i] = layers_[own]; }
+        const AttentionSpec& a = spec_.layers[i].attention;
+        if (spec_.layers[i].kind != LayerSpec::ATTENTION || !a.v_mix) { continue; }
+        layers_[i].v_mix = mixing ? 2 : 1;
+        mixing = true;
+        if (layers_[i].v_mix == 2)
         {
-            L.v_mix = mixing ? 2 : 1;
-            mixing = true;
-            if (L.v_mix == 2)
-            {
-                std::vector<uint16_t> b;
-                if (!s.readBf16(a.vmix, {}, &b, err)) { return false; }
-                L.lambda = widen(b[0]);
-            }
-        }
-        const MlpSpec& m = ls.mlp;
-        if (m.kind == MlpSpec::NONE) { continue; }
-        if (!loadNorm(s, ls.norm2, &L.norm2, err)) { return false; }
-        if (m.kind == MlpSpec::DENSE)
-        {
-            if (!packRows(s, { { m.dense.up, m.dense.ff } }, W, 1, &L.up, err) || !packRows(s, { { m.dense.down, W } }, m.dense.ff, 1, &L.down, err)) { return false; }
-            continue;
-        }
-        parts = { { m.router, (int)m.experts.size() } };
-        if (m.shared.ff) { parts.emplace_back(m.shared_gate, 1); }
-        if (!packRows(s, parts, W, 1, &L.router, err)) { return false; }
-        std::vector<std::pair<std::string, int>> in, out;
-        for (const auto& e : m.experts)
-        {
-            in.emplace_back(e.gate, e.ff);
-            in.emplace_back(e.up, e.ff);
-            out.emplace_back(e.down, W);
-        }
-        if (!packRows(s, in, W, 1, &L.experts_in, err) || !packRows(s, out, m.experts[0].ff, 1, &L.experts_out, err)) { return false; }
-        if (m.shared.ff
-            && (!packRows(s, { { m.shared.gate, m.shared.ff }, { m.shared.up, m.shared.ff } }, W, 1, &L.shared_in, err)
-                || !packRows(s, { { m.shared.down, W } }, m.shared.ff, 1, &L.shared_out, err)))
-        {
-            return false;
+            std::vector<uint16_t> b;
+            if (!s.readBf16(a.vmix, {}, &b, err)) { return false; }
+            layers_[i].lambda = widen(b[0]);
         }
     }
     return true;
 }
 
+bool LayeredDecoder::loadLayer(TensorSource& s, const LayerSpec& ls, Layer* out, std::string* err)
+{
+    const int W = spec_.width;
+    Layer& L = *out;
+    if (!loadNorm(s, ls.norm1, &L.norm1, err) || !loadMixer(s, ls, &L, err)) { return false; }
+    // a branch's norm has no bias
+    if (!ls.norm1b.empty() && !loadVector(s, { { ls.norm1b, W } }, &L.norm1b.w, err)) { return false; }
+    const MlpSpec& m = ls.mlp;
+    if (m.kind == MlpSpec::NONE) { return true; }
+    if (!loadNorm(s, ls.norm2, &L.norm2, err) || (!ls.norm2b.empty() && !loadVector(s, { { ls.norm2b, W } }, &L.norm2b.w, err))) { return false; }
+    if (m.kind == MlpSpec::DENSE)
+    {
+        std::vector<Rows> up = { { m.dense.up, m.dense.ff } };
+        if (!m.dense.gate.empty()) { up.insert(up.begin(), { m.dense.gate, m.dense.ff }); }
+        return packRows(s, up, W, 1, &L.up, err) && packRows(s, { { m.dense.down, W } }, m.dense.ff, 1, &L.down, err);
+    }
+    std::vector<Rows> parts = { { m.router, (int)m.experts.size() } };
+    if (m.shared.ff) { parts.push_back({ m.shared_gate, 1 }); }
+    if (!packRows(s, parts, W, 1, &L.router, err)) { return false; }
+    std::vector<Rows> in, down;
+    for (const auto& e : m.experts)
+    {
+        in.push_back({ e.gate, e.ff });
+        in.push_back({ e.up, e.ff });
+        down.push_back({ e.down, W });
+    }
+    if (!packRows(s, in, W, 1, &L.experts_in, err) || !packRows(s, down, m.experts[0].ff, 1, &L.experts_out, err)) { return false; }
+    return !m.shared.ff
+        || (packRows(s, { { m.shared.gate, m.shared.ff }, { m.shared.up, m.shared.ff } }, W, 1, &L.shared_in, err)
+            && packRows(s, { { m.shared.down, W } }, m.shared.ff, 1, &L.shared_out, err));
+}
+
 bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
 {
-    std::vector<KvLayerShape> shapes;
-    int vdim = 0, qkvg = 0, att = 0, ff = 0, eff = 0, sff = 0, router = 0, first = 0;
+    int ff = 0, eff = 0, sff = 0, router = 0;
+    bool branch = false;
     for (size_t i = 0; i < layers_.size(); i++)
     {
-        const AttentionSpec& a = spec_.layers[i].mixer;
-        const MlpSpec& m = spec_.layers[i].mlp;
-        shapes.push_back({ a.kv_heads, a.dim, a.vdim });
-        vdim = std::max(vdim, a.vdim);
-        qkvg = std::max(qkvg, layers_[i].n_qkvg);
-        att = std::max(att, a.heads * a.vdim);
-        if (a.v_mix) { first = a.kv_heads * a.vdim; }
+        const LayerSpec& ls = spec_.layers[i];
+        const MlpSpec& m = ls.mlp;
+        branch = branch || !ls.norm1b.empty() || !ls.norm2b.empty();
         if (m.kind == MlpSpec::DENSE) { ff = std::max(ff, m.dense.ff); }
         if (m.kind == MlpSpec::MOE)
         {
@@ -220,15 +266,12 @@ bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
             max_experts_ = std::max(max_experts_, (int)m.experts.size());
         }
     }
-    if (!cache_.init(&gpu_, shapes, (int)elem(), o.max_sequences, o.max_context, err)) { return false; }
+    if (!allocateMixers(o, err)) { return false; }
     ldw_ = pad64(spec_.width);
-    ld_qkvg_ = pad64(qkvg);
-    ld_att_ = pad64(att);
     ld_ff_ = pad64(std::max(ff, sff));
     ld_eff_ = pad64(std::max(eff, 1));
     ld_router_ = pad64(std::max(router, 1));
     ld_logits_ = pad64(spec_.vocab);
-    ld_first_ = pad64(std::max(first, 1));
     want_cap_ = std::min(cap_, 256);
     const size_t T = (size_t)cap_, P = T * top_, e = elem();
     bool ok = true;
@@ -239,9 +282,7 @@ bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
     };
     x_ = (float*)get(T * ldw_ * 4);
     xn_ = get(T * ldw_ * e);
-    qkvg_ = get(T * ld_qkvg_ * e);
-    att_ = get(T * ld_att_ * e);
-    v_first_ = get(T * ld_first_ * e);
+    if (branch) { branch_ = (float*)get(T * ldw_ * 4); }
     ff_ = get(T * ld_ff_ * e);
     if (top_)
     {
@@ -262,8 +303,7 @@ bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
     logits_ = (float*)get((size_t)want_cap_ * ld_logits_ * 4);
     d_choice_ = (int*)get((size_t)want_cap_ * 4);
     d_best_ = (float*)get((size_t)want_cap_ * 4);
-    attn_work_ = get(cuda_b200_attention_work_bytes((unsigned int)vdim));
-    const size_t meta = 3 * T + 4 * T;
+    const size_t meta = 3 * T + 4 * T + 2 * windows_.size() * T;
     d_meta_ = (int*)get(meta * 4);
     ok = ok && cudaMallocHost((void**)&h_meta_, meta * 4) == cudaSuccess && cudaMallocHost((void**)&h_choice_, (size_t)want_cap_ * 4) == cudaSuccess
         && cudaMallocHost((void**)&h_logits_, (size_t)want_cap_ * spec_.vocab * 4) == cudaSuccess;
@@ -273,36 +313,69 @@ bool LayeredDecoder::allocate(const ModelOptions& o, std::string* err)
 
 void LayeredDecoder::makePass(const std::vector<StepEntry>& entries, const std::vector<int>& from, const std::vector<int>& count, Pass* p) const
 {
-    std::vector<int> ids, owner, slot, pos, start, n, wants;
-    p->decode = true;
-    for (size_t e = 0; e < entries.size(); e++)
+    std::vector<int> ids, owner, slot, start, wants, order;
+    // entries of a few tokens first; the float mode has one kind of kernel
+    for (int kind = 0; kind < 2; kind++)
     {
-        if (count[e] == 0) { continue; }
+        for (size_t e = 0; e < entries.size(); e++)
+        {
+            const bool few = count[e] <= kFewTokens;
+            if (count[e] != 0 && (kind == 0) == (few || dtype_ == FLOAT)) { order.push_back((int)e); }
+        }
+    }
+    p->decode = true;
+    for (int e : order)
+    {
         const StepEntry& E = entries[e];
         const int first = (int)ids.size(), index = (int)slot.size(), at = cache_.length(E.slot);
+        const bool few = count[e] <= kFewTokens || dtype_ == FLOAT;
+        if (p->parts.empty() || p->parts.back().few != few)
+        {
+            Part part;
+            part.few = few;
+            part.first_entry = index;
+            part.first_token = first;
+            p->parts.push_back(part);
+        }
+        Part& part = p->parts.back();
+        part.entries++;
+        part.tokens += count[e];
+        part.max_n = std::max(part.max_n, count[e]);
+        part.max_len = std::max(part.max_len, at + count[e]);
         slot.push_back(E.slot);
-        pos.push_back(at);
+        p->pos.push_back(at);
         start.push_back(first);
-        n.push_back(count[e]);
+        p->n.push_back(count[e]);
         for (int i = 0; i < count[e]; i++)
         {
             ids.push_back(E.tokens[from[e] + i]);
             owner.push_back(index);
         }
-        size_t before = wants.size();
-        for (int w : E.want)
+        const size_t before = wants.size();
+        for (size_t k = 0; k < E.want.size(); k++)
         {
-            if (w >= from[e] && w < from[e] + count[e]) { wants.push_back(first + w - from[e]); }
+            const int w = E.want[k];
+            if (w >= from[e] && w < from[e] + count[e])
+            {
+                wants.push_back(first + w - from[e]);
+                p->asked.emplace_back(e, (int)k);
+            }
         }
         p->decode = p->decode && count[e] == 1 && wants.size() == before + 1;
-        p->max_n = std::max(p->max_n, count[e]);
-        p->max_len = std::max(p->max_len, at + count[e]);
     }
     p->tokens = (int)ids.size();
     p->entries = (int)slot.size();
     p->wants = (int)wants.size();
     p->decode = p->decode && p->tokens <= kStreamRows;
-    for (auto* v : { &ids, &owner, &slot, &pos, &start, &n, &wants }) { p->host.insert(p->host.end(), v->begin(), v->end()); }
+    for (auto* v : { &ids, &owner, &slot, &p->pos, &start, &p->n, &wants }) { p->host.insert(p->host.end(), v->begin(), v->end()); }
+    if (dtype_ == FLOAT) { return; }
+    for (int window : windows_)
+    {
+        std::vector<int> floor, pos2;
+        expandedFloor(*p, window, &floor, &pos2);
+        p->host.insert(p->host.end(), floor.begin(), floor.end());
+        p->host.insert(p->host.end(), pos2.begin(), pos2.end());
+    }
 }
 
 int LayeredDecoder::issueHead(const Pass& p, int row0, int rows, cudaStream_t st)
@@ -336,6 +409,8 @@ int LayeredDecoder::issueHead(const Pass& p, int row0, int rows, cudaStream_t st
     h.ldx = (unsigned int)ldw_;
     h.ldy = (unsigned int)ld_logits_;
     h.alpha = spec_.logit_scale;
+    h.cap = spec_.logit_softcap;
+    if (h.cap > 0.f) { h.activation = B200_ACT_SOFTCAP; }
     ok(cuda_b200_linear_rows(act(), 1, &h, st, PDL, 0));
     ok(cuda_b200_argmax_f32(logits_, (unsigned int)rows, (unsigned int)spec_.vocab, (unsigned int)ld_logits_, d_choice_, d_best_, st, PDL));
     return bad ? -1 : n;
@@ -345,45 +420,18 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
 {
     const unsigned int PDL = 1u;
     const unsigned int T = (unsigned int)p.tokens, W = (unsigned int)spec_.width;
-    const int out16 = act();
     const bool stream = dtype_ == BFLOAT16 && p.tokens <= kStreamRows;
-    int bad = 0, n = 0;
-    auto ok = [&](int rc) {
-        bad += rc != 0;
-        n++;
-    };
-    cuda_b200_batch b = {};
-    b.slot = devEntries(p, 0);
-    b.pos = devEntries(p, 1);
-    b.start = devEntries(p, 2);
-    b.n = devEntries(p, 3);
-    b.token_entry = devTokenEntry(p);
-    b.entries = (unsigned int)p.entries;
-    b.tokens = T;
-    b.max_n = (unsigned int)p.max_n;
-    b.max_len = (unsigned int)p.max_len;
-    auto dense = [&](const Weight& w, const void* X, int ldx, void* Y, int ldy) {
-        cuda_b200_linear l = {};
-        l.W = w.w;
-        l.X = X;
-        l.Y = Y;
-        l.rows = T;
-        l.N = (unsigned int)w.rows;
-        l.K = (unsigned int)w.k;
-        l.ldw = (unsigned int)w.ld;
-        l.ldx = (unsigned int)ldx;
-        l.ldy = (unsigned int)ldy;
-        l.out_type = out16;
-        l.alpha = 1.0f;
-        return l;
-    };
+    Issue r0{ p, st };
+    auto ok = [&](int rc) { r0.ok(rc); };
+    auto dense = [&](const Weight& w, const void* X, int ldx, void* Y, int ldy) { return this->dense(r0, w, X, ldx, Y, ldy); };
     auto into_stream = [&](const Weight& w, const void* X, int ldx) {
         cuda_b200_linear l = dense(w, X, ldx, x_, ldw_);
         l.out_type = 0;
         l.accumulate = 1;
         return l;
     };
-    unsigned int pending = 0;    // experts' outputs per token that the stream still lacks
+    unsigned int pending = 0;           // experts' outputs per token that the stream still lacks
+    const Norm* branch = nullptr;       // the norm of a branch that the stream still lacks
     auto norm = [&](const Norm& w, void* out) {
         cuda_b200_norm a = {};
         a.X = x_;
@@ -394,6 +442,12 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
         a.slot_row = pair_row_;
         a.slot_weight = pair_weight_;
         a.slots = pending;
+        if (branch)
+        {
+            a.branch = branch_;
+            a.branch_weight = branch->w;
+            a.ldb = (unsigned int)ldw_;
+        }
         a.n = T;
         a.width = W;
         a.ldx = a.ldo = a.ldy = (unsigned int)ldw_;
@@ -401,59 +455,45 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
         a.eps = spec_.eps;
         ok(cuda_b200_norm_rows(act(), &a, st, PDL));
         pending = 0;
+        branch = nullptr;
+    };
+    // a sublayer's last linear: onto the stream, or aside until the next norm
+    auto output = [&](const Weight& w, const void* X, int ldx, const Norm& after) {
+        cuda_b200_linear l = into_stream(w, X, ldx);
+        if (after.w)
+        {
+            l.Y = branch_;
+            l.accumulate = 0;
+            branch = &after;
+        }
+        ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
     };
     ok(cuda_b200_embed_f32(act(), devIds(p), embed_.w, (unsigned int)embed_.ld, x_, (unsigned int)ldw_, T, W, (unsigned int)spec_.vocab, spec_.embed_scale, st,
         PDL));
     for (size_t i = 0; i < layers_.size(); i++)
     {
         const Layer& L = layers_[i];
-        const AttentionSpec& s = spec_.layers[i].mixer;
         const MlpSpec& m = spec_.layers[i].mlp;
         norm(L.norm1, xn_);
-        cuda_b200_linear l = dense(L.qkvg, xn_, ldw_, qkvg_, ld_qkvg_);
-        ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
-        cuda_b200_attention a = {};
-        a.qkvg = qkvg_;
-        a.out = att_;
-        a.k_cache = cache_.k((int)i);
-        a.v_cache = cache_.v((int)i);
-        a.v_first = v_first_;
-        a.work = attn_work_;
-        a.ld = (unsigned int)ld_qkvg_;
-        a.ldo = (unsigned int)ld_att_;
-        a.k_off = (unsigned int)L.k_off;
-        a.v_off = (unsigned int)L.v_off;
-        a.g_off = (unsigned int)L.g_off;
-        a.v_first_ld = (unsigned int)ld_first_;
-        a.H = (unsigned int)s.heads;
-        a.Hkv = (unsigned int)s.kv_heads;
-        a.dim = (unsigned int)s.dim;
-        a.vdim = (unsigned int)s.vdim;
-        a.k_ld = (unsigned int)cache_.kLd((int)i);
-        a.v_ld = (unsigned int)cache_.vLd((int)i);
-        a.T_max = (unsigned int)cache_.rows();
-        a.slots = (unsigned int)cache_.slots();
-        a.v_mix = L.v_mix;
-        a.qk_norm = s.qk_norm;
-        a.gate = !s.gate.empty();
-        a.mix = L.lambda;
-        a.eps = spec_.eps;
-        a.scale = s.scale;
-        ok(cuda_b200_attention_rows(act(), &a, &b, st, PDL, 0));
-        l = into_stream(L.o, att_, ld_att_);
-        ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
+        switch (spec_.layers[i].kind)
+        {
+        case LayerSpec::ATTENTION: issueAttention(r0, (int)i); break;
+        case LayerSpec::LATENT: issueLatent(r0, (int)i); break;
+        case LayerSpec::MLSTM: issueMlstm(r0, (int)i); break;
+        }
+        output(L.o, att_, ld_att_, L.norm1b);
         if (m.kind == MlpSpec::NONE) { continue; }
         norm(L.norm2, xn_);
         if (m.kind == MlpSpec::DENSE)
         {
-            l = dense(L.up, xn_, ldw_, ff_, ld_ff_);
+            cuda_b200_linear l = dense(L.up, xn_, ldw_, ff_, ld_ff_);
             l.activation = m.activation;
+            l.N = l.up_row = (unsigned int)m.dense.ff;
             ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
-            l = into_stream(L.down, ff_, ld_ff_);
-            ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
+            output(L.down, ff_, ld_ff_, L.norm2b);
             continue;
         }
-        l = dense(L.router, xn_, ldw_, router_logits_, ld_router_);
+        cuda_b200_linear l = dense(L.router, xn_, ldw_, router_logits_, ld_router_);
         l.out_type = 0;
         ok(cuda_b200_linear_rows(act(), 1, &l, st, PDL, 0));
         const unsigned int E = (unsigned int)m.experts.size(), top = (unsigned int)m.top;
@@ -507,8 +547,8 @@ int LayeredDecoder::issue(const Pass& p, cudaStream_t st)
         ok(cuda_b200_linear_rows(act(), shared ? 2 : 1, out, st, PDL, 0));
         pending = top;
     }
-    if (pending) { norm(Norm(), nullptr); }
-    return bad ? -1 : n;
+    if (pending || branch) { norm(Norm(), nullptr); }
+    return r0.bad ? -1 : r0.n;
 }
 
 int LayeredDecoder::run(const Pass& p, float* logits, int* choice)
@@ -533,10 +573,11 @@ int LayeredDecoder::run(const Pass& p, float* logits, int* choice)
     {
         // lengths up to a power of two share a graph
         Pass q = p;
-        q.max_len = 64;
-        while (q.max_len < p.max_len) { q.max_len *= 2; }
-        q.max_len = std::min(q.max_len, cache_.rows());
-        auto it = graphs_.find({ p.entries, q.max_len });
+        int& len = q.parts[0].max_len;
+        len = 64;
+        while (len < p.parts[0].max_len) { len *= 2; }
+        len = std::min(len, cache_.rows());
+        auto it = graphs_.find({ p.entries, len });
         if (it != graphs_.end())
         {
             if (cudaGraphLaunch(it->second.first, st) != cudaSuccess) { return 1; }
@@ -560,7 +601,7 @@ int LayeredDecoder::run(const Pass& p, float* logits, int* choice)
             cudaGetLastError();
             return 1;
         }
-        graphs_[{ p.entries, q.max_len }] = { exec, launches };
+        graphs_[{ p.entries, len }] = { exec, launches };
         return 0;
     }
     if (issue(p, st) < 0) { return -1; }
@@ -601,14 +642,7 @@ int LayeredDecoder::step(const std::vector<StepEntry>& entries, float* logits, i
         Pass p;
         makePass(entries, done, count, &p);
         std::vector<int> place;
-        for (size_t e = 0; e < entries.size(); e++)
-        {
-            for (size_t w = 0; w < entries[e].want.size(); w++)
-            {
-                const int at = entries[e].want[w];
-                if (at >= done[e] && at < done[e] + count[e]) { place.push_back(first[e] + (int)w); }
-            }
-        }
+        for (const auto& a : p.asked) { place.push_back(first[a.first] + a.second); }
         std::vector<float> lg(logits && p.wants ? (size_t)p.wants * spec_.vocab : 0);
         std::vector<int> ch(choice ? p.wants : 0);
         const int rc = run(p, logits ? lg.data() : nullptr, choice ? ch.data() : nullptr);
@@ -655,7 +689,7 @@ float LayeredDecoder::timeStep(int entries, int tokens, int context, int inner, 
     {
         for (auto it = graphs_.begin(); it != graphs_.end(); ++it)
         {
-            if (it->first.first == entries && it->first.second >= std::min(p.max_len, cache_.rows()) && (g == graphs_.end() || it->first.second < g->first.second)) { g = it; }
+            if (it->first.first == entries && it->first.second >= std::min(p.parts[0].max_len, cache_.rows()) && (g == graphs_.end() || it->first.second < g->first.second)) { g = it; }
         }
         ok = g != graphs_.end();
     }

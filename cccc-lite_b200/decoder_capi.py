@@ -9,7 +9,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libcccc-b200-decoder.so")
 
 FLOAT, BF16 = 0, 3
-ACT_NONE, ACT_RELU2, ACT_SILU_GATE = 0, 1, 2
+ACT_NONE, ACT_RELU2, ACT_SILU_GATE, ACT_GELU_GATE, ACT_SOFTCAP = 0, 1, 2, 3, 4
 NORM_RMS, NORM_LAYER = 0, 1
 
 _vp, _i, _u, _f = C.c_void_p, C.c_int, C.c_uint, C.c_float
@@ -19,14 +19,19 @@ def _struct(name, pointers, uints, ints=(), floats=()):
     return type(name, (C.Structure,), {"_fields_": [(n, _vp) for n in pointers] + [(n, _u) for n in uints] + [(n, _i) for n in ints] + [(n, _f) for n in floats]})
 
 
-Norm = _struct("Norm", ("X", "weight", "bias", "out", "Y", "slot_row", "slot_weight", "rows"), ("n", "width", "ldx", "ldo", "ldy", "slots"), ("kind",), ("eps",))
-Linear = _struct("Linear", ("W", "X", "Y", "row_scale", "group_offset", "x_row", "active"),
-                 ("rows", "N", "K", "ldw", "ldx", "ldy", "groups", "group_rows", "group_max", "up_row", "active_cap"), ("out_type", "activation", "accumulate"),
-                 ("alpha",))
-Batch = _struct("Batch", ("slot", "pos", "start", "n", "token_entry"), ("entries", "tokens", "max_n", "max_len"))
-Attention = _struct("Attention", ("qkvg", "out", "k_cache", "v_cache", "v_first", "work"),
-                    ("ld", "ldo", "k_off", "v_off", "g_off", "v_first_ld", "H", "Hkv", "dim", "vdim", "k_ld", "v_ld", "T_max", "slots"), ("v_mix", "qk_norm", "gate"),
-                    ("mix", "eps", "scale"))
+Norm = _struct("Norm", ("X", "weight", "bias", "out", "Y", "slot_row", "slot_weight", "rows", "branch", "branch_weight"), ("n", "width", "ldx", "ldo", "ldy", "slots", "ldb"), ("kind",), ("eps",))
+Linear = _struct("Linear", ("W", "X", "Y", "row_scale", "group_offset", "x_row", "active", "head_gate"),
+                 ("rows", "N", "K", "ldw", "ldx", "ldy", "groups", "group_rows", "group_max", "up_row", "active_cap", "blocks", "x_step", "y_step",
+                  "ld_gate"), ("out_type", "activation", "accumulate"), ("alpha", "cap"))
+Batch = _struct("Batch", ("slot", "pos", "start", "n", "token_entry", "floor"), ("entries", "tokens", "max_n", "max_len", "first_entry", "first_token"))
+Attention = _struct("Attention", ("qkvg", "out", "k_cache", "v_cache", "v_first", "work", "q_norm", "k_norm", "rotary", "sink", "head_gate"),
+                    ("ld", "ldo", "k_off", "v_off", "g_off", "v_first_ld", "H", "Hkv", "dim", "vdim", "k_ld", "v_ld", "T_max", "slots", "q_ld", "rot_dims", "ld_gate",
+                     "window"), ("v_mix", "qk_norm", "gate", "rot_interleaved", "no_append"), ("mix", "eps", "scale"))
+Latent = _struct("Latent", ("down", "cq", "cache", "q_norm", "kv_norm", "rotary"), ("ld", "ld_cq", "kv_off", "q_rank", "kv_rank", "rot_dim", "c_ld", "T_max"), (),
+                 ("eps",))
+Expand = _struct("Expand", ("cache", "c", "K", "floor", "pos2"), ("c_ld", "T_max", "kv_rank", "rot_dim", "ld_c", "k_ld", "T", "dim", "heads", "max_rows"))
+Mlstm = _struct("Mlstm", ("qkvg", "gates", "bias", "norm", "out", "state", "work"), ("ld", "ld_gates", "ldo", "k_off", "v_off", "g_off", "heads", "dim", "vdim"), (),
+                ("cap", "eps", "q_scale"))
 Route = _struct("Route", ("logits", "pair_row", "pair_weight", "row_token", "group_offset", "active", "shared_weight", "choice", "counters"),
                 ("n", "ldl", "experts", "top", "active_cap"), ("sg_col",))
 
@@ -36,6 +41,13 @@ SYMBOLS = {
     "cuda_b200_linear_rows": (_i, [_i, _u, C.POINTER(Linear), _vp, _u, _i]),
     "cuda_b200_attention_work_bytes": (C.c_ulonglong, [_u]),
     "cuda_b200_attention_rows": (_i, [_i, C.POINTER(Attention), C.POINTER(Batch), _vp, _u, _i]),
+    "cuda_b200_rotary_table": (_i, [_vp, _u, _u, C.c_double, _vp]),
+    "cuda_b200_latent_down": (_i, [_i, C.POINTER(Latent), C.POINTER(Batch), _vp, _u]),
+    "cuda_b200_latent_query": (_i, [_i, _vp, _u, _u, _u, _vp, _u, _u, _u, _u, _u, _vp, _u, C.POINTER(Batch), _vp, _u]),
+    "cuda_b200_latent_expand": (_i, [_i, C.POINTER(Expand), C.POINTER(Batch), _vp, _u]),
+    "cuda_b200_mlstm_state_floats": (C.c_ulonglong, [_u, _u]),
+    "cuda_b200_mlstm_work_floats": (C.c_ulonglong, [_u, _u, _u, _u]),
+    "cuda_b200_mlstm_rows": (_i, [_i, C.POINTER(Mlstm), C.POINTER(Batch), _vp, _u, _i]),
     "cuda_b200_route_rows": (_i, [C.POINTER(Route), _vp, _u]),
     "cuda_b200_gather_rows": (_i, [_i, _vp, _u, _vp, _vp, _u, _u, _u, _vp, _u]),
     "cuda_b200_argmax_f32": (_i, [_vp, _u, _u, _u, _vp, _vp, _vp, _u]),
@@ -101,6 +113,35 @@ def attention(dtype, desc, batch, flags=0, kernel=0):
 
 def attention_work_bytes(vdim):
     return int(lib().cuda_b200_attention_work_bytes(vdim))
+
+
+def rotary_table(table, rows, dims, base):
+    return lib().cuda_b200_rotary_table(_ptr(table), rows, dims, base, _stream())
+
+
+def latent_down(dtype, desc, batch, flags=0):
+    return lib().cuda_b200_latent_down(dtype, C.byref(desc), C.byref(batch), _stream(), flags)
+
+
+def latent_query(dtype, src, ld_src, src_step, src_off, dst, ld_dst, dst_step, dst_off, heads, rot_dim, rotary, T_max, batch, flags=0):
+    return lib().cuda_b200_latent_query(dtype, _ptr(src), ld_src, src_step, src_off, _ptr(dst), ld_dst, dst_step, dst_off, heads, rot_dim, _ptr(rotary), T_max,
+                                        C.byref(batch), _stream(), flags)
+
+
+def latent_expand(dtype, desc, batch, flags=0):
+    return lib().cuda_b200_latent_expand(dtype, C.byref(desc), C.byref(batch), _stream(), flags)
+
+
+def mlstm_state_floats(dim, vdim):
+    return int(lib().cuda_b200_mlstm_state_floats(dim, vdim))
+
+
+def mlstm_work_floats(tokens, heads, dim, vdim):
+    return int(lib().cuda_b200_mlstm_work_floats(tokens, heads, dim, vdim))
+
+
+def mlstm(dtype, desc, batch, flags=0, kernel=0):
+    return lib().cuda_b200_mlstm_rows(dtype, C.byref(desc), C.byref(batch), _stream(), flags, kernel)
 
 
 def route(desc, flags=0):

@@ -14,7 +14,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 FLOAT32, BFLOAT16 = 0, 3
 DTYPES = {"float32": FLOAT32, "bfloat16": BFLOAT16}
 # architectures made of the decoder library's operations; the others need the quantized path's libraries as well
-DECODER_ARCHITECTURES = ("Fakilorn",)
+DECODER_ARCHITECTURES = ("Fakilorn", "Tazunex")
 
 _vp, _i, _u, _f, _ip, _fp = C.c_void_p, C.c_int, C.c_uint, C.c_float, C.POINTER(C.c_int), C.POINTER(C.c_float)
 SYMBOLS = {

@@ -1,7 +1,8 @@
 /*
  * C-ABI of the layer operations for decoders that keep their weights in BF16 (or float): the residual stream in
- * float, linears with fused epilogues, layer / RMS norm, attention over a KV cache with separate key and value sizes,
- * mixture-of-experts routing, greedy choice over float logits.  Library: libcccc-b200-decoder.so.
+ * float, linears with fused epilogues, layer / RMS norm, attention over a KV cache with separate key and value sizes
+ * (rotary positions, windows, sinks), latent attention, the mLSTM recurrence, mixture-of-experts routing, greedy choice
+ * over float logits.  Library: libcccc-b200-decoder.so.
  *
  * `dtype` says how weights, activations and caches are held: 3 (BF16, float accumulation) or 0 (float, everything in
  * true float).  Pointers are device pointers; `stream` is a cudaStream_t; every call is asynchronous.  flags bit 0:
@@ -16,7 +17,7 @@
 #define C_EXPORT extern "C" __attribute__((visibility("default")))
 #endif
 
-enum { B200_ACT_NONE = 0, B200_ACT_RELU2 = 1, B200_ACT_SILU_GATE = 2 };
+enum { B200_ACT_NONE = 0, B200_ACT_RELU2 = 1, B200_ACT_SILU_GATE = 2, B200_ACT_GELU_GATE = 3, B200_ACT_SOFTCAP = 4 };
 enum { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 };
 
 /* X[i][:] = scale * table[ids[i]][:] into the float residual stream; an id outside [0, vocab) gives zeros. */
@@ -25,9 +26,10 @@ C_EXPORT int cuda_b200_embed_f32(int dtype, const void* ids, const void* table, 
 
 /* Adds pending branch outputs to the float residual stream, then normalises:
  *   X[r][:] += sum_s slot_weight[r * slots + s] * Y[slot_row[r * slots + s]][:]      (slots == 0: nothing)
+ *   X[r][:] += norm(branch[r][:])       (kind's norm without bias, branch_weight; branch NULL: nothing; not with slots)
  *   out[i][:] = norm(X[rows ? rows[i] : i][:])                                       (out NULL: only the addition)
  * kind B200_NORM_LAYER: (x - mean) / sqrt(var + eps) * weight + bias; B200_NORM_RMS: x / sqrt(mean(x^2) + eps) *
- * weight (bias ignored).  weight and bias are float (NULL: 1 and 0).  All sums in float.  `rows` only without slots. */
+ * weight (bias ignored).  weight and bias are float (NULL: 1 and 0).  All sums in float.  `rows` only without slots or branch. */
 typedef struct cuda_b200_norm
 {
     void* X;
@@ -38,7 +40,9 @@ typedef struct cuda_b200_norm
     const void* slot_row;      /* int32 */
     const void* slot_weight;   /* float */
     const void* rows;          /* int32 */
-    unsigned int n, width, ldx, ldo, ldy, slots;
+    const void* branch;        /* float */
+    const void* branch_weight; /* float */
+    unsigned int n, width, ldx, ldo, ldy, slots, ldb;
     int kind;
     float eps;
 } cuda_b200_norm;
@@ -48,7 +52,11 @@ C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* strea
  * Dense (group_offset NULL): rows r = 0..rows-1, xr = r.  Grouped: group g owns the Y rows group_offset[g] ..
  * group_offset[g+1]-1 and the weight rows starting at g * group_rows; xr = x_row ? x_row[r] : r; `rows` is the most rows
  * all groups hold together, group_max the most rows one of them holds.
- * activation B200_ACT_SILU_GATE: feature n uses weight rows n (gate) and up_row + n, Y = silu(gate) * up.
+ * activation B200_ACT_SILU_GATE / _GELU_GATE: feature n uses weight rows n (gate) and up_row + n, Y = act(gate) * up (GELU
+ * in its tanh form); B200_ACT_SOFTCAP: Y = cap * tanh(z / cap).
+ * Block-diagonal (blocks > 1, not grouped): block b is a linear of its own, weight rows from b * group_rows, X columns from
+ * b * x_step, Y columns from b * y_step (X's columns behind K up to the next multiple of 64 hold finite values; x_step a
+ * multiple of 8).  head_gate: block b of row r is multiplied by sigmoid(head_gate[r * ld_gate + b]) (dtype).
  * out_type 0: float (accumulate != 0: Y += row_scale[r] * result), 3: BF16 (float mode: always 0).  row_scale: float per
  * row, or NULL. */
 typedef struct cuda_b200_linear
@@ -60,10 +68,12 @@ typedef struct cuda_b200_linear
     const void* group_offset;   /* int32, groups + 1 */
     const void* x_row;          /* int32 */
     const void* active;         /* int32: ids of the non-empty groups, -1 behind them; `active_cap` entries (NULL: all groups) */
+    const void* head_gate;
     unsigned int rows, N, K, ldw, ldx, ldy;
     unsigned int groups, group_rows, group_max, up_row, active_cap;
+    unsigned int blocks, x_step, y_step, ld_gate;
     int out_type, activation, accumulate;
-    float alpha;
+    float alpha, cap;
 } cuda_b200_linear;
 /* Up to three independent members.  BF16: where no member has more than 32 rows (in one group), one launch of a weight-
  * streaming kernel runs all of them that hold about as many rows; else one tcgen05 launch per member (x_row not taken there).  kernel: 0 = by shape,
@@ -71,7 +81,8 @@ typedef struct cuda_b200_linear
 C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b200_linear* members, void* stream, unsigned int flags, int kernel);
 
 /* A step's ragged batch: entry e brings n[e] tokens, rows start[e].. of the flat token arrays, which continue the
- * sequence in cache slot slot[e] at position pos[e].  token_entry[i] is the entry of token i.  Device int32 arrays. */
+ * sequence in cache slot slot[e] at position pos[e].  token_entry[i] is the entry of token i.  Device int32 arrays.  A call
+ * runs the entries first_entry .. first_entry + entries - 1, whose tokens are first_token .. first_token + tokens - 1. */
 typedef struct cuda_b200_batch
 {
     const void* slot;
@@ -79,26 +90,45 @@ typedef struct cuda_b200_batch
     const void* start;
     const void* n;
     const void* token_entry;
+    const void* floor;                      /* nullable: attention does not let entry e see keys below floor[e] */
     unsigned int entries, tokens, max_n;    /* max_n: the largest n[e]; launch bounds only */
     unsigned int max_len;                   /* no sequence is longer than this after the step; launch bounds only */
+    unsigned int first_entry, first_token;
 } cuda_b200_batch;
 
-/* Attention of a layer from its projections on.  First, for every token of the batch: q heads to unit RMS in place
- * (qk_norm), k heads to unit RMS and v (mixed with v_first: v = (1 - mix) v + mix v_first) appended to the caches,
- * v_first stored.  Caches hold rows of k_ld / v_ld elements (multiples of 8) whose padding is zero.  A batch entry's
- * sequence must fit: pos + n <= T_max.  qkvg, the caches and work are 16-byte aligned. */
+/* cos and sin of p * base^(-2i / dims) for p < rows, i < dims / 2: table[p][i] = (cos, sin), floats, computed in double. */
+C_EXPORT int cuda_b200_rotary_table(void* table, unsigned int rows, unsigned int dims, double base, void* stream);
+
+/* Attention of a layer from its projections on.  First (append), for every token of the batch: q and k are normalised (qk_norm:
+ * every head to unit RMS; q_norm / k_norm: the whole projection to unit RMS, times these weights) and rotated (rotary: the first
+ * rot_dims elements of each head; element i goes with i + rot_dims / 2, or, interleaved, 2i with 2i + 1), q in place, k
+ * appended to its cache; v (mixed with v_first: v = (1 - mix) v + mix v_first) appended as projected, v_first stored.  v_off
+ * may be k_off: the values are the keys as projected.  Caches hold rows of k_ld / v_ld elements (multiples of 8) whose padding
+ * is zero; k_cache and v_cache may be one (vdim <= dim) with append off.  A batch entry's sequence must fit: pos + n <= T_max.
+ * qkvg, the caches and work are 16-byte aligned. */
 typedef struct cuda_b200_attention
 {
-    void* qkvg;                /* [tokens][ld] dtype: q at 0, k at k_off, v at v_off, output gate at g_off */
+    void* qkvg;                /* [tokens][ld] dtype: q at 0 (a head every q_ld), k at k_off, v at v_off, output gate at g_off */
     void* out;                 /* [tokens][ldo] dtype: H * vdim */
     void* k_cache;             /* [slots][Hkv][T_max][k_ld] dtype */
     void* v_cache;             /* [slots][Hkv][T_max][v_ld] dtype */
     void* v_first;             /* [tokens][v_first_ld] dtype: written (v_mix 1) or read (v_mix 2) */
     void* work;                /* float scratch of cuda_b200_attention_work_bytes, zeroed once */
+    const void* q_norm;        /* float [H * dim] */
+    const void* k_norm;        /* float [Hkv * dim] */
+    const void* rotary;        /* cuda_b200_rotary_table of T_max rows */
+    const void* sink;          /* float [H]: a score that takes part in the softmax denominator only */
+    const void* head_gate;     /* [tokens][ld_gate] dtype: head h's output is multiplied by sigmoid(head_gate[h]) */
     unsigned int ld, ldo, k_off, v_off, g_off, v_first_ld;
     unsigned int H, Hkv, dim, vdim, k_ld, v_ld, T_max, slots;
+    unsigned int q_ld;         /* 0: dim.  Others only with append off */
+    unsigned int rot_dims;     /* even */
+    unsigned int ld_gate;
+    unsigned int window;       /* a token sees itself and the window - 1 before it; 0: all */
     int v_mix;                 /* 0: plain, 1: this layer's values are the ones later layers mix in, 2: mix */
-    int qk_norm, gate;         /* 1: unit RMS of q and k; multiply the output by sigmoid(gate) */
+    int qk_norm, gate;         /* 1: unit RMS of q and k heads; multiply the output by sigmoid(gate) */
+    int rot_interleaved;
+    int no_append;             /* 1: the queries are ready and the caches hold the batch's keys and values */
     float mix, eps, scale;
 } cuda_b200_attention;
 C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
@@ -109,6 +139,63 @@ C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
  * tcgen05 (prompts; sizes up to 128, caches 16-byte aligned, `slots` given: the caches end after that many). */
 C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, const cuda_b200_batch* b, void* stream, unsigned int flags,
     int kernel);
+
+/* Latent attention keeps per token one row [latent | rotated key part] for all heads.
+ * _down: for every token of the batch, query latent cq = rms_norm(down[0 .. q_rank)) * q_norm, and the cache row
+ * [rms_norm(down[kv_off .. + kv_rank)) * kv_norm | rotated down[kv_off + kv_rank .. + rot_dim)]; pairs are 2i and 2i + 1.
+ * _query: dst[t][h * dst_step + dst_off ..] = rotated src[t][h * src_step + src_off .. + rot_dim).  src may be dst.
+ * _expand (prompts): the cache rows that entry e's tokens may read, the last n + pos2 - floor of its first pos + n, go one behind
+ * the other to rows floor[e] .. pos2[e] + n[e] - 1: the latents into c, the rotated part beside every head's key, K[h][row][dim
+ * .. dim + rot_dim). */
+typedef struct cuda_b200_latent
+{
+    const void* down;          /* [tokens][ld] dtype */
+    void* cq;                  /* [tokens][ld_cq] dtype */
+    void* cache;               /* [slots][T_max][c_ld] dtype */
+    const void* q_norm;        /* float */
+    const void* kv_norm;       /* float */
+    const void* rotary;        /* cuda_b200_rotary_table of T_max rows */
+    unsigned int ld, ld_cq, kv_off, q_rank, kv_rank, rot_dim, c_ld, T_max;
+    float eps;
+} cuda_b200_latent;
+C_EXPORT int cuda_b200_latent_down(int dtype, const cuda_b200_latent* a, const cuda_b200_batch* b, void* stream, unsigned int flags);
+C_EXPORT int cuda_b200_latent_query(int dtype, const void* src, unsigned int ld_src, unsigned int src_step, unsigned int src_off, void* dst,
+    unsigned int ld_dst, unsigned int dst_step, unsigned int dst_off, unsigned int heads, unsigned int rot_dim, const void* rotary, unsigned int T_max,
+    const cuda_b200_batch* b, void* stream, unsigned int flags);
+typedef struct cuda_b200_expand
+{
+    const void* cache;         /* [slots][T_max][c_ld] dtype */
+    void* c;                   /* [rows][ld_c] dtype */
+    void* K;                   /* [heads][T][k_ld] dtype */
+    const void* floor;         /* int32 per entry */
+    const void* pos2;          /* int32 per entry */
+    unsigned int c_ld, T_max, kv_rank, rot_dim, ld_c, k_ld, T, dim, heads;
+    unsigned int max_rows;     /* the most rows an entry has; launch bounds only */
+} cuda_b200_expand;
+C_EXPORT int cuda_b200_latent_expand(int dtype, const cuda_b200_expand* a, const cuda_b200_batch* b, void* stream, unsigned int flags);
+
+/* The mLSTM recurrence (xLSTM's matrix memory) of a layer from its projections on, per head, in float:
+ *   i = cap tanh((gate_i + i_bias) / cap), f = log sigmoid(cap tanh((gate_f + f_bias) / cap)), m' = max(f + m, i),
+ *   S' = e^(f + m - m') S + e^(i - m') k v^T, n' = e^(f + m - m') n + e^(i - m') k, o = S'^T q / (max(|n' q|, e^-m') + 1e-6),
+ * q times q_scale, then o to unit RMS over the head, times `norm`, times sigmoid(output gate).  A sequence at position 0 starts
+ * from zeros (also m), whatever its slot holds. */
+typedef struct cuda_b200_mlstm
+{
+    const void* qkvg;          /* [tokens][ld] dtype: q at 0 (heads * dim), k at k_off, v at v_off (heads * vdim), gate at g_off */
+    const void* gates;         /* float [tokens][ld_gates]: heads input gates, heads forget gates */
+    const void* bias;          /* float [2 * heads], as the gates */
+    const void* norm;          /* float [heads * vdim] */
+    void* out;                 /* [tokens][ldo] dtype: heads * vdim */
+    void* state;               /* float [slots][heads][cuda_b200_mlstm_state_floats] */
+    void* work;                /* float scratch of cuda_b200_mlstm_work_floats, 16-byte aligned */
+    unsigned int ld, ld_gates, ldo, k_off, v_off, g_off;
+    unsigned int heads, dim, vdim;
+    float cap, eps, q_scale;
+} cuda_b200_mlstm;
+C_EXPORT unsigned long long cuda_b200_mlstm_state_floats(unsigned int dim, unsigned int vdim);
+C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int heads, unsigned int dim, unsigned int vdim);
+/* kernel: 0 = by shape, 1 = token by token, any size. */
+C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cuda_b200_batch* b, void* stream, unsigned int flags, int kernel);
 
 /* Router: the `top` largest of each row of float logits [n][ldl] (ties: the lower expert), softmax over them; the
  * pairs (token, choice) are dealt to groups: pair_row[t * slots + s] = its row in group order, pair_weight, row_token[row]

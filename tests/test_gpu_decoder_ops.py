@@ -240,7 +240,7 @@ def test_a_group_of_members_is_the_separate_launches(D):
 def test_descriptors_that_are_not_taken(D):
     X = padded(np.ones((2, 64)), BF16)
     base = dict(W=X, X=X, Y=X, rows=2, N=2, K=64, ldw=64, ldx=64, ldy=64, alpha=1.0)
-    for bad in (dict(ldw=72), dict(K=65), dict(X=X.data_ptr() + 2), dict(activation=3), dict(accumulate=1, out_type=3), dict(W=None)):
+    for bad in (dict(ldw=72), dict(K=65), dict(X=X.data_ptr() + 2), dict(activation=5), dict(activation=4), dict(blocks=2, x_step=4), dict(accumulate=1, out_type=3), dict(W=None)):
         assert D.linear(BF16, [D.fill(D.Linear, **{**base, **bad})]) == -1, bad
     assert D.linear(FLOAT, [D.fill(D.Linear, **{**base, "out_type": 3})]) == -1
     assert D.linear(7, [D.fill(D.Linear, **base)]) == -1
