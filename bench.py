@@ -22,8 +22,8 @@ With N>1 (launched under torchrun, one rank per GPU) the same token is computed 
 q/k/v/gate/up/lm_head split by output feature, o/down split by input feature with the all-reduce fused
 into their kernel, logits all-gathered; `value` stays whole-job bytes of the unsharded model per second.
 
-`--decoder` instead times decode and prefill steps of Fakilorn models (BF16 weights, random) with layers of a real
-model's size, beside the quantised model's at equal size.
+`--decoder` instead times decode and prefill steps of Fakilorn and Tazunex models (BF16 weights, random) with layers of a
+real model's size, beside the quantised model's at equal size.
 
 `--impl reference` times the reference's CPU form of the path (its types.h decode to float, then
 OpenBLAS sgemm) on all host cores, each step a bounded sample of the same workload.
@@ -735,7 +735,7 @@ def gpu_arm(args):
         os._exit(0)
 
 
-# ---- Fakilorn beside the quantised model (--decoder) ----------------------------------------------------
+# ---- Fakilorn and Tazunex beside the quantised model (--decoder) ----------------------------------------------------
 def decoder_cases(layers):
     """Layers of a real model's size: `dense` has the headline model's own (its linears in BF16), `experts` a routed one's."""
     q = QWEN
@@ -744,7 +744,22 @@ def decoder_cases(layers):
     base = lambda width, vocab, mixer, mlp: dict(architecture="Fakilorn", width=width, vocab=vocab, embedding=dict(scale=8.0), logit_scale=1.0, norm=dict(eps=1e-5),
                                                  layers=[dict(type="attention", mixer=mixer, mlp=mlp)] * layers)
     return {"dense": base(q["HIDDEN"], q["VOCAB"], attn, dict(kind="dense", ff=q["FFN"])),
-            "experts": base(2048, 65536, dict(attn, heads=16, kv_heads=4), moe)}
+            "experts": base(2048, 65536, dict(attn, heads=16, kv_heads=4), moe), **tazunex_cases(layers)}
+
+
+def tazunex_cases(layers):
+    """Tazunex at the dense model's sizes: its three mixers in turn, and each alone."""
+    q = QWEN
+    mask, rot = dict(size=CONTEXT), lambda dims: dict(base=1e6, dims=dims)
+    mixers = {
+        "mlstm": dict(heads=8, dim=256, vdim=512, gate_cap=15.0),
+        "attention": dict(heads=q["HEADS"], kv_heads=q["KVHEADS"], dim=q["HD"], vdim=q["HD"], scale=q["HD"] ** -0.5, mask=mask, rot=rot(q["HD"])),
+        "latent_attention": dict(heads=q["HEADS"], dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, scale=192 ** -0.5, mask=mask, rot=rot(64)),
+    }
+    model = lambda kinds: dict(architecture="Tazunex", width=q["HIDDEN"], vocab=q["VOCAB"], norm=dict(eps=1e-6), logit_softcap=30.0,
+                               layers=[dict(type=k, mixer=mixers[k], mlp=dict(kind="dense", ff=q["FFN"])) for k in kinds])
+    turn = ["mlstm", "attention", "mlstm", "latent_attention"] * layers
+    return {"tazunex": model(turn[:layers]), **{f"tazunex_{k}": model([k] * layers) for k in mixers}}
 
 
 def decoder_work(c, tokens, sequences, context):
@@ -754,6 +769,13 @@ def decoder_work(c, tokens, sequences, context):
     nbytes, flops, aflops = 2 * c["vocab"] * W, 2 * c["vocab"] * W * sequences, 0
     for L in c["layers"]:
         m, f = L["mixer"], L["mlp"]
+        if c["architecture"] == "Tazunex":
+            w, cache, a = tazunex_mixer_work(L["type"], m, W, tokens, context)
+            w += 3 * W * f["ff"]
+            nbytes += 2 * w + cache * sequences
+            flops += 2 * w * T
+            aflops += a * sequences
+            continue
         H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         w = W * (H * d + G * d + G * dv + 2 * H * dv)
         active = w
@@ -770,8 +792,22 @@ def decoder_work(c, tokens, sequences, context):
     return nbytes, flops, aflops
 
 
+def tazunex_mixer_work(kind, m, W, tokens, context):
+    """(weights, bytes of cache or state and flops besides the linears per sequence) of a mixer."""
+    H, d, dv = m["heads"], m["dim"], m["vdim"]
+    pairs = tokens * context + tokens * (tokens + 1) // 2
+    if kind == "mlstm":
+        # state in and out; per token S^T q and k v^T
+        return W * (2 * H * d + 3 * H * dv + 2 * H), 8 * H * d * dv, 4 * H * d * dv * tokens
+    if kind == "attention":
+        return W * (H * d + m["kv_heads"] * d + H * dv), 2 * (context + tokens) * m["kv_heads"] * (d + dv), 2 * H * (d + dv) * pairs
+    R, r = m["kv_rank"], m["rot_dim"]
+    w = W * (m["q_rank"] + R + r + H + H * dv) + m["q_rank"] * H * (d + r) + R * H * (d + dv)
+    return w, 2 * (context + tokens) * (R + r), 2 * H * (d + r + dv) * pairs
+
+
 def decoder_arm(args):
-    """Fakilorn with random weights through the serving interface, and the quantised model's decode step and prefill linears
+    """Fakilorn and Tazunex with random weights through the serving interface, and the quantised model's decode step and prefill linears
     at the same layer sizes, in one JSON line."""
     import importlib
     import tempfile
@@ -794,6 +830,8 @@ def decoder_arm(args):
     sampler.start()
     launches = pkg.decoder_capi.launches()
     for name, c in decoder_cases(layers).items():
+        if args.only and name not in args.only.split(","):
+            continue
         with tempfile.TemporaryDirectory() as d:
             with open(os.path.join(d, "config.json"), "w") as f:
                 json.dump(c, f)
@@ -815,11 +853,12 @@ def decoder_arm(args):
     # the closest model at equal size: FP8 weights, RMSNorm, RoPE, SwiGLU; its decode step, and its prefill linears
     capi, dm = pkg.capi, importlib.import_module("cccc_lite_b200.decode_model")
     dims = model_dims("e5m2", layers)
-    wt, lin, bufs = build_model(torch, capi, dims, 32, "e5m2", 0, 1, dev)
-    model = decode_step_model(torch, capi, dm, dims, wt, lin, 1, 0, 32, dev, bufs)
-    stream = torch.cuda.Stream(dev)
-    out["quantised"] = {f"decode_batch{B}": time_decode_step(torch, None, capi, model, dims, B, "e5m2", 1, 20, dev, stream, 1) for B in (1, 8, 32)}
-    out["quantised"]["prefill_linears_2048"] = prefill_probe(torch, capi, dims, "e5m2", dev, peaks)
+    if not args.only or "quantised" in args.only.split(","):
+        wt, lin, bufs = build_model(torch, capi, dims, 32, "e5m2", 0, 1, dev)
+        model = decode_step_model(torch, capi, dm, dims, wt, lin, 1, 0, 32, dev, bufs)
+        stream = torch.cuda.Stream(dev)
+        out["quantised"] = {f"decode_batch{B}": time_decode_step(torch, None, capi, model, dims, B, "e5m2", 1, 20, dev, stream, 1) for B in (1, 8, 32)}
+        out["quantised"]["prefill_linears_2048"] = prefill_probe(torch, capi, dims, "e5m2", dev, peaks)
     out["gpu_launches"] = pkg.decoder_capi.launches() - launches
     out["clocks"] = sampler.stop()
     print(json.dumps(out), flush=True)
@@ -1139,7 +1178,8 @@ def main():
     ap.add_argument("--watchdog", type=float, default=540.0, help="seconds after which a stuck run exits by itself")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--decoder", action="store_true",
-                    help="instead of the headline: Fakilorn's decode and prefill steps beside the quantised model's at equal layer sizes")
+                    help="instead of the headline: Fakilorn's and Tazunex's decode and prefill steps beside the quantised model's at equal layer sizes")
+    ap.add_argument("--only", default="", help="with --decoder: the cases to time, with commas between them (dense, experts, tazunex, ..., quantised)")
     args = ap.parse_args()
     if args.decoder:
         decoder_arm(args)

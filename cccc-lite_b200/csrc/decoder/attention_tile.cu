@@ -1,5 +1,6 @@
 // BF16 attention of prompts on tcgen05, tensor-bound: 128 packed query rows per CTA (a row is one query head of one token;
-// heads that share a kv head are packed together) against 64-key tiles, two CTAs per SM.
+// heads that share a kv head are packed together) against 64-key tiles, two CTAs per SM (one where keys and values are larger
+// than 128).
 //
 // A TMA lane streams keys and values from the cache (128-byte swizzle) through two-deep rings; the MMA lane issues
 // S = Q K^T (M = 128, N = 64) into tensor memory and, once the softmax warps have turned S into weights, O += P V with P as
@@ -11,6 +12,8 @@
 #include "attention.cuh"
 #include "../gemm_stream.cuh"
 
+#include <type_traits>
+
 namespace b200
 {
 
@@ -19,7 +22,9 @@ constexpr int TA_THREADS = 192;
 constexpr int TA_BLOCK = TA_KT * 128;          // 64 keys x 64 elements
 constexpr int TA_QBLOCK = TA_ROWS * 128;       // 128 rows x 64 elements
 __host__ __device__ constexpr int ta_smem(int dk, int dv) { return 1024 + (dk / 64) * TA_QBLOCK + 2 * (dk / 64 + dv / 64) * TA_BLOCK + 1024; }
-constexpr uint32_t TA_TMEM = 256, TA_O = 128;    // columns: two places of S (64) or P (32 high, 32 low), then O
+constexpr uint32_t TA_O = 128;    // columns: two places of S (64) or P (32 high, 32 low), then O
+__host__ __device__ constexpr uint32_t ta_tmem(int dv) { return dv <= 128 ? 256 : 512; }
+__host__ __device__ constexpr int ta_ctas(int dk, int dv) { return ta_smem(dk, dv) <= 113 * 1024 && dv <= 128 ? 2 : 1; }
 
 // An MN-major operand [k][64 elements] with the 128-byte swizzle: 8-k groups 1024 bytes apart, 64-element blocks TA_BLOCK apart.
 __device__ __forceinline__ uint64_t umma_desc_mnmajor_sw128(uint32_t smem_addr)
@@ -43,7 +48,7 @@ __device__ __forceinline__ float exp2_f32(float x)
 __device__ __forceinline__ float gate_sigmoid(float z) { return __fdividef(1.0f, 1.0f + exp2_f32(-1.44269504088896341f * z)); }
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+__global__ void __launch_bounds__(TA_THREADS, ta_ctas(DK, DV)) attention_tile_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     const __grid_constant__ AttnParams p, unsigned int* status)
 {
     extern __shared__ unsigned char ta_raw[];
@@ -51,8 +56,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
     constexpr int KBY = (DK / 64) * TA_BLOCK, VBY = (DV / 64) * TA_BLOCK;
     uint64_t* k_full = reinterpret_cast<uint64_t*>(smem);
     uint64_t *k_empty = k_full + 2, *v_full = k_full + 4, *v_empty = k_full + 6;
-    uint64_t *s_full = k_full + 8, *p_ready = k_full + 10, *q_ready = k_full + 12, *pv_done = k_full + 13;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 14);
+    uint64_t *s_full = k_full + 8, *p_ready = k_full + 10, *q_ready = k_full + 12, *pv_done = k_full + 13, *o_full = k_full + 14;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 15);
     volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
     unsigned char* qs = smem + 1024;
     unsigned char* ks = qs + (DK / 64) * TA_QBLOCK;
@@ -66,10 +71,11 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
         mbar_init(p_ready, 4);    // one per place: a warp may be a tile ahead of another
         mbar_init(p_ready + 1, 4);
         mbar_init(pv_done, 1);
+        mbar_init(o_full, 1);
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    if (warp == 1) { tmem_alloc(tmem_slot, TA_TMEM); }
+    if (warp == 1) { tmem_alloc(tmem_slot, ta_tmem(DV)); }
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int kvh = blockIdx.y, e = p.e0 + blockIdx.z;
@@ -179,6 +185,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
                 }
                 umma_commit(v_empty + (i & 1u));
                 umma_commit(pv_done);
+                if (i + 1 == tiles) { umma_commit(o_full); }
             }
             __syncwarp();
             // into the place of the weights just issued: products of one thread run in the order of their issue
@@ -302,9 +309,8 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
             __syncwarp();
             if (lane == 0) { mbar_arrive(p_ready + (i & 1u)); }
         }
-        // in turn, since a wait tells only neighbouring phases apart (the scores of the last tile came after product tiles - 3)
-        if (tiles > 1) { ok = ok && __all_sync(0xFFFFFFFFu, wait(pv_done, tiles - 2)); }
-        ok = ok && __all_sync(0xFFFFFFFFu, wait(pv_done, tiles - 1));
+        // a barrier of its own: a wait tells only neighbouring phases apart, and pv_done may be one or two further by now
+        ok = ok && __all_sync(0xFFFFFFFFu, wait(o_full, 0));
         if (ok)
         {
             tc_fence_after();
@@ -366,7 +372,7 @@ __global__ void __launch_bounds__(TA_THREADS, 2) attention_tile_kernel(const __g
     }
     tc_fence_before();
     __syncthreads();
-    if (warp == 1) { tmem_dealloc(tmem, TA_TMEM); }
+    if (warp == 1) { tmem_dealloc(tmem, ta_tmem(DV)); }
 }
 
 template <int DK, int DV>
@@ -382,7 +388,7 @@ int launch_attention_tile(const AttnParams& p, unsigned int slots, unsigned int 
 {
     const unsigned long long rows = (unsigned long long)slots * p.Hkv * p.T_max;
     auto low = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) != 0; };
-    if (p.dim > 128 || p.vdim > 128 || slots == 0 || rows > 0x7FFFFFFFull || low(p.k_cache) || low(p.v_cache) || low(p.qkvg) || low(p.out) || (p.ld % 8)
+    if (p.dim > 256 || p.vdim > 256 || slots == 0 || rows > 0x7FFFFFFFull || low(p.k_cache) || low(p.v_cache) || low(p.qkvg) || low(p.out) || (p.ld % 8)
         || (p.ldo % 8) || entries > 65535u || p.Hkv > 65535u)
     {
         return -1;
@@ -393,8 +399,17 @@ int launch_attention_tile(const AttnParams& p, unsigned int slots, unsigned int 
     {
         return -1;
     }
-    if (p.dim <= 64) { return p.vdim <= 64 ? run_tile<64, 64>(p, tk, tv, entries, max_n, stream, pdl) : run_tile<64, 128>(p, tk, tv, entries, max_n, stream, pdl); }
-    return p.vdim <= 64 ? run_tile<128, 64>(p, tk, tv, entries, max_n, stream, pdl) : run_tile<128, 128>(p, tk, tv, entries, max_n, stream, pdl);
+    auto by_values = [&](auto dk) {
+        constexpr int DK = decltype(dk)::value;
+        if (p.vdim <= 64) { return run_tile<DK, 64>(p, tk, tv, entries, max_n, stream, pdl); }
+        if (p.vdim <= 128) { return run_tile<DK, 128>(p, tk, tv, entries, max_n, stream, pdl); }
+        if (p.vdim <= 192) { return run_tile<DK, 192>(p, tk, tv, entries, max_n, stream, pdl); }
+        return run_tile<DK, 256>(p, tk, tv, entries, max_n, stream, pdl);
+    };
+    if (p.dim <= 64) { return by_values(std::integral_constant<int, 64>()); }
+    if (p.dim <= 128) { return by_values(std::integral_constant<int, 128>()); }
+    if (p.dim <= 192) { return by_values(std::integral_constant<int, 192>()); }
+    return by_values(std::integral_constant<int, 256>());
 }
 
 }    // namespace b200

@@ -103,10 +103,11 @@ __device__ __forceinline__ float rotated(const float* head, unsigned int d, unsi
     return second ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
 }
 
+// A launch in clusters of `cluster` CTAs along x (1: none).
 template <class K, class... Args>
-static int launch_kernel(const char* label, K kernel, dim3 grid, dim3 block, size_t smem, void* stream, bool pdl, Args... args)
+static int launch_cluster(const char* label, K kernel, dim3 grid, dim3 block, size_t smem, unsigned int cluster, void* stream, bool pdl, Args... args)
 {
-    if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     {
         report_launch(label);
         return 1;
@@ -117,11 +118,20 @@ static int launch_kernel(const char* label, K kernel, dim3 grid, dim3 block, siz
     cfg.blockDim = block;
     cfg.dynamicSmemBytes = smem;
     cfg.stream = (cudaStream_t)stream;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cudaLaunchAttribute attr[2];
     cfg.attrs = attr;
-    cfg.numAttrs = pdl ? 1 : 0;
+    if (pdl)
+    {
+        attr[cfg.numAttrs].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[cfg.numAttrs++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 1)
+    {
+        attr[cfg.numAttrs].id = cudaLaunchAttributeClusterDimension;
+        attr[cfg.numAttrs].val.clusterDim.x = cluster;
+        attr[cfg.numAttrs].val.clusterDim.y = 1;
+        attr[cfg.numAttrs++].val.clusterDim.z = 1;
+    }
     count_launch();
     if (cudaLaunchKernelEx(&cfg, kernel, args...) != cudaSuccess)
     {
@@ -129,6 +139,12 @@ static int launch_kernel(const char* label, K kernel, dim3 grid, dim3 block, siz
         return 1;
     }
     return 0;
+}
+
+template <class K, class... Args>
+static int launch_kernel(const char* label, K kernel, dim3 grid, dim3 block, size_t smem, void* stream, bool pdl, Args... args)
+{
+    return launch_cluster(label, kernel, grid, block, smem, 1, stream, pdl, args...);
 }
 
 }    // namespace b200

@@ -128,9 +128,12 @@ using namespace b200;
 
 C_EXPORT unsigned long long cuda_b200_mlstm_state_floats(unsigned int dim, unsigned int vdim) { return mlstm_state_floats(dim, vdim); }
 
-C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int heads, unsigned int dim, unsigned int vdim)
+C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim,
+    unsigned int vdim)
 {
-    return (unsigned long long)tokens * heads * (vdim + dim + 1);
+    const unsigned long long plain = (unsigned long long)tokens * heads * (vdim + dim + 1);
+    const unsigned long long chunks = mlstm_chunk_takes(dim, vdim) ? mlstm_chunk_floats(tokens, entries, heads, dim, vdim) : 0;
+    return plain > chunks ? plain : chunks;
 }
 
 C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cuda_b200_batch* b, void* stream, unsigned int flags, int kernel)
@@ -172,6 +175,16 @@ C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cud
     p.eps = a->eps;
     p.q_scale = a->q_scale;
     const bool pdl = (flags & 1u) != 0;
-    (void)kernel;
+    if (dtype == DT_FLOAT) { kernel = 1; }
+    if (kernel == 3 || (kernel == 0 && b->max_n > 8))
+    {
+        const int rc = launch_mlstm_chunk(p, b->entries, (cudaStream_t)stream, pdl);
+        if (rc != -1 || kernel == 3) { return rc; }
+    }
+    if (kernel == 0 || kernel == 2)
+    {
+        const int rc = launch_mlstm_step(p, b->entries, (cudaStream_t)stream, pdl);
+        if (rc != -1 || kernel == 2) { return rc; }
+    }
     return dtype == DT_BF16 ? mlstm_plain<__nv_bfloat16>(p, b->entries, stream, pdl) : mlstm_plain<float>(p, b->entries, stream, pdl);
 }

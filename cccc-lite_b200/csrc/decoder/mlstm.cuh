@@ -27,6 +27,12 @@ struct MlstmParams
     float cap, eps, q_scale;
 };
 
+// mlstm_step.cu, mlstm_chunk.cu (BF16): -1 where the sizes are not taken
+int launch_mlstm_step(const MlstmParams& p, unsigned int entries, cudaStream_t stream, bool pdl);
+int launch_mlstm_chunk(const MlstmParams& p, unsigned int entries, cudaStream_t stream, bool pdl);
+bool mlstm_chunk_takes(unsigned int dim, unsigned int vdim);
+unsigned long long mlstm_chunk_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim, unsigned int vdim);
+
 __device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
 // Logarithms of the input and the forget gate of a token's head.

@@ -162,7 +162,7 @@ bool LayeredDecoder::allocateMixers(const ModelOptions& o, std::string* err)
             shape.state_floats = (size_t)a.heads * cuda_b200_mlstm_state_floats((unsigned int)a.dim, (unsigned int)a.vdim);
             att = std::max(att, a.heads * a.vdim);
             gates = std::max(gates, 2 * a.heads);
-            mlstm = std::max(mlstm, cuda_b200_mlstm_work_floats((unsigned int)cap_, (unsigned int)a.heads, (unsigned int)a.dim, (unsigned int)a.vdim));
+            mlstm = std::max(mlstm, cuda_b200_mlstm_work_floats((unsigned int)cap_, (unsigned int)std::min(cap_, o.max_sequences), (unsigned int)a.heads, (unsigned int)a.dim, (unsigned int)a.vdim));
         }
         shapes.push_back(shape);
     }

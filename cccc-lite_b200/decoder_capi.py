@@ -46,7 +46,7 @@ SYMBOLS = {
     "cuda_b200_latent_query": (_i, [_i, _vp, _u, _u, _u, _vp, _u, _u, _u, _u, _u, _vp, _u, C.POINTER(Batch), _vp, _u]),
     "cuda_b200_latent_expand": (_i, [_i, C.POINTER(Expand), C.POINTER(Batch), _vp, _u]),
     "cuda_b200_mlstm_state_floats": (C.c_ulonglong, [_u, _u]),
-    "cuda_b200_mlstm_work_floats": (C.c_ulonglong, [_u, _u, _u, _u]),
+    "cuda_b200_mlstm_work_floats": (C.c_ulonglong, [_u, _u, _u, _u, _u]),
     "cuda_b200_mlstm_rows": (_i, [_i, C.POINTER(Mlstm), C.POINTER(Batch), _vp, _u, _i]),
     "cuda_b200_route_rows": (_i, [C.POINTER(Route), _vp, _u]),
     "cuda_b200_gather_rows": (_i, [_i, _vp, _u, _vp, _vp, _u, _u, _u, _vp, _u]),
@@ -136,8 +136,8 @@ def mlstm_state_floats(dim, vdim):
     return int(lib().cuda_b200_mlstm_state_floats(dim, vdim))
 
 
-def mlstm_work_floats(tokens, heads, dim, vdim):
-    return int(lib().cuda_b200_mlstm_work_floats(tokens, heads, dim, vdim))
+def mlstm_work_floats(tokens, entries, heads, dim, vdim):
+    return int(lib().cuda_b200_mlstm_work_floats(tokens, entries, heads, dim, vdim))
 
 
 def mlstm(dtype, desc, batch, flags=0, kernel=0):

@@ -136,7 +136,8 @@ C_EXPORT unsigned long long cuda_b200_attention_work_bytes(unsigned int vdim);
  * kernel: 0 = by shape, 1 = split-KV through shared memory (few query rows), 2 = tiled on mma.sync, 3 = the plain kernel
  * (always in float mode, and for key or value sizes above 256), 4 = split-KV straight into registers (sizes up to 128, k_ld
  * and v_ld multiples of 16, caches 32-byte aligned; with one token per entry the append is part of it), 5 = tiled on
- * tcgen05 (prompts; sizes up to 128, caches 16-byte aligned, `slots` given: the caches end after that many). */
+ * tcgen05 (prompts; sizes up to 256, caches 16-byte aligned, `slots` given: the caches end after that many), 6 = split
+ * over latent rows (k_cache is v_cache, Hkv 1; dim up to 576, vdim up to 512). */
 C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, const cuda_b200_batch* b, void* stream, unsigned int flags,
     int kernel);
 
@@ -193,8 +194,10 @@ typedef struct cuda_b200_mlstm
     float cap, eps, q_scale;
 } cuda_b200_mlstm;
 C_EXPORT unsigned long long cuda_b200_mlstm_state_floats(unsigned int dim, unsigned int vdim);
-C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int heads, unsigned int dim, unsigned int vdim);
-/* kernel: 0 = by shape, 1 = token by token, any size. */
+C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim,
+    unsigned int vdim);
+/* kernel: 0 = by shape, 1 = token by token, any size, 2 = state in registers (BF16; up to 8 tokens per entry, dim and vdim up
+ * to 512), 3 = in chunks of 128 tokens (BF16, prompts; dim up to 256, vdim up to 1024, multiples of 8). */
 C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cuda_b200_batch* b, void* stream, unsigned int flags, int kernel);
 
 /* Router: the `top` largest of each row of float logits [n][ldl] (ties: the lower expert), softmax over them; the

@@ -198,16 +198,26 @@ def tensor_shapes(config):
 
 
 def random_weights(config, seed):
-    """bfloat16-exact float32 tensors: linears N(0, 1 / fan-in), norms near 1, forget gates that mostly keep."""
+    """bfloat16-exact float32 tensors: linears N(0, 1 / fan-in), norms near 1, forget gates that mostly keep.
+
+    An mLSTM's output is divided by its own size, so where its scores q . k cancel, rounding decides its direction.  To keep
+    these models well conditioned, tokens share a direction, the mLSTM's keys resemble its queries and branches are small."""
     rng = np.random.default_rng(seed)
     out = {}
+    shared = 1.5 * rng.standard_normal(config["width"])
     for name, shape in tensor_shapes(config).items():
         a = rng.standard_normal(shape)
         if name.endswith(".f.b"):
             a = 3.0 + 2.0 * a
         elif "norm" in name.rsplit(".", 1)[-1]:
             a = 1.0 + 0.2 * a
+            if name.endswith(("norm1b", "norm2b")):
+                a = 0.3 * a
+        elif name == "embed":
+            a = 0.17 * (a + shared)
         elif len(shape) == 2:
             a = a / np.sqrt(shape[1]) * (3.0 if name.endswith((".mix.i", ".mix.f")) else 1.0)
+        if name.endswith(".mix.k") and name[:-1] + "f" in tensor_shapes(config):
+            a = 0.9 * out[name[:-1] + "q"] + 0.44 * a
         out[name] = bf16_round(np.asarray(a, np.float32)).reshape(shape)
     return out
