@@ -107,7 +107,7 @@ __device__ __forceinline__ float rotated(const float* head, unsigned int d, unsi
 template <class K, class... Args>
 static int launch_cluster(const char* label, K kernel, dim3 grid, dim3 block, size_t smem, unsigned int cluster, void* stream, bool pdl, Args... args)
 {
-    if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (smem > 24 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     {
         report_launch(label);
         return 1;
