@@ -135,6 +135,142 @@ __global__ void __launch_bounds__(512) attention_prepare_kernel(const AttnParams
     }
 }
 
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8])
+{
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = { u.x, u.y, u.z, u.w };
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+    {
+        f[2 * i] = __uint_as_float(w[i] << 16);
+        f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+}
+__device__ __forceinline__ void load8(const float* p, float (&f)[8])
+{
+    const float4 a = load4(p), b = load4(p + 4);
+    const float v[8] = { a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w };
+#pragma unroll
+    for (int i = 0; i < 8; i++) { f[i] = v[i]; }
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8])
+{
+    store4(p, make_float4(f[0], f[1], f[2], f[3]));
+    store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+
+// The same in BF16 by eights, where sizes and offsets allow it: heads and, for pairs that lie apart, half of the rotated part are
+// whole eights.  Without unit RMS of single heads.
+__global__ void __launch_bounds__(512) attention_prepare8_kernel(const AttnParams p)
+{
+    __shared__ float sums[16];
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int i = p.t0 + blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+    const bool is_q = blockIdx.y == 0;
+    const int e = p.token_entry[i];
+    const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
+    if (row >= p.T_max) { return; }
+    __nv_bfloat16* x = (__nv_bfloat16*)p.qkvg + (size_t)i * p.ld;
+    const size_t kv0 = (size_t)p.slot[e] * p.Hkv;
+    const unsigned int per = p.dim / 8, all = (is_q ? p.H : p.Hkv) * per, half = p.rot_dims / 2;
+    const __nv_bfloat16* src = is_q ? x : x + p.k_off;
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    const float2* rot = p.rotary + (size_t)row * half;
+    // the eights of the row that a thread turns, with the ones they are turned with (two rounds keep everything in registers)
+    constexpr int R = 2;
+    float own[R][8], other[R][8], sq = 0.f;
+#pragma unroll
+    for (int r = 0; r < R; r++)
+    {
+        const unsigned int c = tid + r * blockDim.x, d = (c % per) * 8;
+        if (c < all)
+        {
+            load8(src + c * 8, own[r]);
+            if (d < p.rot_dims && !p.rot_interleaved)
+            {
+                const unsigned int o = d < half ? c * 8 + half : c * 8 - half;
+                load8(src + o, other[r]);
+                if (w != nullptr)
+                {
+                    float wo[8];
+                    load8(w + o, wo);
+#pragma unroll
+                    for (int j = 0; j < 8; j++) { other[r][j] *= wo[j]; }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 8; j++) { sq += own[r][j] * own[r][j]; }
+            if (w != nullptr)
+            {
+                float wc[8];
+                load8(w + c * 8, wc);
+#pragma unroll
+                for (int j = 0; j < 8; j++) { own[r][j] *= wc[j]; }
+            }
+        }
+    }
+    sq = warp_sum(sq);
+    if (lane == 0) { sums[warp] = sq; }
+    __syncthreads();    // q: also, every eight has been read
+    const float inv = w != nullptr ? 1.0f / sqrtf(warp_sum(lane < warps ? sums[lane] : 0.f) / (float)(all * 8) + p.eps) : 1.f;
+#pragma unroll
+    for (int r = 0; r < R; r++)
+    {
+        const unsigned int c = tid + r * blockDim.x, h = c / per, d = (c % per) * 8;
+        if (c >= all) { continue; }
+        float out[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) { out[j] = own[r][j] * inv; }
+        if (d < p.rot_dims)
+        {
+            if (p.rot_interleaved)
+            {
+#pragma unroll
+                for (int j = 0; j < 4; j++)
+                {
+                    const float2 cs = rot[d / 2 + j];
+                    const float u = out[2 * j], v = out[2 * j + 1];
+                    out[2 * j] = u * cs.x - v * cs.y;
+                    out[2 * j + 1] = v * cs.x + u * cs.y;
+                }
+            }
+            else
+            {
+                const bool second = d >= half;
+#pragma unroll
+                for (int j = 0; j < 8; j++)
+                {
+                    const float2 cs = rot[(second ? d - half : d) + j];
+                    const float o = other[r][j] * inv;
+                    out[j] = second ? out[j] * cs.x + o * cs.y : out[j] * cs.x - o * cs.y;
+                }
+            }
+        }
+        store8(is_q ? x + c * 8 : (__nv_bfloat16*)p.k_cache + ((kv0 + h) * p.T_max + row) * p.k_ld + d, out);
+    }
+    if (is_q) { return; }
+    for (unsigned int c = tid; c < p.Hkv * (p.vdim / 8); c += blockDim.x)
+    {
+        const unsigned int h = c / (p.vdim / 8), d = (c % (p.vdim / 8)) * 8;
+        float v[8];
+        load8(x + p.v_off + c * 8, v);
+        if (p.v_mix)
+        {
+            __nv_bfloat16* first = (__nv_bfloat16*)p.v_first + (size_t)i * p.v_first_ld + c * 8;
+            if (p.v_mix == 1) { store8(first, v); }
+            else
+            {
+                float f[8];
+                load8(first, f);
+#pragma unroll
+                for (int j = 0; j < 8; j++) { v[j] = (1.0f - p.lambda) * v[j] + p.lambda * f[j]; }
+            }
+        }
+        store8((__nv_bfloat16*)p.v_cache + ((kv0 + h) * p.T_max + row) * p.v_ld + d, v);
+    }
+}
+
 constexpr unsigned int AP_KEYS = 128;
 
 // One CTA per (token, kv head, group of GB query heads): the heads against the cache in chunks of 128 keys with a running
@@ -233,6 +369,13 @@ static int attention_append(const AttnParams& p, unsigned int tokens, void* stre
     {
         const unsigned int most = (p.H > p.Hkv ? p.H : p.Hkv) * p.dim;
         unsigned int threads = 512;
+        const bool eights = Elem<T>::type == DT_BF16 && !p.qk_norm && (p.dim % 8) == 0 && (p.vdim % 8) == 0 && (p.rot_dims % (p.rot_interleaved ? 8 : 16)) == 0
+            && (p.ld % 8) == 0 && (p.k_off % 8) == 0 && (p.v_off % 8) == 0 && (p.v_first_ld % 8) == 0 && most <= 2 * 8 * threads;
+        if (eights)
+        {
+            while (threads > 64 && most <= 2 * 8 * (threads / 2)) { threads /= 2; }
+            return launch_kernel("attention_prepare8", attention_prepare8_kernel, dim3(tokens, 2), dim3(threads), 0, stream, pdl, p);
+        }
         while (threads > 64 && threads / 2 * 4 >= most) { threads /= 2; }
         const DecoderDevice* dev = decoder_device();
         if (!dev || (size_t)most * 4 > (size_t)dev->max_smem - 1024) { return -1; }

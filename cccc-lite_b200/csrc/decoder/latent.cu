@@ -51,6 +51,65 @@ __global__ void __launch_bounds__(512) latent_down_kernel(const LatentParams p)
     }
 }
 
+// The same in BF16 by eights, a thread per eight: ranks, offsets and the rotated part are whole eights.
+__global__ void __launch_bounds__(512) latent_down8_kernel(const LatentParams p)
+{
+    __shared__ float sums[16];
+    grid_dependency_launch();
+    grid_dependency_wait();
+    const unsigned int i = p.t0 + blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+    const bool is_q = blockIdx.y == 0;
+    const int e = p.token_entry[i];
+    const unsigned int row = (unsigned int)(p.pos[e] + ((int)i - p.start[e]));
+    if (row >= p.T_max) { return; }
+    const unsigned int rank = is_q ? p.q_rank : p.kv_rank, all = is_q ? rank : rank + p.rot_dim, d = tid * 8;
+    float f[8], sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) { f[j] = 0.f; }
+    if (d < all)
+    {
+        const uint4 u = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.down + (size_t)i * p.ld + (is_q ? 0u : p.kv_off) + d);
+        const uint32_t w[4] = { u.x, u.y, u.z, u.w };
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+        {
+            f[2 * j] = __uint_as_float(w[j] << 16);
+            f[2 * j + 1] = __uint_as_float(w[j] & 0xFFFF0000u);
+        }
+    }
+    if (d < rank)
+    {
+#pragma unroll
+        for (int j = 0; j < 8; j++) { sq += f[j] * f[j]; }
+    }
+    sq = warp_sum(sq);
+    if (lane == 0) { sums[warp] = sq; }
+    __syncthreads();
+    const float inv = 1.0f / sqrtf(warp_sum(lane < warps ? sums[lane] : 0.f) / (float)rank + p.eps);
+    if (d >= all) { return; }
+    if (d < rank)
+    {
+        const float* w = (is_q ? p.q_norm : p.kv_norm) + d;
+#pragma unroll
+        for (int j = 0; j < 8; j++) { f[j] *= inv * w[j]; }
+    }
+    else
+    {
+        const float2* rot = p.rotary + (size_t)row * (p.rot_dim / 2) + (d - rank) / 2;
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+        {
+            const float2 cs = rot[j];
+            const float u = f[2 * j], v = f[2 * j + 1];
+            f[2 * j] = u * cs.x - v * cs.y;
+            f[2 * j + 1] = v * cs.x + u * cs.y;
+        }
+    }
+    __nv_bfloat16* dst = (is_q ? (__nv_bfloat16*)p.cq + (size_t)i * p.ld_cq : (__nv_bfloat16*)p.cache + ((size_t)p.slot[e] * p.T_max + row) * p.c_ld) + d;
+    store4(dst, make_float4(f[0], f[1], f[2], f[3]));
+    store4(dst + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+
 // A CTA per token, a thread per pair.
 template <class T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const T* src, unsigned int ld_src, unsigned int src_step, unsigned int src_off, T* dst,
@@ -107,6 +166,12 @@ static int latent_down(const LatentParams& p, unsigned int tokens, void* stream,
 {
     const unsigned int most = p.q_rank > p.kv_rank + p.rot_dim ? p.q_rank : p.kv_rank + p.rot_dim;
     unsigned int threads = 512;
+    if (Elem<T>::type == DT_BF16 && (p.q_rank % 8) == 0 && (p.kv_rank % 8) == 0 && (p.rot_dim % 8) == 0 && (p.ld % 8) == 0 && (p.kv_off % 8) == 0
+        && (p.ld_cq % 4) == 0 && (p.c_ld % 4) == 0 && (reinterpret_cast<uintptr_t>(p.down) & 15u) == 0 && most <= 8 * threads)
+    {
+        while (threads > 64 && most <= 8 * (threads / 2)) { threads /= 2; }
+        return launch_kernel("latent_down8", latent_down8_kernel, dim3(tokens, 2), dim3(threads), 0, stream, pdl, p);
+    }
     while (threads > 64 && threads / 2 * 2 >= most) { threads /= 2; }
     const DecoderDevice* dev = decoder_device();
     if (!dev || (size_t)most * 4 > (size_t)dev->max_smem - 1024) { return -1; }

@@ -15,9 +15,11 @@ struct LinearMember
     const float* row_scale;
     const int *group_offset, *x_row, *active;
     const void* head_gate;           // of the launch's dtype
+    float* Y_tail;
     unsigned int rows, N, K, ldw, ldx, ldy;
     unsigned int groups, group_rows, up_row;
     unsigned int blocks, x_step, y_step, ld_gate;    // block-diagonal: 1 or more
+    unsigned int tail, ld_tail;      // first feature of the float tail (none: past all features)
     unsigned int slots;              // groups the launch walks: 1, the blocks, the groups, or the active list's length
     unsigned int block0, fblocks;    // streaming kernel: first CTA, CTAs per group
     int out_type, activation, accumulate;
@@ -36,6 +38,11 @@ __device__ __forceinline__ float linear_row_factor(const LinearMember& m, unsign
 // f: column of Y (the block's first column included)
 __device__ __forceinline__ void linear_store(const LinearMember& m, unsigned int row, unsigned int f, float v)
 {
+    if (f >= m.tail)
+    {
+        m.Y_tail[(size_t)row * m.ld_tail + f - m.tail] = v;
+        return;
+    }
     const size_t i = (size_t)row * m.ldy + f;
     if (m.out_type == DT_BF16) { ((__nv_bfloat16*)m.Y)[i] = __float2bfloat16_rn(v); }
     else if (m.accumulate) { ((float*)m.Y)[i] += v; }

@@ -336,6 +336,7 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         if (a.group_offset && (a.groups == 0 || a.group_max == 0 || a.blocks > 1)) { return -1; }
         if (a.blocks > 1 && ((a.x_step % 8) || a.x_row)) { return -1; }
         if (a.activation == B200_ACT_SOFTCAP && !(a.cap > 0.f)) { return -1; }
+        if (a.tail && (!a.Y_tail || a.accumulate || a.blocks > 1 || a.group_offset || a.activation != B200_ACT_NONE)) { return -1; }
         LinearMember& m = L.m[L.count++];
         m.W = a.W;
         m.X = a.X;
@@ -358,6 +359,9 @@ C_EXPORT int cuda_b200_linear_rows(int dtype, unsigned int count, const cuda_b20
         m.y_step = a.y_step;
         m.head_gate = a.head_gate;
         m.ld_gate = a.ld_gate;
+        m.Y_tail = (float*)a.Y_tail;
+        m.tail = a.tail ? a.tail : 0xFFFFFFFFu;
+        m.ld_tail = a.ld_tail;
         m.cap = a.cap;
         m.slots = a.group_offset ? (a.active ? a.active_cap : a.groups) : m.blocks;
         m.out_type = a.out_type;

@@ -31,7 +31,7 @@ __device__ __forceinline__ void store_row32(const LinearMember& m, unsigned int 
     const float s = linear_row_factor<__nv_bfloat16>(m, row, block);
     const unsigned int ycol = block * m.y_step;
     const size_t i = (size_t)row * m.ldy + ycol + f;
-    if (f + 32 <= m.N && vec)
+    if (f + 32 <= m.N && ycol + f + 32 <= m.tail && vec)
     {
         if (m.out_type == DT_BF16)
         {
@@ -343,8 +343,9 @@ int launch_linear_tile(const LinearMember& m, cudaStream_t stream, bool pdl)
     // the widest tile that still gives every SM one
     const bool gated = activation_gated(m.activation);
     const unsigned long long rt = (m.rows + LT_M - 1) / LT_M;
-    auto tiles = [&](unsigned int bn) {
+    auto tiles = [&](unsigned int bn) -> unsigned long long {
         const unsigned int ft = gated ? bn / 2 : bn;
+        if (m.blocks > 1 && bn > 64 && m.N <= ft / 2) { return 0; }    // a block would not fill half of it
         return rt * m.blocks * ((m.N + ft - 1) / ft);
     };
     if (tiles(256) >= (unsigned long long)dev->sm_count * 8 / 10) { return launch_tile<256>(m, *dev, stream, pdl); }

@@ -164,6 +164,7 @@ C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cud
     p.k_off = a->k_off;
     p.v_off = a->v_off;
     p.g_off = a->g_off;
+    p.f_off = a->f_off;
     p.heads = a->heads;
     p.dim = a->dim;
     p.vdim = a->vdim;

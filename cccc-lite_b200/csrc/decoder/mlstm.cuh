@@ -21,7 +21,7 @@ struct MlstmParams
     void* out;
     float *state, *work;
     const int *slot, *pos, *start, *n, *token_entry;
-    unsigned int ld, ld_gates, ldo, k_off, v_off, g_off;
+    unsigned int ld, ld_gates, ldo, k_off, v_off, g_off, f_off;
     unsigned int heads, dim, vdim;
     unsigned int e0, t0, tokens, max_n;
     float cap, eps, q_scale;
@@ -40,7 +40,7 @@ __device__ __forceinline__ void mlstm_gates(const MlstmParams& p, unsigned int t
 {
     const float* g = p.gates + (size_t)token * p.ld_gates;
     in = p.cap * tanhf((g[head] + p.bias[head]) / p.cap);
-    forget = log_sigmoid_f32(p.cap * tanhf((g[p.heads + head] + p.bias[p.heads + head]) / p.cap));
+    forget = log_sigmoid_f32(p.cap * tanhf((g[p.f_off + head] + p.bias[p.heads + head]) / p.cap));
 }
 
 __device__ __forceinline__ float* mlstm_state_of(const MlstmParams& p, unsigned int e, unsigned int head)

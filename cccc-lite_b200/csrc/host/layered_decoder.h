@@ -143,7 +143,7 @@ private:
         const void* rotary = nullptr;
         Weight uq, absorb, uk, uv;     // latent: a head's queries every q_step columns; absorb: each head's W_uk transposed
         int q_step = 0;
-        Weight gates;                  // mLSTM: input and forget gates
+        int gates = 0, f_off = 0;      // mLSTM: first row of the gates in `in`, and the forget gates' distance from it
         float *gate_bias = nullptr, *head_norm = nullptr;
         int v_mix = 0;    // 1: the first mixing layer, 2: a later one
         float lambda = 0.f;

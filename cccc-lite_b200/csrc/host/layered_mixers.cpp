@@ -112,8 +112,9 @@ bool LayeredDecoder::loadMixer(TensorSource& s, const LayerSpec& ls, Layer* out,
     L.k_off = pad(qk, 8);
     L.v_off = 2 * L.k_off;
     L.g_off = L.v_off + pad(v, 8);
-    return packRows(s, { { a.q, qk }, { a.k, qk }, { a.v, v }, { a.gate, v } }, W, 8, &L.in, err)
-        && packRows(s, { { a.input, a.heads }, { a.forget, a.heads } }, W, 1, &L.gates, err) && packRows(s, { { a.o, W } }, v, 1, &L.o, err)
+    L.gates = L.g_off + pad(v, 8);
+    L.f_off = pad(a.heads, 8);
+    return packRows(s, { { a.q, qk }, { a.k, qk }, { a.v, v }, { a.gate, v }, { a.input, a.heads }, { a.forget, a.heads } }, W, 8, &L.in, err) && packRows(s, { { a.o, W } }, v, 1, &L.o, err)
         && loadVector(s, { { a.input + ".b", a.heads }, { a.forget + ".b", a.heads } }, &L.gate_bias, err) && loadVector(s, { { a.norm, v } }, &L.head_norm, err);
 }
 
@@ -161,7 +162,7 @@ bool LayeredDecoder::allocateMixers(const ModelOptions& o, std::string* err)
             const MlstmSpec& a = ls.mlstm;
             shape.state_floats = (size_t)a.heads * cuda_b200_mlstm_state_floats((unsigned int)a.dim, (unsigned int)a.vdim);
             att = std::max(att, a.heads * a.vdim);
-            gates = std::max(gates, 2 * a.heads);
+            gates = std::max(gates, 2 * layers_[i].f_off);
             mlstm = std::max(mlstm, cuda_b200_mlstm_work_floats((unsigned int)cap_, (unsigned int)std::min(cap_, o.max_sequences), (unsigned int)a.heads, (unsigned int)a.dim, (unsigned int)a.vdim));
         }
         shapes.push_back(shape);
@@ -498,9 +499,11 @@ void LayeredDecoder::issueMlstm(Issue& r, int layer)
 {
     const Layer& L = layers_[layer];
     const MlstmSpec& s = spec_.layers[layer].mlstm;
-    cuda_b200_linear l[2] = { dense(r, L.in, xn_, ldw_, in_, ld_in_), dense(r, L.gates, xn_, ldw_, gates_, ld_gates_) };
-    l[1].out_type = 0;
-    r.ok(cuda_b200_linear_rows(act(), 2, l, r.st, PDL, 0));
+    cuda_b200_linear l = dense(r, L.in, xn_, ldw_, in_, ld_in_);
+    l.Y_tail = gates_;
+    l.tail = (unsigned int)L.gates;
+    l.ld_tail = (unsigned int)ld_gates_;
+    r.ok(cuda_b200_linear_rows(act(), 1, &l, r.st, PDL, 0));
     cuda_b200_mlstm a = {};
     a.qkvg = in_;
     a.gates = gates_;
@@ -515,6 +518,7 @@ void LayeredDecoder::issueMlstm(Issue& r, int layer)
     a.k_off = (unsigned int)L.k_off;
     a.v_off = (unsigned int)L.v_off;
     a.g_off = (unsigned int)L.g_off;
+    a.f_off = (unsigned int)L.f_off;
     a.heads = (unsigned int)s.heads;
     a.dim = (unsigned int)s.dim;
     a.vdim = (unsigned int)s.vdim;

@@ -20,9 +20,9 @@ def _struct(name, pointers, uints, ints=(), floats=()):
 
 
 Norm = _struct("Norm", ("X", "weight", "bias", "out", "Y", "slot_row", "slot_weight", "rows", "branch", "branch_weight"), ("n", "width", "ldx", "ldo", "ldy", "slots", "ldb"), ("kind",), ("eps",))
-Linear = _struct("Linear", ("W", "X", "Y", "row_scale", "group_offset", "x_row", "active", "head_gate"),
+Linear = _struct("Linear", ("W", "X", "Y", "row_scale", "group_offset", "x_row", "active", "head_gate", "Y_tail"),
                  ("rows", "N", "K", "ldw", "ldx", "ldy", "groups", "group_rows", "group_max", "up_row", "active_cap", "blocks", "x_step", "y_step",
-                  "ld_gate"), ("out_type", "activation", "accumulate"), ("alpha", "cap"))
+                  "ld_gate", "tail", "ld_tail"), ("out_type", "activation", "accumulate"), ("alpha", "cap"))
 Batch = _struct("Batch", ("slot", "pos", "start", "n", "token_entry", "floor"), ("entries", "tokens", "max_n", "max_len", "first_entry", "first_token"))
 Attention = _struct("Attention", ("qkvg", "out", "k_cache", "v_cache", "v_first", "work", "q_norm", "k_norm", "rotary", "sink", "head_gate"),
                     ("ld", "ldo", "k_off", "v_off", "g_off", "v_first_ld", "H", "Hkv", "dim", "vdim", "k_ld", "v_ld", "T_max", "slots", "q_ld", "rot_dims", "ld_gate",
@@ -30,8 +30,8 @@ Attention = _struct("Attention", ("qkvg", "out", "k_cache", "v_cache", "v_first"
 Latent = _struct("Latent", ("down", "cq", "cache", "q_norm", "kv_norm", "rotary"), ("ld", "ld_cq", "kv_off", "q_rank", "kv_rank", "rot_dim", "c_ld", "T_max"), (),
                  ("eps",))
 Expand = _struct("Expand", ("cache", "c", "K", "floor", "pos2"), ("c_ld", "T_max", "kv_rank", "rot_dim", "ld_c", "k_ld", "T", "dim", "heads", "max_rows"))
-Mlstm = _struct("Mlstm", ("qkvg", "gates", "bias", "norm", "out", "state", "work"), ("ld", "ld_gates", "ldo", "k_off", "v_off", "g_off", "heads", "dim", "vdim"), (),
-                ("cap", "eps", "q_scale"))
+Mlstm = _struct("Mlstm", ("qkvg", "gates", "bias", "norm", "out", "state", "work"), ("ld", "ld_gates", "ldo", "k_off", "v_off", "g_off", "f_off", "heads", "dim", "vdim"),
+                (), ("cap", "eps", "q_scale"))
 Route = _struct("Route", ("logits", "pair_row", "pair_weight", "row_token", "group_offset", "active", "shared_weight", "choice", "counters"),
                 ("n", "ldl", "experts", "top", "active_cap"), ("sg_col",))
 

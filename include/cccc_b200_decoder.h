@@ -57,6 +57,7 @@ C_EXPORT int cuda_b200_norm_rows(int dtype, const cuda_b200_norm* a, void* strea
  * Block-diagonal (blocks > 1, not grouped): block b is a linear of its own, weight rows from b * group_rows, X columns from
  * b * x_step, Y columns from b * y_step (X's columns behind K up to the next multiple of 64 hold finite values; x_step a
  * multiple of 8).  head_gate: block b of row r is multiplied by sigmoid(head_gate[r * ld_gate + b]) (dtype).
+ * tail > 0 (dense, not gated, not accumulated): the features from `tail` on go to Y_tail[r][n - tail], as floats.
  * out_type 0: float (accumulate != 0: Y += row_scale[r] * result), 3: BF16 (float mode: always 0).  row_scale: float per
  * row, or NULL. */
 typedef struct cuda_b200_linear
@@ -69,9 +70,11 @@ typedef struct cuda_b200_linear
     const void* x_row;          /* int32 */
     const void* active;         /* int32: ids of the non-empty groups, -1 behind them; `active_cap` entries (NULL: all groups) */
     const void* head_gate;
+    void* Y_tail;
     unsigned int rows, N, K, ldw, ldx, ldy;
     unsigned int groups, group_rows, group_max, up_row, active_cap;
     unsigned int blocks, x_step, y_step, ld_gate;
+    unsigned int tail, ld_tail;
     int out_type, activation, accumulate;
     float alpha, cap;
 } cuda_b200_linear;
@@ -183,13 +186,13 @@ C_EXPORT int cuda_b200_latent_expand(int dtype, const cuda_b200_expand* a, const
 typedef struct cuda_b200_mlstm
 {
     const void* qkvg;          /* [tokens][ld] dtype: q at 0 (heads * dim), k at k_off, v at v_off (heads * vdim), gate at g_off */
-    const void* gates;         /* float [tokens][ld_gates]: heads input gates, heads forget gates */
-    const void* bias;          /* float [2 * heads], as the gates */
+    const void* gates;         /* float [tokens][ld_gates]: heads input gates, and from f_off on heads forget gates */
+    const void* bias;          /* float [2 * heads]: input gates, forget gates */
     const void* norm;          /* float [heads * vdim] */
     void* out;                 /* [tokens][ldo] dtype: heads * vdim */
     void* state;               /* float [slots][heads][cuda_b200_mlstm_state_floats] */
     void* work;                /* float scratch of cuda_b200_mlstm_work_floats, 16-byte aligned */
-    unsigned int ld, ld_gates, ldo, k_off, v_off, g_off;
+    unsigned int ld, ld_gates, ldo, k_off, v_off, g_off, f_off;
     unsigned int heads, dim, vdim;
     float cap, eps, q_scale;
 } cuda_b200_mlstm;
