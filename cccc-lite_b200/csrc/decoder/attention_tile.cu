@@ -10,7 +10,7 @@
 // than 2^8, so that O is seldom rescaled.
 // Every wait is bounded; on expiry the status word is raised, the roles drain, tensor memory is freed and the CTA returns.
 #include "attention.cuh"
-#include "../gemm_stream.cuh"
+#include "tile_common.cuh"
 
 #include <type_traits>
 
@@ -25,24 +25,6 @@ __host__ __device__ constexpr int ta_smem(int dk, int dv) { return 1024 + (dk / 
 constexpr uint32_t TA_O = 128;    // columns: two places of S (64) or P (32 high, 32 low), then O
 __host__ __device__ constexpr uint32_t ta_tmem(int dv) { return dv <= 128 ? 256 : 512; }
 __host__ __device__ constexpr int ta_ctas(int dk, int dv) { return ta_smem(dk, dv) <= 113 * 1024 && dv <= 128 ? 2 : 1; }
-
-// An MN-major operand [k][64 elements] with the 128-byte swizzle: 8-k groups 1024 bytes apart, 64-element blocks TA_BLOCK apart.
-__device__ __forceinline__ uint64_t umma_desc_mnmajor_sw128(uint32_t smem_addr)
-{
-    uint64_t d = 0;
-    d |= (uint64_t)((smem_addr & 0x3FFFFu) >> 4);
-    d |= (uint64_t)(TA_BLOCK >> 4) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
-__device__ __forceinline__ float exp2_f32(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 
 // A BF16 gate's sigmoid, by the hardware's exponential and reciprocal.
 __device__ __forceinline__ float gate_sigmoid(float z) { return __fdividef(1.0f, 1.0f + exp2_f32(-1.44269504088896341f * z)); }

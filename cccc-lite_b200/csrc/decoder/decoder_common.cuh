@@ -15,7 +15,8 @@ unsigned int* decoder_status_word();
 enum : unsigned int
 {
     WAIT_LINEAR_TILE = 1,
-    WAIT_ATTENTION_TILE = 2
+    WAIT_ATTENTION_TILE = 2,
+    WAIT_MLSTM_TILE = 3
 };
 __device__ __forceinline__ void note_timeout(unsigned int* status, unsigned int kernel, unsigned int role, unsigned int step)
 {

@@ -170,6 +170,7 @@ C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cud
     p.vdim = a->vdim;
     p.e0 = b->first_entry;
     p.t0 = b->first_token;
+    p.entries = b->entries;
     p.tokens = b->tokens;
     p.max_n = b->max_n;
     p.cap = a->cap;

@@ -23,7 +23,7 @@ struct MlstmParams
     const int *slot, *pos, *start, *n, *token_entry;
     unsigned int ld, ld_gates, ldo, k_off, v_off, g_off, f_off;
     unsigned int heads, dim, vdim;
-    unsigned int e0, t0, tokens, max_n;
+    unsigned int e0, t0, entries, tokens, max_n;
     float cap, eps, q_scale;
 };
 

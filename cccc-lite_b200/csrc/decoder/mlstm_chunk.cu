@@ -1,17 +1,20 @@
-// The mLSTM recurrence over prompts, in chunks of 128 tokens on mma.sync.
+// The mLSTM recurrence over prompts, in chunks of 128 tokens.
 //
 // Inside a chunk, with F the running sum of the log forget gates, a_s = i_s - F_s and M_t = max(m_0, a_s up to t), the running
 // maximum is m_t = F_t + M_t, and unrolled from the chunk's first token
 //   o_t ~ e^(m_0 - M_t) S_0^T q_t + sum_{s <= t} e^(a_s - M_t) (q_t . k_s) v_s,   S_L = e^(m_0 - M_L) S_0 + sum_s e^(a_s - M_L) k_s v_s^T,
 // no exponent above zero.  Three kernels:
 //   gates  : F and a of every chunk.
-//   states : a CTA per 32 value columns of a head walks an entry's chunks, its columns of S as float accumulators in registers;
-//            it leaves the state ahead of every chunk in scratch memory.
-//   outputs: a cluster per (chunk, head), a CTA per 64 or 128 value columns; the head's sum of squares meets in the cluster.
+//   states : a CTA per 32 value columns of a head walks an entry's chunks, its columns of S as float accumulators in registers
+//            (mma.sync); it leaves the state ahead of every chunk in scratch memory.
+//   outputs: a cluster per (chunk, head), a CTA per 64 or 128 value columns, on tcgen05; the head's sum of squares meets in the
+//            cluster.
 // One operand of every product is exact (q, k or v); the other - S, weighted values, weighted scores - enters as the sum of two
 // BF16 numbers.
+#include "../gemm_stream.cuh"
 #include "attention_mma.cuh"
 #include "mlstm.cuh"
+#include "tile_common.cuh"
 
 #include <cooperative_groups.h>
 
@@ -20,29 +23,30 @@ namespace cg = cooperative_groups;
 namespace b200
 {
 
-constexpr unsigned int MC_L = 128, MC_WARPS = 16, MC_THREADS = 32 * MC_WARPS, MC_COLS = 32, MC_SLICE = 32, MC_MAX_DIM = 256, MC_MAX_CLUSTER = 8;
+constexpr unsigned int MC_L = 128, MC_WARPS = 16, MC_THREADS = 32 * MC_WARPS, MC_COLS = 32, MC_MAX_DIM = 256, MC_MAX_CLUSTER = 8;
 
 __host__ __device__ __forceinline__ unsigned int mc_dp(unsigned int dim) { return dim <= 64 ? 64 : (dim <= 128 ? 128 : 256); }
 __host__ __device__ __forceinline__ unsigned int mc_vp(unsigned int vdim) { return (vdim + MC_COLS - 1) / MC_COLS * MC_COLS; }
-// Scratch of a (chunk, head): S high [dp][vp], S low, then n and m ahead of the chunk, n and m behind the entry's last chunk, F, a,
-// the largest a and the last F.
-__host__ __device__ __forceinline__ size_t mc_record(unsigned int dim, unsigned int vdim)
-{
-    return (size_t)mc_dp(dim) * mc_vp(vdim) + 2 * (mc_dp(dim) + 4) + 2 * MC_L + 4;
-}
+// Scratch: of every (chunk, head) S high [dp][vp] and S low; behind all of these, n and m ahead of the chunk, n and m behind the
+// entry's last chunk, F, a, the largest a and the last F.
+__host__ __device__ __forceinline__ size_t mc_matrix(unsigned int dim, unsigned int vdim) { return (size_t)mc_dp(dim) * mc_vp(vdim); }
+__host__ __device__ __forceinline__ size_t mc_record(unsigned int dim) { return 2 * (mc_dp(dim) + 4) + 2 * MC_L + 4; }
+__host__ __device__ __forceinline__ unsigned int mc_slots(unsigned int tokens, unsigned int entries) { return tokens / MC_L + entries; }
 struct ChunkRecord
 {
+    unsigned int at;                  // (chunk, head)
     __nv_bfloat16* S;
     float *n, *last, *F, *a, *top;    // m behind n, the last m behind last
 };
 __device__ __forceinline__ ChunkRecord mc_record_of(const MlstmParams& p, unsigned int e, unsigned int chunk, unsigned int head)
 {
-    const unsigned int at = ((unsigned int)p.start[e] - p.t0) / MC_L + (e - p.e0) + chunk;    // entries' chunks one behind the other
-    const unsigned int dp = mc_dp(p.dim);
-    float* r = p.work + ((size_t)at * p.heads + head) * mc_record(p.dim, p.vdim);
+    // entries' chunks one behind the other
+    const unsigned int at = (((unsigned int)p.start[e] - p.t0) / MC_L + (e - p.e0) + chunk) * p.heads + head, dp = mc_dp(p.dim);
+    const size_t matrix = mc_matrix(p.dim, p.vdim);
     ChunkRecord c;
-    c.S = reinterpret_cast<__nv_bfloat16*>(r);
-    c.n = r + (size_t)dp * mc_vp(p.vdim);
+    c.at = at;
+    c.S = reinterpret_cast<__nv_bfloat16*>(p.work + at * matrix);
+    c.n = p.work + (size_t)mc_slots(p.tokens, p.entries) * p.heads * matrix + at * mc_record(p.dim);
     c.last = c.n + dp + 4;
     c.F = c.last + dp + 4;
     c.a = c.F + MC_L;
@@ -111,9 +115,10 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
     extern __shared__ __align__(16) unsigned char mc_raw[];
     constexpr unsigned int VS = (MC_COLS + 8) * 2, KS = (DP + 8) * 2, KBYTES = MC_L * KS;
     __shared__ float w[MC_L];
+    // weighted values; behind the columns the weights themselves, which make n
     __shared__ __align__(16) __nv_bfloat16 hi[MC_L * (MC_COLS + 8)], lo[MC_L * (MC_COLS + 8)];
     const unsigned int vp = mc_vp(p.vdim);
-    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gc = (lane & 3) * 2, d0 = warp * 16;
+    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gt = lane & 3, gc = gt * 2, d0 = warp * 16;
     const unsigned int c0 = blockIdx.x * MC_COLS, h = blockIdx.y, e = p.e0 + blockIdx.z;
     grid_dependency_launch();
     grid_dependency_wait();
@@ -149,7 +154,24 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
             S[j][2 * half + 1] = v.y;
         }
     }
-    float m = fresh ? 0.f : st_n[mlstm_n_ld(p.dim)], nn = !fresh && tid < p.dim ? st_n[tid] : 0.f;
+    float m = fresh ? 0.f : st_n[mlstm_n_ld(p.dim)];
+    float nn[4] = { 0.f, 0.f, 0.f, 0.f };    // n of rows gr and gr + 8 in the first column's lanes, elements 0 and 2
+    const bool carries = blockIdx.x == 0, holds = carries && gt == 0 && d0 < (unsigned int)DP;
+#pragma unroll
+    for (int half = 0; half < 2; half++)
+    {
+        const unsigned int d = d0 + gr + 8 * half;
+        if (holds && !fresh && d < p.dim) { nn[2 * half] = st_n[d]; }
+    }
+    if (tid < MC_L)
+    {
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+        {
+            reinterpret_cast<uint32_t*>(hi + tid * (MC_COLS + 8) + MC_COLS)[j] = 0u;
+            reinterpret_cast<uint32_t*>(lo + tid * (MC_COLS + 8) + MC_COLS)[j] = 0u;
+        }
+    }
     ChunkRecord rec = mc_record_of(p, e, 0, h);
     float a = tid < MC_L ? rec.a[tid] : 0.f;
     float2 end = *reinterpret_cast<const float2*>(rec.top);
@@ -158,28 +180,56 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
         const unsigned int live = min(MC_L, n - c * MC_L);
         fetch(c + 1);
         const float top = fmaxf(m, end.x), keep = expf(m - top);    // M at the chunk's end
-        if (tid < MC_L) { w[tid] = expf(a - top); }
+        if (tid < MC_L)
+        {
+            const float y = expf(a - top);
+            const __nv_bfloat16 high = __float2bfloat16_rn(y);
+            w[tid] = y;
+            hi[tid * (MC_COLS + 8) + MC_COLS] = high;
+            lo[tid * (MC_COLS + 8) + MC_COLS] = __float2bfloat16_rn(y - __bfloat162float(high));
+        }
         if (d0 < (unsigned int)DP && (!fresh || c > 0))
         {
 #pragma unroll
-            for (int j = 0; j < (int)MC_COLS / 8; j++)
+            for (int half = 0; half < 2; half++)
             {
+                uint32_t part[2][4];    // high, low; of the eight columns of tile j
 #pragma unroll
-                for (int half = 0; half < 2; half++)
+                for (int j = 0; j < 4; j++)
                 {
                     const float s0 = S[j][2 * half], s1 = S[j][2 * half + 1];
-                    const uint32_t high = pack_bf16x2(s0, s1);
-                    uint32_t* y = reinterpret_cast<uint32_t*>(rec.S + (size_t)(d0 + gr + 8 * half) * vp + c0 + j * 8 + gc);
-                    y[0] = high;
-                    y[(size_t)DP * vp / 2] = pack_bf16x2(s0 - __uint_as_float(high << 16), s1 - __uint_as_float(high & 0xFFFF0000u));
+                    part[0][j] = pack_bf16x2(s0, s1);
+                    part[1][j] = pack_bf16x2(s0 - __uint_as_float(part[0][j] << 16), s1 - __uint_as_float(part[0][j] & 0xFFFF0000u));
+                }
+                // the four lanes of a row exchange, so that lane t has all of tile t
+#pragma unroll
+                for (int k = 0; k < 2; k++)
+                {
+                    uint32_t row[4];
+#pragma unroll
+                    for (int step = 0; step < 4; step++)
+                    {
+                        // to lane gt ^ step goes tile gt ^ step
+                        const unsigned int j = gt ^ step;
+                        const uint32_t give = j == 0 ? part[k][0] : (j == 1 ? part[k][1] : (j == 2 ? part[k][2] : part[k][3]));
+                        const uint32_t got = __shfl_xor_sync(0xFFFFFFFFu, give, step);
+#pragma unroll
+                        for (unsigned int i = 0; i < 4; i++)
+                        {
+                            if (i == (gt ^ (unsigned int)step)) { row[i] = got; }
+                        }
+                    }
+                    __nv_bfloat16* y = rec.S + (size_t)(k * DP + d0 + gr + 8 * half) * vp + c0 + gt * 8;
+                    *reinterpret_cast<uint4*>(y) = make_uint4(row[0], row[1], row[2], row[3]);
                 }
             }
         }
-        if (blockIdx.x == 0)
+        if (holds)
         {
-            if (tid < (unsigned int)DP) { rec.n[tid] = nn; }
-            if (tid == 0) { rec.n[DP] = m; }
+            rec.n[d0 + gr] = nn[0];
+            rec.n[d0 + gr + 8] = nn[2];
         }
+        if (carries && tid == 0) { rec.n[DP] = m; }
         m = end.y + top;
         const ChunkRecord now = rec;
         if (c + 1 < chunks)
@@ -201,18 +251,6 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
             *reinterpret_cast<uint32_t*>(hi + at) = u;
             *reinterpret_cast<uint32_t*>(lo + at) = pack_bf16x2(y0 - __uint_as_float(u << 16), y1 - __uint_as_float(u & 0xFFFF0000u));
         }
-        if (blockIdx.x == 0 && tid < p.dim)
-        {
-            const __nv_bfloat16* k = reinterpret_cast<const __nv_bfloat16*>(mc_raw + (c & 1u) * KBYTES) + tid;
-            float part[4] = { 0.f, 0.f, 0.f, 0.f };
-#pragma unroll 4
-            for (unsigned int s = 0; s < MC_L; s += 4)
-            {
-#pragma unroll
-                for (int i = 0; i < 4; i++) { part[i] = fmaf(w[s + i], __bfloat162float(k[(s + i) * (DP + 8)]), part[i]); }
-            }
-            nn = keep * nn + ((part[0] + part[1]) + (part[2] + part[3]));
-        }
         __syncthreads();
         if (d0 < (unsigned int)DP)
         {
@@ -224,10 +262,21 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
 #pragma unroll
                 for (int i = 0; i < 4; i++) { S[j][i] *= keep; }
             }
+#pragma unroll
+            for (int i = 0; i < 4; i++) { nn[i] *= keep; }
 #pragma unroll 4
             for (unsigned int s0 = 0; s0 < live; s0 += 16)
             {
                 uint32_t b[2][MC_COLS / 16][4], k[4];
+                if (carries)
+                {
+                    uint32_t x[4];
+                    ldmatrix_x4_trans(x, (lane < 16 ? hs : ls) + (s0 + (lane & 15)) * VS + MC_COLS * 2);
+                    uint32_t k2[4];
+                    ldmatrix_x4_trans(k2, kb + s0 * KS);
+                    mma_bf16_16816(nn, k2[0], k2[1], k2[2], k2[3], x[0], x[1]);
+                    mma_bf16_16816(nn, k2[0], k2[1], k2[2], k2[3], x[2], x[3]);
+                }
                 ldmatrix_x4_trans(k, kb + s0 * KS);
 #pragma unroll
                 for (int j = 0; j < (int)MC_COLS / 16; j++)
@@ -248,10 +297,14 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
             }
         }
         // other column blocks may still have to read the old n and m: the last kernel puts the new ones in place
-        if (blockIdx.x == 0 && c + 1 == chunks)
+        if (c + 1 == chunks)
         {
-            if (tid < p.dim) { now.last[tid] = nn; }
-            if (tid == 0) { now.last[DP] = m; }
+            if (holds)
+            {
+                now.last[d0 + gr] = nn[0];
+                now.last[d0 + gr + 8] = nn[2];
+            }
+            if (carries && tid == 0) { now.last[DP] = m; }
         }
         __syncthreads();    // the next chunk but one takes this one's place
     }
@@ -269,64 +322,61 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmPar
 }
 
 __host__ __device__ constexpr unsigned int mc_states_smem(unsigned int dp) { return 2 * MC_L * ((dp + 8) * 2 + (MC_COLS + 8) * 2); }
-// q, k, v; two slices of S beside them
-__host__ __device__ constexpr unsigned int mc_slice_bytes(unsigned int vb) { return 2 * MC_SLICE * (vb + 8) * 2; }
-__host__ __device__ constexpr unsigned int mc_outputs_smem(unsigned int dp, unsigned int vb)
-{
-    return 2 * MC_L * (dp + 8) * 2 + MC_L * (vb + 8) * 2 + 2 * mc_slice_bytes(vb);
-}
+// ---- outputs ---------------------------------------------------------------------------------------
+constexpr int MO_THREADS = 32 * 10;
+constexpr int MO_BLOCK = 64 * 128, MO_ROWS = 2 * MO_BLOCK;    // 64 rows x 64 elements; the 128 tokens' block of 64 elements
+constexpr uint32_t MO_P = 128, MO_O = 256, MO_TMEM = 512;      // columns: scores, weighted scores (high, low), what the chunk gives, what S gives
+__host__ __device__ constexpr int mo_slice(int vb) { return 2 * (vb / 64) * MO_BLOCK; }    // 64 rows of S: high, low
+__host__ __device__ constexpr int mo_smem(int dp, int vb) { return 1024 + 2 * (dp / 64) * MO_ROWS + (vb / 64) * MO_ROWS + mo_slice(vb) + 1024; }
 
-// grid (column blocks of VB = the cluster, heads, entries x chunks); a warp owns 16 tokens and half of the columns.  The chunk's own
-// tokens come first; the slices of S then also take the place of k and v.
-template <int DP, int VB>
-__global__ void __launch_bounds__(MC_THREADS) mlstm_outputs_kernel(const MlstmParams p, const unsigned int max_chunks)
+// grid (column blocks of VB = the cluster, heads, entries x chunks).  A TMA lane fetches q, k and v of the chunk and slices of 64 rows of
+// S: the first beside them, the following ones where k was, once the scores are out.  The MMA lane issues q k^T, then q S, then
+// (weighted scores) v.  Eight warps own a row of scores per thread, half of its columns each.
+template <int VB>
+__global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmS,
+    const __grid_constant__ MlstmParams p, const unsigned int max_chunks, unsigned int* status)
 {
-    extern __shared__ __align__(16) unsigned char mc_raw[];
-    __shared__ float F[MC_L], a[MC_L], M[MC_L], maxima[MC_L / 32], sq[2][MC_L], peers[MC_MAX_CLUSTER][MC_L], n0[DP];
-    constexpr unsigned int VS = (VB + 8) * 2, QS = (DP + 8) * 2, SLICE = mc_slice_bytes(VB), SLICES = DP / MC_SLICE, HB = VB / 2;
-    constexpr unsigned int QBYTES = MC_L * QS, VBYTES = MC_L * VS;
-    constexpr unsigned int PLACES = (QBYTES + VBYTES) / SLICE;    // of slices where k and v were
-    const unsigned int vp = mc_vp(p.vdim);
-    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gc = (lane & 3) * 2;
+    extern __shared__ unsigned char mo_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(mo_raw) + 1023) & ~(uintptr_t)1023);
+    __shared__ float F[MC_L], a[MC_L], M[MC_L], maxima[MC_L / 32], sq[2][MC_L], nq[2][MC_L], peers[MC_MAX_CLUSTER][MC_L], n0[MC_MAX_DIM];
+    constexpr int SLICE = mo_slice(VB), HB = VB / 2, MAX_PLACES = 8;
+    const unsigned int dp = mc_dp(p.dim), blocks = dp / 64;
+    uint64_t* qk_full = reinterpret_cast<uint64_t*>(smem);
+    uint64_t *v_full = qk_full + 1, *s_full = qk_full + 2, *p_ready = qk_full + 3, *o_full = qk_full + 4, *slice_full = qk_full + 5,
+             *slice_empty = slice_full + MAX_PLACES;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(slice_empty + MAX_PLACES);
+    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
+    unsigned char* qs = smem + 1024;
+    unsigned char* ks = qs + blocks * MO_ROWS;
+    unsigned char* vs = ks + blocks * MO_ROWS;
+    unsigned char* ss = vs + (VB / 64) * MO_ROWS;
+    const unsigned int places = min((unsigned int)MAX_PLACES, 1u + blocks * MO_ROWS / SLICE);    // of slices
+    auto place = [&](unsigned int i) { return i % places == 0 ? ss : ks + (i % places - 1) * SLICE; };
+
+    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const unsigned int rank = blockIdx.x, h = blockIdx.y, e = p.e0 + blockIdx.z / max_chunks, c = blockIdx.z % max_chunks, c0 = rank * VB;
+    if (tid == 0)
+    {
+        for (int i = 0; i < 5 + 2 * MAX_PLACES; i++) { mbar_init(qk_full + i, i == 3 ? 8 : 1); }
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e];
     if (c * MC_L >= n) { return; }    // the whole cluster
+    if (warp == 1) { tmem_alloc(tmem_slot, MO_TMEM); }
     const unsigned int live = min(MC_L, n - c * MC_L), first = start + c * MC_L;
     const bool fresh = p.pos[e] == 0 && c == 0;
     const ChunkRecord rec = mc_record_of(p, e, c, h);
-    const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg + (size_t)first * p.ld;
-    const uint32_t qs = smem_u32(mc_raw), ks = qs + QBYTES, vs = ks + QBYTES, ss = vs + VBYTES;
-    auto place = [&](unsigned int i) { return i < 2 ? ss + i * SLICE : (i - 2 < PLACES ? ks + (i - 2) * SLICE : ss + (i - 2 - PLACES) * SLICE); };
-    auto fetch_slice = [&](unsigned int i) {
-        if (i < SLICES && !fresh)
-        {
-            constexpr unsigned int PER = VB / 8, ALL = 2 * MC_SLICE * PER;
-            const uint32_t to = place(i);
-            for (unsigned int j = tid; j < ALL; j += MC_THREADS)
-            {
-                const unsigned int part = j / (MC_SLICE * PER), r = j / PER % MC_SLICE, d = j % PER, col = c0 + d * 8;
-                const bool ok = col < vp;
-                cp_async16(to + part * (SLICE / 2) + r * VS + d * 16, rec.S + (ok ? (size_t)part * DP * vp + (size_t)(i * MC_SLICE + r) * vp + col : 0), ok);
-            }
-        }
-        cp_async_commit();
-    };
-    mc_fetch<DP>(qs, x + h * p.dim, p.ld, live, p.dim);
-    mc_fetch<DP>(ks, x + p.k_off + h * p.dim, p.ld, live, p.dim);
-    mc_fetch<VB>(vs, x + p.v_off + h * p.vdim + c0, p.ld, live, min((unsigned int)VB, p.vdim - c0));
-    cp_async_commit();
-    fetch_slice(0);
-    fetch_slice(1);
-    const float m0 = fresh ? 0.f : rec.n[DP];
-    for (unsigned int d = tid; d < (unsigned int)DP; d += MC_THREADS) { n0[d] = fresh ? 0.f : rec.n[d]; }
+    const unsigned int slices = fresh ? 0 : blocks, steps = p.dim / 16;
+    const float m0 = fresh ? 0.f : rec.n[dp];
     float t_max = -INFINITY;
     if (tid < MC_L)    // M: running maxima of a, with m0
     {
         F[tid] = rec.F[tid];
         t_max = rec.a[tid];
-        a[tid] = t_max;
+        a[tid] = t_max * 1.44269504088896341f;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1)
         {
@@ -335,6 +385,7 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_outputs_kernel(const MlstmPa
         }
         if (lane == 31) { maxima[warp] = t_max; }
     }
+    for (unsigned int d = tid; d < dp; d += MO_THREADS) { n0[d] = fresh || d >= p.dim ? 0.f : rec.n[d]; }
     __syncthreads();
     if (tid < MC_L)
     {
@@ -342,218 +393,305 @@ __global__ void __launch_bounds__(MC_THREADS) mlstm_outputs_kernel(const MlstmPa
         for (unsigned int j = 0; j < warp; j++) { t_max = fmaxf(t_max, maxima[j]); }
         M[tid] = t_max;
     }
-    cp_async_wait<2>();
+    tc_fence_before();
     __syncthreads();
-    const unsigned int r0 = (warp & 7u) * 16, ch = warp >> 3;    // tokens, half of the columns
-    const uint32_t qa = qs + (r0 + (lane & 15)) * QS + (lane >> 4) * 16;
-    float o[HB / 8][4], z2[HB / 8][4], nq[2] = { 0.f, 0.f }, mt[2], carry[2];
-#pragma unroll
-    for (int i = 0; i < 2; i++)
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    auto give_up = [&](unsigned int role, unsigned int step) {
+        note_timeout(status, WAIT_MLSTM_TILE, role, step);
+        *abort_flag = 1;
+    };
+    auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
+    const unsigned int quarter = warp & 3u, half = warp >= 2 ? (warp - 2u) >> 2 : 0u, t = quarter * 32 + lane;    // row of an epilogue thread
+    float o[HB], inv = 0.f;
+    bool good = false;
+
+    if (warp == 0)
     {
-        mt[i] = M[r0 + gr + 8 * i];
-        carry[i] = p.q_scale * expf(m0 - mt[i]);
-    }
-#pragma unroll
-    for (int j = 0; j < (int)HB / 8; j++)
-    {
-#pragma unroll
-        for (int i = 0; i < 4; i++) { o[j][i] = z2[j][i] = 0.f; }
-    }
-    {
-        const uint32_t kb = ks + ((lane & 7) + ((lane >> 4) << 3)) * QS + ((lane >> 3) & 1) * 16;
-        const uint32_t vb = vs + (lane & 15) * VS + (lane >> 4) * 16 + ch * HB * 2;
-        for (unsigned int s0 = 0; s0 < r0 + 16; s0 += 32)
+        if (lane == 0)
         {
-            float z[4][4];
-#pragma unroll
-            for (int i = 0; i < 4; i++)
+            const int y = (int)first, xq = (int)(h * p.dim), xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
+            mbar_expect_tx(qk_full, 2 * blocks * MO_ROWS);
+            for (unsigned int b = 0; b < blocks; b++)
             {
-#pragma unroll
-                for (int j = 0; j < 4; j++) { z[i][j] = 0.f; }
-            }
-#pragma unroll 4
-            for (int kk = 0; kk < DP / 16; kk++)
-            {
-                uint32_t q[4], b[2][4];
-                ldmatrix_x4(q, qa + kk * 32);
-                ldmatrix_x4(b[0], kb + s0 * QS + kk * 32);
-                ldmatrix_x4(b[1], kb + (s0 + 16) * QS + kk * 32);
-#pragma unroll
-                for (int i = 0; i < 2; i++)
+                for (int r = 0; r < 2; r++)
                 {
-                    mma_bf16_16816(z[2 * i], q[0], q[1], q[2], q[3], b[i][0], b[i][1]);
-                    mma_bf16_16816(z[2 * i + 1], q[0], q[1], q[2], q[3], b[i][2], b[i][3]);
+                    tma_load_2d(qs + b * MO_ROWS + r * MO_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
+                    tma_load_2d(ks + b * MO_ROWS + r * MO_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
                 }
             }
-#pragma unroll
-            for (int i = 0; i < 4; i++)
+            mbar_arrive(qk_full);
+            mbar_expect_tx(v_full, (VB / 64) * MO_ROWS);
+            for (int r = 0; r < 2; r++)    // 64 rows by 64 rows
             {
-#pragma unroll
-                for (int j = 0; j < 4; j++)
-                {
-                    const unsigned int s = s0 + i * 8 + gc + (j & 1), t = r0 + gr + 8 * (j >> 1);
-                    z[i][j] = s <= t ? z[i][j] * p.q_scale * expf(a[s] - mt[j >> 1]) : 0.f;
-                    nq[j >> 1] += z[i][j];
-                }
+                for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MO_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
             }
-#pragma unroll
-            for (int i = 0; i < 2; i++)
+            mbar_arrive(v_full);
+            bool ok = true;
+            unsigned int issued = 0;
+            for (unsigned int i = 0; i < slices && ok; i++)
             {
-                uint32_t top[4], rest[4];
-#pragma unroll
-                for (int j = 0; j < 4; j++)
-                {
-                    // a0: row g, keys 0-7; a1: row g + 8, keys 0-7; a2, a3: keys 8-15
-                    const float* f = &z[2 * i + (j >> 1)][(j & 1) * 2];
-                    top[j] = pack_bf16x2(f[0], f[1]);
-                    rest[j] = pack_bf16x2(f[0] - __uint_as_float(top[j] << 16), f[1] - __uint_as_float(top[j] & 0xFFFF0000u));
-                }
-#pragma unroll
-                for (int j = 0; j < (int)HB / 16; j++)
-                {
-                    uint32_t b[4];
-                    ldmatrix_x4_trans(b, vb + (s0 + i * 16) * VS + j * 32);
-                    mma_bf16_16816(o[2 * j], top[0], top[1], top[2], top[3], b[0], b[1]);
-                    mma_bf16_16816(o[2 * j + 1], top[0], top[1], top[2], top[3], b[2], b[3]);
-                    mma_bf16_16816(o[2 * j], rest[0], rest[1], rest[2], rest[3], b[0], b[1]);
-                    mma_bf16_16816(o[2 * j + 1], rest[0], rest[1], rest[2], rest[3], b[2], b[3]);
-                }
-            }
-        }
-    }
-    nq[0] += __shfl_xor_sync(0xFFFFFFFFu, nq[0], 1);
-    nq[1] += __shfl_xor_sync(0xFFFFFFFFu, nq[1], 1);
-    nq[0] += __shfl_xor_sync(0xFFFFFFFFu, nq[0], 2);
-    nq[1] += __shfl_xor_sync(0xFFFFFFFFu, nq[1], 2);
-    if (!fresh)
-    {
-        __syncthreads();    // k and v have been read
-#pragma unroll
-        for (unsigned int i = 2; i < SLICES; i++)
-        {
-            if (i < 2 + PLACES) { fetch_slice(i); }
-        }
-        // n0 . q: the four lanes of a row share its elements
-#pragma unroll
-        for (int i = 0; i < 2; i++)
-        {
-            const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(mc_raw) + (size_t)(r0 + gr + 8 * i) * (DP + 8);
-            float s = 0.f;
-#pragma unroll 8
-            for (int d = 0; d < DP; d += 8)
-            {
-                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q + d + gc)), g = *reinterpret_cast<const float2*>(n0 + d + gc);
-                s = fmaf(f.x, g.x, fmaf(f.y, g.y, s));
-            }
-            s += __shfl_xor_sync(0xFFFFFFFFu, s, 1);
-            s += __shfl_xor_sync(0xFFFFFFFFu, s, 2);
-            nq[i] += carry[i] * s;
-        }
-        constexpr int ISSUED = (int)(SLICES < 2 + PLACES ? SLICES : 2 + PLACES);
-#pragma unroll
-        for (int i = 0; i < (int)SLICES; i++)
-        {
-            // groups behind slice i: those issued so far, and one more per slice of the second round
-            constexpr int LATE = (int)SLICES - ISSUED;
-            const int behind = i < ISSUED ? ISSUED - 1 - i + (i < LATE ? i : LATE) : (int)SLICES - 1 - i;
-            switch (behind)
-            {
-            case 0: cp_async_wait<0>(); break;
-            case 1: cp_async_wait<1>(); break;
-            case 2: cp_async_wait<2>(); break;
-            case 3: cp_async_wait<3>(); break;
-            case 4: cp_async_wait<4>(); break;
-            case 5: cp_async_wait<5>(); break;
-            default: cp_async_wait<6>(); break;
-            }
-            __syncthreads();
-            const uint32_t sb = place((unsigned int)i) + (lane & 15) * VS + (lane >> 4) * 16 + ch * HB * 2;
-#pragma unroll
-            for (int kk = 0; kk < (int)MC_SLICE / 16; kk++)
-            {
-                uint32_t q[4];
-                ldmatrix_x4(q, qa + (i * MC_SLICE + kk * 16) * 2);
-#pragma unroll
+                const unsigned int at = i % places;
+                if (i == 1) { ok = wait(s_full, 0); }    // k has been read
+                if (ok && i >= places) { ok = wait(slice_empty + at, i / places - 1); }
+                if (!ok) { break; }
+                mbar_expect_tx(slice_full + at, SLICE);
                 for (int part = 0; part < 2; part++)
                 {
-#pragma unroll
-                    for (int j = 0; j < (int)HB / 16; j++)
+                    for (int b = 0; b < VB / 64; b++)
                     {
-                        uint32_t b[4];
-                        ldmatrix_x4_trans(b, sb + part * (SLICE / 2) + kk * 16 * VS + j * 32);
-                        mma_bf16_16816(z2[2 * j], q[0], q[1], q[2], q[3], b[0], b[1]);
-                        mma_bf16_16816(z2[2 * j + 1], q[0], q[1], q[2], q[3], b[2], b[3]);
+                        tma_load_2d(place(i) + (part * (VB / 64) + b) * MO_BLOCK, &tmS, (int)c0 + b * 64, (int)((rec.at * 2 + part) * dp + i * 64), slice_full + at);
                     }
                 }
+                mbar_arrive(slice_full + at);
+                issued++;
             }
-            if (i < LATE)
+            if (!ok)
             {
-                __syncthreads();    // the place of slice i is free
-                fetch_slice((unsigned int)(ISSUED + i));
+                give_up(0, issued);
+                // wait (bounded) for the copies in flight before the CTA may leave
+                auto drain = [&](uint64_t* bar, unsigned int parity) {
+                    const unsigned long long t0 = global_timer_ns();
+                    while (!mbar_try_wait(bar, parity & 1u) && global_timer_ns() - t0 < 100000ull) {}
+                };
+                drain(qk_full, 0);
+                drain(v_full, 0);
+                for (unsigned int i = issued > places ? issued - places : 0; i < issued; i++) { drain(slice_full + i % places, i / places); }
             }
         }
-#pragma unroll
-        for (int j = 0; j < (int)HB / 8; j++)
-        {
-#pragma unroll
-            for (int i = 0; i < 4; i++) { o[j][i] = fmaf(carry[i >> 1], z2[j][i], o[j][i]); }
-        }
     }
-#pragma unroll
-    for (int i = 0; i < 2; i++)
+    else if (warp == 1)
     {
-        const float inv = 1.0f / (fmaxf(fabsf(nq[i]), expf(-(F[r0 + gr + 8 * i] + mt[i]))) + 1e-6f);
-        float s = 0.f;
-#pragma unroll
-        for (int j = 0; j < (int)HB / 8; j++)
+        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), v_addr = smem_u32(vs);
+        const uint32_t idesc_s = umma_idesc_bf16(MC_L, MC_L), idesc_o = umma_idesc_bf16(MC_L, VB) | (1u << 16);    // B is MN-major
+        unsigned int at = 0;
+        bool ok = wait(qk_full, 0);
+        if (ok)
         {
-            o[j][2 * i] *= inv;
-            o[j][2 * i + 1] *= inv;
-            s += o[j][2 * i] * o[j][2 * i] + o[j][2 * i + 1] * o[j][2 * i + 1];
+            tc_fence_after();
+            if (elect_one())
+            {
+                for (unsigned int k = 0; k < steps; k++)
+                {
+                    const uint32_t off = (k / 4) * MO_ROWS + (k % 4) * 32;
+                    umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + off), umma_desc_kmajor_sw128(k_addr + off), idesc_s, k != 0 ? 1u : 0u);
+                }
+                umma_commit(s_full);
+            }
+            __syncwarp();
         }
-        s += __shfl_xor_sync(0xFFFFFFFFu, s, 1);
-        s += __shfl_xor_sync(0xFFFFFFFFu, s, 2);
-        if ((lane & 3) == 0) { sq[ch][r0 + gr + 8 * i] = s; }
+        for (unsigned int i = 0; i < slices && ok; i++)
+        {
+            at = i + 1;
+            ok = wait(slice_full + i % places, i / places);
+            if (!ok) { break; }
+            tc_fence_after();
+            if (elect_one())
+            {
+                const uint32_t s_addr = smem_u32(place(i));
+                for (unsigned int part = 0; part < 2; part++)
+                {
+                    for (unsigned int k = 0; k < 4 && i * 4 + k < steps; k++)
+                    {
+                        umma_bf16(tmem + MO_O + VB, umma_desc_kmajor_sw128(q_addr + i * MO_ROWS + k * 32),
+                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MO_BLOCK + k * 2048), idesc_o, (i | part | k) != 0 ? 1u : 0u);
+                    }
+                }
+                umma_commit(slice_empty + i % places);
+            }
+            __syncwarp();
+        }
+        if (ok)
+        {
+            at = slices + 1;
+            ok = wait(v_full, 0) && wait(p_ready, 0);
+        }
+        if (ok)
+        {
+            tc_fence_after();
+            if (elect_one())
+            {
+                for (unsigned int part = 0; part < 2; part++)
+                {
+                    for (unsigned int k = 0; k < MC_L / 16; k++)
+                    {
+                        umma_bf16_ts(tmem + MO_O, tmem + MO_P + part * 64 + k * 8, umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MO_BLOCK + (k % 4) * 2048),
+                            idesc_o, (part | k) != 0 ? 1u : 0u);
+                    }
+                }
+                umma_commit(o_full);
+            }
+            __syncwarp();
+        }
+        else
+        {
+            if (lane == 0) { give_up(1, at); }
+            if (elect_one()) { umma_commit(o_full); }    // completes once the MMAs in flight have stopped reading shared memory
+            __syncwarp();
+        }
     }
+    else
+    {
+        const uint32_t lanes = tmem + ((quarter * 32u) << 16);
+        const float mt = M[t], mt2 = mt * 1.44269504088896341f, carry = p.q_scale * expf(m0 - mt);
+        float sum = 0.f;
+        good = __all_sync(0xFFFFFFFFu, wait(s_full, 0));
+        if (good)
+        {
+            tc_fence_after();
+            // this half's 64 keys; none of them where the rows of the warp end before
+#pragma unroll
+            for (int q = 0; q < 2; q++)
+            {
+                const unsigned int s0 = half * 64 + q * 32;
+                uint32_t z[32], hi[16], lo[16];
+#pragma unroll
+                for (int j = 0; j < 16; j++) { hi[j] = lo[j] = 0u; }
+                if (s0 <= quarter * 32 + 31)
+                {
+                    tmem_ld_32x32(lanes + s0, z);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                    {
+                        float w[2];
+#pragma unroll
+                        for (int k = 0; k < 2; k++)
+                        {
+                            const unsigned int s = s0 + 2 * j + k;
+                            w[k] = s <= t ? __uint_as_float(z[2 * j + k]) * p.q_scale * exp2_f32(a[s] - mt2) : 0.f;
+                            sum += w[k];
+                        }
+                        hi[j] = pack_bf16x2(w[0], w[1]);
+                        lo[j] = pack_bf16x2(w[0] - __uint_as_float(hi[j] << 16), w[1] - __uint_as_float(hi[j] & 0xFFFF0000u));
+                    }
+                }
+                tmem_st_32x16(lanes + MO_P + s0 / 2, hi);
+                tmem_st_32x16(lanes + MO_P + 64 + s0 / 2, lo);
+            }
+            tmem_st_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) { mbar_arrive(p_ready); }
+            if (!fresh && wait(qk_full, 0))    // n0 . q over half of the elements
+            {
+                float dot = 0.f;
+                for (unsigned int b = half; b < 2 * blocks; b += 2)    // 32 elements at a time
+                {
+                    const unsigned char* row = qs + (b / 2) * MO_ROWS + t * 128;
+#pragma unroll
+                    for (unsigned int q = 0; q < 4; q++)
+                    {
+                        const unsigned int chunk = (b & 1u) * 4 + q;
+                        const uint4 u = *reinterpret_cast<const uint4*>(row + ((chunk ^ (t & 7u)) * 16));
+                        const uint32_t w[4] = { u.x, u.y, u.z, u.w };
+                        const float* g = n0 + (b / 2) * 64 + chunk * 8;
+#pragma unroll
+                        for (int j = 0; j < 4; j++)
+                        {
+                            dot = fmaf(__uint_as_float(w[j] << 16), g[2 * j], dot);
+                            dot = fmaf(__uint_as_float(w[j] & 0xFFFF0000u), g[2 * j + 1], dot);
+                        }
+                    }
+                }
+                sum = fmaf(carry, dot, sum);
+            }
+            nq[half][t] = sum;
+            bar_sync_named(1, 256);
+            inv = 1.0f / (fmaxf(fabsf(nq[0][t] + nq[1][t]), expf(-(F[t] + mt))) + 1e-6f);
+            good = __all_sync(0xFFFFFFFFu, wait(o_full, 0)) && *abort_flag == 0;
+            good = __all_sync(0xFFFFFFFFu, good);
+        }
+        else { bar_sync_named(1, 256); }
+        float s = 0.f;
+        if (good)
+        {
+            tc_fence_after();
+#pragma unroll
+            for (int d = 0; d < HB; d += 32)
+            {
+                uint32_t x[32];
+                tmem_ld_32x32(lanes + MO_O + half * HB + d, x);
+                tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 32; j++) { o[d + j] = __uint_as_float(x[j]); }
+                if (!fresh)
+                {
+                    tmem_ld_32x32(lanes + MO_O + VB + half * HB + d, x);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 32; j++) { o[d + j] = fmaf(carry, __uint_as_float(x[j]), o[d + j]); }
+                }
+#pragma unroll
+                for (int j = 0; j < 32; j++)
+                {
+                    o[d + j] *= inv;
+                    if (c0 + half * HB + d + j < p.vdim) { s += o[d + j] * o[d + j]; }
+                }
+            }
+        }
+        else if (lane == 0) { give_up(2 + quarter, half); }
+        sq[half][t] = s;
+    }
+    tc_fence_before();
     __syncthreads();
+    if (warp == 1) { tmem_dealloc(tmem, MO_TMEM); }
     cg::cluster_group cluster = cg::this_cluster();
     const unsigned int ranks = cluster.num_blocks();
-    for (unsigned int j = tid; j < ranks * MC_L; j += MC_THREADS)
+    for (unsigned int j = tid; j < ranks * MC_L; j += MO_THREADS)
     {
-        const unsigned int t = j % MC_L;
-        cluster.map_shared_rank(&peers[0][0], j / MC_L)[rank * MC_L + t] = sq[0][t] + sq[1][t];
+        const unsigned int r = j % MC_L;
+        cluster.map_shared_rank(&peers[0][0], j / MC_L)[rank * MC_L + r] = sq[0][r] + sq[1][r];
     }
     cluster.sync();
-#pragma unroll
-    for (int i = 0; i < 2; i++)
+    if (good && t < live)
     {
-        const unsigned int t = r0 + gr + 8 * i;
-        if (t >= live) { continue; }
         float s = 0.f;
         for (unsigned int r = 0; r < ranks; r++) { s += peers[r][t]; }
-        const float inv = 1.0f / sqrtf(s / (float)p.vdim + p.eps);
-        const unsigned int at = h * p.vdim + c0 + ch * HB;
-        const __nv_bfloat16* gate = x + (size_t)t * p.ld + p.g_off + at;
+        const float unit = 1.0f / sqrtf(s / (float)p.vdim + p.eps);
+        const unsigned int at = h * p.vdim + c0 + half * HB;
+        const __nv_bfloat16* gate = (const __nv_bfloat16*)p.qkvg + (size_t)(first + t) * p.ld + p.g_off + at;
         __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)(first + t) * p.ldo + at;
         const float* w = p.norm + at;
 #pragma unroll
-        for (int j = 0; j < (int)HB / 8; j++)
+        for (int d = 0; d < HB; d += 8)
         {
-            const unsigned int col = j * 8 + gc;
-            if (c0 + ch * HB + col < p.vdim)
+            if (c0 + half * HB + d >= p.vdim) { continue; }
+            const uint4 u = *reinterpret_cast<const uint4*>(gate + d);
+            const uint32_t g[4] = { u.x, u.y, u.z, u.w };
+            uint32_t y[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++)
             {
-                const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + col));
-                *reinterpret_cast<uint32_t*>(out + col) =
-                    pack_bf16x2(o[j][2 * i] * inv * w[col] * sigmoid_f32(g.x), o[j][2 * i + 1] * inv * w[col + 1] * sigmoid_f32(g.y));
+                y[j] = pack_bf16x2(o[d + 2 * j] * unit * w[d + 2 * j] * sigmoid_f32(__uint_as_float(g[j] << 16)),
+                    o[d + 2 * j + 1] * unit * w[d + 2 * j + 1] * sigmoid_f32(__uint_as_float(g[j] & 0xFFFF0000u)));
             }
+            *reinterpret_cast<uint4*>(out + d) = make_uint4(y[0], y[1], y[2], y[3]);
         }
     }
     if (rank == 0 && (c + 1) * MC_L >= n)
     {
         float* st_n = mlstm_state_of(p, e, h) + (size_t)p.dim * mlstm_v_ld(p.vdim);
-        for (unsigned int d = tid; d < p.dim; d += MC_THREADS) { st_n[d] = rec.last[d]; }
-        if (tid == 0) { st_n[mlstm_n_ld(p.dim)] = rec.last[DP]; }
+        for (unsigned int d = tid; d < p.dim; d += MO_THREADS) { st_n[d] = rec.last[d]; }
+        if (tid == 0) { st_n[mlstm_n_ld(p.dim)] = rec.last[dp]; }
     }
+}
+
+template <int VB>
+static int run_outputs(const MlstmParams& p, cudaStream_t stream, bool pdl)
+{
+    unsigned int* status = decoder_status_word();
+    if (!status) { return 1; }
+    const unsigned int ranks = (p.vdim + VB - 1) / VB, chunks = (p.max_n + MC_L - 1) / MC_L, dp = mc_dp(p.dim), vp = mc_vp(p.vdim);
+    CUtensorMap tx, ts;
+    if (!make_map_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.qkvg, p.ld, (unsigned long long)p.t0 + p.tokens, (unsigned long long)p.ld * 2, 64, 64, true)
+        || !make_map_2d(&ts, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.work, vp, (unsigned long long)mc_slots(p.tokens, p.entries) * p.heads * 2 * dp,
+            (unsigned long long)vp * 2, 64, 64, true))
+    {
+        return -1;
+    }
+    return launch_cluster("mlstm_outputs", mlstm_outputs_kernel<VB>, dim3(ranks, p.heads, p.entries * chunks), dim3(MO_THREADS), (size_t)mo_smem((int)dp, VB), ranks,
+        stream, pdl, tx, ts, p, chunks, status);
 }
 
 template <int DP>
@@ -565,26 +703,22 @@ static int run_chunks(const MlstmParams& p, unsigned int entries, cudaStream_t s
     rc = launch_kernel("mlstm_states", mlstm_states_kernel<DP>, dim3(mc_vp(p.vdim) / MC_COLS, p.heads, entries), dim3(MC_THREADS), (size_t)mc_states_smem(DP),
         stream, pdl, p);
     if (rc) { return rc; }
-    auto outputs = [&](auto kernel, unsigned int vb) {
-        const unsigned int ranks = (p.vdim + vb - 1) / vb;
-        return launch_cluster("mlstm_outputs", kernel, dim3(ranks, p.heads, entries * chunks), dim3(MC_THREADS), (size_t)mc_outputs_smem(DP, vb), ranks, stream, pdl,
-            p, chunks);
-    };
-    return p.vdim <= 64 ? outputs(mlstm_outputs_kernel<DP, 64>, 64) : outputs(mlstm_outputs_kernel<DP, 128>, 128);
+    return p.vdim <= 64 ? run_outputs<64>(p, stream, pdl) : run_outputs<128>(p, stream, pdl);
 }
 
 unsigned long long mlstm_chunk_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim, unsigned int vdim)
 {
-    return (unsigned long long)(tokens / MC_L + entries) * heads * mc_record(dim, vdim);
+    return (unsigned long long)mc_slots(tokens, entries) * heads * (mc_matrix(dim, vdim) + mc_record(dim));
 }
 
-bool mlstm_chunk_takes(unsigned int dim, unsigned int vdim) { return (dim % 8) == 0 && (vdim % 8) == 0 && dim <= MC_MAX_DIM && vdim <= 128 * MC_MAX_CLUSTER; }
+bool mlstm_chunk_takes(unsigned int dim, unsigned int vdim) { return (dim % 16) == 0 && (vdim % 8) == 0 && dim <= MC_MAX_DIM && vdim <= 128 * MC_MAX_CLUSTER; }
 
 int launch_mlstm_chunk(const MlstmParams& p, unsigned int entries, cudaStream_t stream, bool pdl)
 {
     const unsigned int chunks = (p.max_n + MC_L - 1) / MC_L;
-    if (!mlstm_chunk_takes(p.dim, p.vdim) || (p.ld % 8) || (p.k_off % 8) || (p.v_off % 8) || (p.g_off % 2) || (p.ldo % 2)
-        || (unsigned long long)entries * chunks > 65535ull)
+    auto low = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) != 0; };
+    if (!mlstm_chunk_takes(p.dim, p.vdim) || (p.ld % 8) || (p.k_off % 8) || (p.v_off % 8) || (p.g_off % 8) || (p.ldo % 8)
+        || low(p.qkvg) || low(p.work) || low(p.out) || (unsigned long long)entries * chunks > 65535ull)
     {
         return -1;
     }
