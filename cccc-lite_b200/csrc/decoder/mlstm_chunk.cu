@@ -5,14 +5,13 @@
 //   o_t ~ e^(m_0 - M_t) S_0^T q_t + sum_{s <= t} e^(a_s - M_t) (q_t . k_s) v_s,   S_L = e^(m_0 - M_L) S_0 + sum_s e^(a_s - M_L) k_s v_s^T,
 // no exponent above zero.  Three kernels:
 //   gates  : F and a of every chunk.
-//   states : a CTA per 32 value columns of a head walks an entry's chunks, its columns of S as float accumulators in registers
-//            (mma.sync); it leaves the state ahead of every chunk in scratch memory.
-//   outputs: a cluster per (chunk, head), a CTA per 64 or 128 value columns, on tcgen05; the head's sum of squares meets in the
-//            cluster.
+//   states : a CTA per 64 value columns of a head (and one for n) walks an entry's chunks, its columns of S as the accumulator in
+//            tensor memory; it leaves the state ahead of every chunk in scratch memory.
+//   outputs: a cluster per (chunk, head), a CTA per 64 or 128 value columns; the head's sum of squares meets in the cluster.
 // One operand of every product is exact (q, k or v); the other - S, weighted values, weighted scores - enters as the sum of two
-// BF16 numbers.
+// BF16 numbers.  The products of states and outputs are tcgen05's.  Every wait is bounded; on expiry the status word is raised, the
+// roles drain, tensor memory is freed and the CTA returns.
 #include "../gemm_stream.cuh"
-#include "attention_mma.cuh"
 #include "mlstm.cuh"
 #include "tile_common.cuh"
 
@@ -23,7 +22,8 @@ namespace cg = cooperative_groups;
 namespace b200
 {
 
-constexpr unsigned int MC_L = 128, MC_WARPS = 16, MC_THREADS = 32 * MC_WARPS, MC_COLS = 32, MC_MAX_DIM = 256, MC_MAX_CLUSTER = 8;
+constexpr unsigned int MC_L = 128, MC_COLS = 64, MC_MAX_DIM = 256, MC_MAX_CLUSTER = 8;
+constexpr int MC_BLOCK = 64 * 128, MC_ROWS = 2 * MC_BLOCK;    // 64 rows x 64 elements; the 128 tokens' block of 64 elements
 
 __host__ __device__ __forceinline__ unsigned int mc_dp(unsigned int dim) { return dim <= 64 ? 64 : (dim <= 128 ? 128 : 256); }
 __host__ __device__ __forceinline__ unsigned int mc_vp(unsigned int vdim) { return (vdim + MC_COLS - 1) / MC_COLS * MC_COLS; }
@@ -90,244 +90,334 @@ __global__ void __launch_bounds__(MC_L) mlstm_gates_kernel(const MlstmParams p)
     }
 }
 
-// Rows [0, live) of a projection, `width` elements from `src` on, into padded shared rows of PADDED elements; rows behind and columns
-// past `width` are zero.
-template <unsigned int PADDED>
-__device__ __forceinline__ void mc_fetch(uint32_t dst, const __nv_bfloat16* src, unsigned int ld, unsigned int live, unsigned int width)
-{
-    constexpr unsigned int PER = PADDED / 8, STRIDE = (PADDED + 8) * 2;
-#pragma unroll
-    for (unsigned int i = 0; i < (MC_L * PER + MC_THREADS - 1) / MC_THREADS; i++)
-    {
-        const unsigned int c = threadIdx.x + i * MC_THREADS, r = c / PER, d = c % PER;
-        if (MC_L * PER % MC_THREADS == 0 || c < MC_L * PER)
-        {
-            const bool ok = r < live && d * 8 < width;
-            cp_async16(dst + r * STRIDE + d * 16, src + (ok ? (size_t)r * ld + d * 8 : 0), ok);
-        }
-    }
-}
+// ---- states ----------------------------------------------------------------------------------------
+constexpr int MS_ROLES = 32 * 14;
+constexpr uint32_t MS_TMEM = 128;    // 64 columns for each 128 rows of S
+// header, k twice, v, weighted values (high, low) twice
+__host__ __device__ constexpr int mc_states_smem(int dp) { return 1024 + 2 * (dp / 64) * MC_ROWS + MC_ROWS + 4 * MC_ROWS + 1024; }
 
-// grid (column blocks of 32, heads, entries); a warp owns 16 rows of S
-template <int DP>
-__global__ void __launch_bounds__(MC_THREADS) mlstm_states_kernel(const MlstmParams p)
+// grid (column blocks of 64 and one for n, heads, entries).  A TMA lane fetches k and v of the chunks; four warps weight the values, a
+// token per thread; eight warps own the rows of S, one per thread: between the chunks they take S out of tensor memory, store it
+// for the second kernel and put it back scaled; the MMA lane adds k^T (weighted v) onto it.  The block of n has ones for its
+// values' first column.
+__global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ MlstmParams p,
+    unsigned int* status)
 {
-    extern __shared__ __align__(16) unsigned char mc_raw[];
-    constexpr unsigned int VS = (MC_COLS + 8) * 2, KS = (DP + 8) * 2, KBYTES = MC_L * KS;
-    __shared__ float w[MC_L];
-    // weighted values; behind the columns the weights themselves, which make n
-    __shared__ __align__(16) __nv_bfloat16 hi[MC_L * (MC_COLS + 8)], lo[MC_L * (MC_COLS + 8)];
-    const unsigned int vp = mc_vp(p.vdim);
-    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gt = lane & 3, gc = gt * 2, d0 = warp * 16;
-    const unsigned int c0 = blockIdx.x * MC_COLS, h = blockIdx.y, e = p.e0 + blockIdx.z;
+    extern __shared__ unsigned char ms_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(ms_raw) + 1023) & ~(uintptr_t)1023);
+    const unsigned int dp = mc_dp(p.dim), vp = mc_vp(p.vdim), blocks = dp / 64;
+    uint64_t* k_full = reinterpret_cast<uint64_t*>(smem);
+    uint64_t *k_empty = k_full + 2, *vp_full = k_full + 4, *vp_empty = k_full + 6, *v_full = k_full + 8, *v_empty = k_full + 9, *s_ready = k_full + 10,
+             *s_done = k_full + 11;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 12);
+    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
+    unsigned char* ks = smem + 1024;
+    unsigned char* vs = ks + 2 * blocks * MC_ROWS;
+    unsigned char* ws = vs + MC_ROWS;    // [buffer][high, low]
+
+    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const bool is_n = blockIdx.x == gridDim.x - 1;
+    const unsigned int c0 = is_n ? 0u : blockIdx.x * MC_COLS, h = blockIdx.y, e = p.e0 + blockIdx.z;
+    if (tid == 0)
+    {
+        for (int i = 0; i < 12; i++) { mbar_init(k_full + i, i == 4 || i == 5 || i == 9 ? 4 : (i == 10 ? 8 : 1)); }
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) { tmem_alloc(tmem_slot, MS_TMEM); }
     grid_dependency_launch();
     grid_dependency_wait();
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], chunks = (n + MC_L - 1) / MC_L;
     const bool fresh = p.pos[e] == 0;
+    const ChunkRecord first = mc_record_of(p, e, 0, h);
+    // of chunk c: its largest a and its last F
+    auto end_of = [&](unsigned int c) { return *reinterpret_cast<const float2*>(first.top + (size_t)c * p.heads * mc_record(p.dim)); };
     float* st = mlstm_state_of(p, e, h);
-    const unsigned int v_ld = mlstm_v_ld(p.vdim), vw = min(MC_COLS, p.vdim - c0);
+    const unsigned int v_ld = mlstm_v_ld(p.vdim);
     float* st_n = st + (size_t)p.dim * v_ld;
-    const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg + (size_t)start * p.ld;
-    const uint32_t ks = smem_u32(mc_raw), vs = ks + 2 * KBYTES, hs = smem_u32(hi), ls = smem_u32(lo);
-    const __nv_bfloat16* v_raw = reinterpret_cast<const __nv_bfloat16*>(mc_raw + 2 * KBYTES);
-    auto fetch = [&](unsigned int c) {
-        if (c < chunks)
-        {
-            const unsigned int live = min(MC_L, n - c * MC_L);
-            mc_fetch<DP>(ks + (c & 1u) * KBYTES, x + (size_t)c * MC_L * p.ld + p.k_off + h * p.dim, p.ld, live, p.dim);
-            mc_fetch<MC_COLS>(vs + (c & 1u) * MC_L * VS, x + (size_t)c * MC_L * p.ld + p.v_off + h * p.vdim + c0, p.ld, live, vw);
-        }
-        cp_async_commit();
+    const float m_start = fresh ? 0.f : st_n[mlstm_n_ld(p.dim)];
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    auto give_up = [&](unsigned int role, unsigned int step) {
+        note_timeout(status, WAIT_MLSTM_STATES, role, step);
+        *abort_flag = 1;
     };
-    fetch(0);
-    float S[MC_COLS / 8][4];
-#pragma unroll
-    for (int j = 0; j < (int)MC_COLS / 8; j++)
+    auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
+
+    if (warp == 0)
     {
-#pragma unroll
-        for (int half = 0; half < 2; half++)
+        if (lane == 0)
         {
-            const unsigned int d = d0 + gr + 8 * half, col = c0 + j * 8 + gc;
-            float2 v = make_float2(0.f, 0.f);
-            if (!fresh && d < p.dim && col < p.vdim) { v = *reinterpret_cast<const float2*>(st + (size_t)d * v_ld + col); }
-            S[j][2 * half] = v.x;
-            S[j][2 * half + 1] = v.y;
-        }
-    }
-    float m = fresh ? 0.f : st_n[mlstm_n_ld(p.dim)];
-    float nn[4] = { 0.f, 0.f, 0.f, 0.f };    // n of rows gr and gr + 8 in the first column's lanes, elements 0 and 2
-    const bool carries = blockIdx.x == 0, holds = carries && gt == 0 && d0 < (unsigned int)DP;
-#pragma unroll
-    for (int half = 0; half < 2; half++)
-    {
-        const unsigned int d = d0 + gr + 8 * half;
-        if (holds && !fresh && d < p.dim) { nn[2 * half] = st_n[d]; }
-    }
-    if (tid < MC_L)
-    {
-#pragma unroll
-        for (int j = 0; j < 4; j++)
-        {
-            reinterpret_cast<uint32_t*>(hi + tid * (MC_COLS + 8) + MC_COLS)[j] = 0u;
-            reinterpret_cast<uint32_t*>(lo + tid * (MC_COLS + 8) + MC_COLS)[j] = 0u;
-        }
-    }
-    ChunkRecord rec = mc_record_of(p, e, 0, h);
-    float a = tid < MC_L ? rec.a[tid] : 0.f;
-    float2 end = *reinterpret_cast<const float2*>(rec.top);
-    for (unsigned int c = 0; c < chunks; c++)
-    {
-        const unsigned int live = min(MC_L, n - c * MC_L);
-        fetch(c + 1);
-        const float top = fmaxf(m, end.x), keep = expf(m - top);    // M at the chunk's end
-        if (tid < MC_L)
-        {
-            const float y = expf(a - top);
-            const __nv_bfloat16 high = __float2bfloat16_rn(y);
-            w[tid] = y;
-            hi[tid * (MC_COLS + 8) + MC_COLS] = high;
-            lo[tid * (MC_COLS + 8) + MC_COLS] = __float2bfloat16_rn(y - __bfloat162float(high));
-        }
-        if (d0 < (unsigned int)DP && (!fresh || c > 0))
-        {
-#pragma unroll
-            for (int half = 0; half < 2; half++)
+            const int xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
+            unsigned int k_issued = 0, v_issued = 0;
+            bool ok = true;
+            for (unsigned int c = 0; c < chunks && ok; c++)
             {
-                uint32_t part[2][4];    // high, low; of the eight columns of tile j
-#pragma unroll
-                for (int j = 0; j < 4; j++)
+                const unsigned int s = c & 1u;
+                const int y = (int)(start + c * MC_L);
+                if (c >= 2 && !wait(k_empty + s, (c >> 1) - 1)) { ok = false; break; }
+                mbar_expect_tx(k_full + s, blocks * MC_ROWS);
+                for (unsigned int r = 0; r < 2; r++)    // 64 tokens by 64 tokens
                 {
-                    const float s0 = S[j][2 * half], s1 = S[j][2 * half + 1];
-                    part[0][j] = pack_bf16x2(s0, s1);
-                    part[1][j] = pack_bf16x2(s0 - __uint_as_float(part[0][j] << 16), s1 - __uint_as_float(part[0][j] & 0xFFFF0000u));
-                }
-                // the four lanes of a row exchange, so that lane t has all of tile t
-#pragma unroll
-                for (int k = 0; k < 2; k++)
-                {
-                    uint32_t row[4];
-#pragma unroll
-                    for (int step = 0; step < 4; step++)
+                    for (unsigned int b = 0; b < blocks; b++)
                     {
-                        // to lane gt ^ step goes tile gt ^ step
-                        const unsigned int j = gt ^ step;
-                        const uint32_t give = j == 0 ? part[k][0] : (j == 1 ? part[k][1] : (j == 2 ? part[k][2] : part[k][3]));
-                        const uint32_t got = __shfl_xor_sync(0xFFFFFFFFu, give, step);
+                        tma_load_2d(ks + ((s * 2 + r) * blocks + b) * MC_BLOCK, &tmX, xk + (int)b * 64, y + (int)r * 64, k_full + s);
+                    }
+                }
+                mbar_arrive(k_full + s);
+                k_issued++;
+                if (is_n) { continue; }
+                if (c >= 1 && !wait(v_empty, c - 1)) { ok = false; break; }
+                mbar_expect_tx(v_full, MC_ROWS);
+                for (unsigned int r = 0; r < 2; r++) { tma_load_2d(vs + r * MC_BLOCK, &tmX, xv, y + (int)r * 64, v_full); }
+                mbar_arrive(v_full);
+                v_issued++;
+            }
+            if (!ok)
+            {
+                give_up(0, k_issued);
+                // wait (bounded) for the copies in flight before the CTA may leave
+                auto drain = [&](uint64_t* bar, unsigned int parity) {
+                    const unsigned long long t0 = global_timer_ns();
+                    while (!mbar_try_wait(bar, parity & 1u) && global_timer_ns() - t0 < 100000ull) {}
+                };
+                for (unsigned int i = k_issued > 2 ? k_issued - 2 : 0; i < k_issued; i++) { drain(k_full + (i & 1u), i >> 1); }
+                if (v_issued != 0) { drain(v_full, v_issued - 1); }
+            }
+        }
+    }
+    else if (warp == 1)
+    {
+        const uint32_t k_addr = smem_u32(ks), w_addr = smem_u32(ws);
+        const uint32_t idesc = umma_idesc_bf16(128, MC_COLS) | (1u << 15) | (1u << 16);    // both operands lie with their k outermost
+        bool ok = true;
+        unsigned int c = 0;
+        for (; c < chunks && ok; c++)
+        {
+            const unsigned int s = c & 1u;
+            ok = wait(k_full + s, c >> 1) && wait(vp_full + s, c >> 1) && wait(s_ready, c);
+            if (!ok) { break; }
+            tc_fence_after();
+            if (elect_one())
+            {
+                for (unsigned int mb = 0; mb < (dp + 127) / 128; mb++)
+                {
+                    for (unsigned int part = 0; part < 2; part++)
+                    {
 #pragma unroll
-                        for (unsigned int i = 0; i < 4; i++)
+                        for (unsigned int k = 0; k < MC_L / 16; k++)
                         {
-                            if (i == (gt ^ (unsigned int)step)) { row[i] = got; }
+                            umma_bf16(tmem + mb * MC_COLS,
+                                umma_desc_mnmajor_sw128(k_addr + ((s * 2 + k / 4) * blocks + mb * 2) * MC_BLOCK + (k % 4) * 2048),
+                                umma_desc_mnmajor_sw128(w_addr + (s * 2 + part) * MC_ROWS + (k / 4) * MC_BLOCK + (k % 4) * 2048), idesc, 1u);
                         }
                     }
-                    __nv_bfloat16* y = rec.S + (size_t)(k * DP + d0 + gr + 8 * half) * vp + c0 + gt * 8;
-                    *reinterpret_cast<uint4*>(y) = make_uint4(row[0], row[1], row[2], row[3]);
                 }
+                umma_commit(k_empty + s);
+                umma_commit(vp_empty + s);
+                umma_commit(s_done);
             }
+            __syncwarp();
         }
-        if (holds)
+        if (!ok)
         {
-            rec.n[d0 + gr] = nn[0];
-            rec.n[d0 + gr + 8] = nn[2];
+            if (lane == 0) { give_up(1, c); }
+            if (elect_one()) { umma_commit(s_done); }    // completes once the MMAs in flight have stopped reading shared memory
+            __syncwarp();
         }
-        if (carries && tid == 0) { rec.n[DP] = m; }
-        m = end.y + top;
-        const ChunkRecord now = rec;
-        if (c + 1 < chunks)
-        {
-            rec = mc_record_of(p, e, c + 1, h);
-            if (tid < MC_L) { a = rec.a[tid]; }
-            end = *reinterpret_cast<const float2*>(rec.top);
-        }
-        cp_async_wait<1>();
-        __syncthreads();
-        const __nv_bfloat16* v = v_raw + (c & 1u) * MC_L * (MC_COLS + 8);
+    }
+    else if (warp < 10)
+    {
+        const unsigned int quarter = warp & 3u, mb = (warp - 2) >> 2, d = mb * 128 + quarter * 32 + lane;
+        const uint32_t mine = tmem + ((quarter * 32u) << 16) + mb * MC_COLS;
+        const bool some = mb * 128 + quarter * 32 < dp;    // does the warp have rows
+        float m = m_start;
+        bool ok = true;
+        uint32_t S[MC_COLS];
 #pragma unroll
-        for (unsigned int i = tid; i < MC_L * MC_COLS / 2; i += MC_THREADS)
+        for (int j = 0; j < (int)MC_COLS; j++) { S[j] = 0u; }
+        if (!fresh && d < p.dim)
         {
-            const unsigned int s = i / (MC_COLS / 2), at = s * (MC_COLS + 8) + (i % (MC_COLS / 2)) * 2;
-            const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v + at));
-            const float y0 = w[s] * f.x, y1 = w[s] * f.y;
-            const uint32_t u = pack_bf16x2(y0, y1);
-            *reinterpret_cast<uint32_t*>(hi + at) = u;
-            *reinterpret_cast<uint32_t*>(lo + at) = pack_bf16x2(y0 - __uint_as_float(u << 16), y1 - __uint_as_float(u & 0xFFFF0000u));
-        }
-        __syncthreads();
-        if (d0 < (unsigned int)DP)
-        {
-            const uint32_t kb = ks + (c & 1u) * KBYTES + ((lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 16 + d0 * 2;
-            const uint32_t vb = (lane & 15) * VS + (lane >> 4) * 16;
-#pragma unroll
-            for (int j = 0; j < (int)MC_COLS / 8; j++)
+            if (is_n) { S[0] = __float_as_uint(st_n[d]); }
+            else
             {
 #pragma unroll
-                for (int i = 0; i < 4; i++) { S[j][i] *= keep; }
-            }
-#pragma unroll
-            for (int i = 0; i < 4; i++) { nn[i] *= keep; }
-#pragma unroll 4
-            for (unsigned int s0 = 0; s0 < live; s0 += 16)
-            {
-                uint32_t b[2][MC_COLS / 16][4], k[4];
-                if (carries)
+                for (int j = 0; j < (int)MC_COLS; j += 4)
                 {
-                    uint32_t x[4];
-                    ldmatrix_x4_trans(x, (lane < 16 ? hs : ls) + (s0 + (lane & 15)) * VS + MC_COLS * 2);
-                    uint32_t k2[4];
-                    ldmatrix_x4_trans(k2, kb + s0 * KS);
-                    mma_bf16_16816(nn, k2[0], k2[1], k2[2], k2[3], x[0], x[1]);
-                    mma_bf16_16816(nn, k2[0], k2[1], k2[2], k2[3], x[2], x[3]);
-                }
-                ldmatrix_x4_trans(k, kb + s0 * KS);
-#pragma unroll
-                for (int j = 0; j < (int)MC_COLS / 16; j++)
-                {
-                    ldmatrix_x4_trans(b[0][j], hs + vb + s0 * VS + j * 32);
-                    ldmatrix_x4_trans(b[1][j], ls + vb + s0 * VS + j * 32);
-                }
-#pragma unroll
-                for (int part = 0; part < 2; part++)
-                {
-#pragma unroll
-                    for (int j = 0; j < (int)MC_COLS / 16; j++)
+                    if (c0 + j < p.vdim)
                     {
-                        mma_bf16_16816(S[2 * j], k[0], k[1], k[2], k[3], b[part][j][0], b[part][j][1]);
-                        mma_bf16_16816(S[2 * j + 1], k[0], k[1], k[2], k[3], b[part][j][2], b[part][j][3]);
+                        const uint4 u = *reinterpret_cast<const uint4*>(st + (size_t)d * v_ld + c0 + j);
+                        S[j] = u.x;
+                        S[j + 1] = u.y;
+                        S[j + 2] = u.z;
+                        S[j + 3] = u.w;
                     }
                 }
             }
         }
-        // other column blocks may still have to read the old n and m: the last kernel puts the new ones in place
-        if (c + 1 == chunks)
+        float2 end = end_of(0);
+        for (unsigned int c = 0; c < chunks; c++)
         {
-            if (holds)
+            const float top = fmaxf(m, end.x), keep = expf(m - top), m_before = m;
+            m = end.y + top;
+            if (c + 1 < chunks) { end = end_of(c + 1); }
+            if (c > 0)
             {
-                now.last[d0 + gr] = nn[0];
-                now.last[d0 + gr + 8] = nn[2];
+                ok = __all_sync(0xFFFFFFFFu, wait(s_done, c - 1));
+                if (!ok) { break; }
+                tc_fence_after();
+                if (some)
+                {
+                    tmem_ld_32x32(mine, *reinterpret_cast<uint32_t(*)[32]>(S));
+                    tmem_ld_32x32(mine + 32, *reinterpret_cast<uint32_t(*)[32]>(S + 32));
+                    tmem_ld_wait();
+                }
             }
-            if (carries && tid == 0) { now.last[DP] = m; }
+            if (some)
+            {
+                uint32_t scaled[MC_COLS];
+#pragma unroll
+                for (int j = 0; j < (int)MC_COLS; j++) { scaled[j] = __float_as_uint(__uint_as_float(S[j]) * keep); }
+#pragma unroll
+                for (int j = 0; j < (int)MC_COLS; j += 16) { tmem_st_32x16(mine + j, scaled + j); }
+                tmem_st_wait();
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) { mbar_arrive(s_ready); }
+            // the state ahead of the chunk, while the products run
+            if (d < dp && (is_n || !fresh || c > 0))
+            {
+                if (is_n)
+                {
+                    float* out = first.n + (size_t)c * p.heads * mc_record(p.dim);
+                    out[d] = __uint_as_float(S[0]);
+                    if (d == 0) { out[dp] = m_before; }
+                }
+                else
+                {
+                    __nv_bfloat16* out = first.S + (size_t)c * p.heads * 2 * mc_matrix(p.dim, p.vdim) + (size_t)d * vp + c0;
+#pragma unroll
+                    for (int j = 0; j < (int)MC_COLS; j += 8)
+                    {
+                        uint32_t hi[4], lo[4];
+#pragma unroll
+                        for (int i = 0; i < 4; i++)
+                        {
+                            const float a = __uint_as_float(S[j + 2 * i]), b = __uint_as_float(S[j + 2 * i + 1]);
+                            hi[i] = pack_bf16x2(a, b);
+                            lo[i] = pack_bf16x2(a - __uint_as_float(hi[i] << 16), b - __uint_as_float(hi[i] & 0xFFFF0000u));
+                        }
+                        *reinterpret_cast<uint4*>(out + j) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                        *reinterpret_cast<uint4*>(out + (size_t)dp * vp + j) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                    }
+                }
+            }
         }
-        __syncthreads();    // the next chunk but one takes this one's place
-    }
-    cp_async_wait<0>();
-#pragma unroll
-    for (int j = 0; j < (int)MC_COLS / 8; j++)
-    {
-#pragma unroll
-        for (int half = 0; half < 2; half++)
+        ok = ok && __all_sync(0xFFFFFFFFu, wait(s_done, chunks - 1));
+        if (ok)
         {
-            const unsigned int d = d0 + gr + 8 * half, col = c0 + j * 8 + gc;
-            if (d < p.dim && col < p.vdim) { *reinterpret_cast<float2*>(st + (size_t)d * v_ld + col) = make_float2(S[j][2 * half], S[j][2 * half + 1]); }
+            tc_fence_after();
+            if (some)
+            {
+                tmem_ld_32x32(mine, *reinterpret_cast<uint32_t(*)[32]>(S));
+                tmem_ld_32x32(mine + 32, *reinterpret_cast<uint32_t(*)[32]>(S + 32));
+                tmem_ld_wait();
+            }
+            if (is_n)
+            {
+                // other column blocks may still have to read the old m: the last kernel puts the new n and m in place
+                float* out = first.last + (size_t)(chunks - 1) * p.heads * mc_record(p.dim);
+                if (d < dp) { out[d] = __uint_as_float(S[0]); }
+                if (d == 0) { out[dp] = m; }
+            }
+            else if (d < p.dim)
+            {
+#pragma unroll
+                for (int j = 0; j < (int)MC_COLS; j += 4)
+                {
+                    if (c0 + j < p.vdim) { *reinterpret_cast<uint4*>(st + (size_t)d * v_ld + c0 + j) = make_uint4(S[j], S[j + 1], S[j + 2], S[j + 3]); }
+                }
+            }
         }
+        else if (lane == 0) { give_up(2 + quarter, mb); }
     }
+    else
+    {
+        const unsigned int t = tid - 320;    // token of the chunk
+        float m = m_start;
+        bool ok = true;
+        float2 end = end_of(0);
+        float a = first.a[t];
+        unsigned int c = 0;
+        for (; c < chunks; c++)
+        {
+            const unsigned int s = c & 1u;
+            const float top = fmaxf(m, end.x), w = expf(a - top);
+            m = end.y + top;
+            if (c + 1 < chunks)
+            {
+                end = end_of(c + 1);
+                a = first.a[(size_t)(c + 1) * p.heads * mc_record(p.dim) + t];
+            }
+            ok = (is_n || wait(v_full, c)) && (c < 2 || wait(vp_empty + s, (c >> 1) - 1));
+            ok = __all_sync(0xFFFFFFFFu, ok);
+            if (!ok) { break; }
+            const unsigned char* src = vs + t * 128;
+            unsigned char* dst = ws + s * 2 * MC_ROWS + t * 128;
+#pragma unroll
+            for (unsigned int q = 0; q < 8; q++)
+            {
+                const unsigned int at = (q ^ (t & 7u)) * 16;
+                float f[8];
+                if (is_n)
+                {
+#pragma unroll
+                    for (int i = 0; i < 8; i++) { f[i] = q == 0 && i == 0 ? w : 0.f; }
+                }
+                else
+                {
+                    const uint4 u = *reinterpret_cast<const uint4*>(src + at);
+                    const uint32_t x[4] = { u.x, u.y, u.z, u.w };
+#pragma unroll
+                    for (int i = 0; i < 4; i++)
+                    {
+                        f[2 * i] = w * __uint_as_float(x[i] << 16);
+                        f[2 * i + 1] = w * __uint_as_float(x[i] & 0xFFFF0000u);
+                    }
+                }
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                {
+                    hi[i] = pack_bf16x2(f[2 * i], f[2 * i + 1]);
+                    lo[i] = pack_bf16x2(f[2 * i] - __uint_as_float(hi[i] << 16), f[2 * i + 1] - __uint_as_float(hi[i] & 0xFFFF0000u));
+                }
+                *reinterpret_cast<uint4*>(dst + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                *reinterpret_cast<uint4*>(dst + MC_ROWS + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+            fence_proxy_async();
+            __syncwarp();
+            if (lane == 0)
+            {
+                mbar_arrive(vp_full + s);
+                if (!is_n) { mbar_arrive(v_empty); }
+            }
+        }
+        if (!ok && lane == 0) { give_up(6, c); }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) { tmem_dealloc(tmem, MS_TMEM); }
 }
 
-__host__ __device__ constexpr unsigned int mc_states_smem(unsigned int dp) { return 2 * MC_L * ((dp + 8) * 2 + (MC_COLS + 8) * 2); }
 // ---- outputs ---------------------------------------------------------------------------------------
 constexpr int MO_THREADS = 32 * 10;
-constexpr int MO_BLOCK = 64 * 128, MO_ROWS = 2 * MO_BLOCK;    // 64 rows x 64 elements; the 128 tokens' block of 64 elements
 constexpr uint32_t MO_P = 128, MO_O = 256, MO_TMEM = 512;      // columns: scores, weighted scores (high, low), what the chunk gives, what S gives
-__host__ __device__ constexpr int mo_slice(int vb) { return 2 * (vb / 64) * MO_BLOCK; }    // 64 rows of S: high, low
-__host__ __device__ constexpr int mo_smem(int dp, int vb) { return 1024 + 2 * (dp / 64) * MO_ROWS + (vb / 64) * MO_ROWS + mo_slice(vb) + 1024; }
+__host__ __device__ constexpr int mo_slice(int vb) { return 2 * (vb / 64) * MC_BLOCK; }    // 64 rows of S: high, low
+__host__ __device__ constexpr int mo_smem(int dp, int vb) { return 1024 + 2 * (dp / 64) * MC_ROWS + (vb / 64) * MC_ROWS + mo_slice(vb) + 1024; }
 
 // grid (column blocks of VB = the cluster, heads, entries x chunks).  A TMA lane fetches q, k and v of the chunk and slices of 64 rows of
 // S: the first beside them, the following ones where k was, once the scores are out.  The MMA lane issues q k^T, then q S, then
@@ -347,10 +437,10 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(slice_empty + MAX_PLACES);
     volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
     unsigned char* qs = smem + 1024;
-    unsigned char* ks = qs + blocks * MO_ROWS;
-    unsigned char* vs = ks + blocks * MO_ROWS;
-    unsigned char* ss = vs + (VB / 64) * MO_ROWS;
-    const unsigned int places = min((unsigned int)MAX_PLACES, 1u + blocks * MO_ROWS / SLICE);    // of slices
+    unsigned char* ks = qs + blocks * MC_ROWS;
+    unsigned char* vs = ks + blocks * MC_ROWS;
+    unsigned char* ss = vs + (VB / 64) * MC_ROWS;
+    const unsigned int places = min((unsigned int)MAX_PLACES, 1u + blocks * MC_ROWS / SLICE);    // of slices
     auto place = [&](unsigned int i) { return i % places == 0 ? ss : ks + (i % places - 1) * SLICE; };
 
     const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -398,7 +488,7 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
     auto give_up = [&](unsigned int role, unsigned int step) {
-        note_timeout(status, WAIT_MLSTM_TILE, role, step);
+        note_timeout(status, WAIT_MLSTM_OUTPUTS, role, step);
         *abort_flag = 1;
     };
     auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
@@ -411,20 +501,20 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
         if (lane == 0)
         {
             const int y = (int)first, xq = (int)(h * p.dim), xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
-            mbar_expect_tx(qk_full, 2 * blocks * MO_ROWS);
+            mbar_expect_tx(qk_full, 2 * blocks * MC_ROWS);
             for (unsigned int b = 0; b < blocks; b++)
             {
                 for (int r = 0; r < 2; r++)
                 {
-                    tma_load_2d(qs + b * MO_ROWS + r * MO_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
-                    tma_load_2d(ks + b * MO_ROWS + r * MO_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
+                    tma_load_2d(qs + b * MC_ROWS + r * MC_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
+                    tma_load_2d(ks + b * MC_ROWS + r * MC_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
                 }
             }
             mbar_arrive(qk_full);
-            mbar_expect_tx(v_full, (VB / 64) * MO_ROWS);
+            mbar_expect_tx(v_full, (VB / 64) * MC_ROWS);
             for (int r = 0; r < 2; r++)    // 64 rows by 64 rows
             {
-                for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MO_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
+                for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MC_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
             }
             mbar_arrive(v_full);
             bool ok = true;
@@ -440,7 +530,7 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                 {
                     for (int b = 0; b < VB / 64; b++)
                     {
-                        tma_load_2d(place(i) + (part * (VB / 64) + b) * MO_BLOCK, &tmS, (int)c0 + b * 64, (int)((rec.at * 2 + part) * dp + i * 64), slice_full + at);
+                        tma_load_2d(place(i) + (part * (VB / 64) + b) * MC_BLOCK, &tmS, (int)c0 + b * 64, (int)((rec.at * 2 + part) * dp + i * 64), slice_full + at);
                     }
                 }
                 mbar_arrive(slice_full + at);
@@ -473,7 +563,7 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
             {
                 for (unsigned int k = 0; k < steps; k++)
                 {
-                    const uint32_t off = (k / 4) * MO_ROWS + (k % 4) * 32;
+                    const uint32_t off = (k / 4) * MC_ROWS + (k % 4) * 32;
                     umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + off), umma_desc_kmajor_sw128(k_addr + off), idesc_s, k != 0 ? 1u : 0u);
                 }
                 umma_commit(s_full);
@@ -493,8 +583,8 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                 {
                     for (unsigned int k = 0; k < 4 && i * 4 + k < steps; k++)
                     {
-                        umma_bf16(tmem + MO_O + VB, umma_desc_kmajor_sw128(q_addr + i * MO_ROWS + k * 32),
-                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MO_BLOCK + k * 2048), idesc_o, (i | part | k) != 0 ? 1u : 0u);
+                        umma_bf16(tmem + MO_O + VB, umma_desc_kmajor_sw128(q_addr + i * MC_ROWS + k * 32),
+                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MC_BLOCK + k * 2048), idesc_o, (i | part | k) != 0 ? 1u : 0u);
                     }
                 }
                 umma_commit(slice_empty + i % places);
@@ -515,7 +605,7 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                 {
                     for (unsigned int k = 0; k < MC_L / 16; k++)
                     {
-                        umma_bf16_ts(tmem + MO_O, tmem + MO_P + part * 64 + k * 8, umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MO_BLOCK + (k % 4) * 2048),
+                        umma_bf16_ts(tmem + MO_O, tmem + MO_P + part * 64 + k * 8, umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MC_BLOCK + (k % 4) * 2048),
                             idesc_o, (part | k) != 0 ? 1u : 0u);
                     }
                 }
@@ -578,7 +668,7 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                 float dot = 0.f;
                 for (unsigned int b = half; b < 2 * blocks; b += 2)    // 32 elements at a time
                 {
-                    const unsigned char* row = qs + (b / 2) * MO_ROWS + t * 128;
+                    const unsigned char* row = qs + (b / 2) * MC_ROWS + t * 128;
 #pragma unroll
                     for (unsigned int q = 0; q < 4; q++)
                     {
@@ -678,32 +768,18 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
 }
 
 template <int VB>
-static int run_outputs(const MlstmParams& p, cudaStream_t stream, bool pdl)
+static int run_outputs(const MlstmParams& p, const CUtensorMap& tx, unsigned int* status, cudaStream_t stream, bool pdl)
+
 {
-    unsigned int* status = decoder_status_word();
-    if (!status) { return 1; }
     const unsigned int ranks = (p.vdim + VB - 1) / VB, chunks = (p.max_n + MC_L - 1) / MC_L, dp = mc_dp(p.dim), vp = mc_vp(p.vdim);
-    CUtensorMap tx, ts;
-    if (!make_map_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.qkvg, p.ld, (unsigned long long)p.t0 + p.tokens, (unsigned long long)p.ld * 2, 64, 64, true)
-        || !make_map_2d(&ts, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.work, vp, (unsigned long long)mc_slots(p.tokens, p.entries) * p.heads * 2 * dp,
+    CUtensorMap ts;
+    if (!make_map_2d(&ts, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.work, vp, (unsigned long long)mc_slots(p.tokens, p.entries) * p.heads * 2 * dp,
             (unsigned long long)vp * 2, 64, 64, true))
     {
         return -1;
     }
     return launch_cluster("mlstm_outputs", mlstm_outputs_kernel<VB>, dim3(ranks, p.heads, p.entries * chunks), dim3(MO_THREADS), (size_t)mo_smem((int)dp, VB), ranks,
         stream, pdl, tx, ts, p, chunks, status);
-}
-
-template <int DP>
-static int run_chunks(const MlstmParams& p, unsigned int entries, cudaStream_t stream, bool pdl)
-{
-    const unsigned int chunks = (p.max_n + MC_L - 1) / MC_L;
-    int rc = launch_kernel("mlstm_gates", mlstm_gates_kernel, dim3(chunks, p.heads, entries), dim3(MC_L), 0, stream, pdl, p);
-    if (rc) { return rc; }
-    rc = launch_kernel("mlstm_states", mlstm_states_kernel<DP>, dim3(mc_vp(p.vdim) / MC_COLS, p.heads, entries), dim3(MC_THREADS), (size_t)mc_states_smem(DP),
-        stream, pdl, p);
-    if (rc) { return rc; }
-    return p.vdim <= 64 ? run_outputs<64>(p, stream, pdl) : run_outputs<128>(p, stream, pdl);
 }
 
 unsigned long long mlstm_chunk_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim, unsigned int vdim)
@@ -722,9 +798,19 @@ int launch_mlstm_chunk(const MlstmParams& p, unsigned int entries, cudaStream_t 
     {
         return -1;
     }
-    if (p.dim <= 64) { return run_chunks<64>(p, entries, stream, pdl); }
-    if (p.dim <= 128) { return run_chunks<128>(p, entries, stream, pdl); }
-    return run_chunks<256>(p, entries, stream, pdl);
+    unsigned int* status = decoder_status_word();
+    if (!status) { return 1; }
+    CUtensorMap tx;
+    if (!make_map_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.qkvg, p.ld, (unsigned long long)p.t0 + p.tokens, (unsigned long long)p.ld * 2, 64, 64, true))
+    {
+        return -1;
+    }
+    int rc = launch_kernel("mlstm_gates", mlstm_gates_kernel, dim3(chunks, p.heads, entries), dim3(MC_L), 0, stream, pdl, p);
+    if (rc) { return rc; }
+    rc = launch_kernel("mlstm_states", mlstm_states_kernel, dim3(mc_vp(p.vdim) / MC_COLS + 1, p.heads, entries), dim3(MS_ROLES),
+        (size_t)mc_states_smem((int)mc_dp(p.dim)), stream, pdl, tx, p, status);
+    if (rc) { return rc; }
+    return p.vdim <= 64 ? run_outputs<64>(p, tx, status, stream, pdl) : run_outputs<128>(p, tx, status, stream, pdl);
 }
 
 }    // namespace b200
