@@ -93,8 +93,8 @@ __global__ void __launch_bounds__(MC_L) mlstm_gates_kernel(const MlstmParams p)
 // ---- states ----------------------------------------------------------------------------------------
 constexpr int MS_ROLES = 32 * 14;
 constexpr uint32_t MS_TMEM = 128;    // 64 columns for each 128 rows of S
-// header, k twice, v, weighted values (high, low) twice
-__host__ __device__ constexpr int mc_states_smem(int dp) { return 1024 + 2 * (dp / 64) * MC_ROWS + MC_ROWS + 4 * MC_ROWS + 1024; }
+// header, k twice, v, weighted values (high, low), 32 rows of S per warp on their way out
+__host__ __device__ constexpr int mc_states_smem(int dp) { return 1024 + 2 * (dp / 64) * MC_ROWS + MC_ROWS + 2 * MC_ROWS + 8 * 32 * 128 + 1024; }
 
 // grid (column blocks of 64 and one for n, heads, entries).  A TMA lane fetches k and v of the chunks; four warps weight the values, a
 // token per thread; eight warps own the rows of S, one per thread: between the chunks they take S out of tensor memory, store it
@@ -107,20 +107,20 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(ms_raw) + 1023) & ~(uintptr_t)1023);
     const unsigned int dp = mc_dp(p.dim), vp = mc_vp(p.vdim), blocks = dp / 64;
     uint64_t* k_full = reinterpret_cast<uint64_t*>(smem);
-    uint64_t *k_empty = k_full + 2, *vp_full = k_full + 4, *vp_empty = k_full + 6, *v_full = k_full + 8, *v_empty = k_full + 9, *s_ready = k_full + 10,
-             *s_done = k_full + 11;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 12);
+    uint64_t *k_empty = k_full + 2, *w_full = k_full + 4, *v_full = k_full + 5, *v_empty = k_full + 6, *s_ready = k_full + 7, *s_done = k_full + 8;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 9);
     volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
     unsigned char* ks = smem + 1024;
     unsigned char* vs = ks + 2 * blocks * MC_ROWS;
-    unsigned char* ws = vs + MC_ROWS;    // [buffer][high, low]
+    unsigned char* ws = vs + MC_ROWS;    // high, low
+    unsigned char* out_rows = ws + 2 * MC_ROWS;
 
     const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const bool is_n = blockIdx.x == gridDim.x - 1;
     const unsigned int c0 = is_n ? 0u : blockIdx.x * MC_COLS, h = blockIdx.y, e = p.e0 + blockIdx.z;
     if (tid == 0)
     {
-        for (int i = 0; i < 12; i++) { mbar_init(k_full + i, i == 4 || i == 5 || i == 9 ? 4 : (i == 10 ? 8 : 1)); }
+        for (int i = 0; i < 9; i++) { mbar_init(k_full + i, i == 4 || i == 6 ? 4 : (i == 7 ? 8 : 1)); }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
         for (; c < chunks && ok; c++)
         {
             const unsigned int s = c & 1u;
-            ok = wait(k_full + s, c >> 1) && wait(vp_full + s, c >> 1) && wait(s_ready, c);
+            ok = wait(k_full + s, c >> 1) && wait(w_full, c) && wait(s_ready, c);
             if (!ok) { break; }
             tc_fence_after();
             if (elect_one())
@@ -211,12 +211,11 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
                         {
                             umma_bf16(tmem + mb * MC_COLS,
                                 umma_desc_mnmajor_sw128(k_addr + ((s * 2 + k / 4) * blocks + mb * 2) * MC_BLOCK + (k % 4) * 2048),
-                                umma_desc_mnmajor_sw128(w_addr + (s * 2 + part) * MC_ROWS + (k / 4) * MC_BLOCK + (k % 4) * 2048), idesc, 1u);
+                                umma_desc_mnmajor_sw128(w_addr + part * MC_ROWS + (k / 4) * MC_BLOCK + (k % 4) * 2048), idesc, 1u);
                         }
                     }
                 }
                 umma_commit(k_empty + s);
-                umma_commit(vp_empty + s);
                 umma_commit(s_done);
             }
             __syncwarp();
@@ -277,18 +276,21 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
             }
             if (some)
             {
-                uint32_t scaled[MC_COLS];
 #pragma unroll
-                for (int j = 0; j < (int)MC_COLS; j++) { scaled[j] = __float_as_uint(__uint_as_float(S[j]) * keep); }
+                for (int j = 0; j < (int)MC_COLS; j += 16)
+                {
+                    uint32_t scaled[16];
 #pragma unroll
-                for (int j = 0; j < (int)MC_COLS; j += 16) { tmem_st_32x16(mine + j, scaled + j); }
+                    for (int i = 0; i < 16; i++) { scaled[i] = __float_as_uint(__uint_as_float(S[j + i]) * keep); }
+                    tmem_st_32x16(mine + j, scaled);
+                }
                 tmem_st_wait();
             }
             tc_fence_before();
             __syncwarp();
             if (lane == 0) { mbar_arrive(s_ready); }
             // the state ahead of the chunk, while the products run
-            if (d < dp && (is_n || !fresh || c > 0))
+            if (some && (is_n || !fresh || c > 0))
             {
                 if (is_n)
                 {
@@ -298,20 +300,34 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
                 }
                 else
                 {
-                    __nv_bfloat16* out = first.S + (size_t)c * p.heads * 2 * mc_matrix(p.dim, p.vdim) + (size_t)d * vp + c0;
-#pragma unroll
-                    for (int j = 0; j < (int)MC_COLS; j += 8)
+                    // through shared memory, so that a store covers whole rows
+                    __nv_bfloat16* out = first.S + (size_t)c * p.heads * 2 * mc_matrix(p.dim, p.vdim) + (size_t)(d - lane) * vp + c0;
+                    unsigned char* stage = out_rows + (warp - 2) * 32 * 128;
+#pragma unroll 1
+                    for (int part = 0; part < 2; part++)
                     {
-                        uint32_t hi[4], lo[4];
+                        __syncwarp();
 #pragma unroll
-                        for (int i = 0; i < 4; i++)
+                        for (int q = 0; q < 8; q++)
                         {
-                            const float a = __uint_as_float(S[j + 2 * i]), b = __uint_as_float(S[j + 2 * i + 1]);
-                            hi[i] = pack_bf16x2(a, b);
-                            lo[i] = pack_bf16x2(a - __uint_as_float(hi[i] << 16), b - __uint_as_float(hi[i] & 0xFFFF0000u));
+                            uint32_t y[4];
+#pragma unroll
+                            for (int i = 0; i < 4; i++)
+                            {
+                                const float a = __uint_as_float(S[q * 8 + 2 * i]), b = __uint_as_float(S[q * 8 + 2 * i + 1]);
+                                y[i] = pack_bf16x2(a, b);
+                                if (part == 1) { y[i] = pack_bf16x2(a - __uint_as_float(y[i] << 16), b - __uint_as_float(y[i] & 0xFFFF0000u)); }
+                            }
+                            *reinterpret_cast<uint4*>(stage + lane * 128 + ((q ^ (lane & 7u)) * 16)) = make_uint4(y[0], y[1], y[2], y[3]);
                         }
-                        *reinterpret_cast<uint4*>(out + j) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                        *reinterpret_cast<uint4*>(out + (size_t)dp * vp + j) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                        __syncwarp();
+#pragma unroll
+                        for (unsigned int i = 0; i < 8; i++)
+                        {
+                            const unsigned int r = i * 4 + lane / 8, q = lane % 8;
+                            *reinterpret_cast<uint4*>(out + (size_t)(part * dp + r) * vp + q * 8) =
+                                *reinterpret_cast<const uint4*>(stage + r * 128 + ((q ^ (r & 7u)) * 16));
+                        }
                     }
                 }
             }
@@ -354,7 +370,6 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
         unsigned int c = 0;
         for (; c < chunks; c++)
         {
-            const unsigned int s = c & 1u;
             const float top = fmaxf(m, end.x), w = expf(a - top);
             m = end.y + top;
             if (c + 1 < chunks)
@@ -362,11 +377,11 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
                 end = end_of(c + 1);
                 a = first.a[(size_t)(c + 1) * p.heads * mc_record(p.dim) + t];
             }
-            ok = (is_n || wait(v_full, c)) && (c < 2 || wait(vp_empty + s, (c >> 1) - 1));
+            ok = (is_n || wait(v_full, c)) && (c == 0 || wait(s_done, c - 1));    // the products have read the weighted values before
             ok = __all_sync(0xFFFFFFFFu, ok);
             if (!ok) { break; }
             const unsigned char* src = vs + t * 128;
-            unsigned char* dst = ws + s * 2 * MC_ROWS + t * 128;
+            unsigned char* dst = ws + t * 128;
 #pragma unroll
             for (unsigned int q = 0; q < 8; q++)
             {
@@ -402,7 +417,7 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
             __syncwarp();
             if (lane == 0)
             {
-                mbar_arrive(vp_full + s);
+                mbar_arrive(w_full);
                 if (!is_n) { mbar_arrive(v_empty); }
             }
         }
@@ -459,6 +474,27 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     const unsigned int live = min(MC_L, n - c * MC_L), first = start + c * MC_L;
     const bool fresh = p.pos[e] == 0 && c == 0;
     const ChunkRecord rec = mc_record_of(p, e, c, h);
+    if (tid == 0)
+    {
+        fence_proxy_async();    // the barriers
+        const int y = (int)first, xq = (int)(h * p.dim), xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
+        mbar_expect_tx(qk_full, 2 * blocks * MC_ROWS);
+        for (unsigned int b = 0; b < blocks; b++)
+        {
+            for (int r = 0; r < 2; r++)
+            {
+                tma_load_2d(qs + b * MC_ROWS + r * MC_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
+                tma_load_2d(ks + b * MC_ROWS + r * MC_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
+            }
+        }
+        mbar_arrive(qk_full);
+        mbar_expect_tx(v_full, (VB / 64) * MC_ROWS);
+        for (int r = 0; r < 2; r++)    // 64 rows by 64 rows
+        {
+            for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MC_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
+        }
+        mbar_arrive(v_full);
+    }
     const unsigned int slices = fresh ? 0 : blocks, steps = p.dim / 16;
     const float m0 = fresh ? 0.f : rec.n[dp];
     float t_max = -INFINITY;
@@ -500,23 +536,6 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     {
         if (lane == 0)
         {
-            const int y = (int)first, xq = (int)(h * p.dim), xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
-            mbar_expect_tx(qk_full, 2 * blocks * MC_ROWS);
-            for (unsigned int b = 0; b < blocks; b++)
-            {
-                for (int r = 0; r < 2; r++)
-                {
-                    tma_load_2d(qs + b * MC_ROWS + r * MC_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
-                    tma_load_2d(ks + b * MC_ROWS + r * MC_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
-                }
-            }
-            mbar_arrive(qk_full);
-            mbar_expect_tx(v_full, (VB / 64) * MC_ROWS);
-            for (int r = 0; r < 2; r++)    // 64 rows by 64 rows
-            {
-                for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MC_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
-            }
-            mbar_arrive(v_full);
             bool ok = true;
             unsigned int issued = 0;
             for (unsigned int i = 0; i < slices && ok; i++)
@@ -769,7 +788,6 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
 
 template <int VB>
 static int run_outputs(const MlstmParams& p, const CUtensorMap& tx, unsigned int* status, cudaStream_t stream, bool pdl)
-
 {
     const unsigned int ranks = (p.vdim + VB - 1) / VB, chunks = (p.max_n + MC_L - 1) / MC_L, dp = mc_dp(p.dim), vp = mc_vp(p.vdim);
     CUtensorMap ts;
