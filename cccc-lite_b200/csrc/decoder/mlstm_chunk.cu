@@ -430,39 +430,39 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
 
 // ---- outputs ---------------------------------------------------------------------------------------
 constexpr int MO_THREADS = 32 * 10;
-constexpr uint32_t MO_P = 128, MO_O = 256, MO_TMEM = 512;      // columns: scores, weighted scores (high, low), what the chunk gives, what S gives
-__host__ __device__ constexpr int mo_slice(int vb) { return 2 * (vb / 64) * MC_BLOCK; }    // 64 rows of S: high, low
-__host__ __device__ constexpr int mo_smem(int dp, int vb) { return 1024 + 2 * (dp / 64) * MC_ROWS + (vb / 64) * MC_ROWS + mo_slice(vb) + 1024; }
+constexpr uint32_t MO_O = 128, MO_TMEM = 256;    // columns: scores, in their place weighted scores (64 keys: 32 high, 32 low), then the output
+// a block of 64 elements: q, k, and 64 rows of S (high, low)
+__host__ __device__ constexpr int mo_stage(int vb) { return 2 * MC_ROWS + 2 * (vb / 64) * MC_BLOCK; }
+__host__ __device__ constexpr int mo_smem(int vb) { return 1024 + mo_stage(vb) + (vb / 64) * MC_ROWS + 1024; }
 
-// grid (column blocks of VB = the cluster, heads, entries x chunks).  A TMA lane fetches q, k and v of the chunk and slices of 64 rows of
-// S: the first beside them, the following ones where k was, once the scores are out.  The MMA lane issues q k^T, then q S, then
-// (weighted scores) v.  Eight warps own a row of scores per thread, half of its columns each.
+// grid (column blocks of VB = the cluster, heads, entries x chunks), two CTAs per SM.  A TMA lane fetches v, then q, k and S in blocks of
+// 64 elements; the MMA lane adds up q k^T and q S over the blocks and, once eight warps (half a row of scores per thread) have weighted
+// the scores and scaled what S gives, (weighted scores) v on top.  The results leave through shared memory, so that gates and
+// outputs are read and written in whole rows.
 template <int VB>
-__global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmS,
+__global__ void __launch_bounds__(MO_THREADS, 2) mlstm_outputs_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmS,
     const __grid_constant__ MlstmParams p, const unsigned int max_chunks, unsigned int* status)
 {
     extern __shared__ unsigned char mo_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(mo_raw) + 1023) & ~(uintptr_t)1023);
-    __shared__ float F[MC_L], a[MC_L], M[MC_L], maxima[MC_L / 32], sq[2][MC_L], nq[2][MC_L], peers[MC_MAX_CLUSTER][MC_L], n0[MC_MAX_DIM];
-    constexpr int SLICE = mo_slice(VB), HB = VB / 2, MAX_PLACES = 8;
+    __shared__ float F[MC_L], a[MC_L], M[MC_L], maxima[MC_L / 32], sq[2][MC_L], nq[2][MC_L], peers[MC_MAX_CLUSTER][MC_L];
+    __shared__ __align__(16) float n0[MC_MAX_DIM];
+    constexpr int HB = VB / 2;
     const unsigned int dp = mc_dp(p.dim), blocks = dp / 64;
-    uint64_t* qk_full = reinterpret_cast<uint64_t*>(smem);
-    uint64_t *v_full = qk_full + 1, *s_full = qk_full + 2, *p_ready = qk_full + 3, *o_full = qk_full + 4, *slice_full = qk_full + 5,
-             *slice_empty = slice_full + MAX_PLACES;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(slice_empty + MAX_PLACES);
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem);
+    uint64_t *empty = full + 1, *v_full = full + 2, *s_full = full + 3, *p_ready = full + 4, *o_full = full + 5;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(full + 6);
     volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
     unsigned char* qs = smem + 1024;
-    unsigned char* ks = qs + blocks * MC_ROWS;
-    unsigned char* vs = ks + blocks * MC_ROWS;
-    unsigned char* ss = vs + (VB / 64) * MC_ROWS;
-    const unsigned int places = min((unsigned int)MAX_PLACES, 1u + blocks * MC_ROWS / SLICE);    // of slices
-    auto place = [&](unsigned int i) { return i % places == 0 ? ss : ks + (i % places - 1) * SLICE; };
+    unsigned char* ks = qs + MC_ROWS;
+    unsigned char* ss = ks + MC_ROWS;
+    unsigned char* vs = qs + mo_stage(VB);
 
     const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const unsigned int rank = blockIdx.x, h = blockIdx.y, e = p.e0 + blockIdx.z / max_chunks, c = blockIdx.z % max_chunks, c0 = rank * VB;
     if (tid == 0)
     {
-        for (int i = 0; i < 5 + 2 * MAX_PLACES; i++) { mbar_init(qk_full + i, i == 3 ? 8 : 1); }
+        for (int i = 0; i < 6; i++) { mbar_init(full + i, i == 4 ? 8 : 1); }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -474,28 +474,40 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     const unsigned int live = min(MC_L, n - c * MC_L), first = start + c * MC_L;
     const bool fresh = p.pos[e] == 0 && c == 0;
     const ChunkRecord rec = mc_record_of(p, e, c, h);
-    if (tid == 0)
-    {
-        fence_proxy_async();    // the barriers
-        const int y = (int)first, xq = (int)(h * p.dim), xk = (int)(p.k_off + h * p.dim), xv = (int)(p.v_off + h * p.vdim + c0);
-        mbar_expect_tx(qk_full, 2 * blocks * MC_ROWS);
-        for (unsigned int b = 0; b < blocks; b++)
+    const unsigned int steps = p.dim / 16;
+    auto load_block = [&](unsigned int b) {
+        const int y = (int)first, xq = (int)(h * p.dim + b * 64), xk = (int)(p.k_off + h * p.dim + b * 64);
+        mbar_expect_tx(full, fresh ? 2 * MC_ROWS : mo_stage(VB));
+        for (int r = 0; r < 2; r++)
         {
-            for (int r = 0; r < 2; r++)
+            tma_load_2d(qs + r * MC_BLOCK, &tmX, xq, y + r * 64, full);
+            tma_load_2d(ks + r * MC_BLOCK, &tmX, xk, y + r * 64, full);
+        }
+        if (!fresh)
+        {
+            for (int part = 0; part < 2; part++)
             {
-                tma_load_2d(qs + b * MC_ROWS + r * MC_BLOCK, &tmX, xq + (int)b * 64, y + r * 64, qk_full);
-                tma_load_2d(ks + b * MC_ROWS + r * MC_BLOCK, &tmX, xk + (int)b * 64, y + r * 64, qk_full);
+                for (int j = 0; j < VB / 64; j++)
+                {
+                    tma_load_2d(ss + (part * (VB / 64) + j) * MC_BLOCK, &tmS, (int)c0 + j * 64, (int)((rec.at * 2 + part) * dp + b * 64), full);
+                }
             }
         }
-        mbar_arrive(qk_full);
+        mbar_arrive(full);
+    };
+    if (tid == 0)
+    {
+        load_block(0);
         mbar_expect_tx(v_full, (VB / 64) * MC_ROWS);
         for (int r = 0; r < 2; r++)    // 64 rows by 64 rows
         {
-            for (int b = 0; b < VB / 64; b++) { tma_load_2d(vs + (r * (VB / 64) + b) * MC_BLOCK, &tmX, xv + b * 64, y + r * 64, v_full); }
+            for (int j = 0; j < VB / 64; j++)
+            {
+                tma_load_2d(vs + (r * (VB / 64) + j) * MC_BLOCK, &tmX, (int)(p.v_off + h * p.vdim + c0) + j * 64, (int)first + r * 64, v_full);
+            }
         }
         mbar_arrive(v_full);
     }
-    const unsigned int slices = fresh ? 0 : blocks, steps = p.dim / 16;
     const float m0 = fresh ? 0.f : rec.n[dp];
     float t_max = -INFINITY;
     if (tid < MC_L)    // M: running maxima of a, with m0
@@ -529,92 +541,67 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
     };
     auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
     const unsigned int quarter = warp & 3u, half = warp >= 2 ? (warp - 2u) >> 2 : 0u, t = quarter * 32 + lane;    // row of an epilogue thread
-    float o[HB], inv = 0.f;
+    const uint32_t lanes = tmem + ((quarter * 32u) << 16);
+    const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg + (size_t)first * p.ld;
+    float inv = 0.f;
     bool good = false;
 
     if (warp == 0)
     {
         if (lane == 0)
         {
+            unsigned int b = 1;
             bool ok = true;
-            unsigned int issued = 0;
-            for (unsigned int i = 0; i < slices && ok; i++)
+            for (; b < blocks && ok; b++)
             {
-                const unsigned int at = i % places;
-                if (i == 1) { ok = wait(s_full, 0); }    // k has been read
-                if (ok && i >= places) { ok = wait(slice_empty + at, i / places - 1); }
-                if (!ok) { break; }
-                mbar_expect_tx(slice_full + at, SLICE);
-                for (int part = 0; part < 2; part++)
-                {
-                    for (int b = 0; b < VB / 64; b++)
-                    {
-                        tma_load_2d(place(i) + (part * (VB / 64) + b) * MC_BLOCK, &tmS, (int)c0 + b * 64, (int)((rec.at * 2 + part) * dp + i * 64), slice_full + at);
-                    }
-                }
-                mbar_arrive(slice_full + at);
-                issued++;
+                ok = wait(empty, b - 1);
+                if (ok) { load_block(b); }
+                else { break; }
             }
             if (!ok)
             {
-                give_up(0, issued);
+                give_up(0, b);
                 // wait (bounded) for the copies in flight before the CTA may leave
                 auto drain = [&](uint64_t* bar, unsigned int parity) {
                     const unsigned long long t0 = global_timer_ns();
                     while (!mbar_try_wait(bar, parity & 1u) && global_timer_ns() - t0 < 100000ull) {}
                 };
-                drain(qk_full, 0);
                 drain(v_full, 0);
-                for (unsigned int i = issued > places ? issued - places : 0; i < issued; i++) { drain(slice_full + i % places, i / places); }
+                drain(full, b - 1);
             }
         }
     }
     else if (warp == 1)
     {
-        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), v_addr = smem_u32(vs);
+        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), s_addr = smem_u32(ss), v_addr = smem_u32(vs);
         const uint32_t idesc_s = umma_idesc_bf16(MC_L, MC_L), idesc_o = umma_idesc_bf16(MC_L, VB) | (1u << 16);    // B is MN-major
-        unsigned int at = 0;
-        bool ok = wait(qk_full, 0);
-        if (ok)
+        bool ok = true;
+        unsigned int b = 0;
+        for (; b < blocks && ok; b++)
         {
-            tc_fence_after();
-            if (elect_one())
-            {
-                for (unsigned int k = 0; k < steps; k++)
-                {
-                    const uint32_t off = (k / 4) * MC_ROWS + (k % 4) * 32;
-                    umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + off), umma_desc_kmajor_sw128(k_addr + off), idesc_s, k != 0 ? 1u : 0u);
-                }
-                umma_commit(s_full);
-            }
-            __syncwarp();
-        }
-        for (unsigned int i = 0; i < slices && ok; i++)
-        {
-            at = i + 1;
-            ok = wait(slice_full + i % places, i / places);
+            ok = wait(full, b);
             if (!ok) { break; }
             tc_fence_after();
             if (elect_one())
             {
-                const uint32_t s_addr = smem_u32(place(i));
-                for (unsigned int part = 0; part < 2; part++)
+                for (unsigned int k = 0; k < 4 && b * 4 + k < steps; k++)
                 {
-                    for (unsigned int k = 0; k < 4 && i * 4 + k < steps; k++)
+                    umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + k * 32), umma_desc_kmajor_sw128(k_addr + k * 32), idesc_s, (b | k) != 0 ? 1u : 0u);
+                }
+                for (unsigned int part = 0; part < 2 && !fresh; part++)
+                {
+                    for (unsigned int k = 0; k < 4 && b * 4 + k < steps; k++)
                     {
-                        umma_bf16(tmem + MO_O + VB, umma_desc_kmajor_sw128(q_addr + i * MC_ROWS + k * 32),
-                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MC_BLOCK + k * 2048), idesc_o, (i | part | k) != 0 ? 1u : 0u);
+                        umma_bf16(tmem + MO_O, umma_desc_kmajor_sw128(q_addr + k * 32),
+                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MC_BLOCK + k * 2048), idesc_o, (b | part | k) != 0 ? 1u : 0u);
                     }
                 }
-                umma_commit(slice_empty + i % places);
+                if (b + 1 < blocks) { umma_commit(empty); }
+                else { umma_commit(s_full); }
             }
             __syncwarp();
         }
-        if (ok)
-        {
-            at = slices + 1;
-            ok = wait(v_full, 0) && wait(p_ready, 0);
-        }
+        if (ok) { ok = wait(v_full, 0) && wait(p_ready, 0); }
         if (ok)
         {
             tc_fence_after();
@@ -624,8 +611,8 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                 {
                     for (unsigned int k = 0; k < MC_L / 16; k++)
                     {
-                        umma_bf16_ts(tmem + MO_O, tmem + MO_P + part * 64 + k * 8, umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MC_BLOCK + (k % 4) * 2048),
-                            idesc_o, (part | k) != 0 ? 1u : 0u);
+                        umma_bf16_ts(tmem + MO_O, tmem + (k / 4) * 64 + part * 32 + (k % 4) * 8,
+                            umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MC_BLOCK + (k % 4) * 2048), idesc_o, !fresh || (part | k) != 0 ? 1u : 0u);
                     }
                 }
                 umma_commit(o_full);
@@ -634,28 +621,43 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
         }
         else
         {
-            if (lane == 0) { give_up(1, at); }
+            if (lane == 0) { give_up(1, b); }
             if (elect_one()) { umma_commit(o_full); }    // completes once the MMAs in flight have stopped reading shared memory
             __syncwarp();
         }
     }
     else
     {
-        const uint32_t lanes = tmem + ((quarter * 32u) << 16);
         const float mt = M[t], mt2 = mt * 1.44269504088896341f, carry = p.q_scale * expf(m0 - mt);
         float sum = 0.f;
+        if (!fresh && t < live)    // n0 . q over half of the eights
+        {
+            const __nv_bfloat16* q = x + (size_t)t * p.ld + h * p.dim;
+#pragma unroll 4
+            for (unsigned int d = half * 8; d < p.dim; d += 16)
+            {
+                const uint4 u = *reinterpret_cast<const uint4*>(q + d);
+                const float4 g0 = *reinterpret_cast<const float4*>(n0 + d), g1 = *reinterpret_cast<const float4*>(n0 + d + 4);
+                sum = fmaf(__uint_as_float(u.x << 16), g0.x, fmaf(__uint_as_float(u.x & 0xFFFF0000u), g0.y, sum));
+                sum = fmaf(__uint_as_float(u.y << 16), g0.z, fmaf(__uint_as_float(u.y & 0xFFFF0000u), g0.w, sum));
+                sum = fmaf(__uint_as_float(u.z << 16), g1.x, fmaf(__uint_as_float(u.z & 0xFFFF0000u), g1.y, sum));
+                sum = fmaf(__uint_as_float(u.w << 16), g1.z, fmaf(__uint_as_float(u.w & 0xFFFF0000u), g1.w, sum));
+            }
+            sum *= carry;
+        }
         good = __all_sync(0xFFFFFFFFu, wait(s_full, 0));
         if (good)
         {
             tc_fence_after();
-            // this half's 64 keys; none of them where the rows of the warp end before
+            // this half's 64 keys, their weights in the place of their scores; none where the rows of the warp end before
+            uint32_t hi[32], lo[32];
 #pragma unroll
             for (int q = 0; q < 2; q++)
             {
                 const unsigned int s0 = half * 64 + q * 32;
-                uint32_t z[32], hi[16], lo[16];
+                uint32_t z[32];
 #pragma unroll
-                for (int j = 0; j < 16; j++) { hi[j] = lo[j] = 0u; }
+                for (int j = 0; j < 16; j++) { hi[q * 16 + j] = lo[q * 16 + j] = 0u; }
                 if (s0 <= quarter * 32 + 31)
                 {
                     tmem_ld_32x32(lanes + s0, z);
@@ -671,47 +673,42 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
                             w[k] = s <= t ? __uint_as_float(z[2 * j + k]) * p.q_scale * exp2_f32(a[s] - mt2) : 0.f;
                             sum += w[k];
                         }
-                        hi[j] = pack_bf16x2(w[0], w[1]);
-                        lo[j] = pack_bf16x2(w[0] - __uint_as_float(hi[j] << 16), w[1] - __uint_as_float(hi[j] & 0xFFFF0000u));
+                        const uint32_t u = pack_bf16x2(w[0], w[1]);
+                        hi[q * 16 + j] = u;
+                        lo[q * 16 + j] = pack_bf16x2(w[0] - __uint_as_float(u << 16), w[1] - __uint_as_float(u & 0xFFFF0000u));
                     }
                 }
-                tmem_st_32x16(lanes + MO_P + s0 / 2, hi);
-                tmem_st_32x16(lanes + MO_P + 64 + s0 / 2, lo);
+            }
+#pragma unroll
+            for (int q = 0; q < 2; q++)
+            {
+                tmem_st_32x16(lanes + half * 64 + q * 16, hi + q * 16);
+                tmem_st_32x16(lanes + half * 64 + 32 + q * 16, lo + q * 16);
+            }
+            if (!fresh)
+            {
+#pragma unroll
+                for (int d = 0; d < HB; d += 32)
+                {
+                    uint32_t o[32];
+                    tmem_ld_32x32(lanes + MO_O + half * HB + d, o);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 32; j++) { o[j] = __float_as_uint(__uint_as_float(o[j]) * carry); }
+                    tmem_st_32x16(lanes + MO_O + half * HB + d, o);
+                    tmem_st_32x16(lanes + MO_O + half * HB + d + 16, o + 16);
+                }
             }
             tmem_st_wait();
             tc_fence_before();
             __syncwarp();
             if (lane == 0) { mbar_arrive(p_ready); }
-            if (!fresh && wait(qk_full, 0))    // n0 . q over half of the elements
-            {
-                float dot = 0.f;
-                for (unsigned int b = half; b < 2 * blocks; b += 2)    // 32 elements at a time
-                {
-                    const unsigned char* row = qs + (b / 2) * MC_ROWS + t * 128;
-#pragma unroll
-                    for (unsigned int q = 0; q < 4; q++)
-                    {
-                        const unsigned int chunk = (b & 1u) * 4 + q;
-                        const uint4 u = *reinterpret_cast<const uint4*>(row + ((chunk ^ (t & 7u)) * 16));
-                        const uint32_t w[4] = { u.x, u.y, u.z, u.w };
-                        const float* g = n0 + (b / 2) * 64 + chunk * 8;
-#pragma unroll
-                        for (int j = 0; j < 4; j++)
-                        {
-                            dot = fmaf(__uint_as_float(w[j] << 16), g[2 * j], dot);
-                            dot = fmaf(__uint_as_float(w[j] & 0xFFFF0000u), g[2 * j + 1], dot);
-                        }
-                    }
-                }
-                sum = fmaf(carry, dot, sum);
-            }
-            nq[half][t] = sum;
-            bar_sync_named(1, 256);
-            inv = 1.0f / (fmaxf(fabsf(nq[0][t] + nq[1][t]), expf(-(F[t] + mt))) + 1e-6f);
-            good = __all_sync(0xFFFFFFFFu, wait(o_full, 0)) && *abort_flag == 0;
-            good = __all_sync(0xFFFFFFFFu, good);
         }
-        else { bar_sync_named(1, 256); }
+        nq[half][t] = sum;
+        bar_sync_named(1, 256);
+        inv = 1.0f / (fmaxf(fabsf(nq[0][t] + nq[1][t]), expf(-(F[t] + mt))) + 1e-6f);
+        good = __all_sync(0xFFFFFFFFu, good && wait(o_full, 0)) && *abort_flag == 0;
+        good = __all_sync(0xFFFFFFFFu, good);
         float s = 0.f;
         if (good)
         {
@@ -719,32 +716,21 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
 #pragma unroll
             for (int d = 0; d < HB; d += 32)
             {
-                uint32_t x[32];
-                tmem_ld_32x32(lanes + MO_O + half * HB + d, x);
+                uint32_t o[32];
+                tmem_ld_32x32(lanes + MO_O + half * HB + d, o);
                 tmem_ld_wait();
-#pragma unroll
-                for (int j = 0; j < 32; j++) { o[d + j] = __uint_as_float(x[j]); }
-                if (!fresh)
-                {
-                    tmem_ld_32x32(lanes + MO_O + VB + half * HB + d, x);
-                    tmem_ld_wait();
-#pragma unroll
-                    for (int j = 0; j < 32; j++) { o[d + j] = fmaf(carry, __uint_as_float(x[j]), o[d + j]); }
-                }
 #pragma unroll
                 for (int j = 0; j < 32; j++)
                 {
-                    o[d + j] *= inv;
-                    if (c0 + half * HB + d + j < p.vdim) { s += o[d + j] * o[d + j]; }
+                    const float v = __uint_as_float(o[j]) * inv;
+                    if (c0 + half * HB + d + j < p.vdim) { s = fmaf(v, v, s); }
                 }
             }
         }
         else if (lane == 0) { give_up(2 + quarter, half); }
         sq[half][t] = s;
     }
-    tc_fence_before();
     __syncthreads();
-    if (warp == 1) { tmem_dealloc(tmem, MO_TMEM); }
     cg::cluster_group cluster = cg::this_cluster();
     const unsigned int ranks = cluster.num_blocks();
     for (unsigned int j = tid; j < ranks * MC_L; j += MO_THREADS)
@@ -753,31 +739,58 @@ __global__ void __launch_bounds__(MO_THREADS, 1) mlstm_outputs_kernel(const __gr
         cluster.map_shared_rank(&peers[0][0], j / MC_L)[rank * MC_L + r] = sq[0][r] + sq[1][r];
     }
     cluster.sync();
-    if (good && t < live)
+    if (warp >= 2)
     {
-        float s = 0.f;
-        for (unsigned int r = 0; r < ranks; r++) { s += peers[r][t]; }
-        const float unit = 1.0f / sqrtf(s / (float)p.vdim + p.eps);
-        const unsigned int at = h * p.vdim + c0 + half * HB;
-        const __nv_bfloat16* gate = (const __nv_bfloat16*)p.qkvg + (size_t)(first + t) * p.ld + p.g_off + at;
-        __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)(first + t) * p.ldo + at;
-        const float* w = p.norm + at;
-#pragma unroll
-        for (int d = 0; d < HB; d += 8)
+        float* rows = reinterpret_cast<float*>(qs);    // [128][VB], sixteen bytes at a time in an order of the row's own
+        if (good)
         {
-            if (c0 + half * HB + d >= p.vdim) { continue; }
-            const uint4 u = *reinterpret_cast<const uint4*>(gate + d);
+            float s = 0.f;
+            for (unsigned int r = 0; r < ranks; r++) { s += peers[r][t]; }
+            const float unit = inv / sqrtf(s / (float)p.vdim + p.eps);
+#pragma unroll
+            for (int d = 0; d < HB; d += 32)
+            {
+                uint32_t o[32];
+                tmem_ld_32x32(lanes + MO_O + half * HB + d, o);
+                tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 32; j += 4)
+                {
+                    const unsigned int q = (half * HB + d + j) / 4;
+                    *reinterpret_cast<float4*>(rows + t * VB + ((q ^ (t & 15u)) * 4)) = make_float4(__uint_as_float(o[j]) * unit, __uint_as_float(o[j + 1]) * unit,
+                        __uint_as_float(o[j + 2]) * unit, __uint_as_float(o[j + 3]) * unit);
+                }
+            }
+        }
+        const bool all_good = *abort_flag == 0;
+        bar_sync_named(1, 256);
+        const __nv_bfloat16* gate = x + p.g_off + h * p.vdim + c0;
+        __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)first * p.ldo + h * p.vdim + c0;
+        const float* w = p.norm + h * p.vdim + c0;
+        constexpr unsigned int PER = VB / 8;
+#pragma unroll 4
+        for (unsigned int j = tid - 64; j < MC_L * PER; j += 256)
+        {
+            const unsigned int r = j / PER, col = j % PER * 8;
+            if (r >= live || c0 + col >= p.vdim || !all_good) { continue; }
+            const uint4 u = *reinterpret_cast<const uint4*>(gate + (size_t)r * p.ld + col);
+            const float4 v0 = *reinterpret_cast<const float4*>(rows + r * VB + ((col / 4 ^ (r & 15u)) * 4));
+            const float4 v1 = *reinterpret_cast<const float4*>(rows + r * VB + (((col / 4 + 1) ^ (r & 15u)) * 4));
+            const float4 w0 = *reinterpret_cast<const float4*>(w + col), w1 = *reinterpret_cast<const float4*>(w + col + 4);
+            const float v[8] = { v0.x * w0.x, v0.y * w0.y, v0.z * w0.z, v0.w * w0.w, v1.x * w1.x, v1.y * w1.y, v1.z * w1.z, v1.w * w1.w };
             const uint32_t g[4] = { u.x, u.y, u.z, u.w };
             uint32_t y[4];
 #pragma unroll
-            for (int j = 0; j < 4; j++)
+            for (int k = 0; k < 4; k++)
             {
-                y[j] = pack_bf16x2(o[d + 2 * j] * unit * w[d + 2 * j] * sigmoid_f32(__uint_as_float(g[j] << 16)),
-                    o[d + 2 * j + 1] * unit * w[d + 2 * j + 1] * sigmoid_f32(__uint_as_float(g[j] & 0xFFFF0000u)));
+                y[k] = pack_bf16x2(v[2 * k] * sigmoid_f32(__uint_as_float(g[k] << 16)), v[2 * k + 1] * sigmoid_f32(__uint_as_float(g[k] & 0xFFFF0000u)));
             }
-            *reinterpret_cast<uint4*>(out + d) = make_uint4(y[0], y[1], y[2], y[3]);
+            *reinterpret_cast<uint4*>(out + (size_t)r * p.ldo + col) = make_uint4(y[0], y[1], y[2], y[3]);
         }
     }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) { tmem_dealloc(tmem, MO_TMEM); }
     if (rank == 0 && (c + 1) * MC_L >= n)
     {
         float* st_n = mlstm_state_of(p, e, h) + (size_t)p.dim * mlstm_v_ld(p.vdim);
@@ -796,7 +809,7 @@ static int run_outputs(const MlstmParams& p, const CUtensorMap& tx, unsigned int
     {
         return -1;
     }
-    return launch_cluster("mlstm_outputs", mlstm_outputs_kernel<VB>, dim3(ranks, p.heads, p.entries * chunks), dim3(MO_THREADS), (size_t)mo_smem((int)dp, VB), ranks,
+    return launch_cluster("mlstm_outputs", mlstm_outputs_kernel<VB>, dim3(ranks, p.heads, p.entries * chunks), dim3(MO_THREADS), (size_t)mo_smem(VB), ranks,
         stream, pdl, tx, ts, p, chunks, status);
 }
 
