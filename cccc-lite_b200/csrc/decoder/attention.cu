@@ -475,7 +475,7 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     if (dtype == DT_FLOAT) { kernel = 3; }
     if (kernel == 0)
     {
-        if (p.k_cache == p.v_cache && p.Hkv == 1 && p.k_ld == p.v_ld && p.dim <= 576 && p.vdim <= 512) { kernel = 6; }
+        if (p.k_cache == p.v_cache && p.Hkv == 1 && p.k_ld == p.v_ld && p.dim <= 576 && p.vdim <= 512 && a->slots != 0) { kernel = 6; }
         else if (p.dim > 256 || p.vdim > 256) { kernel = 3; }
         else if (b->max_n * p.G <= 64 || b->max_n <= 4) { kernel = direct ? 4 : 1; }
         else { kernel = a->slots != 0 ? 5 : 2; }
@@ -492,7 +492,7 @@ C_EXPORT int cuda_b200_attention_rows(int dtype, const cuda_b200_attention* a, c
     {
     case 1: return launch_attention_split(p, b->entries, b->max_n, b->max_len, st, pdl);
     case 2: return launch_attention_tiled(p, b->entries, b->max_n, st, pdl);
-    case 6: return launch_attention_latent(p, b->entries, b->max_n, b->max_len, st, pdl);
+    case 6: return launch_attention_latent(p, a->slots, b->entries, b->max_n, b->max_len, st, pdl);
     case 5: return launch_attention_tile(p, a->slots, b->entries, b->max_n, st, pdl);
     case 4: return launch_attention_direct(p, b->entries, b->max_n, b->max_len, st, pdl);
     default: return dtype == DT_BF16 ? attention_plain<__nv_bfloat16>(p, b->tokens, st, pdl) : attention_plain<float>(p, b->tokens, st, pdl);

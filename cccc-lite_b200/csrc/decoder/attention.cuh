@@ -47,7 +47,7 @@ bool plan_splits(AttnParams& p, unsigned int entries, unsigned int max_n, unsign
 // attention_direct.cu, attention_mma.cu: -1 where the sizes are not taken
 int launch_attention_direct(const AttnParams& p, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream, bool pdl);
 // attention_latent.cu: k_cache is v_cache, one kv head
-int launch_attention_latent(const AttnParams& p, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream, bool pdl);
+int launch_attention_latent(const AttnParams& p, unsigned int slots, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream, bool pdl);
 // attention_tile.cu
 int launch_attention_tile(const AttnParams& p, unsigned int slots, unsigned int entries, unsigned int max_n, cudaStream_t stream, bool pdl);
 int launch_attention_split(const AttnParams& p, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream, bool pdl);

@@ -1,29 +1,32 @@
-// BF16 attention of few query rows over latent rows: one key/value head for all query heads, whose values are the first columns
-// of the key rows, so that a cache row is read once for both products.
+// BF16 attention of few query rows over latent rows (decoding), HBM-bound, on tcgen05: one key/value head for all query heads, whose
+// values are the first columns of the key rows, so that a cache row is read once for both products.
 //
-// A CTA holds 32 query rows (a row is one head of one token) against a split of the sequence, in tiles of 64 rows that arrive
-// through cp.async, two deep.  Scores: sixteen warps share 4 quarters of the row elements x 2 x 16 query rows x 2 x 32 keys,
-// their queries as fragments in registers; the quarters meet in shared memory.  Softmax: sixteen threads per query row, running
-// maximum; the weights enter the value product as the sum of two BF16 numbers.  Values: a warp owns a sixteenth of the columns.
-// Partial results of the splits are combined by a second kernel, in split order.
+// A CTA holds 32 query rows (a row is one head of one token) against a split of the sequence, in tiles of 64 cache rows that a TMA
+// lane fetches, two deep.  Both products are turned so that the 32 query rows are the short side: scores = K Q^T (64 x 32) and
+// O^T += K^T P^T (128 latent columns x 32, the tile as an operand with its keys outermost).  Eight warps turn scores into weights:
+// scores go through shared memory, eight threads then own a query row; the weights enter as the sum of two BF16 numbers.  The
+// running maximum only moves when it grows by more than 2^8, so that O is seldom rescaled.  Partial results of the splits are
+// combined by a second kernel, in split order.
+// Every wait is bounded; on expiry the status word is raised, the roles drain, tensor memory is freed and the CTA returns.
 #include "attention_mma.cuh"
+#include "tile_common.cuh"
 
 namespace b200
 {
 
-constexpr int AL_WARPS = 16, AL_THREADS = 32 * AL_WARPS, AL_ROWS = 32, AL_KT = 64, AL_PARTS = 4, AL_SS = AL_KT + 4, AL_PS = AL_KT + 8;
-__host__ __device__ constexpr int al_stride(int dv) { return dv + 64 + 8; }    // elements of a shared row
-// queries, then in their place partial scores and weights
-__host__ __device__ constexpr int al_front(int dv)
+constexpr int AL_THREADS = 32 * 10, AL_ROWS = 32, AL_KT = 64, AL_SS = AL_KT + 4;
+constexpr int AL_BLOCK = AL_KT * 128, AL_QBLOCK = AL_ROWS * 128;    // 64 elements of 64 cache rows, of 32 query rows
+constexpr uint32_t AL_O = 64, AL_TMEM = 256;                          // columns: two places of scores, then O^T (32 for each 128 columns)
+// 64-element blocks of a cache row: what the scores take, and what the value product touches
+__host__ __device__ constexpr int al_key_blocks(int dim) { return (dim + 63) / 64; }
+__host__ __device__ constexpr int al_blocks(int dim, int vdim)
 {
-    const int q = AL_ROWS * al_stride(dv) * 2, s = AL_PARTS * AL_ROWS * AL_SS * 4 + 2 * AL_ROWS * AL_PS * 2;
-    return q > s ? q : s;
+    const int k = al_key_blocks(dim), v = 2 * ((vdim + 127) / 128);
+    return k > v ? k : v;
 }
-__host__ __device__ constexpr int al_smem(int dv) { return al_front(dv) + 2 * AL_KT * al_stride(dv) * 2; }
-
-__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t (&r)[4], uint32_t addr)
+__host__ __device__ constexpr int al_smem(int dim, int vdim)
 {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+    return 1024 + al_key_blocks(dim) * AL_QBLOCK + 2 * al_blocks(dim, vdim) * AL_BLOCK + 2 * AL_QBLOCK + AL_ROWS * AL_SS * 4 + 1024;
 }
 
 __device__ __forceinline__ unsigned int al_value_ld(const AttnParams& p) { return (p.vdim + 15) / 16 * 16; }
@@ -34,249 +37,306 @@ __device__ __forceinline__ float* al_partial(const AttnParams& p, unsigned int u
 }
 
 // grid (splits, row tiles, entries)
-template <int DV>
-__global__ void __launch_bounds__(AL_THREADS, 1) attention_latent_kernel(const AttnParams p)
+__global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ AttnParams p,
+    unsigned int* status)
 {
-    extern __shared__ __align__(16) unsigned char al_raw[];
-    // k steps of a warp, column tiles of 8 per warp, in pairs
-    constexpr int DK = DV + 64, KS = al_stride(DV) * 2, STEPS = DK / 64, CT = DV / 128, CP = CT > 1 ? CT / 2 : 1;
+    extern __shared__ unsigned char al_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(al_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ float corr[AL_ROWS], ml[AL_ROWS][2];
+    // by parity of the tile, so that a warp may be a barrier ahead of another: does any row rescale, has any wait run out
+    __shared__ int moved[2], stop[2];
+    const int kblocks = al_key_blocks((int)p.dim), tile_bytes = al_blocks((int)p.dim, (int)p.vdim) * AL_BLOCK, vparts = ((int)p.vdim + 127) / 128;
+    uint64_t* k_full = reinterpret_cast<uint64_t*>(smem);
+    uint64_t *k_empty = k_full + 2, *s_full = k_full + 4, *q_ready = k_full + 6, *p_ready = k_full + 7, *pv_done = k_full + 8, *o_full = k_full + 9;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_full + 10);
+    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(tmem_slot + 1);
+    unsigned char* ks = smem + 1024;
+    unsigned char* qs = ks + 2 * tile_bytes;
+    unsigned char* pw = qs + kblocks * AL_QBLOCK;                              // [high, low][row][key]
+    float* sc = reinterpret_cast<float*>(pw + 2 * AL_QBLOCK);                  // [row][key]
+
+    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const unsigned int split = blockIdx.x, rt = blockIdx.y, e = p.e0 + blockIdx.z;
+    if (tid == 0)
+    {
+        for (int i = 0; i < 10; i++) { mbar_init(k_full + i, i == 6 || i == 7 ? 8 : 1); }
+        *abort_flag = 0;
+        moved[0] = moved[1] = stop[0] = stop[1] = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) { tmem_alloc(tmem_slot, AL_TMEM); }
     grid_dependency_launch();
     grid_dependency_wait();
-    const unsigned int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gc = (lane & 3) * 2;
-    const unsigned int split = blockIdx.x, rt = blockIdx.y, e = p.e0 + blockIdx.z;
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e], rows = n * p.G, r0 = rt * AL_ROWS;
-    if (r0 >= rows) { return; }
+    const bool idle = r0 >= rows;    // a shorter entry than the longest one
     const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg;
-    const __nv_bfloat16* K = (const __nv_bfloat16*)p.k_cache + (size_t)p.slot[e] * p.T_max * p.k_ld;
-    const unsigned int last_row = min(r0 + AL_ROWS - 1u, rows - 1);
-    const unsigned int T = min(pos + last_row / p.G + 1, p.T_max), begin = first_key(p, e, pos + r0 / p.G + 1) / AL_KT;
-    const unsigned int tiles = (T + AL_KT - 1) / AL_KT, per = (tiles - begin + p.splits - 1) / p.splits;
-    const unsigned int tile0 = min(begin + split * per, tiles), tile1 = min(tile0 + per, tiles);
-    const uint32_t qs = smem_u32(al_raw), ks = qs + al_front(DV);
-    float* sc = reinterpret_cast<float*>(al_raw);                                               // [part][row][key]
-    __nv_bfloat16* pw = reinterpret_cast<__nv_bfloat16*>(sc + AL_PARTS * AL_ROWS * AL_SS);      // [high, low][row][key]
-    auto fetch = [&](unsigned int tile) {
-        if (tile < tile1)
+    const unsigned int last_row = idle ? 0 : min(r0 + AL_ROWS - 1u, rows - 1);
+    const unsigned int T = idle ? 0 : min(pos + last_row / p.G + 1, p.T_max), begin = idle ? 0 : first_key(p, e, pos + r0 / p.G + 1) / AL_KT;
+    const unsigned int all = (T + AL_KT - 1) / AL_KT, per = (all - begin + p.splits - 1) / p.splits;
+    const unsigned int tile0 = min(begin + split * per, all), tiles = min(tile0 + per, all) - tile0;
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    auto give_up = [&](unsigned int role, unsigned int step) {
+        note_timeout(status, WAIT_ATTENTION_LATENT, role, step);
+        *abort_flag = 1;
+    };
+    auto wait = [&](uint64_t* bar, unsigned int parity) { return *abort_flag == 0 && mbar_wait_bounded(bar, parity & 1u); };
+
+    if (warp == 0)
+    {
+        if (lane == 0)
         {
-            const uint32_t dst = ks + (tile & 1u) * AL_KT * KS;
-            const __nv_bfloat16* src = K + (size_t)tile * AL_KT * p.k_ld;
-#pragma unroll
-            for (int c = 0; c < AL_KT * (DK / 8) / AL_THREADS; c++)
+            const unsigned int seq = (unsigned int)p.slot[e] * p.T_max;
+            unsigned int i = 0;
+            bool ok = true;
+            for (; i < tiles; i++)
             {
-                const unsigned int at = tid + c * AL_THREADS, r = at / (DK / 8), d = at % (DK / 8);
-                const bool ok = tile * AL_KT + r < T && d * 8 < p.k_ld;
-                cp_async16(dst + r * KS + d * 16, src + (ok ? r * p.k_ld + d * 8 : 0u), ok);
+                const unsigned int s = i & 1u;
+                if (i >= 2 && !wait(k_empty + s, (i >> 1) - 1)) { ok = false; break; }
+                mbar_expect_tx(k_full + s, (unsigned int)kblocks * AL_BLOCK);
+                for (int b = 0; b < kblocks; b++) { tma_load_2d(ks + s * tile_bytes + b * AL_BLOCK, &tmK, b * 64, (int)(seq + (tile0 + i) * AL_KT), k_full + s); }
+                mbar_arrive(k_full + s);
+            }
+            if (!ok)
+            {
+                give_up(0, i);
+                // wait (bounded) for the copies in flight before the CTA may leave
+                for (unsigned int j = i > 2 ? i - 2 : 0; j < i; j++)
+                {
+                    const unsigned long long t = global_timer_ns();
+                    while (!mbar_try_wait(k_full + (j & 1u), (j >> 1) & 1u) && global_timer_ns() - t < 100000ull) {}
+                }
             }
         }
-        cp_async_commit();
-    };
-    // a tile's lines on their way to L2
-    auto prefetch = [&](unsigned int tile) {
-        if (tile < tile1 && (tile + 1) * AL_KT <= T)
-        {
-            const char* src = reinterpret_cast<const char*>(K + (size_t)tile * AL_KT * p.k_ld);
-            for (unsigned int line = tid; line * 128 < AL_KT * p.k_ld * 2; line += AL_THREADS) { asm volatile("prefetch.global.L2 [%0];" ::"l"(src + line * 128)); }
-        }
-    };
-    if ((p.q_ld % 8) == 0 && (p.ld % 8) == 0)
+    }
+    else if (warp == 1)
     {
-        for (unsigned int c = tid; c < AL_ROWS * (DK / 8); c += AL_THREADS)
+        const uint32_t idesc_s = umma_idesc_bf16(AL_KT, AL_ROWS), idesc_o = umma_idesc_bf16(128, AL_ROWS) | (1u << 15);    // A has its keys outermost
+        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), p_addr = smem_u32(pw);
+        auto scores = [&](unsigned int i) {
+            if (!wait(k_full + (i & 1u), i >> 1)) { return false; }
+            tc_fence_after();
+            if (elect_one())
+            {
+                for (int k = 0; k * 16 < (int)p.dim; k++)
+                {
+                    umma_bf16(tmem + (i & 1u) * AL_ROWS, umma_desc_kmajor_sw128(k_addr + (i & 1u) * tile_bytes + (k / 4) * AL_BLOCK + (k % 4) * 32),
+                        umma_desc_kmajor_sw128(q_addr + (k / 4) * AL_QBLOCK + (k % 4) * 32), idesc_s, k != 0 ? 1u : 0u);
+                }
+                umma_commit(s_full + (i & 1u));
+            }
+            __syncwarp();
+            return true;
+        };
+        unsigned int i = 0;
+        bool ok = tiles == 0 || (wait(q_ready, 0) && scores(0) && (tiles == 1 || scores(1)));
+        for (; i < tiles && ok; i++)
         {
-            const unsigned int r = c / (DK / 8), d = c % (DK / 8), row = r0 + r;
-            const bool ok = row < rows && d * 8 < p.q_ld;
-            cp_async16(qs + r * KS + d * 16, x + (ok ? (size_t)(start + row / p.G) * p.ld + (size_t)(row % p.G) * p.q_ld + d * 8 : 0), ok);
+            ok = wait(p_ready, i);
+            if (!ok) { break; }
+            tc_fence_after();
+            if (elect_one())
+            {
+                for (int v = 0; v < vparts; v++)
+                {
+#pragma unroll
+                    for (int part = 0; part < 2; part++)    // the high halves of the weights, then the low ones
+                    {
+#pragma unroll
+                        for (int k = 0; k < AL_KT / 16; k++)
+                        {
+                            umma_bf16(tmem + AL_O + v * AL_ROWS, umma_desc_mnmajor_sw128(k_addr + (i & 1u) * tile_bytes + v * 2 * AL_BLOCK + k * 2048),
+                                umma_desc_kmajor_sw128(p_addr + part * AL_QBLOCK + k * 32), idesc_o, (i | (unsigned int)part | (unsigned int)k) != 0 ? 1u : 0u);
+                        }
+                    }
+                }
+                umma_commit(k_empty + (i & 1u));
+                umma_commit(pv_done);
+                if (i + 1 == tiles) { umma_commit(o_full); }
+            }
+            __syncwarp();
+            if (i + 2 < tiles && !scores(i + 2)) { ok = false; }
+        }
+        if (!ok)
+        {
+            if (lane == 0) { give_up(1, i); }
+            if (elect_one()) { umma_commit(o_full); }    // completes once the MMAs in flight have stopped reading shared memory
+            __syncwarp();
         }
     }
     else
     {
-        for (unsigned int j = tid; j < AL_ROWS * DK; j += AL_THREADS)
+        const unsigned int st = tid - 64, sw = warp - 2, quarter = warp & 3u, side = sw >> 2;
+        // queries, in eights
+        if (!idle)
         {
-            const unsigned int r = j / DK, d = j % DK, row = r0 + r;
-            __nv_bfloat16 v = __float2bfloat16_rn(0.f);
-            if (row < rows && d < p.dim) { v = x[(size_t)(start + row / p.G) * p.ld + (size_t)(row % p.G) * p.q_ld + d]; }
-            reinterpret_cast<__nv_bfloat16*>(al_raw)[r * al_stride(DV) + d] = v;
-        }
-    }
-    cp_async_commit();
-    fetch(tile0);
-    prefetch(tile0 + 1);
-    cp_async_wait<1>();
-    __syncthreads();
-    // scores: this warp's quarter of the elements, query rows, keys
-    const unsigned int part = warp >> 2, mr = (warp >> 1) & 1u, kg = warp & 1u;
-    uint32_t q[STEPS][4];
-    {
-        const uint32_t qa = qs + (mr * 16 + (lane & 15)) * KS + (lane >> 4) * 16 + part * STEPS * 32;
-#pragma unroll
-        for (int i = 0; i < STEPS; i++) { ldmatrix_x4(q[i], qa + i * 32); }
-    }
-    const uint32_t kb = (kg * 32 + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 16 + part * STEPS * 32;
-    // softmax: query row tid / 16, keys tid % 16 + 16 j
-    const unsigned int sr = tid >> 4, sk = tid & 15u, end = pos + (r0 + sr) / p.G + 1;
-    const bool real = r0 + sr < rows;
-    const unsigned int low = first_key(p, e, end), lim = real ? min(end, T) : 0u;
-    const float scale2 = p.scale * 1.44269504088896341f;
-    float m = -INFINITY, l = 0.f;
-    // values
-    const uint32_t vb = (lane & 15) * KS + (CT > 1 ? (lane >> 4) * 16 : 0u) + warp * CT * 16;
-    const uint32_t pa = smem_u32(pw) + (lane & 15) * (AL_PS * 2) + (lane >> 4) * 16;
-    float o[2][CT][4];
-#pragma unroll
-    for (int i = 0; i < 2; i++)
-    {
-#pragma unroll
-        for (int j = 0; j < CT; j++)
-        {
-#pragma unroll
-            for (int k = 0; k < 4; k++) { o[i][j][k] = 0.f; }
-        }
-    }
-    for (unsigned int tile = tile0; tile < tile1; tile++)
-    {
-        cp_async_wait<0>();
-        __syncthreads();
-        fetch(tile + 1);
-        prefetch(tile + 2);
-        const uint32_t at = ks + (tile & 1u) * AL_KT * KS;
-        {
-            float s[4][4];
-#pragma unroll
-            for (int i = 0; i < 4; i++)
+            const bool vec = (p.q_ld % 8) == 0 && (p.ld % 8) == 0;
+            for (unsigned int c = st; c < AL_ROWS * (unsigned int)kblocks * 8; c += 256)
             {
-#pragma unroll
-                for (int j = 0; j < 4; j++) { s[i][j] = 0.f; }
-            }
-#pragma unroll
-            for (int i = 0; i < STEPS; i++)
-            {
-#pragma unroll
-                for (int j = 0; j < 2; j++)
+                const unsigned int r = c / (kblocks * 8), q = c % (kblocks * 8), d = q * 8, row = r0 + r;
+                uint4 u = make_uint4(0, 0, 0, 0);
+                if (row < rows && d < p.dim)
                 {
-                    uint32_t b[4];
-                    ldmatrix_x4(b, at + kb + j * 16 * KS + i * 32);
-                    mma_bf16_16816(s[2 * j], q[i][0], q[i][1], q[i][2], q[i][3], b[0], b[1]);
-                    mma_bf16_16816(s[2 * j + 1], q[i][0], q[i][1], q[i][2], q[i][3], b[2], b[3]);
-                }
-            }
-            float* dst = sc + (part * AL_ROWS + mr * 16 + gr) * AL_SS + kg * 32 + gc;
-#pragma unroll
-            for (int i = 0; i < 4; i++)
-            {
-                *reinterpret_cast<float2*>(dst + i * 8) = make_float2(s[i][0], s[i][1]);
-                *reinterpret_cast<float2*>(dst + 8 * AL_SS + i * 8) = make_float2(s[i][2], s[i][3]);
-            }
-        }
-        __syncthreads();
-        {
-            float z[4], mx = -INFINITY;
-#pragma unroll
-            for (int j = 0; j < 4; j++)
-            {
-                const unsigned int key = tile * AL_KT + sk + 16 * j;
-                const float* src = sc + sr * AL_SS + sk + 16 * j;
-                z[j] = ((src[0] + src[AL_ROWS * AL_SS]) + (src[2 * AL_ROWS * AL_SS] + src[3 * AL_ROWS * AL_SS])) * scale2;
-                if (key < low || key >= lim) { z[j] = -INFINITY; }
-                mx = fmaxf(mx, z[j]);
-            }
-#pragma unroll
-            for (int i = 1; i < 16; i *= 2) { mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, i)); }
-            const float mn = fmaxf(m, mx), base = mn == -INFINITY ? 0.f : mn, c = exp2f(m - base);
-            m = mn;
-            l *= c;
-#pragma unroll
-            for (int j = 0; j < 4; j++)
-            {
-                const float w = exp2f(z[j] - base);
-                l += w;
-                const __nv_bfloat16 hi = __float2bfloat16_rn(w);
-                pw[sr * AL_PS + sk + 16 * j] = hi;
-                pw[(AL_ROWS + sr) * AL_PS + sk + 16 * j] = __float2bfloat16_rn(w - __bfloat162float(hi));
-            }
-            if (sk == 0) { corr[sr] = c; }
-        }
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < 2; i++)
-        {
-            const float c0 = corr[i * 16 + gr], c1 = corr[i * 16 + gr + 8];
-#pragma unroll
-            for (int j = 0; j < CT; j++)
-            {
-                o[i][j][0] *= c0;
-                o[i][j][1] *= c0;
-                o[i][j][2] *= c1;
-                o[i][j][3] *= c1;
-            }
-        }
-#pragma unroll
-        for (int k = 0; k < AL_KT / 16; k++)
-        {
-            uint32_t b[CP][4];
-#pragma unroll
-            for (int j = 0; j < CP; j++)
-            {
-                if constexpr (CT > 1) { ldmatrix_x4_trans(b[j], at + vb + k * 16 * KS + j * 32); }
-                else { ldmatrix_x2_trans(b[j], at + vb + k * 16 * KS); }
-            }
-#pragma unroll
-            for (int i = 0; i < 2; i++)
-            {
-#pragma unroll
-                for (int low = 0; low < 2; low++)
-                {
-                    uint32_t w[4];
-                    ldmatrix_x4(w, pa + (low * AL_ROWS + i * 16) * (AL_PS * 2) + k * 32);
-#pragma unroll
-                    for (int j = 0; j < CP; j++)
+                    const __nv_bfloat16* src = x + (size_t)(start + row / p.G) * p.ld + (size_t)(row % p.G) * p.q_ld + d;
+                    if (vec && d + 8 <= p.dim) { u = *reinterpret_cast<const uint4*>(src); }
+                    else
                     {
-                        mma_bf16_16816(o[i][2 * j], w[0], w[1], w[2], w[3], b[j][0], b[j][1]);
-                        if constexpr (CT > 1) { mma_bf16_16816(o[i][2 * j + 1], w[0], w[1], w[2], w[3], b[j][2], b[j][3]); }
+                        uint32_t w[8];
+#pragma unroll
+                        for (int j = 0; j < 8; j++) { w[j] = d + j < p.dim ? __bfloat16_as_ushort(src[j]) : 0u; }
+                        u = make_uint4(w[0] | (w[1] << 16), w[2] | (w[3] << 16), w[4] | (w[5] << 16), w[6] | (w[7] << 16));
                     }
                 }
+                *reinterpret_cast<uint4*>(qs + (q / 8) * AL_QBLOCK + r * 128 + (((q % 8) ^ (r & 7u)) * 16)) = u;
             }
         }
-    }
-    cp_async_wait<0>();
-#pragma unroll
-    for (int i = 1; i < 16; i *= 2) { l += __shfl_xor_sync(0xFFFFFFFFu, l, i); }
-    if (sk == 0)
-    {
-        if (p.splits == 1 && p.sink != nullptr && real) { l += exp2f(p.sink[(r0 + sr) % p.G] * 1.44269504088896341f - m); }
-        ml[sr][0] = m;
-        ml[sr][1] = l;
-    }
-    __syncthreads();
-    const unsigned int vl = al_value_ld(p);
-    float* mine = al_partial(p, blockIdx.z * gridDim.y + rt, split);
-    if (p.splits > 1 && tid < AL_ROWS)
-    {
-        mine[2 * tid] = ml[tid][0];
-        mine[2 * tid + 1] = ml[tid][1];
-    }
-#pragma unroll
-    for (int i = 0; i < 2; i++)
-    {
-#pragma unroll
-        for (int hf = 0; hf < 2; hf++)
+        fence_proxy_async();
+        __syncwarp();
+        if (lane == 0) { mbar_arrive(q_ready); }
+        // softmax: query row st / 8, keys 8 (st % 8) ..
+        const unsigned int sr = st >> 3, sk = st & 7u, end = pos + (r0 + sr) / p.G + 1;
+        const bool real = r0 + sr < rows;
+        const unsigned int low = first_key(p, e, end), lim = real ? min(end, T) : 0u;
+        const float scale2 = p.scale * 1.44269504088896341f;
+        const uint32_t lanes = tmem + ((quarter * 32u) << 16);
+        float m = -INFINITY, l = 0.f;
+        bool ok = true;
+        unsigned int i = 0;
+        for (; i < tiles; i++)
         {
-            const unsigned int r = i * 16 + gr + 8 * hf;
-            if (r0 + r >= rows) { continue; }
-            const float inv = 1.0f / ml[r][1];
-#pragma unroll
-            for (int j = 0; j < CT; j++)
+            ok = __all_sync(0xFFFFFFFFu, wait(s_full + (i & 1u), i >> 1));
+            // sixteen keys per quarter of tensor memory; half of the query rows for each of its two warps
+            if (ok)
             {
-                const unsigned int d = (warp * CT + j) * 8 + gc;
-                if (p.splits > 1)
+                tc_fence_after();
+                uint32_t z[16];
+                tmem_ld_32x16(lanes + (i & 1u) * AL_ROWS + side * 16, z);
+                tmem_ld_wait();
+                if (lane < 16)
                 {
-                    if (d < vl) { *reinterpret_cast<float2*>(mine + 2 * AL_ROWS + (size_t)r * vl + d) = make_float2(o[i][j][2 * hf], o[i][j][2 * hf + 1]); }
-                    continue;
+#pragma unroll
+                    for (int j = 0; j < 16; j++) { sc[(side * 16 + j) * AL_SS + quarter * 16 + lane] = __uint_as_float(z[j]); }
                 }
-                if (d < p.vdim) { attention_store(p, x, start, 0, r0 + r, d, o[i][j][2 * hf] * inv); }
-                if (d + 1 < p.vdim) { attention_store(p, x, start, 0, r0 + r, d + 1, o[i][j][2 * hf + 1] * inv); }
+            }
+            bar_sync_named(1, 256);    // also: every warp is past the tile before
+            if (st == 0) { moved[(i + 1) & 1u] = 0; }
+            float w[8], mx = -INFINITY;
+            const unsigned int key0 = (tile0 + i) * AL_KT + sk * 8;
+            const float4 z0 = *reinterpret_cast<const float4*>(sc + sr * AL_SS + sk * 8), z1 = *reinterpret_cast<const float4*>(sc + sr * AL_SS + sk * 8 + 4);
+            w[0] = z0.x, w[1] = z0.y, w[2] = z0.z, w[3] = z0.w, w[4] = z1.x, w[5] = z1.y, w[6] = z1.z, w[7] = z1.w;
+#pragma unroll
+            for (int j = 0; j < 8; j++)
+            {
+                w[j] = key0 + j < low || key0 + j >= lim ? -INFINITY : w[j] * scale2;
+                mx = fmaxf(mx, w[j]);
+            }
+#pragma unroll
+            for (int k = 1; k < 8; k *= 2) { mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, k)); }
+            float c = 1.f;
+            if (mx > m + 8.f)
+            {
+                c = exp2_f32(m - mx);    // 0 at the first keys
+                m = mx;
+                l *= c;
+                if (i > 0) { moved[i & 1u] = 1; }
+            }
+            if (sk == 0) { corr[sr] = c; }
+            const float base = m == -INFINITY ? 0.f : m;
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+            {
+                const float a = exp2_f32(w[2 * j] - base), b = exp2_f32(w[2 * j + 1] - base);
+                l += a + b;
+                hi[j] = pack_bf16x2(a, b);
+                lo[j] = pack_bf16x2(a - __uint_as_float(hi[j] << 16), b - __uint_as_float(hi[j] & 0xFFFF0000u));
+            }
+            // the product before has read its weights (and left O alone) before they are written over
+            if (i > 0) { ok = __all_sync(0xFFFFFFFFu, ok && wait(pv_done, i - 1)); }
+            unsigned char* dst = pw + sr * 128 + ((sk ^ (sr & 7u)) * 16);
+            *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(dst + AL_QBLOCK) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            fence_proxy_async();
+            if (!ok && lane == 0) { stop[i & 1u] = 1; }
+            bar_sync_named(1, 256);
+            if (stop[i & 1u] != 0)    // all eight warps or none
+            {
+                ok = false;
+                break;
+            }
+            if (moved[i & 1u] != 0)
+            {
+                tc_fence_after();
+                for (int v = (int)side; v < vparts; v += 2)
+                {
+                    uint32_t o[32];
+                    tmem_ld_32x32(lanes + AL_O + v * AL_ROWS, o);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 32; j++) { o[j] = __float_as_uint(__uint_as_float(o[j]) * corr[j]); }
+                    tmem_st_32x16(lanes + AL_O + v * AL_ROWS, o);
+                    tmem_st_32x16(lanes + AL_O + v * AL_ROWS + 16, o + 16);
+                }
+                tmem_st_wait();
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) { mbar_arrive(p_ready); }
+        }
+        ok = ok && (tiles == 0 || wait(o_full, 0));
+        ok = __all_sync(0xFFFFFFFFu, ok);
+#pragma unroll
+        for (int k = 1; k < 8; k *= 2) { l += __shfl_xor_sync(0xFFFFFFFFu, l, k); }
+        if (sk == 0)
+        {
+            if (p.splits == 1 && p.sink != nullptr && real) { l += exp2f(p.sink[(r0 + sr) % p.G] * 1.44269504088896341f - m); }
+            ml[sr][0] = m;
+            ml[sr][1] = l;
+        }
+        bar_sync_named(1, 256);
+        if (!ok)
+        {
+            if (lane == 0) { give_up(2 + quarter, i); }
+        }
+        else if (!idle)
+        {
+            const unsigned int vl = al_value_ld(p), live = min((unsigned int)AL_ROWS, rows - r0);
+            float* mine = al_partial(p, blockIdx.z * gridDim.y + rt, split);
+            if (p.splits > 1 && st < AL_ROWS)
+            {
+                mine[2 * st] = ml[st][0];
+                mine[2 * st + 1] = ml[st][1];
+            }
+            tc_fence_after();
+            for (int v = (int)side; v < vparts; v += 2)
+            {
+                const unsigned int d = v * 128 + quarter * 32 + lane;
+                uint32_t o[32];
+#pragma unroll
+                for (int j = 0; j < 32; j++) { o[j] = 0u; }
+                if (tiles != 0)
+                {
+                    tmem_ld_32x32(lanes + AL_O + v * AL_ROWS, o);
+                    tmem_ld_wait();
+                }
+#pragma unroll
+                for (unsigned int r = 0; r < AL_ROWS; r++)
+                {
+                    if (r >= live) { continue; }
+                    if (p.splits > 1)
+                    {
+                        if (d < vl) { mine[2 * AL_ROWS + (size_t)r * vl + d] = __uint_as_float(o[r]); }
+                    }
+                    else if (d < p.vdim) { attention_store(p, x, start, 0, r0 + r, d, __uint_as_float(o[r]) / ml[r][1]); }
+                }
             }
         }
     }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) { tmem_dealloc(tmem, AL_TMEM); }
 }
 
 // grid (rows of a tile, row tiles, entries); a thread per four columns
@@ -324,37 +384,41 @@ __global__ void __launch_bounds__(128) attention_latent_combine_kernel(const Att
     }
 }
 
-int launch_attention_latent(const AttnParams& p0, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream, bool pdl)
+int launch_attention_latent(const AttnParams& p0, unsigned int slots, unsigned int entries, unsigned int max_n, unsigned int max_len, cudaStream_t stream,
+    bool pdl)
 {
     AttnParams p = p0;
     const DecoderDevice* dev = decoder_device();
-    if (!dev) { return 1; }
+    unsigned int* status = decoder_status_word();
+    if (!dev || !status) { return 1; }
     const unsigned int row_tiles = (max_n * p.G + AL_ROWS - 1) / AL_ROWS;
-    if (p.Hkv != 1 || p.k_cache != p.v_cache || p.k_ld != p.v_ld || p.dim > 576 || p.vdim > 512 || (p.k_ld % 8) || row_tiles > 65535u || entries > 65535u)
+    const unsigned long long cache_rows = (unsigned long long)slots * p.T_max;
+    if (p.Hkv != 1 || p.k_cache != p.v_cache || p.k_ld != p.v_ld || p.dim > 576 || p.vdim > 512 || (p.k_ld % 8) || slots == 0 || cache_rows > 0x7FFFFFFFull
+        || row_tiles > 65535u || entries > 65535u)
     {
         return -1;
     }
+    CUtensorMap tk;
+    if (!make_map_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.k_cache, p.k_ld, cache_rows, (unsigned long long)p.k_ld * 2, 64, AL_KT, true)) { return -1; }
     if (p.window != 0 && max_len > p.window + max_n) { max_len = p.window + max_n; }
-    const unsigned long long units = (unsigned long long)entries * row_tiles;
+    const size_t smem = (size_t)al_smem((int)p.dim, (int)p.vdim);
+    const unsigned int per_sm = smem > 100 * 1024 ? 1u : 2u;    // tensor memory holds two
+    const unsigned long long units = (unsigned long long)entries * row_tiles, places = (unsigned long long)dev->sm_count * per_sm;
     const unsigned int tiles = (max_len + AL_KT - 1) / AL_KT + (p.window != 0 ? 1 : 0);
-    // the fewest tiles in a row, over all waves of CTAs; a split costs its start and the combining
+    // the fewest tiles in a row, over all waves of CTAs; a CTA costs its start, splits the combining
     double best = 1e30;
     p.splits = 1;
     for (unsigned int s = 1; s <= kMaxSplits && (s == 1 || (units * s * 2 <= kAttnPartials && s <= tiles)); s++)
     {
-        const double waves = (double)((units * s + dev->sm_count - 1) / dev->sm_count);
-        const double t = waves * ((double)((tiles + s - 1) / s) + 1.0) + (s > 1 ? 1.0 + 0.03 * s : 0.0);
+        const double waves = (double)((units * s + places - 1) / places);
+        const double t = waves * ((double)((tiles + s - 1) / s) + 2.0) + (s > 1 ? 2.0 + 0.05 * s : 0.0);
         if (t < best)
         {
             best = t;
             p.splits = s;
         }
     }
-    const dim3 grid(p.splits, row_tiles, entries);
-    int rc;
-    if (p.vdim <= 128 && p.dim <= 192) { rc = launch_kernel("attention_latent", attention_latent_kernel<128>, grid, dim3(AL_THREADS), (size_t)al_smem(128), stream, pdl, p); }
-    else if (p.vdim <= 256 && p.dim <= 320) { rc = launch_kernel("attention_latent", attention_latent_kernel<256>, grid, dim3(AL_THREADS), (size_t)al_smem(256), stream, pdl, p); }
-    else { rc = launch_kernel("attention_latent", attention_latent_kernel<512>, grid, dim3(AL_THREADS), (size_t)al_smem(512), stream, pdl, p); }
+    const int rc = launch_kernel("attention_latent", attention_latent_kernel, dim3(p.splits, row_tiles, entries), dim3(AL_THREADS), smem, stream, pdl, tk, p, status);
     if (rc || p.splits == 1) { return rc; }
     return launch_kernel("attention_latent_combine", attention_latent_combine_kernel, dim3(AL_ROWS, row_tiles, entries), dim3(128), 0, stream, pdl, p);
 }

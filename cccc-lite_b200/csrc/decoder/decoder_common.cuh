@@ -17,7 +17,8 @@ enum : unsigned int
     WAIT_LINEAR_TILE = 1,
     WAIT_ATTENTION_TILE = 2,
     WAIT_MLSTM_STATES = 3,
-    WAIT_MLSTM_OUTPUTS = 4
+    WAIT_MLSTM_OUTPUTS = 4,
+    WAIT_ATTENTION_LATENT = 5
 };
 __device__ __forceinline__ void note_timeout(unsigned int* status, unsigned int kernel, unsigned int role, unsigned int step)
 {
