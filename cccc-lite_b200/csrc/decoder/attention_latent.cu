@@ -91,9 +91,19 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
             const unsigned int seq = (unsigned int)p.slot[e] * p.T_max;
             unsigned int i = 0;
             bool ok = true;
+            // tiles further on, on their way to L2
+            auto prefetch = [&](unsigned int t) {
+                for (int b = 0; b < kblocks && t < tiles; b++)
+                {
+                    asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];" ::"l"(&tmK), "r"(b * 64), "r"((int)(seq + (tile0 + t) * AL_KT))
+                                 : "memory");
+                }
+            };
+            prefetch(2);
             for (; i < tiles; i++)
             {
                 const unsigned int s = i & 1u;
+                if (i >= 1) { prefetch(i + 2); }
                 if (i >= 2 && !wait(k_empty + s, (i >> 1) - 1)) { ok = false; break; }
                 mbar_expect_tx(k_full + s, (unsigned int)kblocks * AL_BLOCK);
                 for (int b = 0; b < kblocks; b++) { tma_load_2d(ks + s * tile_bytes + b * AL_BLOCK, &tmK, b * 64, (int)(seq + (tile0 + i) * AL_KT), k_full + s); }
@@ -114,50 +124,66 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
     else if (warp == 1)
     {
         const uint32_t idesc_s = umma_idesc_bf16(AL_KT, AL_ROWS), idesc_o = umma_idesc_bf16(128, AL_ROWS) | (1u << 15);    // A has its keys outermost
-        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), p_addr = smem_u32(pw);
-        auto scores = [&](unsigned int i) {
-            if (!wait(k_full + (i & 1u), i >> 1)) { return false; }
-            tc_fence_after();
-            if (elect_one())
-            {
-                for (int k = 0; k * 16 < (int)p.dim; k++)
-                {
-                    umma_bf16(tmem + (i & 1u) * AL_ROWS, umma_desc_kmajor_sw128(k_addr + (i & 1u) * tile_bytes + (k / 4) * AL_BLOCK + (k % 4) * 32),
-                        umma_desc_kmajor_sw128(q_addr + (k / 4) * AL_QBLOCK + (k % 4) * 32), idesc_s, k != 0 ? 1u : 0u);
-                }
-                umma_commit(s_full + (i & 1u));
-            }
-            __syncwarp();
-            return true;
-        };
-        unsigned int i = 0;
-        bool ok = tiles == 0 || (wait(q_ready, 0) && scores(0) && (tiles == 1 || scores(1)));
-        for (; i < tiles && ok; i++)
+        const uint32_t k_addr = smem_u32(ks);
+        const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(qs)), p_desc = umma_desc_kmajor_sw128(smem_u32(pw));
+        const int steps = ((int)p.dim + 15) / 16;
+        // whatever is ready first: the scores of a tile that has arrived, or the value product of one whose weights are there (the
+        // scores two tiles on take the place of scores that have been read by then)
+        unsigned int si = 0, i = 0;
+        bool ok = tiles == 0 || wait(q_ready, 0);
+        unsigned long long since = global_timer_ns();
+        while (ok && i < tiles)
         {
-            ok = wait(p_ready, i);
-            if (!ok) { break; }
-            tc_fence_after();
-            if (elect_one())
+            if (si < tiles && si < i + 2 && mbar_test(k_full + (si & 1u), (si >> 1) & 1u))
             {
-                for (int v = 0; v < vparts; v++)
+                tc_fence_after();
+                if (elect_one())
                 {
-#pragma unroll
-                    for (int part = 0; part < 2; part++)    // the high halves of the weights, then the low ones
+                    uint64_t a = umma_desc_kmajor_sw128(k_addr + (si & 1u) * tile_bytes), b = q_desc;
+                    for (int k0 = 0; k0 < steps; k0 += 4, a += AL_BLOCK >> 4, b += AL_QBLOCK >> 4)
                     {
 #pragma unroll
-                        for (int k = 0; k < AL_KT / 16; k++)
+                        for (int k = 0; k < 4; k++)
                         {
-                            umma_bf16(tmem + AL_O + v * AL_ROWS, umma_desc_mnmajor_sw128(k_addr + (i & 1u) * tile_bytes + v * 2 * AL_BLOCK + k * 2048),
-                                umma_desc_kmajor_sw128(p_addr + part * AL_QBLOCK + k * 32), idesc_o, (i | (unsigned int)part | (unsigned int)k) != 0 ? 1u : 0u);
+                            if (k0 + k < steps) { umma_bf16(tmem + (si & 1u) * AL_ROWS, a + k * 2, b + k * 2, idesc_s, (k0 | k) != 0 ? 1u : 0u); }
                         }
                     }
+                    umma_commit(s_full + (si & 1u));
                 }
-                umma_commit(k_empty + (i & 1u));
-                umma_commit(pv_done);
-                if (i + 1 == tiles) { umma_commit(o_full); }
+                __syncwarp();
+                si++;
+                since = global_timer_ns();
+                continue;
             }
-            __syncwarp();
-            if (i + 2 < tiles && !scores(i + 2)) { ok = false; }
+            if (i < si && mbar_test(p_ready, i & 1u))
+            {
+                tc_fence_after();
+                if (elect_one())
+                {
+                    uint64_t a = umma_desc_mnmajor_sw128(k_addr + (i & 1u) * tile_bytes);
+                    for (int v = 0; v < vparts; v++, a += 2 * AL_BLOCK >> 4)
+                    {
+#pragma unroll
+                        for (int part = 0; part < 2; part++)    // the high halves of the weights, then the low ones
+                        {
+#pragma unroll
+                            for (int k = 0; k < AL_KT / 16; k++)
+                            {
+                                umma_bf16(tmem + AL_O + v * AL_ROWS, a + (k * 2048 >> 4), p_desc + (part * AL_QBLOCK + k * 32 >> 4), idesc_o,
+                                    (i | (unsigned int)part | (unsigned int)k) != 0 ? 1u : 0u);
+                            }
+                        }
+                    }
+                    umma_commit(k_empty + (i & 1u));
+                    umma_commit(pv_done);
+                    if (i + 1 == tiles) { umma_commit(o_full); }
+                }
+                __syncwarp();
+                i++;
+                since = global_timer_ns();
+                continue;
+            }
+            ok = __all_sync(0xFFFFFFFFu, *abort_flag == 0 && global_timer_ns() - since < kWaitLimitNs);
         }
         if (!ok)
         {
@@ -169,27 +195,41 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
     else
     {
         const unsigned int st = tid - 64, sw = warp - 2, quarter = warp & 3u, side = sw >> 2;
-        // queries, in eights
+        // queries in eights, four rows per warp
         if (!idle)
         {
-            const bool vec = (p.q_ld % 8) == 0 && (p.ld % 8) == 0;
-            for (unsigned int c = st; c < AL_ROWS * (unsigned int)kblocks * 8; c += 256)
+            const bool vec = (p.q_ld % 8) == 0 && (p.ld % 8) == 0 && (p.dim % 8) == 0;
+            uint4 u[4][3];
+#pragma unroll
+            for (unsigned int r = 0; r < 4; r++)
             {
-                const unsigned int r = c / (kblocks * 8), q = c % (kblocks * 8), d = q * 8, row = r0 + r;
-                uint4 u = make_uint4(0, 0, 0, 0);
-                if (row < rows && d < p.dim)
+                const unsigned int row = r0 + sw * 4 + r;
+                const __nv_bfloat16* src = x + (size_t)(start + (row < rows ? row / p.G : 0u)) * p.ld + (size_t)(row < rows ? row % p.G : 0u) * p.q_ld;
+#pragma unroll
+                for (unsigned int j = 0; j < 3; j++)
                 {
-                    const __nv_bfloat16* src = x + (size_t)(start + row / p.G) * p.ld + (size_t)(row % p.G) * p.q_ld + d;
-                    if (vec && d + 8 <= p.dim) { u = *reinterpret_cast<const uint4*>(src); }
+                    const unsigned int d = (lane + j * 32) * 8;
+                    u[r][j] = make_uint4(0, 0, 0, 0);
+                    if (row >= rows || d >= p.dim) { continue; }
+                    if (vec) { u[r][j] = *reinterpret_cast<const uint4*>(src + d); }
                     else
                     {
                         uint32_t w[8];
 #pragma unroll
-                        for (int j = 0; j < 8; j++) { w[j] = d + j < p.dim ? __bfloat16_as_ushort(src[j]) : 0u; }
-                        u = make_uint4(w[0] | (w[1] << 16), w[2] | (w[3] << 16), w[4] | (w[5] << 16), w[6] | (w[7] << 16));
+                        for (int k = 0; k < 8; k++) { w[k] = d + k < p.dim ? __bfloat16_as_ushort(src[d + k]) : 0u; }
+                        u[r][j] = make_uint4(w[0] | (w[1] << 16), w[2] | (w[3] << 16), w[4] | (w[5] << 16), w[6] | (w[7] << 16));
                     }
                 }
-                *reinterpret_cast<uint4*>(qs + (q / 8) * AL_QBLOCK + r * 128 + (((q % 8) ^ (r & 7u)) * 16)) = u;
+            }
+#pragma unroll
+            for (unsigned int r = 0; r < 4; r++)
+            {
+#pragma unroll
+                for (unsigned int j = 0; j < 3; j++)
+                {
+                    const unsigned int q = lane + j * 32, at = sw * 4 + r;
+                    if (q < (unsigned int)kblocks * 8) { *reinterpret_cast<uint4*>(qs + (q / 8) * AL_QBLOCK + at * 128 + (((q % 8) ^ (at & 7u)) * 16)) = u[r][j]; }
+                }
             }
         }
         fence_proxy_async();
@@ -321,15 +361,23 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
                     tmem_ld_32x32(lanes + AL_O + v * AL_ROWS, o);
                     tmem_ld_wait();
                 }
-#pragma unroll
-                for (unsigned int r = 0; r < AL_ROWS; r++)
+                if (p.splits > 1)
                 {
-                    if (r >= live) { continue; }
-                    if (p.splits > 1)
+                    float* out = mine + 2 * AL_ROWS + d;
+#pragma unroll
+                    for (unsigned int r = 0; r < AL_ROWS; r++)
                     {
-                        if (d < vl) { mine[2 * AL_ROWS + (size_t)r * vl + d] = __uint_as_float(o[r]); }
+                        if (r < live && d < vl) { out[r * vl] = __uint_as_float(o[r]); }
                     }
-                    else if (d < p.vdim) { attention_store(p, x, start, 0, r0 + r, d, __uint_as_float(o[r]) / ml[r][1]); }
+                    continue;
+                }
+#pragma unroll 1
+                for (unsigned int r = 0; r < live; r++)
+                {
+                    float y = 0.f;
+#pragma unroll
+                    for (unsigned int k = 0; k < AL_ROWS; k++) { y = k == r ? __uint_as_float(o[k]) : y; }
+                    if (d < p.vdim) { attention_store(p, x, start, 0, r0 + r, d, y / ml[r][1]); }
                 }
             }
         }

@@ -190,7 +190,8 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
     }
     else if (warp == 1)
     {
-        const uint32_t k_addr = smem_u32(ks), w_addr = smem_u32(ws);
+        const uint32_t k_addr = smem_u32(ks);
+        const uint64_t w_desc = umma_desc_mnmajor_sw128(smem_u32(ws));
         const uint32_t idesc = umma_idesc_bf16(128, MC_COLS) | (1u << 15) | (1u << 16);    // both operands lie with their k outermost
         bool ok = true;
         unsigned int c = 0;
@@ -204,14 +205,15 @@ __global__ void __launch_bounds__(MS_ROLES, 1) mlstm_states_kernel(const __grid_
             {
                 for (unsigned int mb = 0; mb < (dp + 127) / 128; mb++)
                 {
+                    const uint64_t a = umma_desc_mnmajor_sw128(k_addr + (s * 2 * blocks + mb * 2) * MC_BLOCK), later = a + (blocks * MC_BLOCK >> 4);
+#pragma unroll
                     for (unsigned int part = 0; part < 2; part++)
                     {
 #pragma unroll
                         for (unsigned int k = 0; k < MC_L / 16; k++)
                         {
-                            umma_bf16(tmem + mb * MC_COLS,
-                                umma_desc_mnmajor_sw128(k_addr + ((s * 2 + k / 4) * blocks + mb * 2) * MC_BLOCK + (k % 4) * 2048),
-                                umma_desc_mnmajor_sw128(w_addr + part * MC_ROWS + (k / 4) * MC_BLOCK + (k % 4) * 2048), idesc, 1u);
+                            umma_bf16(tmem + mb * MC_COLS, (k < 4 ? a : later) + ((k % 4) * 2048 >> 4),
+                                w_desc + (part * MC_ROWS + (k / 4) * MC_BLOCK + (k % 4) * 2048 >> 4), idesc, 1u);
                         }
                     }
                 }
@@ -573,7 +575,8 @@ __global__ void __launch_bounds__(MO_THREADS, 2) mlstm_outputs_kernel(const __gr
     }
     else if (warp == 1)
     {
-        const uint32_t q_addr = smem_u32(qs), k_addr = smem_u32(ks), s_addr = smem_u32(ss), v_addr = smem_u32(vs);
+        const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(qs)), k_desc = umma_desc_kmajor_sw128(smem_u32(ks)),
+                       s_desc = umma_desc_mnmajor_sw128(smem_u32(ss)), v_desc = umma_desc_mnmajor_sw128(smem_u32(vs));
         const uint32_t idesc_s = umma_idesc_bf16(MC_L, MC_L), idesc_o = umma_idesc_bf16(MC_L, VB) | (1u << 16);    // B is MN-major
         bool ok = true;
         unsigned int b = 0;
@@ -584,16 +587,21 @@ __global__ void __launch_bounds__(MO_THREADS, 2) mlstm_outputs_kernel(const __gr
             tc_fence_after();
             if (elect_one())
             {
-                for (unsigned int k = 0; k < 4 && b * 4 + k < steps; k++)
+#pragma unroll
+                for (unsigned int k = 0; k < 4; k++)
                 {
-                    umma_bf16(tmem, umma_desc_kmajor_sw128(q_addr + k * 32), umma_desc_kmajor_sw128(k_addr + k * 32), idesc_s, (b | k) != 0 ? 1u : 0u);
+                    if (b * 4 + k < steps) { umma_bf16(tmem, q_desc + k * 2, k_desc + k * 2, idesc_s, (b | k) != 0 ? 1u : 0u); }
                 }
-                for (unsigned int part = 0; part < 2 && !fresh; part++)
+#pragma unroll
+                for (unsigned int part = 0; part < 2; part++)
                 {
-                    for (unsigned int k = 0; k < 4 && b * 4 + k < steps; k++)
+#pragma unroll
+                    for (unsigned int k = 0; k < 4; k++)
                     {
-                        umma_bf16(tmem + MO_O, umma_desc_kmajor_sw128(q_addr + k * 32),
-                            umma_desc_mnmajor_sw128(s_addr + part * (VB / 64) * MC_BLOCK + k * 2048), idesc_o, (b | part | k) != 0 ? 1u : 0u);
+                        if (!fresh && b * 4 + k < steps)
+                        {
+                            umma_bf16(tmem + MO_O, q_desc + k * 2, s_desc + (part * (VB / 64) * MC_BLOCK + k * 2048 >> 4), idesc_o, (b | part | k) != 0 ? 1u : 0u);
+                        }
                     }
                 }
                 if (b + 1 < blocks) { umma_commit(empty); }
@@ -607,12 +615,14 @@ __global__ void __launch_bounds__(MO_THREADS, 2) mlstm_outputs_kernel(const __gr
             tc_fence_after();
             if (elect_one())
             {
+#pragma unroll
                 for (unsigned int part = 0; part < 2; part++)
                 {
+#pragma unroll
                     for (unsigned int k = 0; k < MC_L / 16; k++)
                     {
                         umma_bf16_ts(tmem + MO_O, tmem + (k / 4) * 64 + part * 32 + (k % 4) * 8,
-                            umma_desc_mnmajor_sw128(v_addr + (k / 4) * (VB / 64) * MC_BLOCK + (k % 4) * 2048), idesc_o, !fresh || (part | k) != 0 ? 1u : 0u);
+                            v_desc + ((k / 4) * (VB / 64) * MC_BLOCK + (k % 4) * 2048 >> 4), idesc_o, !fresh || (part | k) != 0 ? 1u : 0u);
                     }
                 }
                 umma_commit(o_full);
