@@ -66,7 +66,7 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
     }
     if (warp == 1) { tmem_alloc(tmem_slot, AL_TMEM); }
     grid_dependency_launch();
-    grid_dependency_wait();
+    // (the batch's arrays are written before the step's first launch)
     const unsigned int n = (unsigned int)p.n[e], start = (unsigned int)p.start[e], pos = (unsigned int)p.pos[e], rows = n * p.G, r0 = rt * AL_ROWS;
     const bool idle = r0 >= rows;    // a shorter entry than the longest one
     const __nv_bfloat16* x = (const __nv_bfloat16*)p.qkvg;
@@ -74,6 +74,20 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
     const unsigned int T = idle ? 0 : min(pos + last_row / p.G + 1, p.T_max), begin = idle ? 0 : first_key(p, e, pos + r0 / p.G + 1) / AL_KT;
     const unsigned int all = (T + AL_KT - 1) / AL_KT, per = (all - begin + p.splits - 1) / p.splits;
     const unsigned int tile0 = min(begin + split * per, all), tiles = min(tile0 + per, all) - tile0;
+    const int seq_row = (int)((unsigned int)p.slot[e] * p.T_max + tile0 * AL_KT);
+    // tiles on their way to L2
+    auto prefetch = [&](unsigned int t) {
+        for (int b = 0; b < kblocks && t < tiles; b++)
+        {
+            asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];" ::"l"(&tmK), "r"(b * 64), "r"(seq_row + (int)t * AL_KT) : "memory");
+        }
+    };
+    if (tid == 0)
+    {
+        prefetch(0);
+        prefetch(1);
+    }
+    grid_dependency_wait();
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -88,26 +102,16 @@ __global__ void __launch_bounds__(AL_THREADS) attention_latent_kernel(const __gr
     {
         if (lane == 0)
         {
-            const unsigned int seq = (unsigned int)p.slot[e] * p.T_max;
             unsigned int i = 0;
             bool ok = true;
-            // tiles further on, on their way to L2
-            auto prefetch = [&](unsigned int t) {
-                for (int b = 0; b < kblocks && t < tiles; b++)
-                {
-                    asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];" ::"l"(&tmK), "r"(b * 64), "r"((int)(seq + (tile0 + t) * AL_KT))
-                                 : "memory");
-                }
-            };
-            prefetch(2);
             for (; i < tiles; i++)
             {
                 const unsigned int s = i & 1u;
-                if (i >= 1) { prefetch(i + 2); }
                 if (i >= 2 && !wait(k_empty + s, (i >> 1) - 1)) { ok = false; break; }
                 mbar_expect_tx(k_full + s, (unsigned int)kblocks * AL_BLOCK);
-                for (int b = 0; b < kblocks; b++) { tma_load_2d(ks + s * tile_bytes + b * AL_BLOCK, &tmK, b * 64, (int)(seq + (tile0 + i) * AL_KT), k_full + s); }
+                for (int b = 0; b < kblocks; b++) { tma_load_2d(ks + s * tile_bytes + b * AL_BLOCK, &tmK, b * 64, seq_row + (int)i * AL_KT, k_full + s); }
                 mbar_arrive(k_full + s);
+                prefetch(i + 2);
             }
             if (!ok)
             {

@@ -4,6 +4,7 @@
 #include "../../../include/cccc_b200_decoder.h"
 #include "../common.cuh"
 
+#include <atomic>
 #include <cstring>
 
 namespace b200
@@ -106,6 +107,16 @@ __device__ __forceinline__ float rotated(const float* head, unsigned int d, unsi
     return second ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
 }
 
+// Once per kernel (its own `done`) and device: of an SM's memory, a quarter as shared memory is enough.
+template <class K>
+static void prefer_l1(K kernel, std::atomic<unsigned long long>& done)
+{
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64 || (done.load(std::memory_order_relaxed) >> dev & 1ull)) { return; }
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, 25) != cudaSuccess) { cudaGetLastError(); }
+    done.fetch_or(1ull << dev, std::memory_order_relaxed);
+}
+
 // A launch in clusters of `cluster` CTAs along x (1: none).
 template <class K, class... Args>
 static int launch_cluster(const char* label, K kernel, dim3 grid, dim3 block, size_t smem, unsigned int cluster, void* stream, bool pdl, Args... args)
@@ -127,6 +138,11 @@ static int launch_cluster(const char* label, K kernel, dim3 grid, dim3 block, si
     {
         attr[cfg.numAttrs].id = cudaLaunchAttributeProgrammaticStreamSerialization;
         attr[cfg.numAttrs++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 8 && cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess)
+    {
+        report_launch(label);
+        return 1;
     }
     if (cluster > 1)
     {

@@ -299,6 +299,9 @@ static int launch_stream_wk(LinearLaunch& L, cudaStream_t st, bool pdl)
         m.block0 = blocks;
         blocks += m.fblocks * m.slots;
     }
+    // The rows of X are read through L1, of which a kernel with much shared memory just before would otherwise leave little.
+    static std::atomic<unsigned long long> done{ 0 };
+    prefer_l1(linear_stream_kernel<NT, RT, U, WK>, done);
     return launch_kernel("linear_stream", linear_stream_kernel<NT, RT, U, WK>, dim3(blocks), dim3(32 * LS_WARPS), 0, st, pdl, L);
 }
 

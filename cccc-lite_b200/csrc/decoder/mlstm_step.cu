@@ -13,11 +13,11 @@ namespace cg = cooperative_groups;
 namespace b200
 {
 
-constexpr unsigned int MS_THREADS = 256, MS_WARPS = MS_THREADS / 32, MS_TOKENS = 8, MS_COLS = 64, MS_MAX_DIM = 512, MS_MAX_CLUSTER = 8;
+constexpr unsigned int MS_THREADS = 256, MS_WARPS = MS_THREADS / 32, MS_TOKENS = 8, MS_COLS = 64, MS_MAX_DIM = 512, MS_MAX_CLUSTER = 16;
 
 // ROWS: key rows per thread; QUADS: threads side by side (four columns each)
 template <int ROWS, int QUADS>
-__global__ void __launch_bounds__(MS_THREADS, ROWS <= 16 ? 2 : 1) mlstm_step_kernel(const MlstmParams p, const unsigned int cols)
+__global__ void __launch_bounds__(MS_THREADS, ROWS <= 8 ? 3 : (ROWS <= 16 ? 2 : 1)) mlstm_step_kernel(const MlstmParams p, const unsigned int cols)
 {
     constexpr unsigned int RG = MS_THREADS / QUADS;
     extern __shared__ __align__(16) float ms_smem[];
@@ -221,8 +221,12 @@ static int step_rows(const MlstmParams& p, unsigned int entries, unsigned int ra
 int launch_mlstm_step(const MlstmParams& p, unsigned int entries, cudaStream_t stream, bool pdl)
 {
     if (p.max_n > MS_TOKENS || p.dim > MS_MAX_DIM || p.vdim > MS_COLS * MS_MAX_CLUSTER) { return -1; }
+    const DecoderDevice* dev = decoder_device();
+    if (!dev) { return 1; }
+    // slices of 16 columns, of more in clusters of eight; clusters of sixteen where they are needed, or all fit at once
     unsigned int ranks = (p.vdim + 15) / 16;
-    if (ranks > MS_MAX_CLUSTER) { ranks = MS_MAX_CLUSTER; }
+    const bool wide = p.vdim > 8 * MS_COLS || (p.vdim > 256 && entries * p.heads * 16 <= (unsigned int)dev->sm_count);
+    if (ranks > 8) { ranks = wide ? 16 : 8; }
     const unsigned int cols = ((p.vdim + ranks - 1) / ranks + 3) / 4 * 4;
     ranks = (p.vdim + cols - 1) / cols;
     if (cols <= 16) { return step_rows<4>(p, entries, ranks, cols, stream, pdl); }
