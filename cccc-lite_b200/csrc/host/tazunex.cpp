@@ -12,7 +12,7 @@ bool positive(const Json& j, const std::vector<std::string>& names, const std::s
 {
     for (const auto& n : names)
     {
-        if (j[n].type() != Json::NUMBER || j[n].number() <= 0) { return configError(err, at + "." + n + " must be positive"); }
+        if (j[n].type() != Json::NUMBER || j[n].number() <= 0) { return configError(err, (at.empty() ? "" : at + ".") + n + " must be positive"); }
     }
     return true;
 }
@@ -104,10 +104,8 @@ bool readMixer(const Json& j, const std::string& at, const std::string& p, Layer
 bool readSpec(const Json& c, DecoderSpec* s, std::string* err)
 {
     warnUnknown(c, "", { "architecture", "layers", "logit_softcap", "norm", "vocab", "width" });
-    if (!c["layers"].size() || !positive(c, { "vocab", "width", "logit_softcap" }, "", err) || c["norm"]["eps"].type() != Json::NUMBER)
-    {
-        return configError(err, "vocab, width, norm.eps, logit_softcap and layers are needed");
-    }
+    if (!positive(c, { "vocab", "width", "logit_softcap" }, "", err)) { return false; }
+    if (!c["layers"].size() || c["norm"]["eps"].type() != Json::NUMBER) { return configError(err, "norm.eps and layers are needed"); }
     s->vocab = (int)c["vocab"].number();
     s->width = (int)c["width"].number();
     s->eps = (float)c["norm"]["eps"].number();
