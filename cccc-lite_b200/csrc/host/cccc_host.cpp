@@ -306,7 +306,7 @@ void Matrix::quantizeWeights(DataType target, const std::function<float(float)>&
     if (!Cublas::isQuantized(target) || !owns_ || !gpu_) { return; }
     if (dt_ != FLOAT && dt_ != BFLOAT16) { return; }
     gpu_->setAsCurrent();
-    gpu_->synchronize();
+    cudaDeviceSynchronize();    // the tensor may have come through the default stream
     const size_t n = getDataSize();
     // Matrix.cpp:310-318: work from a float copy
     float* fbuf = (float*)gpu_->malloc(n * sizeof(float));
@@ -318,6 +318,8 @@ void Matrix::quantizeWeights(DataType target, const std::function<float(float)>&
     }
     if (dt_ == FLOAT) { cudaMemcpy(fbuf, data_, n * sizeof(float), cudaMemcpyDeviceToDevice); }
     else { cuda_convert(data_, (int)dt_, fbuf, (int)FLOAT, (unsigned)n, 1.0f); }
+    // a copy within the device returns before it is done, and the control's stream does not wait for the default one
+    cudaDeviceSynchronize();
     if (target == FP4_E2M1)
     {
         // Matrix.cpp:321-335: block 16, E4M3 dequant multipliers

@@ -199,8 +199,9 @@ typedef struct cuda_b200_mlstm
 C_EXPORT unsigned long long cuda_b200_mlstm_state_floats(unsigned int dim, unsigned int vdim);
 C_EXPORT unsigned long long cuda_b200_mlstm_work_floats(unsigned int tokens, unsigned int entries, unsigned int heads, unsigned int dim,
     unsigned int vdim);
-/* kernel: 0 = by shape, 1 = token by token, any size, 2 = state in registers (BF16; up to 8 tokens per entry, dim and vdim up
- * to 512), 3 = in chunks of 128 tokens (BF16, prompts; dim up to 256, vdim up to 1024, multiples of 8). */
+/* kernel: 0 = by shape, 1 = token by token, any size, 2 = state in registers (BF16; up to 8 tokens per entry, dim up to 512,
+ * vdim up to 1024), 3 = in chunks of 128 tokens on tcgen05 (BF16, prompts; dim up to 256 and a multiple of 16, vdim up to 1024 and a
+ * multiple of 8; qkvg's offsets and strides multiples of 8). */
 C_EXPORT int cuda_b200_mlstm_rows(int dtype, const cuda_b200_mlstm* a, const cuda_b200_batch* b, void* stream, unsigned int flags, int kernel);
 
 /* Router: the `top` largest of each row of float logits [n][ldl] (ties: the lower expert), softmax over them; the
