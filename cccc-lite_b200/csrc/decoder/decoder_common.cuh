@@ -79,20 +79,44 @@ __device__ __forceinline__ float warp_sum(float v)
 
 __host__ __device__ __forceinline__ bool activation_gated(int activation) { return activation == B200_ACT_SILU_GATE || activation == B200_ACT_GELU_GATE; }
 
-__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
-
-// The part of a linear's epilogue that does not depend on where the result goes.
-__device__ __forceinline__ float linear_activation(int activation, float a, float up, float cap)
+// sigmoid by the hardware's exponential and reciprocal (a few units in the last place), for results that become BF16
+__device__ __forceinline__ float sigmoid_fast(float z)
 {
-    if (activation == B200_ACT_RELU2)
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(-1.44269504088896341f * z));
+    return __fdividef(1.0f, 1.0f + y);
+}
+
+// The part of a linear's epilogue that does not depend on where the result goes.  GELU in its tanh form: (1 + tanh u) / 2 is the sigmoid
+// of 2u.
+template <int ACT, bool FAST>
+__device__ __forceinline__ float activate(float a, float up, float cap)
+{
+    if constexpr (ACT == B200_ACT_RELU2)
     {
         a = fmaxf(a, 0.f);
         return a * a;
     }
-    if (activation == B200_ACT_SILU_GATE) { return a * sigmoid_f32(a) * up; }
-    if (activation == B200_ACT_GELU_GATE) { return gelu_tanh_f32(a) * up; }
-    if (activation == B200_ACT_SOFTCAP) { return cap * tanhf(a / cap); }
-    return a;
+    else if constexpr (ACT == B200_ACT_SILU_GATE) { return a * (FAST ? sigmoid_fast(a) : sigmoid_f32(a)) * up; }
+    else if constexpr (ACT == B200_ACT_GELU_GATE)
+    {
+        const float u = 0.7978845608028654f * (a + 0.044715f * a * a * a);
+        return FAST ? a * sigmoid_fast(2.0f * u) * up : 0.5f * a * (1.0f + tanhf(u)) * up;
+    }
+    else if constexpr (ACT == B200_ACT_SOFTCAP) { return cap * tanhf(a / cap); }
+    else { return a; }
+}
+template <bool FAST>
+__device__ __forceinline__ float linear_activation(int activation, float a, float up, float cap)
+{
+    switch (activation)
+    {
+    case B200_ACT_RELU2: return activate<B200_ACT_RELU2, FAST>(a, up, cap);
+    case B200_ACT_SILU_GATE: return activate<B200_ACT_SILU_GATE, FAST>(a, up, cap);
+    case B200_ACT_GELU_GATE: return activate<B200_ACT_GELU_GATE, FAST>(a, up, cap);
+    case B200_ACT_SOFTCAP: return activate<B200_ACT_SOFTCAP, FAST>(a, up, cap);
+    default: return a;
+    }
 }
 
 // Element d of a head after its first `dims` elements have been turned pair by pair (element i goes with i + dims / 2, or,

@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(32 * LS_WARPS, NT == 4 ? 1 : 2) linear_stream_
 #pragma unroll
                 for (int w = 0; w < WK; w++) { up += red[w0 + w][n][16 + fl]; }
             }
-            const float y = linear_activation(m.activation, m.alpha * v, m.alpha * up, m.cap);
+            const float y = linear_activation<true>(m.activation, m.alpha * v, m.alpha * up, m.cap);
             linear_store(m, row0 + n0 + n, ycol + fc + f, y * linear_row_factor<__nv_bfloat16>(m, row0 + n0 + n, group));
         }
     }
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearMember m)
             const unsigned int r = r0 + ty + 16 * i, f = f0 + tx + 16 * j;
             if (r < count && f < m.N)
             {
-                const float y = linear_activation(m.activation, m.alpha * acc[0][i][j], GATED ? m.alpha * acc[GATED ? 1 : 0][i][j] : 0.f, m.cap);
+                const float y = linear_activation<false>(m.activation, m.alpha * acc[0][i][j], GATED ? m.alpha * acc[GATED ? 1 : 0][i][j] : 0.f, m.cap);
                 linear_store(m, row0 + r, ycol + f, y * linear_row_factor<float>(m, row0 + r, group));
             }
         }

@@ -11,6 +11,8 @@
 #include "../gemm_prefill.cuh"
 #include "linear.cuh"
 
+#include <type_traits>
+
 namespace b200
 {
 
@@ -283,22 +285,29 @@ __global__ void __launch_bounds__(LT_THREADS, 1) linear_tile_kernel(const __grid
                 float v[32];
                 tmem_ld_32x32(lanes + c, r);
                 tmem_ld_wait();
+                // one activation's code for all columns at a time
+                auto plain = [&](auto act) {
+#pragma unroll
+                    for (int j = 0; j < 32; j++) { v[j] = activate<decltype(act)::value, true>(m.alpha * __uint_as_float(r[j]), 0.f, m.cap); }
+                };
                 if (gated)
                 {
                     uint32_t u[32];
                     tmem_ld_32x32(lanes + BN / 2 + c, u);
                     tmem_ld_wait();
+                    auto both = [&](auto act) {
 #pragma unroll
-                    for (int j = 0; j < 32; j++)
-                    {
-                        v[j] = linear_activation(m.activation, m.alpha * __uint_as_float(r[j]), m.alpha * __uint_as_float(u[j]), m.cap);
-                    }
+                        for (int j = 0; j < 32; j++)
+                        {
+                            v[j] = activate<decltype(act)::value, true>(m.alpha * __uint_as_float(r[j]), m.alpha * __uint_as_float(u[j]), m.cap);
+                        }
+                    };
+                    if (m.activation == B200_ACT_SILU_GATE) { both(std::integral_constant<int, B200_ACT_SILU_GATE>()); }
+                    else { both(std::integral_constant<int, B200_ACT_GELU_GATE>()); }
                 }
-                else
-                {
-#pragma unroll
-                    for (int j = 0; j < 32; j++) { v[j] = linear_activation(m.activation, m.alpha * __uint_as_float(r[j]), 0.f, m.cap); }
-                }
+                else if (m.activation == B200_ACT_NONE) { plain(std::integral_constant<int, B200_ACT_NONE>()); }
+                else if (m.activation == B200_ACT_RELU2) { plain(std::integral_constant<int, B200_ACT_RELU2>()); }
+                else { plain(std::integral_constant<int, B200_ACT_SOFTCAP>()); }
                 if (rl < live) { store_row32(m, r0 + rl, block, f0 + c, v, vec != 0); }
                 __syncwarp();
             }
