@@ -8,7 +8,7 @@
 // choice, gate+up of the chosen experts and the shared one, down of both.  The mixer is q+k+v+gate, append and attention (which
 // applies the output gate); or, for latent attention, both down projections, their norms and the cache row, the queries, the
 // queries against the latent (or, in prompts, keys and values of all heads from the cached latents), attention, the values'
-// projection and gate; or q+k+v+gate, the gates of the recurrence, and the recurrence.
+// projection and gate; or q+k+v+gate with the recurrence's own gates beside them as floats, and the recurrence.
 #pragma once
 
 #include "language_model.h"
